@@ -273,19 +273,58 @@ int b200_rejection_sample(int64_t* out, int64_t B, int S, const int64_t* draft_i
                           const uint8_t* is_greedy, const float* uniform, const float* recover_q, uint64_t seed,
                           uint64_t step, cudaStream_t st);
 
+// ---- layer norm / post-norm residual stream / unit-norm split (elementwise/layernorm.cu) ----------
+int b200_embed_layernorm(float* x, void* h, const int64_t* ids, const int64_t* positions, const void* table,
+                         const double* freq, const float* w, int64_t T, int H, int ld, int64_t rows, float eps,
+                         int dtype, cudaStream_t st);
+int b200_layernorm_residual(float* x, void* h, const void* y1, int64_t y1_stride, float s1, const void* y2,
+                            int64_t y2_stride, float s2, const float* w, int64_t T, int H, int ld, float eps, int add,
+                            int dtype, cudaStream_t st);
+int b200_gated_group_rmsnorm(void* out, int64_t out_stride, const float* o, int64_t o_stride, const void* gate,
+                             int64_t gate_stride, const float* w, int64_t T, int groups, int D, float eps, int dtype,
+                             cudaStream_t st);
+int b200_qk_unit_norm_cache(void* q_out, const void* q, const void* k, const void* v, int64_t stride, void* kv_cache,
+                            const int64_t* slots, int64_t T, int Hq, int Hkv, int D, int Dv, int Dc, int block_size,
+                            int64_t num_blocks, float eps, int dtype, cudaStream_t st);
+
+// ---- fp32 GEMM on the CUDA cores (gemm/gemm_f32.cu): out[T, N] = x[T, K] . w[N, K]^T (+ bias) -----------------
+int b200_gemm_f32(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, int64_t ldw, const float* bias,
+                  int64_t T, int N, int K, cudaStream_t st);
+
+// ---- paged attention for any head size and for fp32 (attention/paged_generic.cu) -----------------
+int b200_paged_attention_generic(void* out, const void* q, const void* kv_cache, const int* block_tables,
+                                 const int* seq_lens, const int* qsl, const float* sinks, int64_t T, int B, int Hq,
+                                 int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks, int max_query_len,
+                                 int window, float scale, int dtype, cudaStream_t st);
+
 // ---- gated delta net / conv / MTP glue --------------------------------------------------------
 int b200_causal_conv1d_fwd(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w,
                            const void* bias, const int* cu, int R, void* states, const int* slots,
                            const uint8_t* has_init, int C, int W, int act, int64_t T_, int dtype, cudaStream_t st);
 int b200_causal_conv1d_update(void* out, int64_t out_stride, const void* x, int64_t x_stride, void* states,
-                              const void* w, const void* bias, const int* slots, int64_t B, int C, int W, int act,
-                              int dtype, cudaStream_t st);
+                              const void* w, const void* bias, const int* slots, const int* has_init, int64_t B, int C,
+                              int W, int act, int dtype, cudaStream_t st);
 int b200_gdn_gating(float* g, float* beta, const void* a, int64_t a_stride, const void* b, int64_t b_stride,
                     const float* A_log, const float* dt_bias, int H, int64_t T_, int dtype, cudaStream_t st);
 int b200_gdn_recurrent(void* out, int64_t o_stride, const void* q, const void* k, int64_t qk_stride, const void* v,
                        int64_t v_stride, const float* g, const float* beta, float* states, const int* cu,
                        const int* slots, const uint8_t* has_init, int R, int Hk, int Hv, int Dk, int Dv, float scale,
                        int l2norm, int dtype, cudaStream_t st);
+// Linear recurrences with a matrix state (linear_attn/recurrence.cu); kind 0 = delta rule with a decay per key channel,
+// 1 = fixed decay per head.  q, k: [T][Hk][Dk], v: [T][H][Dv] column slices of one row-strided tensor.
+typedef struct RecurrenceArgs {
+  float* out;                // [T][H][Dv], rows out_stride apart
+  const void *q, *k, *v;     // raw (kind 1) or convolved (kind 0) projections, rows qkv_stride apart
+  const void *a, *b;         // kind 0: raw decay [T][H][Dk] and step-size [T][H] projections
+  const float *A_log, *dt_bias;  // kind 0: [H], [H][Dk]
+  const float* decay;        // kind 1: [H]
+  float* states;             // [slots][H][Dv][Dks]
+  const int *cu, *slots, *has_init;
+  int64_t out_stride, qkv_stride, a_stride, b_stride;
+  int R, Hk, H, Dk, Dks, Dv, kind;
+  float scale, unit_eps;
+} RecurrenceArgs;
+int b200_linear_recurrence(const RecurrenceArgs* a, int dtype, cudaStream_t st);
 int b200_sigmoid_gate_mul(void* out, const void* o, const void* gate, int64_t gate_stride, int D, int64_t T_,
                           int dtype, cudaStream_t st);
 int b200_mtp_concat_norm(void* out, const void* embed, const void* hidden, const void* we, const void* wh,

@@ -1331,11 +1331,13 @@ void causal_conv1d_fwd(at::Tensor out, const at::Tensor& x, const at::Tensor& w,
 }
 
 void causal_conv1d_update(at::Tensor out, const at::Tensor& x, at::Tensor states, const at::Tensor& w,
-                          const c10::optional<at::Tensor>& bias, const at::Tensor& slots, bool act) {
+                          const c10::optional<at::Tensor>& bias, const at::Tensor& slots, bool act,
+                          const c10::optional<at::Tensor>& has_init) {
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.stride(1) == 1 && w.is_contiguous() && states.is_contiguous());
+  if (has_init.has_value()) TORCH_CHECK(has_init->scalar_type() == at::kInt && has_init->numel() >= x.size(0));
   check(b200_causal_conv1d_update(out.data_ptr(), out.stride(0), x.data_ptr(), x.stride(0), states.data_ptr(), w.data_ptr(),
-                                  opt_ptr(bias), slots.data_ptr<int>(), x.size(0), (int)x.size(1), (int)w.size(1), act,
-                                  dtype_code(x), stream()), "causal_conv1d_update");
+                                  opt_ptr(bias), slots.data_ptr<int>(), optp<int>(has_init), x.size(0), (int)x.size(1),
+                                  (int)w.size(1), act, dtype_code(x), stream()), "causal_conv1d_update");
 }
 
 void gdn_gating(at::Tensor g, at::Tensor beta, const at::Tensor& a, const at::Tensor& b, const at::Tensor& A_log,
@@ -1372,6 +1374,121 @@ void sigmoid_gate_mul(at::Tensor out, const at::Tensor& o, const at::Tensor& gat
   TORCH_CHECK(o.is_contiguous() && out.is_contiguous() && gate.stride(1) == 1 && o.dim() == 2);
   check(b200_sigmoid_gate_mul(out.data_ptr(), o.data_ptr(), gate.data_ptr(), gate.stride(0), (int)o.size(1), o.size(0),
                               dtype_code(o), stream()), "sigmoid_gate_mul");
+}
+
+// ------------------------------------------------------- fp32 residual stream, linear recurrences, fp32 models
+// x [T, ld] fp32 stream, h its copy in the model's dtype (the same tensor for fp32 models); width = w.numel() <= ld.
+void embed_layernorm(at::Tensor x, at::Tensor h, const at::Tensor& ids, const at::Tensor& positions, const at::Tensor& table,
+                     const at::Tensor& freq, const at::Tensor& w, double eps) {
+  TORCH_CHECK(x.is_contiguous() && h.is_contiguous() && table.is_contiguous() && x.scalar_type() == at::kFloat);
+  TORCH_CHECK(h.sizes() == x.sizes() && table.size(1) == x.size(1) && table.scalar_type() == h.scalar_type());
+  TORCH_CHECK(freq.scalar_type() == at::kDouble && freq.numel() >= (w.numel() + 1) / 2 && w.scalar_type() == at::kFloat);
+  TORCH_CHECK(ids.numel() == x.size(0) && positions.numel() == x.size(0) && w.numel() <= x.size(1));
+  check(b200_embed_layernorm(x.data_ptr<float>(), h.data_ptr(), ids.data_ptr<int64_t>(), positions.data_ptr<int64_t>(),
+                             table.data_ptr(), freq.data_ptr<double>(), w.data_ptr<float>(), x.size(0), (int)w.numel(),
+                             (int)x.size(1), table.size(0), (float)eps, dtype_code(h), stream()), "embed_layernorm");
+}
+void layernorm_residual(at::Tensor x, at::Tensor h, const c10::optional<at::Tensor>& y1, double s1,
+                        const c10::optional<at::Tensor>& y2, double s2, const at::Tensor& w, double eps) {
+  TORCH_CHECK(x.is_contiguous() && h.is_contiguous() && x.scalar_type() == at::kFloat && h.sizes() == x.sizes());
+  TORCH_CHECK(w.scalar_type() == at::kFloat && w.numel() <= x.size(1));
+  for (const auto* y : {&y1, &y2})
+    if (y->has_value())
+      TORCH_CHECK((*y)->dim() == 2 && (*y)->sizes() == x.sizes() && (*y)->stride(1) == 1 && (*y)->scalar_type() == h.scalar_type());
+  TORCH_CHECK(y1.has_value() || !y2.has_value());
+  check(b200_layernorm_residual(x.data_ptr<float>(), h.data_ptr(), opt_ptr(y1), y1.has_value() ? y1->stride(0) : 0, (float)s1,
+                                opt_ptr(y2), y2.has_value() ? y2->stride(0) : 0, (float)s2, w.data_ptr<float>(), x.size(0),
+                                (int)w.numel(), (int)x.size(1), (float)eps, y1.has_value() ? 1 : 0, dtype_code(h), stream()),
+        "layernorm_residual");
+}
+// out, gate [T, groups * D] (row-strided), o fp32; w [D]
+void gated_group_rmsnorm(at::Tensor out, const at::Tensor& o, const at::Tensor& gate, const at::Tensor& w, double eps) {
+  TORCH_CHECK(out.dim() == 2 && o.dim() == 2 && gate.dim() == 2 && out.stride(1) == 1 && o.stride(1) == 1 && gate.stride(1) == 1);
+  TORCH_CHECK(o.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && gate.scalar_type() == out.scalar_type());
+  TORCH_CHECK(o.size(1) % w.numel() == 0 && gate.sizes() == o.sizes() && out.size(0) == o.size(0) && out.size(1) >= o.size(1));
+  check(b200_gated_group_rmsnorm(out.data_ptr(), out.stride(0), o.data_ptr<float>(), o.stride(0), gate.data_ptr(),
+                                 gate.stride(0), w.data_ptr<float>(), o.size(0), (int)(o.size(1) / w.numel()), (int)w.numel(),
+                                 (float)eps, dtype_code(out), stream()), "gated_group_rmsnorm");
+}
+// q, k, v: column slices [T, heads * head size] of one row-strided tensor; q_out [T, Hq, Dc]
+void qk_unit_norm_cache(at::Tensor q_out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at::Tensor kv_cache,
+                        const at::Tensor& slots, int64_t num_heads, int64_t num_kv_heads, double eps) {
+  TORCH_CHECK(q_out.is_contiguous() && kv_cache.is_contiguous() && kv_cache.dim() == 5 && kv_cache.size(2) == num_kv_heads);
+  TORCH_CHECK(q.stride(1) == 1 && k.stride(1) == 1 && v.stride(1) == 1 && q.stride(0) == k.stride(0) && q.stride(0) == v.stride(0));
+  TORCH_CHECK(q.scalar_type() == q_out.scalar_type() && q.scalar_type() == kv_cache.scalar_type());
+  const int64_t D = q.size(1) / num_heads, Dv = v.size(1) / num_kv_heads, Dc = kv_cache.size(4);
+  TORCH_CHECK(k.size(1) == D * num_kv_heads && q_out.numel() == q.size(0) * num_heads * Dc && slots.numel() == q.size(0));
+  check(b200_qk_unit_norm_cache(q_out.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), kv_cache.data_ptr(),
+                                slots.data_ptr<int64_t>(), q.size(0), (int)num_heads, (int)num_kv_heads, (int)D, (int)Dv,
+                                (int)Dc, (int)kv_cache.size(3), kv_cache.size(0), (float)eps, dtype_code(q), stream()),
+        "qk_unit_norm_cache");
+}
+void fill_recurrence(RecurrenceArgs& a, at::Tensor& out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v,
+                     at::Tensor& states, const at::Tensor& cu, const at::Tensor& slots, const at::Tensor& has_init) {
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && out.dim() == 3 && states.dim() == 4);
+  for (const at::Tensor* t : {&q, &k, &v}) TORCH_CHECK(t->stride(2) == 1 && t->stride(1) == t->size(2));
+  TORCH_CHECK(q.stride(0) == k.stride(0) && q.stride(0) == v.stride(0) && q.sizes() == k.sizes());
+  TORCH_CHECK(out.scalar_type() == at::kFloat && out.stride(2) == 1 && out.stride(1) == out.size(2) && out.sizes() == v.sizes());
+  TORCH_CHECK(states.scalar_type() == at::kFloat && states.is_contiguous() && states.size(1) == v.size(1) &&
+              states.size(2) == v.size(2));
+  TORCH_CHECK(cu.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && has_init.scalar_type() == at::kInt);
+  TORCH_CHECK(cu.numel() == slots.numel() + 1 && has_init.numel() == slots.numel());
+  memset(&a, 0, sizeof(a));
+  a.out = out.data_ptr<float>();
+  a.q = q.data_ptr(); a.k = k.data_ptr(); a.v = v.data_ptr();
+  a.states = states.data_ptr<float>();
+  a.cu = cu.data_ptr<int>(); a.slots = slots.data_ptr<int>(); a.has_init = has_init.data_ptr<int>();
+  a.out_stride = out.stride(0); a.qkv_stride = q.stride(0);
+  a.R = (int)slots.numel(); a.Hk = (int)q.size(1); a.H = (int)v.size(1);
+  a.Dk = (int)q.size(2); a.Dks = (int)states.size(3); a.Dv = (int)v.size(2);
+}
+void channel_delta_rule(at::Tensor out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& a_,
+                        const at::Tensor& b, const at::Tensor& A_log, const at::Tensor& dt_bias, at::Tensor states,
+                        const at::Tensor& cu, const at::Tensor& slots, const at::Tensor& has_init, double scale,
+                        double unit_eps) {
+  RecurrenceArgs a;
+  fill_recurrence(a, out, q, k, v, states, cu, slots, has_init);
+  TORCH_CHECK(a_.stride(1) == 1 && b.stride(1) == 1 && a_.size(1) == a.H * a.Dk && b.size(1) == a.H);
+  TORCH_CHECK(a_.scalar_type() == q.scalar_type() && b.scalar_type() == q.scalar_type());
+  TORCH_CHECK(A_log.scalar_type() == at::kFloat && A_log.numel() == a.H && dt_bias.scalar_type() == at::kFloat &&
+              dt_bias.numel() == a.H * a.Dk);
+  a.a = a_.data_ptr(); a.b = b.data_ptr(); a.a_stride = a_.stride(0); a.b_stride = b.stride(0);
+  a.A_log = A_log.data_ptr<float>(); a.dt_bias = dt_bias.data_ptr<float>();
+  a.kind = 0; a.scale = (float)scale; a.unit_eps = (float)unit_eps;
+  check(b200_linear_recurrence(&a, dtype_code(q), stream()), "channel_delta_rule");
+}
+void fixed_decay_attention(at::Tensor out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v,
+                           const at::Tensor& decay, at::Tensor states, const at::Tensor& cu, const at::Tensor& slots,
+                           const at::Tensor& has_init) {
+  RecurrenceArgs a;
+  fill_recurrence(a, out, q, k, v, states, cu, slots, has_init);
+  TORCH_CHECK(a.Hk == a.H && decay.scalar_type() == at::kFloat && decay.numel() == a.H);
+  a.decay = decay.data_ptr<float>();
+  a.kind = 1;
+  check(b200_linear_recurrence(&a, dtype_code(q), stream()), "fixed_decay_attention");
+}
+void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& bias) {
+  TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1);
+  TORCH_CHECK(x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && out.scalar_type() == at::kFloat);
+  TORCH_CHECK(x.size(1) == w.size(1) && out.size(0) == x.size(0) && out.size(1) == w.size(0));
+  if (bias.has_value()) TORCH_CHECK(bias->scalar_type() == at::kFloat && bias->numel() == w.size(0));
+  check(b200_gemm_f32(out.data_ptr<float>(), out.stride(0), x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(), w.stride(0),
+                      bias.has_value() ? bias->data_ptr<float>() : nullptr, x.size(0), (int)w.size(0), (int)w.size(1),
+                      stream()), "gemm_f32");
+}
+void paged_attention_generic(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
+                             const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
+                             int64_t max_query_len, int64_t window, double scale) {
+  TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && kv_cache.dim() == 5);
+  TORCH_CHECK(q.size(2) == kv_cache.size(4) && out.sizes() == q.sizes() && q.scalar_type() == kv_cache.scalar_type());
+  TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && qsl.scalar_type() == at::kInt);
+  TORCH_CHECK(block_tables.stride(1) == 1);
+  check(b200_paged_attention_generic(out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(), block_tables.data_ptr<int>(),
+                                     seq_lens.data_ptr<int>(), qsl.data_ptr<int>(),
+                                     sinks.has_value() ? sinks->data_ptr<float>() : nullptr, q.size(0), (int)seq_lens.size(0),
+                                     (int)q.size(1), (int)kv_cache.size(2), (int)q.size(2), (int)kv_cache.size(3),
+                                     (int)block_tables.stride(0), kv_cache.size(0), (int)max_query_len, (int)window,
+                                     (float)scale, dtype_code(q), stream()), "paged_attention_generic");
 }
 
 // ------------------------------------------------------------------- expert-parallel dispatch / combine
@@ -1479,6 +1596,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rejection_sample", &rejection_sample);
   m.def("causal_conv1d_fwd", &causal_conv1d_fwd);
   m.def("causal_conv1d_update", &causal_conv1d_update);
+  m.def("embed_layernorm", &embed_layernorm);
+  m.def("layernorm_residual", &layernorm_residual);
+  m.def("gated_group_rmsnorm", &gated_group_rmsnorm);
+  m.def("qk_unit_norm_cache", &qk_unit_norm_cache);
+  m.def("channel_delta_rule", &channel_delta_rule);
+  m.def("fixed_decay_attention", &fixed_decay_attention);
+  m.def("gemm_f32", &gemm_f32);
+  m.def("paged_attention_generic", &paged_attention_generic);
   m.def("gdn_gating", &gdn_gating);
   m.def("gdn_recurrent", &gdn_recurrent);
   m.def("mtp_concat_norm", &mtp_concat_norm);

@@ -7,14 +7,15 @@
 // fused_recurrent_gated_delta_rule (ops/fla/fused_recurrent.py:52-155) and the chunked form
 // (ops/fla/chunk.py:23-140), which is numerically the same recurrence.
 #include "../api.h"
+#include "../common/launch.cuh"
 #include "../common/utils.cuh"
 
 namespace b200 {
 namespace {
 
-constexpr int kMaxW = 8;
-
-__device__ __forceinline__ float silu(float v) { return v / (1.f + __expf(-v)); }
+// fp32 tensors keep full fp32 accuracy (this file is compiled without fast-math); 16-bit outputs use the fast forms
+template <typename T> __device__ __forceinline__ float silu(float v) { return __fdividef(v, 1.f + __expf(-v)); }
+template <> __device__ __forceinline__ float silu<float>(float v) { return v / (1.f + expf(-v)); }
 
 __device__ __forceinline__ int find_seq(const int* __restrict__ cu, int R, int t) {
   int lo = 0, hi = R;  // largest r with cu[r] <= t
@@ -88,7 +89,7 @@ __global__ void __launch_bounds__(128) conv1d_fwd_kernel(T* __restrict__ out, in
       float acc = bv[e];
 #pragma unroll
       for (int j = 0; j < W; ++j) acc += wv[j][e] * win[j][e];
-      o.v[e] = from_f<T>(act ? silu(acc) : acc);
+      o.v[e] = from_f<T>(act ? silu<T>(acc) : acc);
     }
     st_vec(out + t * out_stride + c0, o);
 #pragma unroll
@@ -99,7 +100,31 @@ __global__ void __launch_bounds__(128) conv1d_fwd_kernel(T* __restrict__ out, in
   }
 }
 
-// states[slot] <- last W-1 rows of (old state ++ x[seq]); one thread owns a channel column.
+// Any number of taps: one thread per (token, channel), every input row read from memory.
+template <typename T>
+__global__ void conv1d_fwd_generic_kernel(T* __restrict__ out, int64_t out_stride, const T* __restrict__ x, int64_t x_stride,
+                                          const T* __restrict__ w, const T* __restrict__ bias, const int* __restrict__ cu,
+                                          int R, const T* __restrict__ states, const int* __restrict__ slots,
+                                          const uint8_t* __restrict__ has_init, int C, int W, int act, int64_t Ttot) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int64_t t = blockIdx.y;
+  if (c >= C || t >= Ttot) return;
+  const int r = find_seq(cu, R, (int)t);
+  const int p = (int)t - cu[r], slot = slots[r];
+  const bool init = has_init[r] != 0 && slot >= 0;
+  float acc = bias ? to_f(bias[c]) : 0.f;
+  for (int j = 0; j < W; ++j) {
+    const int q = p - (W - 1) + j;
+    float v = 0.f;
+    if (q >= 0) v = to_f(x[(t - (W - 1) + j) * x_stride + c]);
+    else if (init) v = to_f(states[((int64_t)slot * (W - 1) + (W - 1 + q)) * C + c]);
+    acc += to_f(w[(int64_t)c * W + j]) * v;
+  }
+  out[t * out_stride + c] = from_f<T>(act ? silu<T>(acc) : acc);
+}
+
+// states[slot] <- last W-1 rows of (old state ++ x[seq]); one thread owns a channel column.  Row j takes old row
+// j + L (or an input row): ascending j never reads a row it has already overwritten.
 template <typename T>
 __global__ void conv1d_state_kernel(T* __restrict__ states, const T* __restrict__ x, int64_t x_stride,
                                     const int* __restrict__ cu, const int* __restrict__ slots,
@@ -110,35 +135,40 @@ __global__ void conv1d_state_kernel(T* __restrict__ states, const T* __restrict_
   const int s = cu[r], L = cu[r + 1] - s, slot = slots[r];
   if (L == 0 || slot < 0) return;
   const bool init = has_init[r] != 0;
-  float keep[kMaxW];
+  T* st = states + (int64_t)slot * (W - 1) * C + c;
   for (int j = 0; j < W - 1; ++j) {
     const int q = L - (W - 1) + j;
-    if (q >= 0) keep[j] = to_f(x[(int64_t)(s + q) * x_stride + c]);
-    else keep[j] = init ? to_f(states[((int64_t)slot * (W - 1) + (W - 1 + q)) * C + c]) : 0.f;
+    T v = from_f<T>(0.f);
+    if (q >= 0) v = x[(int64_t)(s + q) * x_stride + c];
+    else if (init) v = st[(int64_t)(j + L) * C];
+    st[(int64_t)j * C] = v;
   }
-  for (int j = 0; j < W - 1; ++j) states[((int64_t)slot * (W - 1) + j) * C + c] = from_f<T>(keep[j]);
 }
 
+// One token per sequence.  `has_init` (optional): a row whose flag is 0 starts from zeros, whatever its slot holds.
 template <typename T>
 __global__ void conv1d_update_kernel(T* __restrict__ out, int64_t out_stride, const T* __restrict__ x, int64_t x_stride,
                                      T* __restrict__ states, const T* __restrict__ w, const T* __restrict__ bias,
-                                     const int* __restrict__ slots, int C, int W, int act) {
+                                     const int* __restrict__ slots, const int* __restrict__ has_init, int C, int W, int act) {
+  griddep_launch();
+  griddep_wait();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   const int b = blockIdx.y;
   if (c >= C) return;
   const int slot = slots[b];
   if (slot < 0) { out[(int64_t)b * out_stride + c] = from_f<T>(0.f); return; }
+  const bool init = has_init == nullptr || has_init[b] != 0;
   T* st = states + (int64_t)slot * (W - 1) * C + c;
   float acc = bias ? to_f(bias[c]) : 0.f;
   float cur = to_f(x[(int64_t)b * x_stride + c]);
   for (int j = 0; j < W - 1; ++j) {
-    float v = to_f(st[(int64_t)j * C]);
+    float v = init ? to_f(st[(int64_t)j * C]) : 0.f;
     acc += to_f(w[(int64_t)c * W + j]) * v;
     if (j > 0) st[(int64_t)(j - 1) * C] = from_f<T>(v);
   }
   acc += to_f(w[(int64_t)c * W + W - 1]) * cur;
-  st[(int64_t)(W - 2) * C] = from_f<T>(cur);
-  out[(int64_t)b * out_stride + c] = from_f<T>(act ? silu(acc) : acc);
+  if (W > 1) st[(int64_t)(W - 2) * C] = from_f<T>(cur);
+  out[(int64_t)b * out_stride + c] = from_f<T>(act ? silu<T>(acc) : acc);
 }
 
 // g = -exp(A_log) * softplus(a + dt_bias), beta = sigmoid(b)
@@ -153,7 +183,7 @@ __global__ void gdn_gating_kernel(float* __restrict__ g, float* __restrict__ bet
   float xa = to_f(a[t * a_stride + h]) + dt_bias[h];
   float sp = xa > 20.f ? xa : log1pf(__expf(xa));
   g[i] = -__expf(A_log[h]) * sp;
-  beta[i] = 1.f / (1.f + __expf(-to_f(b[t * b_stride + h])));
+  beta[i] = __fdividef(1.f, 1.f + __expf(-to_f(b[t * b_stride + h])));
 }
 
 // Sequential gated delta rule.  Block = 128 threads = 32 state rows (of Dv) x 4 quarters of Dk; grid
@@ -315,7 +345,7 @@ __global__ void sigmoid_gate_mul_kernel(T* __restrict__ out, const T* __restrict
   int64_t t = i / D;
   int c = (int)(i % D);
   float gv = to_f(gate[t * gate_stride + c]);
-  out[i] = from_f<T>(to_f(o[i]) / (1.f + __expf(-gv)));
+  out[i] = from_f<T>(__fdividef(to_f(o[i]), 1.f + __expf(-gv)));
 }
 
 }  // namespace
@@ -334,15 +364,22 @@ int launch_conv_fwd(void* out, int64_t out_stride, const void* x, int64_t x_stri
   conv1d_fwd_kernel<T, WW><<<g1, 128, 0, st>>>((T*)out, out_stride, (const T*)x, x_stride, (const T*)w, (const T*)bias, cu, \
                                                R, (const T*)states, slots, has_init, C, act, T_)
   switch (W) {
+    case 1: B200_CONV_W(1); break;
     case 2: B200_CONV_W(2); break;
     case 3: B200_CONV_W(3); break;
     case 4: B200_CONV_W(4); break;
     case 5: B200_CONV_W(5); break;
     case 6: B200_CONV_W(6); break;
     case 7: B200_CONV_W(7); break;
-    default: B200_CONV_W(8); break;
+    case 8: B200_CONV_W(8); break;
+    default:
+      if (T_ > 65535) return 3;
+      conv1d_fwd_generic_kernel<T><<<dim3((C + 127) / 128, (unsigned)T_), 128, 0, st>>>(
+          (T*)out, out_stride, (const T*)x, x_stride, (const T*)w, (const T*)bias, cu, R, (const T*)states, slots, has_init, C,
+          W, act, T_);
   }
 #undef B200_CONV_W
+  if (W == 1) return cudaGetLastError() != cudaSuccess;  // no history to keep
   conv1d_state_kernel<T><<<g2, 256, 0, st>>>((T*)states, (const T*)x, x_stride, cu, slots, has_init, C, W);
   return cudaGetLastError() != cudaSuccess;
 }
@@ -352,7 +389,7 @@ int launch_conv_fwd(void* out, int64_t out_stride, const void* x, int64_t x_stri
 extern "C" int b200_causal_conv1d_fwd(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w,
                                       const void* bias, const int* cu, int R, void* states, const int* slots,
                                       const uint8_t* has_init, int C, int W, int act, int64_t T_, int dtype, cudaStream_t st) {
-  if (W > b200::kMaxW || W < 2) return 3;
+  if (W < 1) return 3;
   if (T_ == 0) return 0;
   B200_DISPATCH_DTYPE(dtype, return (b200::launch_conv_fwd<T>(out, out_stride, x, x_stride, w, bias, cu, R, states, slots,
                                                               has_init, C, W, act, T_, st)));
@@ -360,14 +397,14 @@ extern "C" int b200_causal_conv1d_fwd(void* out, int64_t out_stride, const void*
 }
 
 extern "C" int b200_causal_conv1d_update(void* out, int64_t out_stride, const void* x, int64_t x_stride, void* states,
-                                         const void* w, const void* bias, const int* slots, int64_t B, int C, int W, int act,
-                                         int dtype, cudaStream_t st) {
-  if (W > b200::kMaxW || W < 2) return 3;
+                                         const void* w, const void* bias, const int* slots, const int* has_init,
+                                         int64_t B, int C, int W, int act, int dtype, cudaStream_t st) {
+  if (W < 1) return 3;
   if (B == 0) return 0;
   dim3 g((C + 255) / 256, (unsigned)B);
-  B200_DISPATCH_DTYPE(dtype, (b200::conv1d_update_kernel<T><<<g, 256, 0, st>>>((T*)out, out_stride, (const T*)x, x_stride,
-                                                                              (T*)states, (const T*)w, (const T*)bias, slots,
-                                                                              C, W, act)));
+  B200_DISPATCH_DTYPE(dtype, (b200::launch_pdl(b200::conv1d_update_kernel<T>, g, dim3(256), 0, st, (T*)out, out_stride,
+                                               (const T*)x, x_stride, (T*)states, (const T*)w, (const T*)bias, slots, has_init,
+                                               C, W, act)));
   return cudaGetLastError() != cudaSuccess;
 }
 

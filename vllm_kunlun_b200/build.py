@@ -24,6 +24,10 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v",
               "-DNDEBUG"]
 
+# Kernels that also serve fp32 models: exp / log / division / square root at full fp32 accuracy.
+PRECISE = {"linear_attn/gdn.cu", "linear_attn/recurrence.cu", "elementwise/layernorm.cu", "gemm/gemm_f32.cu",
+           "attention/paged_generic.cu"}
+
 
 def _nvcc() -> str:
     for c in (os.environ.get("CUDA_HOME", ""), "/usr/local/cuda"):
@@ -91,7 +95,10 @@ def build(verbose: bool = False, force: bool = False) -> str:
     for s in cu:
         obj = os.path.join(BUILD, os.path.relpath(s, CSRC).replace(os.sep, "_") + ".o")
         objs.append(obj)
-        jobs.append((s, [nvcc, *NVCC_FLAGS, "-c", s, "-o", obj], obj))
+        flags = NVCC_FLAGS
+        if os.path.relpath(s, CSRC).replace(os.sep, "/") in PRECISE:
+            flags = [f for f in NVCC_FLAGS if f != "--use_fast_math"]
+        jobs.append((s, [nvcc, *flags, "-c", s, "-o", obj], obj))
     torch_inc = [f"-I{p}" for p in ce.include_paths()]
     py_inc = f"-I{sysconfig.get_paths()['include']}"
     abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)

@@ -65,12 +65,19 @@ class DecodeGraphs:
         # plan attention splits for the longest context this graph may ever see
         md.max_seq_len = self.runner.cfg.scheduler.max_model_len
         md.max_query_len = self.tokens_per_req
+        # the warm-up passes run on this step's inputs: rewriting K / V is harmless, but a recurrent state would be
+        # advanced once per pass, so the state kernels see no slots until the replay
+        slots = None if md.state_indices is None else md.state_indices.clone()
+        if slots is not None:
+            md.state_indices.fill_(-1)
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s):
             for _ in range(2):  # warm-up: lazy allocations, tensor-map cache, function attributes
                 self._forward(md, input_ids)
         torch.cuda.current_stream().wait_stream(s)
+        if slots is not None:
+            md.state_indices.copy_(slots)
         torch.cuda.synchronize()
         from ..ops import _ext
         g = torch.cuda.CUDAGraph()
@@ -109,7 +116,8 @@ class DecodeGraphs:
                 dist.barrier(group=g)
 
     @torch.inference_mode()
-    def run(self, md: AttentionMetadata, input_ids, sp):
+    def replay(self, md: AttentionMetadata, input_ids):
+        """Capture on first use, then replay: ``(logits, hidden)`` of every row of the padded batch."""
         key = md.num_reqs
         if key not in self.graphs:
             self._capture(md, input_ids)
@@ -118,8 +126,12 @@ class DecodeGraphs:
             self.watcher.check(str(key), self._watched(md, input_ids))
         self.graphs[key].replay()
         self.replayed_kernels += self.kernels_per_graph[key]
-        tokens = self.runner.sampler(self.logits[key], sp)
-        return tokens, self.hidden[key]
+        return self.logits[key], self.hidden[key]
+
+    @torch.inference_mode()
+    def run(self, md: AttentionMetadata, input_ids, sp):
+        logits, hidden = self.replay(md, input_ids)
+        return self.runner.sampler(logits, sp), hidden
 
     @staticmethod
     def _watched(md, input_ids) -> dict:

@@ -35,6 +35,15 @@ class RopeScaling:
 
 
 @dataclass
+class LayerSpec:
+    """One entry of an explicit layer list (designs whose layers differ in kind and size)."""
+
+    type: str                   # name of the mixer (``models/mixers.py``)
+    mixer: dict                 # its sizes and constants
+    mlp: Optional[dict] = None  # {"kind": "dense", "ff": width}, or None: the layer has no feed-forward
+
+
+@dataclass
 class ModelConfig:
     """Architecture description shared by every model family."""
 
@@ -119,6 +128,7 @@ class ModelConfig:
     global_head_dim: Optional[int] = None  # head size of the full-attention layers when it differs (Gemma-4)
     num_global_kv_heads: Optional[int] = None  # their KV head count when values are the keys (attention_k_eq_v)
     attention_k_eq_v: bool = False  # full-attention layers have no v_proj: V is the (un-normalised, un-rotated) K
+    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel); the flat fields above then hold the largest sizes
     attn_output_gate: bool = False  # q_proj carries a sigmoid output gate (Qwen3-Next full-attention layers)
     # quantization of the checkpoint
     quantization: Optional[str] = None  # None | "fp8" | "int8" | "awq" | "gptq" | "w4a16"
@@ -167,6 +177,16 @@ class ModelConfig:
             return False
         return (i + 1) % self.linear_attn_pattern != 0
 
+    @property
+    def has_recurrent_state(self) -> bool:
+        """Some layer keeps a per-request state besides (or instead of) the paged cache."""
+        if self.linear_attn_pattern > 0:
+            return True
+        if not self.layer_specs:
+            return False
+        from .models.mixers import MIXERS
+        return any(MIXERS[spec.type].has_state for spec in self.layer_specs)
+
     def num_params(self) -> int:
         """Rough parameter count (used for memory planning)."""
         h = self.hidden_size
@@ -191,6 +211,8 @@ class ModelConfig:
     @classmethod
     def from_hf_config(cls, cfg: dict) -> "ModelConfig":
         """Build from a Hugging Face ``config.json`` dict (same checkpoints the reference serves)."""
+        if isinstance(cfg.get("layers"), list) and cfg.get("architecture"):
+            return cls._from_layer_list(cfg)
         arch = (cfg.get("architectures") or ["LlamaForCausalLM"])[0]
         if isinstance(cfg.get("thinker_config"), dict):     # Qwen3-Omni: the served part is the "thinker"
             cfg = {**cfg["thinker_config"], "architectures": [arch], "quantization_config": cfg.get("quantization_config")}
@@ -440,9 +462,42 @@ class ModelConfig:
         return out
 
     @classmethod
+    def _from_layer_list(cls, cfg: dict) -> "ModelConfig":
+        """Configurations that list their layers one by one (``architecture``, ``width``, ``vocab``, ``norm.eps``,
+        ``layers: [{type, mixer, mlp}]``)."""
+        from .models.mixers import MIXERS
+        specs = []
+        for i, entry in enumerate(cfg["layers"]):
+            if entry["type"] not in MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}; known: {sorted(MIXERS)}")
+            mlp = entry.get("mlp")
+            if mlp is not None and mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            specs.append(LayerSpec(entry["type"], dict(entry["mixer"]), None if mlp is None else dict(mlp)))
+        arch = cfg["architecture"]
+        return cls(architecture=arch, name=cfg.get("_name_or_path", arch), vocab_size=int(cfg["vocab"]),
+                   hidden_size=int(cfg["width"]), num_layers=len(specs), num_heads=1, num_kv_heads=1, head_dim=1,
+                   intermediate_size=max([1] + [int(s.mlp["ff"]) for s in specs if s.mlp]),
+                   rms_norm_eps=float(cfg["norm"]["eps"]), max_position=1 << 30, layer_specs=tuple(specs),
+                   dtype=str(cfg.get("torch_dtype", "bfloat16")))
+
+    def complete_from_shapes(self, shapes: dict) -> "ModelConfig":
+        """Sizes that only the checkpoint's tensors tell (``shapes``: name -> shape): the low-rank widths of mixers."""
+        from .models.mixers import MIXERS
+        for i, spec in enumerate(self.layer_specs):
+            prefix = f"l{i}.mix."
+            MIXERS[spec.type].complete_sizes(spec.mixer, {n.removeprefix(prefix): s for n, s in shapes.items()
+                                                          if n.startswith(prefix)})
+        return self
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
-            return cls.from_hf_config(json.load(f))
+            out = cls.from_hf_config(json.load(f))
+        if out.layer_specs:
+            from .models.loader import tensor_shapes
+            out.complete_from_shapes(tensor_shapes(path))
+        return out
 
 
 def _leading_dense(cfg: dict) -> int:
@@ -538,11 +593,11 @@ class EngineConfig:
             self.cache.cache_dtype = "bfloat16"
         if self.device == "cpu":
             self.compilation.mode = "none"
-        if m.linear_attn_pattern:
+        if m.has_recurrent_state:
             # the recurrent state of a cached prefix is not kept, and a rejected draft cannot be rolled back
             self.cache.enable_prefix_caching = False
             if self.speculative.num_speculative_tokens:
-                raise ValueError("speculative decoding is not supported with linear-attention layers")
+                raise ValueError("speculative decoding is not supported with recurrent layers")
         if self.speculative.method == "eagle3":
             self.compilation.mode = "none"  # the auxiliary hidden states are not carried through captured graphs
         if self.speculative.method == "mtp" and not m.num_mtp_layers:

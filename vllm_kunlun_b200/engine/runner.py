@@ -42,6 +42,7 @@ class StepHandle:
     logprobs_cpu: Optional[torch.Tensor] = None  # log p of every sampled row (when a request asked for it)
     status_cpu: Optional[torch.Tensor] = None    # device status words copied with the tokens (0 = all waits were met)
     status_names: tuple = ()
+    logits: Optional[torch.Tensor] = None        # fp32, on the host: wanted rows of a ``return_logits`` step
 
     def wait(self) -> torch.Tensor:
         if self.event is not None:
@@ -89,11 +90,14 @@ class ModelRunner:
         self.kv_caches = self._alloc_kv()
         self.num_state_slots = 0
         if getattr(self.model, "uses_state_cache", False):
-            # one slot per running request for the linear-attention (conv + recurrent) state
+            # one slot per running request for the linear-attention (conv + recurrent) state; a layer that also has
+            # paged tensors holds them in front: (paged ..., state ...)
             self.num_state_slots = self.max_bs
             for i, specs in self.model.state_cache_spec().items():
-                self.kv_caches[i] = tuple(torch.zeros((self.num_state_slots, *shp), dtype=dt, device=self.device)
-                                          for shp, dt in specs)
+                paged = self.kv_caches.get(i, ())
+                paged = paged if isinstance(paged, tuple) else (paged,)
+                self.kv_caches[i] = paged + tuple(torch.zeros((self.num_state_slots, *shp), dtype=dt, device=self.device)
+                                                  for shp, dt in specs)
         self._alloc_staging()
         self.graphs = None
         self.is_vl = hasattr(self.model, "embed_multimodal")
@@ -173,8 +177,10 @@ class ModelRunner:
             return None
         from ..ops.attention_cuda import AttnWorkspace
         m = self.cfg.model
-        heads = m.num_heads // self.pstate.tp_size
-        return AttnWorkspace(self.max_bs * (1 + self.num_spec), heads, m.head_dim, 16, self.device)
+        heads, dim = m.num_heads // self.pstate.tp_size, m.head_dim
+        if hasattr(self.model, "attn_workspace_size"):   # layers of different sizes: the largest of each
+            heads, dim = self.model.attn_workspace_size()
+        return AttnWorkspace(self.max_bs * (1 + self.num_spec), heads, dim, 16, self.device)
 
     def _alloc_staging(self):
         T, B, MB = self.max_tokens, self.max_bs, self.max_blocks_per_seq
@@ -338,7 +344,13 @@ class ModelRunner:
             if sr.is_decode:
                 num_decodes += 1
                 num_decode_tokens += n
-            if sr.samples:
+            if sched.return_logits:
+                # a captured step computes the logits of every request; the caller picks the wanted ones
+                rows = [0] if pad_reqs else sr.logit_rows
+                logits_idx[n_logits:n_logits + len(rows)] = t + np.asarray(rows, dtype=np.int64)
+                lora_row[n_logits:n_logits + len(rows)] = lslot
+                n_logits += len(rows)
+            elif sr.samples:
                 rows = n if (sr.is_decode and n_spec) else 1
                 logits_idx[n_logits:n_logits + rows] = np.arange(t + n - rows, t + n)
                 lora_row[n_logits:n_logits + rows] = lslot
@@ -428,6 +440,8 @@ class ModelRunner:
                      and self.graphs.supports(len(srs), sched.num_tokens))
         pad = self.graphs.padded_batch(len(srs)) if use_graph else 0
         md, input_ids, (sample_reqs, rows_per_req, n_logits) = self.prepare(sched, pad)
+        if sched.return_logits:
+            return self._execute_logits(sched, md, input_ids, use_graph, t0)
         sp = self.sampler.make_params([r.sampling for r in sample_reqs], rows_per_req, n_logits, reqs=sample_reqs)
         from ..models.layers import set_sp_mode
         if use_graph:
@@ -482,6 +496,29 @@ class ModelRunner:
         return StepHandle(sched, sample_reqs, rows_per_req, tokens, tokens_cpu, ev, hidden, t0, md, input_ids, full,
                           lp_cpu, status_cpu, names)
 
+    def _execute_logits(self, sched: SchedulerOutput, md, input_ids, use_graph: bool, t0: float) -> StepHandle:
+        """Tail of :meth:`execute` for a step that returns logits: the same model step (captured or eager), no sampling.
+        ``StepHandle.logits`` holds the wanted rows in the order of ``sched.scheduled``."""
+        if use_graph:
+            logits, _ = self.graphs.replay(md, input_ids)
+            keep = [i for i, sr in enumerate(sched.scheduled) if sr.logit_rows]
+            logits = logits[torch.tensor(keep, dtype=torch.int64, device=self.device)]
+        else:
+            logits, _ = self.forward_logits(md, input_ids)
+        for sr in sched.scheduled:
+            sr.req.num_computed_tokens += sr.num_new_tokens
+        self.last_rows, self.last_tokens = {}, None
+        logits_cpu = logits.float().cpu()
+        names, status_cpu, ev = (), None, None
+        if self.is_cuda:
+            words = self._status_words()
+            if words:
+                names = tuple(n for n, _ in words)
+                status_cpu = torch.cat([w.view(-1)[:1] for _, w in words]).cpu()
+        none = torch.empty(0, dtype=torch.int64)
+        return StepHandle(sched, [], [], none, none, ev, launch_time=t0, md=md, input_ids=input_ids, logits=logits_cpu,
+                          status_cpu=status_cpu, status_names=names)
+
     def _status_words(self) -> list:
         """``(name, int32 device tensor)`` of every status word a kernel of this process may have set."""
         st = self.pstate
@@ -523,6 +560,16 @@ class ModelRunner:
             if st.pp_size > 1:
                 st.pp_comm.broadcast(tokens, src=st.pp_size - 1)
         return tokens, sel
+
+    def forward_logits(self, md: AttentionMetadata, input_ids):
+        """The model step up to the logits of ``md.logits_indices`` (no sampling, one pipeline stage)."""
+        assert self.pstate.pp_size == 1, "logits are returned by single-stage models"
+        ctx = ForwardContext(attn=md, kv_caches=self.kv_caches, pstate=self.pstate,
+                             lora=None if self.lora is None else self.lora.punica, extras=self._step_extras)
+        with set_forward_context(ctx):
+            hidden = self.run_model(input_ids, md)
+            sel = hidden.index_select(0, md.logits_indices.long())
+            return self.model.compute_logits(sel), sel
 
     def run_model(self, input_ids, md):
         """One pipeline stage: receive from the previous stage, run, send on (NCCL p2p)."""

@@ -105,6 +105,7 @@ class ScheduledRequest:
     num_new_tokens: int  # tokens fed this step (prefill chunk, or 1 + drafts)
     is_decode: bool
     samples: bool  # logits wanted for this request this step
+    logit_rows: Optional[tuple] = None  # replayed portions: the places within the portion whose logits are wanted
 
 
 @dataclass
@@ -112,6 +113,7 @@ class SchedulerOutput:
     scheduled: list = field(default_factory=list)
     num_tokens: int = 0
     preempted: list = field(default_factory=list)
+    return_logits: bool = False  # the step returns logits of the ``logit_rows`` instead of sampled tokens
 
     @property
     def empty(self) -> bool:
@@ -230,6 +232,28 @@ class Scheduler:
         out.scheduled = decodes + prefills
         out.num_tokens = sum(s.num_new_tokens for s in out.scheduled)
         return out
+
+    def schedule_portions(self, portions) -> SchedulerOutput:
+        """A step with a prescribed composition: ``portions`` is a list of ``(request, tokens, logit_rows)`` that run
+        together whatever the policy would have chosen.  Requests seen for the first time are admitted (they take
+        blocks and a state slot as usual); nothing is preempted - a pool without room is an error."""
+        decodes, prefills = [], []
+        for req, n, rows in portions:
+            if req not in self.running:
+                if len(self.running) >= self.max_num_seqs or (self.uses_state and not self.free_state_slots):
+                    raise RuntimeError(f"request {req.request_id}: all {self.max_num_seqs} request slots are taken")
+                if self.uses_state:
+                    req.state_slot = self.free_state_slots.pop()
+                req.status = RequestStatus.RUNNING
+                self.running.append(req)
+            if not self._ensure_blocks(req, req.num_computed_tokens + n):
+                raise RuntimeError(f"request {req.request_id}: no free cache blocks for {n} more tokens")
+            # one token on top of computed ones is a decode step; anything else runs as a prompt portion
+            is_decode = n == 1 and req.num_computed_tokens > 0
+            (decodes if is_decode else prefills).append(
+                ScheduledRequest(req, n, is_decode, len(rows) > 0, logit_rows=tuple(rows)))
+        scheduled = decodes + prefills
+        return SchedulerOutput(scheduled=scheduled, num_tokens=sum(s.num_new_tokens for s in scheduled), return_logits=True)
 
     def finish(self, req: Request) -> None:
         if req in self.running:

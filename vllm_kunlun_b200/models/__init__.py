@@ -37,6 +37,8 @@ _REGISTRY = {
     "Qwen3_5MoeForConditionalGeneration": "vision:Qwen3_5ForConditionalGeneration",
     "Qwen3_5ForCausalLM": "qwen3_next:Qwen3NextForCausalLM",          # the text-only classes of the same checkpoints
     "Qwen3_5MoeForCausalLM": "qwen3_next:Qwen3NextForCausalLM",
+    # layers listed one by one: windowed attention beside linear attention, channel-wise delta rule
+    "Bolopel": "bolopel:BolopelForCausalLM",
     # asymmetric V / sliding window with sinks
     "MiMoV2FlashForCausalLM": "mimo_v2_flash:MiMoV2FlashForCausalLM",
     # Gemma family

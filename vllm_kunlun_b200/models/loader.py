@@ -14,8 +14,7 @@ from typing import Iterator
 import torch
 
 
-def load_safetensors(path: str, device: str = "cpu") -> Iterator[tuple[str, torch.Tensor]]:
-    from safetensors import safe_open
+def _files(path: str) -> list:
     index = os.path.join(path, "model.safetensors.index.json")
     if os.path.exists(index):
         with open(index) as f:
@@ -24,7 +23,23 @@ def load_safetensors(path: str, device: str = "cpu") -> Iterator[tuple[str, torc
         files = sorted(os.path.basename(p) for p in glob.glob(os.path.join(path, "*.safetensors")))
     if not files:
         raise FileNotFoundError(f"no safetensors files under {path}")
-    for fn in files:
+    return files
+
+
+def tensor_shapes(path: str) -> dict:
+    """Name -> shape of every tensor of a checkpoint directory (headers only)."""
+    from safetensors import safe_open
+    out = {}
+    for fn in _files(path):
+        with safe_open(os.path.join(path, fn), framework="pt") as f:
+            for name in f.keys():
+                out[name] = tuple(f.get_slice(name).get_shape())
+    return out
+
+
+def load_safetensors(path: str, device: str = "cpu") -> Iterator[tuple[str, torch.Tensor]]:
+    from safetensors import safe_open
+    for fn in _files(path):
         with safe_open(os.path.join(path, fn), framework="pt", device=device) as f:
             for name in f.keys():
                 yield name, f.get_tensor(name)

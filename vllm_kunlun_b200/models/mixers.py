@@ -1,0 +1,323 @@
+"""Sequence mixers of designs that list their layers one by one, with every size and constant a parameter.
+
+A mixer reads the residual stream's 16-bit (or fp32) copy ``h [T, ld]`` and returns the summands of its output as
+``[(y, scale), ...]`` for :func:`ops.layernorm_residual`.  It declares what it keeps between steps - paged tensors
+(``kv_cache_spec``) and per-request state (``state_spec``) - and finds both in the forward context:
+``kv_caches[layer] = (paged ..., state ...)``.
+
+* :class:`WindowAttention`   softmax attention, unit-RMS q / k heads, optional sliding window, optional constant sink
+* :class:`LightningAttention` linear attention with a fixed decay per head, jointly normed and gated output
+* :class:`ParallelMixer`     both of them on the same input, one input projection, scaled sum
+* :class:`ChannelDelta`      short convolutions + delta rule with one decay per head and key channel
+
+Checkpoint rows are padded so that every column slice of a fused projection starts on a 16-byte boundary; padding rows
+and columns are zero.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+import torch.nn as nn
+
+from .. import ops
+from ..attention.metadata import get_forward_context
+from ..config import round_up
+from .layers import ReplicatedLinear, param
+
+ALIGN = 8                       # elements: 16 bytes of a 16-bit row
+_TENSOR_CORE_HEADS = (64, 128, 256)
+UNIT_NORM_EPS = 1e-6            # inside the root of the delta rule's unit vectors
+
+
+def align(n: int) -> int:
+    return round_up(n, ALIGN)
+
+
+def cache_head_dim(dim: int, vdim: int, dtype: torch.dtype) -> int:
+    """Head size of the paged cache: keys and values share it, zero-padded to one the attention kernels serve."""
+    n = max(dim, vdim)
+    if dtype == torch.float32:
+        return round_up(n, 4)
+    return next((d for d in _TENSOR_CORE_HEADS if d >= n), align(n))
+
+
+def padded(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+    if tuple(w.shape) == (rows, cols):
+        return w
+    out = w.new_zeros(rows, cols)
+    out[:w.shape[0], :w.shape[1]] = w
+    return out
+
+
+class FusedProjection(ReplicatedLinear):
+    """Several projections of the same input in one GEMM; part ``i`` is a column slice starting at a multiple of 8."""
+
+    def __init__(self, in_features: int, sizes: dict, dtype, device):
+        self.parts, off = {}, 0
+        for name, n in sizes.items():
+            self.parts[name] = (off, n)
+            off += align(n)
+        super().__init__(in_features, off, dtype=dtype, device=device)
+        self.weight.data.zero_()
+
+    def load_part(self, name: str, w: torch.Tensor):
+        off, n = self.parts[name]
+        if w.shape[0] != n or w.shape[1] > self.in_features:
+            raise ValueError(f"projection {name}: checkpoint shape {tuple(w.shape)}, expected [{n}, <= {self.in_features}]")
+        self.weight.data[off:off + n, :w.shape[1]].copy_(w)
+
+    def slice(self, y: torch.Tensor, name: str) -> torch.Tensor:
+        off, n = self.parts[name]
+        return y[:, off:off + n]
+
+
+def output_projection(in_features: int, width: int, dtype, device) -> ReplicatedLinear:
+    lin = ReplicatedLinear(in_features, width, dtype=dtype, device=device)
+    lin.weight.data.zero_()
+    return lin
+
+
+def _rows(T: int, n: int, dtype, device) -> torch.Tensor:
+    """Buffer ``[T, align(n)]`` whose padding columns are zero (they meet zero weight columns)."""
+    return torch.empty(T, n, dtype=dtype, device=device) if align(n) == n else \
+        torch.zeros(T, align(n), dtype=dtype, device=device)
+
+
+class WindowAttention(nn.Module):
+    """Causal softmax attention over the paged cache; no rotation.  Every q / k head is divided by its root mean
+    square.  ``window``: position i sees the last ``window`` positions up to itself (None = all of them).  ``sink``: a
+    constant score without a value that joins the softmax denominator (None = no sink)."""
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: Optional[int],
+                 sink: Optional[float], eps: float, dtype, device):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"{heads} query heads do not divide over {kv_heads} key / value heads")
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.window, self.eps = float(scale), window, eps
+        self.cache_dim = cache_head_dim(dim, vdim, dtype)
+        self.sinks = None if sink is None else param(heads, dtype=torch.float32, device=device)
+        if sink is not None:
+            self.sinks.data.fill_(sink)
+        self.o = output_projection(heads * self.cache_dim, width, dtype, device)
+
+    def proj_sizes(self) -> dict:
+        return {"q": self.heads * self.dim, "k": self.kv_heads * self.dim, "v": self.kv_heads * self.vdim}
+
+    def kv_cache_spec(self, block_size: int, dtype):
+        return ((2, self.kv_heads, block_size, self.cache_dim), dtype)
+
+    def load_o(self, w: torch.Tensor):
+        """Columns are spread to the cache's head size (the padded value dims are zero)."""
+        g = self.o.weight.data.view(self.o.out_features, self.heads, self.cache_dim)
+        g[:w.shape[0], :, :self.vdim].copy_(w.reshape(w.shape[0], self.heads, self.vdim))
+
+    def forward(self, q, k, v, kv_cache, md):
+        T = q.shape[0]
+        qn = ops.qk_unit_norm_cache(q, k, v, kv_cache, md.slot_mapping, self.heads, self.kv_heads, self.eps)
+        span = md.max_seq_len if self.window is None else min(md.max_seq_len, self.window + 127)
+        o = ops.paged_attention(
+            qn, kv_cache, md.block_tables, md.seq_lens, md.query_start_loc, self.scale, md.max_query_len, span,
+            self.window, self.sinks, md.seq_lens_cpu, md.query_start_loc_cpu, workspace=md.workspace,
+            num_decodes=md.num_decodes, decode_query_len=1 + md.num_spec_tokens,
+            num_decode_tokens=md.num_decode_tokens, stable_metadata=True)
+        return self.o(o.reshape(T, self.heads * self.cache_dim))
+
+
+class LightningAttention(nn.Module):
+    """``S <- decay_h S + k v^T``, ``o = S^T q`` with SiLU on q, k and v; the concatenated heads are RMS-normed together,
+    multiplied by ``sigmoid`` of the gate projection and projected."""
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, decay, eps: float, dtype, device):
+        super().__init__()
+        if len(decay) != heads:
+            raise ValueError(f"{len(decay)} decay constants for {heads} heads")
+        self.heads, self.dim, self.vdim, self.eps = heads, dim, vdim, eps
+        self.register_buffer("decay", torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device))
+        self.norm = nn.Module()
+        self.norm.weight = param(heads * vdim, dtype=torch.float32, device=device)
+        self.o = output_projection(align(heads * vdim), width, dtype, device)
+
+    def proj_sizes(self) -> dict:
+        n = self.heads * self.vdim
+        return {"q": self.heads * self.dim, "k": self.heads * self.dim, "v": n, "g": n}
+
+    def state_spec(self):
+        return [((self.heads, self.vdim, round_up(self.dim, 4)), torch.float32)]
+
+    def load_o(self, w: torch.Tensor):
+        self.o.weight.data[:w.shape[0], :w.shape[1]].copy_(w)
+
+    def forward(self, q, k, v, g, state, md):
+        T, H = q.shape[0], self.heads
+        o = ops.fixed_decay_attention(_heads(q, H, self.dim), _heads(k, H, self.dim), _heads(v, H, self.vdim), self.decay,
+                                      state, md.query_start_loc, md.state_indices, md.has_initial_state)
+        n = H * self.vdim
+        y = ops.gated_group_rmsnorm(o.reshape(T, n), g, self.norm.weight, self.eps, _rows(T, n, q.dtype, q.device))
+        return self.o(y)
+
+
+def _heads(x: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
+    """``[T, heads * dim]`` column slice -> ``[T, heads, dim]`` view."""
+    return x.as_strided((x.shape[0], heads, dim), (x.stride(0), dim, 1))
+
+
+class ParallelMixer(nn.Module):
+    """Windowed softmax attention and lightning attention on the same input, added with constant scales."""
+
+    has_state = True
+    sink_score = 0.0            # one unit in the softmax denominator
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        pass
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        super().__init__()
+        a, b = sizes["left"], sizes["right"]
+        self.layer_idx = layer_idx
+        mask = a.get("mask") or {}
+        window = mask.get("size")
+        self.left = WindowAttention(width, a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["scale"],
+                                    None if window is None else int(window), self.sink_score, eps, dtype, device)
+        self.right = LightningAttention(width, b["heads"], b["dim"], b["vdim"], b["decay"], eps, dtype, device)
+        self.scales = (float(sizes["left_scale"]), float(sizes["right_scale"]))
+        self.in_proj = FusedProjection(width, {**{f"left.{k}": n for k, n in self.left.proj_sizes().items()},
+                                               **{f"right.{k}": n for k, n in self.right.proj_sizes().items()}}, dtype, device)
+
+    @staticmethod
+    def tensor_shapes(sizes: dict, width: int) -> dict:
+        a, b = sizes["left"], sizes["right"]
+        n = b["heads"] * b["vdim"]
+        return {"left.q": (a["heads"] * a["dim"], width), "left.k": (a["kv_heads"] * a["dim"], width),
+                "left.v": (a["kv_heads"] * a["vdim"], width), "left.o": (width, a["heads"] * a["vdim"]),
+                "right.q": (b["heads"] * b["dim"], width), "right.k": (b["heads"] * b["dim"], width), "right.v": (n, width),
+                "right.g": (n, width), "right.o": (width, n), "right.norm": (n,)}
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        if key == "left.o":
+            self.left.load_o(w)
+        elif key == "right.o":
+            self.right.load_o(w)
+        elif key == "right.norm":
+            self.right.norm.weight.data.copy_(w)
+        else:
+            self.in_proj.load_part(key, w)
+
+    def kv_cache_spec(self, block_size: int, dtype):
+        return self.left.kv_cache_spec(block_size, dtype)
+
+    def state_spec(self, dtype):
+        return self.right.state_spec()
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md = ctx.attn
+        kv_cache, state = ctx.kv_caches[self.layer_idx]
+        p = self.in_proj
+        y = p(h)
+        yl = self.left(p.slice(y, "left.q"), p.slice(y, "left.k"), p.slice(y, "left.v"), kv_cache, md)
+        yr = self.right(p.slice(y, "right.q"), p.slice(y, "right.k"), p.slice(y, "right.v"), p.slice(y, "right.g"), state, md)
+        return [(yl, self.scales[0]), (yr, self.scales[1])]
+
+
+class ChannelDelta(nn.Module):
+    """Gated delta rule with one decay per head and key channel.  ``q | k | v`` pass one short causal convolution and
+    SiLU; q and k become unit vectors inside the recurrence kernel; decay and output gate come from low-rank pairs
+    whose second factors run as one block-diagonal GEMM."""
+
+    has_state = True
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        for key, name in (("decay_rank", "a1"), ("gate_rank", "g1")):
+            if name in shapes:
+                sizes[key] = int(shapes[name][0])
+
+    @staticmethod
+    def _ranks(sizes: dict) -> tuple:
+        return int(sizes.get("decay_rank", sizes["dim"])), int(sizes.get("gate_rank", sizes["vdim"]))
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        super().__init__()
+        self.layer_idx, self.eps = layer_idx, eps
+        self.heads, self.kv_heads, self.dim, self.vdim = sizes["heads"], sizes["kv_heads"], sizes["dim"], sizes["vdim"]
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} value heads do not divide over {self.kv_heads} key heads")
+        self.taps = int(sizes["conv"])
+        ra, rg = self._ranks(sizes)
+        H, nk, nv = self.heads, self.kv_heads * self.dim, self.heads * self.vdim
+        self.in_proj = FusedProjection(width, {"q": nk, "k": nk, "v": nv, "a1": ra, "g1": rg, "b": H}, dtype, device)
+        self.conv_dim = self.in_proj.parts["v"][0] + align(nv)          # q | k | v with their padding
+        self.conv_weight = param(self.conv_dim, self.taps, dtype=dtype, device=device)
+        self.conv_weight.data.zero_()
+        self.low = (self.in_proj.parts["a1"][0], align(ra) + align(rg))  # columns of a1 | g1
+        self.rank_a, self.n_decay = align(ra), align(H * self.dim)
+        self.up = ReplicatedLinear(self.low[1], self.n_decay + align(nv), dtype=dtype, device=device)
+        self.up.weight.data.zero_()
+        self.A_log = param(H, dtype=torch.float32, device=device)
+        self.dt_bias = param(H * self.dim, dtype=torch.float32, device=device)
+        self.norm = nn.Module()
+        self.norm.weight = param(self.vdim, dtype=torch.float32, device=device)
+        self.o = output_projection(align(nv), width, dtype, device)
+
+    @classmethod
+    def tensor_shapes(cls, sizes: dict, width: int) -> dict:
+        H, nk, nv = sizes["heads"], sizes["kv_heads"] * sizes["dim"], sizes["heads"] * sizes["vdim"]
+        ra, rg = cls._ranks(sizes)
+        W = sizes["conv"]
+        return {"q": (nk, width), "q.conv": (nk, W), "k": (nk, width), "k.conv": (nk, W), "v": (nv, width),
+                "v.conv": (nv, W), "b": (H, width), "A_log": (H,), "norm": (sizes["vdim"],), "a1": (ra, width),
+                "a2": (H * sizes["dim"], ra), "dt_bias": (H * sizes["dim"],), "g1": (rg, width), "g2": (nv, rg),
+                "o": (width, nv)}
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        if key.endswith(".conv"):
+            off, n = self.in_proj.parts[key.removesuffix(".conv")]
+            self.conv_weight.data[off:off + n].copy_(w)
+        elif key == "a2":
+            self.up.weight.data[:w.shape[0], :w.shape[1]].copy_(w)
+        elif key == "g2":
+            self.up.weight.data[self.n_decay:self.n_decay + w.shape[0], self.rank_a:self.rank_a + w.shape[1]].copy_(w)
+        elif key in ("A_log", "dt_bias"):
+            getattr(self, key).data.copy_(w)
+        elif key == "norm":
+            self.norm.weight.data.copy_(w)
+        elif key == "o":
+            self.o.weight.data[:w.shape[0], :w.shape[1]].copy_(w)
+        else:
+            self.in_proj.load_part(key, w)
+
+    def kv_cache_spec(self, block_size: int, dtype):
+        return None
+
+    def state_spec(self, dtype):
+        return [((self.taps - 1, self.conv_dim), dtype),
+                ((self.heads, self.vdim, round_up(self.dim, 4)), torch.float32)]
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md = ctx.attn
+        conv_state, state = ctx.kv_caches[self.layer_idx]
+        T, H, p = h.shape[0], self.heads, self.in_proj
+        y = p(h)
+        if md.max_query_len == 1:
+            x = ops.causal_conv1d_update(y[:, :self.conv_dim], conv_state, self.conv_weight, None, md.state_indices, True,
+                                         md.has_initial_state)
+        else:
+            x = ops.causal_conv1d_fn(y[:, :self.conv_dim], self.conv_weight, None, md.query_start_loc, conv_state,
+                                     md.state_indices, md.has_initial_state, True)
+        up = self.up(y[:, self.low[0]:self.low[0] + self.low[1]])
+        q, k, v = (_heads(p.slice(x, n), m, d) for n, m, d in
+                   (("q", self.kv_heads, self.dim), ("k", self.kv_heads, self.dim), ("v", H, self.vdim)))
+        o = ops.channel_delta_rule(q, k, v, up[:, :H * self.dim], p.slice(y, "b"), self.A_log, self.dt_bias, state,
+                                   md.query_start_loc, md.state_indices, md.has_initial_state, self.dim ** -0.5,
+                                   UNIT_NORM_EPS)
+        n = H * self.vdim
+        z = ops.gated_group_rmsnorm(o.reshape(T, n), up[:, self.n_decay:self.n_decay + n], self.norm.weight, self.eps,
+                                    _rows(T, n, h.dtype, h.device))
+        return [(self.o(z), 1.0)]
+
+
+MIXERS = {"channel_delta": ChannelDelta, "parallel": ParallelMixer}

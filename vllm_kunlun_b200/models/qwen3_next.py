@@ -66,7 +66,8 @@ class GatedDeltaNet(nn.Module):
         mixed = qkvz[:, : self.conv_dim]
         z = qkvz[:, self.conv_dim:]
         if md.max_query_len == 1:
-            mixed = ops.causal_conv1d_update(mixed, conv_state, self.conv_weight, None, md.state_indices, True)
+            mixed = ops.causal_conv1d_update(mixed, conv_state, self.conv_weight, None, md.state_indices, True,
+                                             md.has_initial_state)
         else:
             mixed = ops.causal_conv1d_fn(mixed, self.conv_weight, None, md.query_start_loc, conv_state, md.state_indices,
                                          md.has_initial_state, True)

@@ -15,6 +15,7 @@ import torch
 from . import _ext
 from .reference import attention as _ra
 from .reference import basic as _rb
+from .reference import linear_recurrence as _rl
 from .reference import misc as _rx
 from .reference import moe as _rm
 
@@ -229,8 +230,16 @@ def merge_attn_states(o1, lse1, o2, lse2):
 # ----------------------------------------------------------------------------- GEMM
 
 def linear(x, weight, bias=None, out=None):
-    """``y = x @ W.T (+ b)``, ``W [N, K]`` as stored in checkpoints.  CUDA: the tcgen05 GEMM."""
+    """``y = x @ W.T (+ b)``, ``W [N, K]`` as stored in checkpoints.  CUDA: the tcgen05 GEMM; fp32 models run on the
+    CUDA-core GEMM with true 32-bit products."""
     if x.is_cuda:
+        if x.dtype == torch.float32:
+            x2 = x.reshape(-1, x.shape[-1])
+            if x2.stride(-1) != 1:
+                x2 = x2.contiguous()
+            y = torch.empty(x2.shape[0], weight.shape[0], dtype=x.dtype, device=x.device) if out is None else out
+            _c().gemm_f32(y, x2, weight, bias)
+            return y.reshape(*x.shape[:-1], -1)
         from .gemm_cuda import gemm_bf16
         return gemm_bf16(x, weight, bias, out)
     return _rb.linear(x, weight, bias)
@@ -551,12 +560,15 @@ def causal_conv1d_fn(x, weight, bias, cu_seqlens, conv_states, state_indices, ha
     return _rx.causal_conv1d_fn(x, weight, bias, cu_seqlens, conv_states, state_indices, has_initial_state, activation)
 
 
-def causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation=True):
+def causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation=True, has_initial_state=None):
+    """One token per sequence.  Rows whose ``has_initial_state`` is 0 (a prompt of one token, or a slot that another
+    request used before) start from zeros instead of the slot's contents."""
     if x.is_cuda:
         out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
-        _c().causal_conv1d_update(out, x, conv_states, weight, bias, state_indices.int(), activation)
+        _c().causal_conv1d_update(out, x, conv_states, weight, bias, state_indices.int(), activation,
+                                  None if has_initial_state is None else has_initial_state.int())
         return out
-    return _rx.causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation)
+    return _rx.causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation, has_initial_state)
 
 
 def fused_gdn_gating(A_log, a, b, dt_bias):
@@ -635,6 +647,80 @@ def mtp_concat_norm(embed, hidden, enorm_w, hnorm_w, eps, positions=None):
         return out
     e = embed if positions is None else torch.where((positions == 0).unsqueeze(-1), torch.zeros_like(embed), embed)
     return torch.cat([_rb.rmsnorm(e, enorm_w, eps), _rb.rmsnorm(hidden, hnorm_w, eps)], -1)
+
+
+# ----------------------------------------------------------------- fp32 residual stream / linear recurrences
+
+def embed_positions_layernorm(ids, positions, table, freq, weight, eps: float):
+    """Token rows plus sinusoidal position vectors through a LayerNorm: ``(stream fp32, copy in table.dtype)``, both
+    ``[T, ld]`` with ``ld = table.shape[1] >= weight.numel()`` (the padding columns stay zero).  ``freq`` (float64)
+    holds the turns per position of every column pair."""
+    T, ld = ids.shape[0], table.shape[1]
+    x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
+    h = x if table.dtype == torch.float32 else torch.empty(T, ld, dtype=table.dtype, device=table.device)
+    if table.is_cuda:
+        _c().embed_layernorm(x, h, ids, positions, table, freq, weight, eps)
+    else:
+        _rl.embed_positions_layernorm(x, h, ids, positions, table, freq, weight, eps)
+    return x, h
+
+
+def layernorm_residual(x, dtype, parts, weight, eps: float):
+    """Post-norm residual step ``x += LayerNorm(sum of scale * y)`` in place on the fp32 stream, ``parts`` being one or
+    two ``(y, scale)``; with no parts the stream itself is normalised and left as it is.  Returns the stream's (or the
+    normalised stream's) copy in ``dtype``."""
+    h = x if (dtype == torch.float32 and parts) else torch.empty(x.shape, dtype=dtype, device=x.device)
+    (y1, s1), (y2, s2) = (list(parts) + [(None, 0.0)] * 2)[:2]
+    if x.is_cuda:
+        _c().layernorm_residual(x, h, y1, s1, y2, s2, weight, eps)
+    else:
+        _rl.layernorm_residual(x, h, y1, s1, y2, s2, weight, eps)
+    return h
+
+
+def gated_group_rmsnorm(o, gate, weight, eps: float, out):
+    """``o / rms(o) * weight * sigmoid(gate)`` over groups of ``weight.numel()`` columns into ``out``; ``o`` fp32
+    ``[T, n]``, ``gate [T, n]`` (may be a column slice), ``out [T, >= n]``."""
+    if o.is_cuda:
+        _c().gated_group_rmsnorm(out, o, gate, weight, eps)
+    else:
+        _rl.gated_group_rmsnorm(out, o, gate, weight, eps)
+    return out
+
+
+def qk_unit_norm_cache(q, k, v, kv_cache, slot_mapping, num_heads: int, num_kv_heads: int, eps: float):
+    """Scale every q / k head to unit root mean square (no weight, no rotation), write K and V into the paged cache and
+    return ``q [T, Hq, Dc]``; heads are zero-padded to the cache's head size.  ``q, k, v`` are column slices of one
+    projection."""
+    if q.is_cuda:
+        out = torch.empty(q.shape[0], num_heads, kv_cache.shape[-1], dtype=q.dtype, device=q.device)
+        _c().qk_unit_norm_cache(out, q, k, v, kv_cache, slot_mapping, num_heads, num_kv_heads, eps)
+        return out
+    return _rl.qk_unit_norm_cache(q, k, v, kv_cache, slot_mapping, num_heads, num_kv_heads, eps)
+
+
+def channel_delta_rule(q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_indices, has_initial_state, scale: float,
+                       unit_eps: float = 1e-6):
+    """Varlen delta rule with one decay per key channel over a state cache ``[slots, H, Dv, >= Dk]`` (fp32, in place).
+    ``q, k [T, Hk, Dk]``, ``v [T, H, Dv]`` (convolved), ``a [T, H * Dk]`` / ``b [T, H]`` the raw decay and step-size
+    projections.  The decays, step sizes and unit norms are computed in fp32 inside.  Returns fp32 ``[T, H, Dv]``."""
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    if q.is_cuda:
+        _c().channel_delta_rule(out, q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_indices, has_initial_state,
+                                scale, unit_eps)
+        return out
+    return _rl.channel_delta_rule(out, q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_indices, has_initial_state,
+                                  scale, unit_eps)
+
+
+def fixed_decay_attention(q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state):
+    """Varlen linear attention with a fixed decay per head: ``S <- decay S + silu(k) silu(v)^T``, ``o = S^T silu(q)``
+    over a state cache ``[slots, H, Dv, >= D]`` (fp32, in place).  Returns fp32 ``[T, H, Dv]``."""
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    if q.is_cuda:
+        _c().fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state)
+        return out
+    return _rl.fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state)
 
 
 # ----------------------------------------------------------------------------- LoRA

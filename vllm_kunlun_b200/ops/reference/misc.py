@@ -117,11 +117,11 @@ def causal_conv1d_fn(x, weight, bias, cu_seqlens, conv_states, state_indices, ha
         if activation:
             y = torch.nn.functional.silu(y)
         out[s:e] = y.to(x.dtype)
-        conv_states[slot] = seq[-(W - 1):].to(conv_states.dtype)
+        conv_states[slot] = seq[seq.shape[0] - (W - 1):].to(conv_states.dtype)
     return out
 
 
-def causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation: bool = True):
+def causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation: bool = True, has_initial_state=None):
     """``kunlun_ops.causal_conv1d_update`` (``ops/mamba/causal_conv1d.py:118-225``): one token per
     sequence.  ``x [B, C]``."""
     out = torch.empty_like(x)
@@ -130,7 +130,10 @@ def causal_conv1d_update(x, conv_states, weight, bias, state_indices, activation
         if slot < 0:
             out[b] = 0
             continue
-        seq = torch.cat([conv_states[slot].float(), x[b:b + 1].float()], 0)  # [W, C]
+        old = conv_states[slot].float()
+        if has_initial_state is not None and not bool(has_initial_state[b]):
+            old = torch.zeros_like(old)
+        seq = torch.cat([old, x[b:b + 1].float()], 0)  # [W, C]
         y = (seq.T * weight.float()).sum(-1)
         if bias is not None:
             y = y + bias.float()
