@@ -239,7 +239,7 @@ def linear(x, weight, bias=None, out=None):
                 x2 = x2.contiguous()
             y = torch.empty(x2.shape[0], weight.shape[0], dtype=x.dtype, device=x.device) if out is None else out
             _c().gemm_f32(y, x2, weight, bias)
-            return y.reshape(*x.shape[:-1], -1)
+            return y.reshape(*x.shape[:-1], weight.shape[0])
         from .gemm_cuda import gemm_bf16
         return gemm_bf16(x, weight, bias, out)
     return _rb.linear(x, weight, bias)
