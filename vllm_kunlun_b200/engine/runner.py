@@ -515,6 +515,10 @@ class ModelRunner:
             if words:
                 names = tuple(n for n, _ in words)
                 status_cpu = torch.cat([w.view(-1)[:1] for _, w in words]).cpu()
+            # a step without wanted rows copies nothing back: the event keeps the host from refilling staging buffers
+            # whose copies are still queued
+            ev = torch.cuda.Event()
+            ev.record()
         none = torch.empty(0, dtype=torch.int64)
         return StepHandle(sched, [], [], none, none, ev, launch_time=t0, md=md, input_ids=input_ids, logits=logits_cpu,
                           status_cpu=status_cpu, status_names=names)
