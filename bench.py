@@ -77,6 +77,11 @@ def parse():
                          "the concurrent requests")
     ap.add_argument("--layers", type=int, default=0,
                     help="debugging only: run with this many layers (the JSON line then says so and is not a result)")
+    ap.add_argument("--layer-bench", nargs="?", const="all", default=None, metavar="SIZE",
+                    help="instead of the headline run: prefill and decode throughput of Bolopel layers beside the "
+                         "closest existing hybrid (Qwen3-Next with dense feed-forwards) at equal sizes; one JSON line "
+                         "per size and model (SIZE: small | large | all)")
+    ap.add_argument("--layer-bench-model", default="both", choices=["both", "bolopel", "qwen3-next"])
     a = ap.parse_args()
     c = CONFIGS[a.config]
     a.model = a.model or c["model"]
@@ -158,8 +163,107 @@ def reference_arm(args):
     return 0
 
 
+# Sizes of the layer benchmark: width, feed-forward, query / key-value heads of the softmax attention, heads of the
+# recurrent layers (head size 128 throughout), layers (every 4th one differs in kind).
+LAYER_SIZES = {
+    "small": dict(width=2048, ff=6144, heads=16, kv_heads=4, lin_heads=16, layers=8, window=1024),
+    "large": dict(width=4096, ff=12288, heads=32, kv_heads=8, lin_heads=32, layers=8, window=1024),
+}
+LAYER_VOCAB = 32000
+
+
+def layer_models(size):
+    """The two models of one size: Bolopel (3 of 4 layers 'parallel', 1 'channel_delta') and the existing hybrid (3 of
+    4 layers gated delta net, 1 gated full attention), both with dense feed-forwards of the same width."""
+    from vllm_kunlun_b200.config import LayerSpec, ModelConfig
+    z = LAYER_SIZES[size]
+    H = z["lin_heads"]
+    par = dict(left=dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5,
+                         mask=dict(size=z["window"])),
+               right=dict(heads=H, dim=128, vdim=128, decay=[1 - 2.0 ** -(3 + 5 * i / H) for i in range(H)]),
+               left_scale=1.0, right_scale=0.5)
+    delta = dict(heads=H, kv_heads=H, dim=128, vdim=128, conv=4)
+    specs = tuple(LayerSpec("channel_delta" if i % 4 == 3 else "parallel", dict(delta if i % 4 == 3 else par),
+                            dict(kind="dense", ff=z["ff"])) for i in range(z["layers"]))
+    own = ModelConfig(architecture="Bolopel", name=f"bolopel-{size}", vocab_size=LAYER_VOCAB, hidden_size=z["width"],
+                      num_layers=z["layers"], num_heads=1, num_kv_heads=1, head_dim=1, intermediate_size=z["ff"],
+                      rms_norm_eps=1e-5, max_position=1 << 30, layer_specs=specs)
+    like = ModelConfig(architecture="Qwen3NextForCausalLM", name=f"qwen3-next-dense-{size}", vocab_size=LAYER_VOCAB,
+                       hidden_size=z["width"], num_layers=z["layers"], num_heads=z["heads"], num_kv_heads=z["kv_heads"],
+                       head_dim=128, intermediate_size=z["ff"], rms_norm_eps=1e-6, qk_norm=True, gemma_norm=True,
+                       attn_output_gate=True, max_position=1 << 16, linear_attn_pattern=4, gdn_num_k_heads=H,
+                       gdn_num_v_heads=H, gdn_head_k_dim=128, gdn_head_v_dim=128, gdn_conv_kernel=4)
+    return {"bolopel": own, "qwen3-next": like}
+
+
+def layer_bench(args):
+    """Device-timed prefill and decode of the layer models: CUDA events around the engine's steps, after ``--warmup``
+    rounds; a prefill step is 4 prompts of 2048 tokens, a decode round is 32 steps of 16 / 64 requests at a context of
+    2048 tokens.  Weights and activations of a step exceed L2 (126 MB)."""
+    import torch
+
+    from vllm_kunlun_b200 import LLM, SamplingParams
+    g = torch.Generator().manual_seed(7)
+    sizes = list(LAYER_SIZES) if args.layer_bench == "all" else [args.layer_bench]
+    W, K, IN, DEC = max(3, args.warmup), max(1, args.steps), 2048, 32
+    for size in sizes:
+        for name, cfg in layer_models(size).items():
+            if args.layer_bench_model not in ("both", name):
+                continue
+            llm = LLM(cfg, device="cuda", block_size=64, max_model_len=IN + 2 * DEC + 64, max_num_seqs=64,
+                      max_num_batched_tokens=4 * IN, gpu_memory_utilization=0.5)
+            eng = llm.engine
+            out = {"layer_bench": size, "model": cfg.name, "config": LAYER_SIZES[size], "dtype": "bf16",
+                   "data": "synthetic (uniform random token ids, random weights)", "warmup": W, "steps": K}
+            clocks = ClockSampler(0)
+            clocks.start()
+            ev = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+
+            def requests(n, max_tokens):
+                sp = SamplingParams(max_tokens=max_tokens, ignore_eos=True)
+                for _ in range(n):
+                    eng.add_request(torch.randint(0, LAYER_VOCAB, (IN,), generator=g).tolist(), sp)
+
+            times = []
+            for i in range(W + K):
+                requests(4, 1)
+                torch.cuda.synchronize()
+                ev[0].record()
+                eng.run_until_done()
+                ev[1].record()
+                torch.cuda.synchronize()
+                if i >= W:
+                    times.append(ev[0].elapsed_time(ev[1]))
+            ms = statistics.median(times)
+            out["prefill"] = {"tokens": 4 * IN, "ms": round(ms, 3), "tok_per_s": round(4 * IN / ms * 1e3)}
+            for batch in (16, 64):
+                requests(batch, 2 * DEC + 8)
+                while eng.scheduler.waiting or any(r.in_prefill for r in eng.scheduler.running):
+                    eng.step()
+                for _ in range(DEC // 2):
+                    eng.step()
+                torch.cuda.synchronize()
+                ev[0].record()
+                for _ in range(DEC):
+                    eng.step()
+                ev[1].record()
+                torch.cuda.synchronize()
+                ms = ev[0].elapsed_time(ev[1]) / DEC
+                eng.run_until_done()
+                out[f"decode_{batch}"] = {"ms_per_step": round(ms, 4), "tok_per_s": round(batch / ms * 1e3)}
+            out["clocks"] = clocks.stop()
+            print(json.dumps(out), flush=True)
+            del eng, llm
+            torch.cuda.empty_cache()
+    from vllm_kunlun_b200.ops.gemm_cuda import check_status
+    check_status()
+    return 0
+
+
 def main():
     args = parse()
+    if args.layer_bench:
+        return layer_bench(args)
     if args.impl == "reference":
         return reference_arm(args)
     import torch

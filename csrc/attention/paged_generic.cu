@@ -17,8 +17,8 @@ constexpr int kGenWarps = 4;
 
 template <typename T, int ND>  // ND: value dims per lane, D <= 32 ND
 __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel(
-    T* __restrict__ out, const T* __restrict__ q, const T* __restrict__ cache, const int* __restrict__ block_tables,
-    const int* __restrict__ seq_lens, const int* __restrict__ qsl, const float* __restrict__ sinks, int B, int Hq, int Hkv,
+    T* out, const T* q, const T* cache, const int* block_tables,
+    const int* seq_lens, const int* qsl, const float* sinks, int B, int Hq, int Hkv,
     int D, int block_size, int max_blocks, int64_t num_blocks, int window, float scale) {
   extern __shared__ float sm_gen[];
   float* sq = sm_gen;                       // [D]

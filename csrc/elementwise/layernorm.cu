@@ -3,6 +3,9 @@
 //   layernorm_residual     stream += LayerNorm(s1 y1 [+ s2 y2]) (or the final norm of the stream) + 16-bit copy
 //   gated_group_rmsnorm    RMS norm over groups of a mixer's output, times weight and sigmoid(gate)
 //   qk_unit_norm_cache     split a fused projection, scale q / k to unit RMS per head, K / V into the paged cache
+// These kernels are launched with programmatic dependent launch, so they may be resident while the producer of their
+// inputs still runs: the pointers carry no __restrict__, which would let the compiler read them through the
+// non-coherent path.
 // All statistics in fp32 (this file is compiled without fast-math).  `ld` is the row length of stream and copy: the
 // width rounded up so that rows stay 16-byte aligned; the padding columns are kept at zero.
 #include "../api.h"
@@ -29,7 +32,7 @@ template <typename T> __device__ __forceinline__ void store4(T* p, const float (
 
 // Normalise NV x 4 values per thread (columns 4 (i kLnThreads + tid) ..), zero beyond H.
 template <int NV>
-__device__ __forceinline__ void layer_norm_regs(float (&y)[NV][4], int H, float eps, const float* __restrict__ w, float* red) {
+__device__ __forceinline__ void layer_norm_regs(float (&y)[NV][4], int H, float eps, const float* w, float* red) {
   float s = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i)
@@ -59,12 +62,12 @@ __device__ __forceinline__ void layer_norm_regs(float (&y)[NV][4], int H, float 
 // freq[i]: turns (angle / 2 pi) per position of column pair i.  The product and the reduction to one turn are in
 // double, so the angle keeps fp32 accuracy at any position.
 template <typename T, int NV>
-__global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(float* __restrict__ x, T* __restrict__ h,
-                                                                    const int64_t* __restrict__ ids,
-                                                                    const int64_t* __restrict__ positions,
-                                                                    const T* __restrict__ table,
-                                                                    const double* __restrict__ freq,
-                                                                    const float* __restrict__ w, int H, int ld,
+__global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(float* x, T* h,
+                                                                    const int64_t* ids,
+                                                                    const int64_t* positions,
+                                                                    const T* table,
+                                                                    const double* freq,
+                                                                    const float* w, int H, int ld,
                                                                     int64_t rows, float eps) {
   __shared__ float red[32];
   griddep_launch();
@@ -101,10 +104,10 @@ __global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(float* __re
 }
 
 template <typename T, int NV>
-__global__ void __launch_bounds__(kLnThreads) layernorm_residual_kernel(float* __restrict__ x, T* h,
-                                                                       const T* __restrict__ y1, int64_t y1_stride, float s1,
-                                                                       const T* __restrict__ y2, int64_t y2_stride, float s2,
-                                                                       const float* __restrict__ w, int H, int ld, float eps,
+__global__ void __launch_bounds__(kLnThreads) layernorm_residual_kernel(float* x, T* h,
+                                                                       const T* y1, int64_t y1_stride, float s1,
+                                                                       const T* y2, int64_t y2_stride, float s2,
+                                                                       const float* w, int H, int ld, float eps,
                                                                        int add) {
   __shared__ float red[32];
   griddep_launch();
@@ -152,10 +155,10 @@ __global__ void __launch_bounds__(kLnThreads) layernorm_residual_kernel(float* _
 
 // out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) over groups of D columns; RT threads per group.
 template <typename T, int RT, bool VEC>
-__global__ void __launch_bounds__(256) gated_group_rmsnorm_kernel(T* __restrict__ out, int64_t out_stride,
-                                                                  const float* __restrict__ o, int64_t o_stride,
-                                                                  const T* __restrict__ gate, int64_t gate_stride,
-                                                                  const float* __restrict__ w, int64_t rows, int groups,
+__global__ void __launch_bounds__(256) gated_group_rmsnorm_kernel(T* out, int64_t out_stride,
+                                                                  const float* o, int64_t o_stride,
+                                                                  const T* gate, int64_t gate_stride,
+                                                                  const float* w, int64_t rows, int groups,
                                                                   int D, float eps) {
   constexpr int V = VEC ? 4 : 1;
   __shared__ float red[32];
@@ -199,10 +202,10 @@ __global__ void __launch_bounds__(256) gated_group_rmsnorm_kernel(T* __restrict_
 // One warp per (token, head) of q, k and v.  Head sizes D (q, k) and Dv (v) are zero-padded to Dc in q_out and in the
 // cache [block][2][Hkv][slot][Dc].
 template <typename T>
-__global__ void __launch_bounds__(256) qk_unit_norm_cache_kernel(T* __restrict__ q_out, const T* __restrict__ q,
-                                                                 const T* __restrict__ k, const T* __restrict__ v,
-                                                                 int64_t stride, T* __restrict__ cache,
-                                                                 const int64_t* __restrict__ slots, int Hq, int Hkv, int D,
+__global__ void __launch_bounds__(256) qk_unit_norm_cache_kernel(T* q_out, const T* q,
+                                                                 const T* k, const T* v,
+                                                                 int64_t stride, T* cache,
+                                                                 const int64_t* slots, int Hq, int Hkv, int D,
                                                                  int Dv, int Dc, int block_size, int64_t num_blocks,
                                                                  float eps, int vec) {
   griddep_launch();

@@ -11,9 +11,9 @@ namespace {
 
 constexpr int kRows = 8;
 
-__global__ void __launch_bounds__(256) gemm_f32_rows_kernel(float* __restrict__ out, int64_t ldo, const float* __restrict__ x,
-                                                            int64_t ldx, const float* __restrict__ w, int64_t ldw,
-                                                            const float* __restrict__ bias, int64_t T_, int N, int K) {
+__global__ void __launch_bounds__(256) gemm_f32_rows_kernel(float* out, int64_t ldo, const float* x,
+                                                            int64_t ldx, const float* w, int64_t ldw,
+                                                            const float* bias, int64_t T_, int N, int K) {
   griddep_launch();
   griddep_wait();
   const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -36,9 +36,9 @@ __global__ void __launch_bounds__(256) gemm_f32_rows_kernel(float* __restrict__ 
   }
 }
 
-__global__ void __launch_bounds__(256) gemm_f32_tile_kernel(float* __restrict__ out, int64_t ldo, const float* __restrict__ x,
-                                                            int64_t ldx, const float* __restrict__ w, int64_t ldw,
-                                                            const float* __restrict__ bias, int64_t T_, int N, int K) {
+__global__ void __launch_bounds__(256) gemm_f32_tile_kernel(float* out, int64_t ldo, const float* x,
+                                                            int64_t ldx, const float* w, int64_t ldw,
+                                                            const float* bias, int64_t T_, int N, int K) {
   __shared__ __align__(16) float sx[16][68], sw[16][68];
   griddep_launch();
   griddep_wait();

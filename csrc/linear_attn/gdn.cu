@@ -147,9 +147,9 @@ __global__ void conv1d_state_kernel(T* __restrict__ states, const T* __restrict_
 
 // One token per sequence.  `has_init` (optional): a row whose flag is 0 starts from zeros, whatever its slot holds.
 template <typename T>
-__global__ void conv1d_update_kernel(T* __restrict__ out, int64_t out_stride, const T* __restrict__ x, int64_t x_stride,
-                                     T* __restrict__ states, const T* __restrict__ w, const T* __restrict__ bias,
-                                     const int* __restrict__ slots, const int* __restrict__ has_init, int C, int W, int act) {
+__global__ void conv1d_update_kernel(T* out, int64_t out_stride, const T* x, int64_t x_stride,
+                                     T* states, const T* w, const T* bias,
+                                     const int* slots, const int* has_init, int C, int W, int act) {
   griddep_launch();
   griddep_wait();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
