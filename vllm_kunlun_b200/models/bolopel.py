@@ -120,9 +120,9 @@ class BolopelForCausalLM(DenseForCausalLM):
         return self.cfg.has_recurrent_state
 
     def attn_workspace_size(self) -> tuple:
-        """(heads, head size) whose product covers every layer's split-KV partials."""
+        """(heads, head size) that cover every layer's split-KV partials (heads x size) and log-sum-exps (heads)."""
         left = [m.left for m in (self.layers[str(i)].mixer for i in range(self.last_layer)) if isinstance(m, ParallelMixer)]
-        return (1, max([1] + [a.heads * a.cache_dim for a in left]))
+        return max([1] + [a.heads for a in left]), max([1] + [a.cache_dim for a in left])
 
     # ---- weights
     def tensor_shapes(self) -> dict:
