@@ -325,6 +325,7 @@ typedef struct RecurrenceArgs {
   float scale, unit_eps;
 } RecurrenceArgs;
 int b200_linear_recurrence(const RecurrenceArgs* a, int dtype, cudaStream_t st);
+int b200_chunk_decay(const RecurrenceArgs* a, int dtype, cudaStream_t st);  // kind 1, prompt portions (linear_attn/chunk_decay.cu)
 int b200_sigmoid_gate_mul(void* out, const void* o, const void* gate, int64_t gate_stride, int D, int64_t T_,
                           int dtype, cudaStream_t st);
 int b200_mtp_concat_norm(void* out, const void* embed, const void* hidden, const void* we, const void* wh,

@@ -1459,13 +1459,14 @@ void channel_delta_rule(at::Tensor out, const at::Tensor& q, const at::Tensor& k
 }
 void fixed_decay_attention(at::Tensor out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v,
                            const at::Tensor& decay, at::Tensor states, const at::Tensor& cu, const at::Tensor& slots,
-                           const at::Tensor& has_init) {
+                           const at::Tensor& has_init, bool chunked) {
   RecurrenceArgs a;
   fill_recurrence(a, out, q, k, v, states, cu, slots, has_init);
   TORCH_CHECK(a.Hk == a.H && decay.scalar_type() == at::kFloat && decay.numel() == a.H);
   a.decay = decay.data_ptr<float>();
   a.kind = 1;
-  check(b200_linear_recurrence(&a, dtype_code(q), stream()), "fixed_decay_attention");
+  if (chunked) check(b200_chunk_decay(&a, dtype_code(q), stream()), "fixed_decay_attention (chunked)");
+  else check(b200_linear_recurrence(&a, dtype_code(q), stream()), "fixed_decay_attention");
 }
 void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& bias) {
   TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1);

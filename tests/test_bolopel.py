@@ -336,7 +336,7 @@ def test_fixed_decay_attention(device, dtype, H, D, Dv):
 
         for cuts in CUTS:
             got, other = _recur(device, dtype, lambda a, st, cu, sl, ini: ops.fixed_decay_attention(
-                *a, dec.to(device), st, cu, sl, ini), T, cuts, args, (H, Dv, -(-D // 4) * 4))
+                *a, dec.to(device), st, cu, sl, ini, max(1, int((cu[1:] - cu[:-1]).max())), 1), T, cuts, args, (H, Dv, -(-D // 4) * 4))
             close(got, want, dtype, f"portions {cuts[:4]}")
             close(other, want[:len(cuts)], dtype, "neighbour")
 

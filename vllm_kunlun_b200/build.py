@@ -25,7 +25,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-DNDEBUG"]
 
 # Kernels that also serve fp32 models: exp / log / division / square root at full fp32 accuracy.
-PRECISE = {"linear_attn/gdn.cu", "linear_attn/recurrence.cu", "elementwise/layernorm.cu", "gemm/gemm_f32.cu",
+PRECISE = {"linear_attn/gdn.cu", "linear_attn/recurrence.cu", "linear_attn/chunk_decay.cu", "elementwise/layernorm.cu", "gemm/gemm_f32.cu",
            "attention/paged_generic.cu"}
 
 

@@ -152,7 +152,8 @@ class LightningAttention(nn.Module):
     def forward(self, q, k, v, g, state, md):
         T, H = q.shape[0], self.heads
         o = ops.fixed_decay_attention(_heads(q, H, self.dim), _heads(k, H, self.dim), _heads(v, H, self.vdim), self.decay,
-                                      state, md.query_start_loc, md.state_indices, md.has_initial_state)
+                                      state, md.query_start_loc, md.state_indices, md.has_initial_state, md.max_query_len,
+                                      md.num_decodes)
         n = H * self.vdim
         y = ops.gated_group_rmsnorm(o.reshape(T, n), g, self.norm.weight, self.eps, _rows(T, n, q.dtype, q.device))
         return self.o(y)

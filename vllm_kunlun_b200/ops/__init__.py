@@ -713,14 +713,27 @@ def channel_delta_rule(q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_
                                   scale, unit_eps)
 
 
-def fixed_decay_attention(q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state):
+LINEAR_CHUNK_MIN = 16      # longest portion of a step from which its prompt portions take the chunked kernels
+
+
+def fixed_decay_attention(q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state, max_query_len: int = 0,
+                          num_decodes: int = 0):
     """Varlen linear attention with a fixed decay per head: ``S <- decay S + silu(k) silu(v)^T``, ``o = S^T silu(q)``
-    over a state cache ``[slots, H, Dv, >= D]`` (fp32, in place).  Returns fp32 ``[T, H, Dv]``."""
+    over a state cache ``[slots, H, Dv, >= D]`` (fp32, in place).  Returns fp32 ``[T, H, Dv]``.  bf16 prompt portions run
+    chunk by chunk on the tensor cores (``csrc/linear_attn/chunk_decay.cu``); the ``num_decodes`` single-token requests
+    at the front of the batch, fp32 models and other head sizes take the token-by-token kernel."""
     out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
-    if q.is_cuda:
-        _c().fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state)
-        return out
-    return _rl.fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state)
+    if not q.is_cuda:
+        return _rl.fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens, state_indices, has_initial_state)
+    D, Dv = q.shape[2], v.shape[2]
+    chunked = (max_query_len >= LINEAR_CHUNK_MIN and q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128
+               and q.stride(0) % 8 == 0 and not any(t.data_ptr() % 16 for t in (q, k, v)))
+    R, nd = state_indices.shape[0], num_decodes if chunked else state_indices.shape[0]
+    for lo, hi, chunk in ((0, nd, False), (nd, R, True)):
+        if lo < hi:
+            _c().fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens[lo:hi + 1], state_indices[lo:hi],
+                                       has_initial_state[lo:hi], chunk)
+    return out
 
 
 # ----------------------------------------------------------------------------- LoRA
