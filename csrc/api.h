@@ -275,7 +275,7 @@ int b200_rejection_sample(int64_t* out, int64_t B, int S, const int64_t* draft_i
 
 // ---- layer norm / post-norm residual stream / unit-norm split (elementwise/layernorm.cu) ----------
 int b200_embed_layernorm(float* x, void* h, const int64_t* ids, const int64_t* positions, const void* table,
-                         const double* freq, const float* w, int64_t T, int H, int ld, int64_t rows, float eps,
+                         const int64_t* freq, const float* w, int64_t T, int H, int ld, int64_t rows, float eps,
                          int dtype, cudaStream_t st);
 int b200_layernorm_residual(float* x, void* h, const void* y1, int64_t y1_stride, float s1, const void* y2,
                             int64_t y2_stride, float s2, const float* w, int64_t T, int H, int ld, float eps, int add,
@@ -322,6 +322,7 @@ typedef struct RecurrenceArgs {
   const int *cu, *slots, *has_init;
   int64_t out_stride, qkv_stride, a_stride, b_stride;
   int R, Hk, H, Dk, Dks, Dv, kind;
+  int decode;                // the requests have one token each (any number is correct, one is fast)
   float scale, unit_eps;
 } RecurrenceArgs;
 int b200_linear_recurrence(const RecurrenceArgs* a, int dtype, cudaStream_t st);

@@ -1382,10 +1382,10 @@ void embed_layernorm(at::Tensor x, at::Tensor h, const at::Tensor& ids, const at
                      const at::Tensor& freq, const at::Tensor& w, double eps) {
   TORCH_CHECK(x.is_contiguous() && h.is_contiguous() && table.is_contiguous() && x.scalar_type() == at::kFloat);
   TORCH_CHECK(h.sizes() == x.sizes() && table.size(1) == x.size(1) && table.scalar_type() == h.scalar_type());
-  TORCH_CHECK(freq.scalar_type() == at::kDouble && freq.numel() >= (w.numel() + 1) / 2 && w.scalar_type() == at::kFloat);
+  TORCH_CHECK(freq.scalar_type() == at::kLong && freq.numel() >= (w.numel() + 1) / 2 && w.scalar_type() == at::kFloat);
   TORCH_CHECK(ids.numel() == x.size(0) && positions.numel() == x.size(0) && w.numel() <= x.size(1));
   check(b200_embed_layernorm(x.data_ptr<float>(), h.data_ptr(), ids.data_ptr<int64_t>(), positions.data_ptr<int64_t>(),
-                             table.data_ptr(), freq.data_ptr<double>(), w.data_ptr<float>(), x.size(0), (int)w.numel(),
+                             table.data_ptr(), freq.data_ptr<int64_t>(), w.data_ptr<float>(), x.size(0), (int)w.numel(),
                              (int)x.size(1), table.size(0), (float)eps, dtype_code(h), stream()), "embed_layernorm");
 }
 void layernorm_residual(at::Tensor x, at::Tensor h, const c10::optional<at::Tensor>& y1, double s1,
@@ -1445,7 +1445,7 @@ void fill_recurrence(RecurrenceArgs& a, at::Tensor& out, const at::Tensor& q, co
 void channel_delta_rule(at::Tensor out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& a_,
                         const at::Tensor& b, const at::Tensor& A_log, const at::Tensor& dt_bias, at::Tensor states,
                         const at::Tensor& cu, const at::Tensor& slots, const at::Tensor& has_init, double scale,
-                        double unit_eps) {
+                        double unit_eps, bool decode) {
   RecurrenceArgs a;
   fill_recurrence(a, out, q, k, v, states, cu, slots, has_init);
   TORCH_CHECK(a_.stride(1) == 1 && b.stride(1) == 1 && a_.size(1) == a.H * a.Dk && b.size(1) == a.H);
@@ -1454,17 +1454,17 @@ void channel_delta_rule(at::Tensor out, const at::Tensor& q, const at::Tensor& k
               dt_bias.numel() == a.H * a.Dk);
   a.a = a_.data_ptr(); a.b = b.data_ptr(); a.a_stride = a_.stride(0); a.b_stride = b.stride(0);
   a.A_log = A_log.data_ptr<float>(); a.dt_bias = dt_bias.data_ptr<float>();
-  a.kind = 0; a.scale = (float)scale; a.unit_eps = (float)unit_eps;
+  a.kind = 0; a.scale = (float)scale; a.unit_eps = (float)unit_eps; a.decode = decode;
   check(b200_linear_recurrence(&a, dtype_code(q), stream()), "channel_delta_rule");
 }
 void fixed_decay_attention(at::Tensor out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v,
                            const at::Tensor& decay, at::Tensor states, const at::Tensor& cu, const at::Tensor& slots,
-                           const at::Tensor& has_init, bool chunked) {
+                           const at::Tensor& has_init, bool chunked, bool decode) {
   RecurrenceArgs a;
   fill_recurrence(a, out, q, k, v, states, cu, slots, has_init);
   TORCH_CHECK(a.Hk == a.H && decay.scalar_type() == at::kFloat && decay.numel() == a.H);
   a.decay = decay.data_ptr<float>();
-  a.kind = 1;
+  a.kind = 1; a.decode = decode;
   if (chunked) check(b200_chunk_decay(&a, dtype_code(q), stream()), "fixed_decay_attention (chunked)");
   else check(b200_linear_recurrence(&a, dtype_code(q), stream()), "fixed_decay_attention");
 }

@@ -59,14 +59,14 @@ __device__ __forceinline__ void layer_norm_regs(float (&y)[NV][4], int H, float 
     }
 }
 
-// freq[i]: turns (angle / 2 pi) per position of column pair i.  The product and the reduction to one turn are in
-// double, so the angle keeps fp32 accuracy at any position.
+// freq[i]: turns (angle / 2 pi) per position of column pair i as a 64-bit fixed-point fraction.  The product with the
+// position wraps modulo one turn by itself, so the angle keeps fp32 accuracy at any position.
 template <typename T, int NV>
 __global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(float* x, T* h,
                                                                     const int64_t* ids,
                                                                     const int64_t* positions,
                                                                     const T* table,
-                                                                    const double* freq,
+                                                                    const int64_t* freq,
                                                                     const float* w, int H, int ld,
                                                                     int64_t rows, float eps) {
   __shared__ float red[32];
@@ -74,7 +74,7 @@ __global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(float* x, T
   griddep_wait();
   const int64_t t = blockIdx.x, id = ids[t];
   const bool ok = id >= 0 && id < rows;
-  const double pos = (double)positions[t];
+  const uint64_t pos = (uint64_t)positions[t];
   float y[NV][4];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -85,10 +85,9 @@ __global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(float* x, T
 #pragma unroll
     for (int j = 0; j < 4; j += 2) {
       if (c + j >= H) continue;
-      double turns = pos * freq[(c + j) >> 1];
-      turns -= rint(turns);
+      const int64_t turns = (int64_t)(pos * (uint64_t)freq[(c + j) >> 1]);  // [-1/2, 1/2) of a turn in units of 2^-64
       float sn, cs;
-      sincospif(2.f * (float)turns, &sn, &cs);
+      sincospif((float)turns * 0x1p-63f, &sn, &cs);
       y[i][j] += sn;
       if (c + j + 1 < H) y[i][j + 1] += cs;
     }
@@ -271,7 +270,7 @@ __global__ void __launch_bounds__(256) qk_unit_norm_cache_kernel(T* q_out, const
 using namespace b200;
 
 extern "C" int b200_embed_layernorm(float* x, void* h, const int64_t* ids, const int64_t* positions, const void* table,
-                                    const double* freq, const float* w, int64_t T_, int H, int ld, int64_t rows, float eps,
+                                    const int64_t* freq, const float* w, int64_t T_, int H, int ld, int64_t rows, float eps,
                                     int dtype, cudaStream_t st) {
   if (T_ == 0) return 0;
   if (ld % 4 || H > ld) return 3;

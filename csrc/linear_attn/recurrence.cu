@@ -24,14 +24,15 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + lo
 
 enum RecurrenceKind : int { kChannelDelta = 0, kFixedDecay = 1 };
 
-template <typename T, int DK, int TPR, int KIND>
-__global__ void __launch_bounds__(kThreads) linear_recurrence_kernel(const RecurrenceArgs p) {
+// CH: tokens per staged chunk.  CH = 1 is the decode instance: few registers, so that enough state rows are in flight to
+// stream the states at memory rate.
+template <typename T, int DK, int TPR, int KIND, int CH>
+__global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kChannelDelta ? 4 : 6) : 1) linear_recurrence_kernel(const RecurrenceArgs p) {
   constexpr int RB = kThreads / TPR;                 // state rows of a block
   constexpr int QW = DK / TPR;                       // key channels of a thread
-  constexpr int CH = DK <= 128 ? 16 : (DK <= 256 ? 8 : 4);
-  constexpr int QK_PER = CH * DK / kThreads;
+  constexpr int QK_PER = (CH * DK + kThreads - 1) / kThreads;
   constexpr int V_PER = (CH * RB + kThreads - 1) / kThreads;
-  static_assert(QW % 4 == 0 && CH * DK % kThreads == 0, "tile");
+  static_assert(QW % 4 == 0, "tile");
   constexpr bool kDelta = KIND == kChannelDelta;
   __shared__ __align__(16) float sk[CH][DK];
   __shared__ __align__(16) float sq[CH][DK];
@@ -68,7 +69,7 @@ __global__ void __launch_bounds__(kThreads) linear_recurrence_kernel(const Recur
 #pragma unroll
     for (int i = 0; i < QK_PER; ++i) {
       const int e = i * kThreads + tid, t = e / DK, d = e % DK;
-      const bool ok = c0 + t < L && d < p.Dk;
+      const bool ok = t < CH && c0 + t < L && d < p.Dk;
       const int64_t tok = s + c0 + t;
       rk_[i] = ok ? to_f(k[tok * p.qkv_stride + d]) : 0.f;
       rq_[i] = ok ? to_f(q[tok * p.qkv_stride + d]) : 0.f;
@@ -172,14 +173,20 @@ __global__ void __launch_bounds__(kThreads) linear_recurrence_kernel(const Recur
       *reinterpret_cast<float4*>(sp + j * TPR) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
 }
 
+template <typename T, int DK, int TPR, int CH>
+void launch_ch(const RecurrenceArgs& a, dim3 grid, cudaStream_t st) {
+  if (a.kind == kChannelDelta)
+    launch_pdl(linear_recurrence_kernel<T, DK, TPR, kChannelDelta, CH>, grid, dim3(kThreads), 0, st, a);
+  else
+    launch_pdl(linear_recurrence_kernel<T, DK, TPR, kFixedDecay, CH>, grid, dim3(kThreads), 0, st, a);
+}
+
 template <typename T, int DK, int TPR>
 int launch(const RecurrenceArgs& a, cudaStream_t st) {
   constexpr int RB = kThreads / TPR;
   dim3 grid((a.Dv + RB - 1) / RB, a.H, a.R);
-  if (a.kind == kChannelDelta)
-    launch_pdl(linear_recurrence_kernel<T, DK, TPR, kChannelDelta>, grid, dim3(kThreads), 0, st, a);
-  else
-    launch_pdl(linear_recurrence_kernel<T, DK, TPR, kFixedDecay>, grid, dim3(kThreads), 0, st, a);
+  if (a.decode) launch_ch<T, DK, TPR, 1>(a, grid, st);
+  else launch_ch<T, DK, TPR, DK <= 128 ? 16 : (DK <= 256 ? 8 : 4)>(a, grid, st);
   return (int)cudaGetLastError();
 }
 

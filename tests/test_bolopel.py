@@ -122,8 +122,7 @@ def test_embedding_positions_and_norms(device, dtype, width):
     ids = torch.randint(0, V, (T,), generator=g)
     start = 70001                                   # positions far out: the angle must not lose bits
     pos = torch.arange(start, start + T)
-    i = torch.arange((width + 1) // 2, dtype=torch.float64)
-    freq = 10000.0 ** (-2 * i / width) / (2 * math.pi)
+    freq = ops.position_turns(width, 10000.0)
     x, h = ops.embed_positions_layernorm(ids.to(device), pos.to(device), table.to(DT[dtype]).to(device), freq.to(device),
                                          w.to(device), 1e-5)
     want = oracle.layer_norm(table[ids].double()[:, :width] + oracle.position_vectors(T, width, start), w.double(), 1e-5)
@@ -370,7 +369,7 @@ def test_channel_delta_rule(device, dtype, H, G, D, Dv):
 
     for cuts in CUTS:
         got, other = _recur(device, dtype, lambda z, st, cu, sl, ini: ops.channel_delta_rule(
-            *z, A_log.to(device), dt.to(device), st, cu, sl, ini, D ** -0.5, 1e-6), T, cuts, args, (H, Dv, -(-D // 4) * 4))
+            *z, A_log.to(device), dt.to(device), st, cu, sl, ini, D ** -0.5, 1e-6, max(1, int((cu[1:] - cu[:-1]).max())), 1), T, cuts, args, (H, Dv, -(-D // 4) * 4))
         close(got, want, dtype, f"portions {cuts[:4]}")
         close(other, want[:len(cuts)], dtype, "neighbour")
 

@@ -14,7 +14,6 @@ Checkpoint names: ``embed``, ``embed.norm``, ``l<i>.norm1``, ``l<i>.mix.*``, ``l
 """
 from __future__ import annotations
 
-import math
 from typing import Iterable, Optional
 
 import torch
@@ -93,12 +92,11 @@ class BolopelForCausalLM(DenseForCausalLM):
         self.layers = nn.ModuleDict({str(i): self.layer_cls(cfg, i, self.dtype, device) for i in range(cfg.num_layers)})
         self.norm = LayerNormWeight(self.width, device)
         self.lm_head = ParallelLMHead(cfg.vocab_size, self.ld, self.dtype, device)
-        i = torch.arange((self.width + 1) // 2, dtype=torch.float64)
-        self.register_buffer("freq", (POSITION_BASE ** (-2.0 * i / self.width) / (2.0 * math.pi)).to(device))
+        self.register_buffer("turns", ops.position_turns(self.width, POSITION_BASE).to(device))
 
     def forward(self, input_ids, hidden=None, residual=None):
         md = get_forward_context().attn
-        x, h = ops.embed_positions_layernorm(input_ids, md.positions, self.embed_tokens.weight, self.freq,
+        x, h = ops.embed_positions_layernorm(input_ids, md.positions, self.embed_tokens.weight, self.turns,
                                              self.embed_norm.weight, self.eps)
         for i in range(self.last_layer):
             h = self.layers[str(i)](x, h)

@@ -314,7 +314,7 @@ class ChannelDelta(nn.Module):
                    (("q", self.kv_heads, self.dim), ("k", self.kv_heads, self.dim), ("v", H, self.vdim)))
         o = ops.channel_delta_rule(q, k, v, up[:, :H * self.dim], p.slice(y, "b"), self.A_log, self.dt_bias, state,
                                    md.query_start_loc, md.state_indices, md.has_initial_state, self.dim ** -0.5,
-                                   UNIT_NORM_EPS)
+                                   UNIT_NORM_EPS, md.max_query_len, md.num_decodes)
         n = H * self.vdim
         z = ops.gated_group_rmsnorm(o.reshape(T, n), up[:, self.n_decay:self.n_decay + n], self.norm.weight, self.eps,
                                     _rows(T, n, h.dtype, h.device))

@@ -651,10 +651,18 @@ def mtp_concat_norm(embed, hidden, enorm_w, hnorm_w, eps, positions=None):
 
 # ----------------------------------------------------------------- fp32 residual stream / linear recurrences
 
+def position_turns(width: int, base: float):
+    """Angle per position of column pair i, ``base ** (-2 i / width)`` radians, as a fraction of a turn in units of
+    2^-64 (two's complement, so that ``position * fraction`` in 64 bits is the angle modulo one turn)."""
+    import math
+    vals = [round(base ** (-2.0 * i / width) / (2.0 * math.pi) * 2.0 ** 64) for i in range((width + 1) // 2)]
+    return torch.tensor([v - (1 << 64) if v >= (1 << 63) else v for v in vals], dtype=torch.int64)
+
+
 def embed_positions_layernorm(ids, positions, table, freq, weight, eps: float):
     """Token rows plus sinusoidal position vectors through a LayerNorm: ``(stream fp32, copy in table.dtype)``, both
-    ``[T, ld]`` with ``ld = table.shape[1] >= weight.numel()`` (the padding columns stay zero).  ``freq`` (float64)
-    holds the turns per position of every column pair."""
+    ``[T, ld]`` with ``ld = table.shape[1] >= weight.numel()`` (the padding columns stay zero).  ``freq`` (int64)
+    holds the turns per position of every column pair as 64-bit fixed-point fractions (:func:`position_turns`)."""
     T, ld = ids.shape[0], table.shape[1]
     x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
     h = x if table.dtype == torch.float32 else torch.empty(T, ld, dtype=table.dtype, device=table.device)
@@ -700,14 +708,18 @@ def qk_unit_norm_cache(q, k, v, kv_cache, slot_mapping, num_heads: int, num_kv_h
 
 
 def channel_delta_rule(q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_indices, has_initial_state, scale: float,
-                       unit_eps: float = 1e-6):
+                       unit_eps: float = 1e-6, max_query_len: int = 0, num_decodes: int = 0):
     """Varlen delta rule with one decay per key channel over a state cache ``[slots, H, Dv, >= Dk]`` (fp32, in place).
     ``q, k [T, Hk, Dk]``, ``v [T, H, Dv]`` (convolved), ``a [T, H * Dk]`` / ``b [T, H]`` the raw decay and step-size
     projections.  The decays, step sizes and unit norms are computed in fp32 inside.  Returns fp32 ``[T, H, Dv]``."""
     out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
     if q.is_cuda:
-        _c().channel_delta_rule(out, q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_indices, has_initial_state,
-                                scale, unit_eps)
+        R = state_indices.shape[0]
+        nd = R if max_query_len == 1 else num_decodes
+        for lo, hi in ((0, nd), (nd, R)):
+            if lo < hi:
+                _c().channel_delta_rule(out, q, k, v, a, b, A_log, dt_bias, states, cu_seqlens[lo:hi + 1],
+                                        state_indices[lo:hi], has_initial_state[lo:hi], scale, unit_eps, lo == 0 and nd > 0)
         return out
     return _rl.channel_delta_rule(out, q, k, v, a, b, A_log, dt_bias, states, cu_seqlens, state_indices, has_initial_state,
                                   scale, unit_eps)
@@ -728,11 +740,12 @@ def fixed_decay_attention(q, k, v, decay, states, cu_seqlens, state_indices, has
     D, Dv = q.shape[2], v.shape[2]
     chunked = (max_query_len >= LINEAR_CHUNK_MIN and q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128
                and q.stride(0) % 8 == 0 and not any(t.data_ptr() % 16 for t in (q, k, v)))
-    R, nd = state_indices.shape[0], num_decodes if chunked else state_indices.shape[0]
-    for lo, hi, chunk in ((0, nd, False), (nd, R, True)):
+    R = state_indices.shape[0]
+    nd = R if max_query_len == 1 else num_decodes
+    for lo, hi, decode in ((0, nd, True), (nd, R, False)):
         if lo < hi:
             _c().fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens[lo:hi + 1], state_indices[lo:hi],
-                                       has_initial_state[lo:hi], chunk)
+                                       has_initial_state[lo:hi], chunked and not decode, decode)
     return out
 
 

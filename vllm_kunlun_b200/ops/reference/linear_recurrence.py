@@ -17,8 +17,8 @@ def _layer_norm(y, weight, eps):
 
 def embed_positions_layernorm(x, h, ids, positions, table, freq, weight, eps):
     n = weight.numel()
-    turns = positions.double().unsqueeze(1) * freq.double()
-    angle = (2 * math.pi * (turns - turns.round())).float()
+    turns = positions.long().unsqueeze(1) * freq           # 64-bit fractions of a turn: the product wraps by itself
+    angle = (turns.double() * (2 * math.pi * 2.0 ** -64)).float()
     pe = torch.stack([angle.sin(), angle.cos()], -1).reshape(len(ids), -1)[:, :n]
     y = table[ids.long()].float()
     y[:, :n] += pe
