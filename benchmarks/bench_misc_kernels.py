@@ -1,7 +1,7 @@
 """Device timings of the sampling, gated-delta-net, conv, LoRA and MTP-glue kernels (CUDA events, L2 flushed
 between iterations, 3 warm-ups), reported against the algorithmic bytes and the measured copy bandwidth.
 
-    python benchmarks/bench_misc_kernels.py [--case sample|gdn|conv|lora|all] [--small]
+    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|conv|lora|all] [--small]
 
 ``--small`` shrinks every case to a few hundred MB so that a profiler capture of one launch ends quickly."""
 import argparse
@@ -87,6 +87,52 @@ def case_gdn(small):
         report(f"gdn_recurrent_kernel({name})", sec, nbytes, f"R={R} L={L}; {T * Hv * 3 * D * D * 2 / sec / 1e12:.2f} TFLOP/s fp32 FMA")
 
 
+def case_recurrence(small):
+    """Linear recurrences of the layer-list designs: fixed decay per head and delta rule with a decay per key channel."""
+    H, D = 32, 128
+    for name, R, L in (("decode", 16, 1), ("prefill", 4, 2048 if not small else 512)):
+        T = R * L
+        mixed = torch.randn(T, 3 * H * D, device="cuda").to(torch.bfloat16)
+        q, k, v = (mixed[:, i * H * D:(i + 1) * H * D].as_strided((T, H, D), (3 * H * D, D, 1), i * H * D) for i in range(3))
+        states = torch.zeros(R, H, D, D, device="cuda")
+        cu = (torch.arange(R + 1, device="cuda") * L).int()
+        idx, init = torch.arange(R, device="cuda").int(), torch.ones(R, device="cuda").int()
+        nd = R if L == 1 else 0
+        decay = torch.linspace(0.9, 0.999, H, device="cuda")
+        nbytes = 2 * states.numel() * 4 + T * 3 * H * D * 2 + T * H * D * 4
+        sec = timeit(lambda: ops.fixed_decay_attention(q, k, v, decay, states, cu, idx, init, L, nd))
+        report(f"fixed_decay_attention({name})", sec, nbytes, f"R={R} L={L}")
+        a = torch.randn(T, H * D, device="cuda").to(torch.bfloat16)
+        b = torch.randn(T, H, device="cuda").to(torch.bfloat16)
+        A_log, dt = torch.zeros(H, device="cuda"), torch.full((H * D,), -3.0, device="cuda")
+        sec = timeit(lambda: ops.channel_delta_rule(q, k, v, a, b, A_log, dt, states, cu, idx, init, D ** -0.5, 1e-6, L, nd))
+        report(f"channel_delta_rule({name})", sec, nbytes + T * H * D * 2, f"R={R} L={L}")
+
+
+def case_stream(small):
+    """fp32-stream kernels: post-norm residual step, unit-RMS split with cache write, gated group norm."""
+    T, W, H, G, D = (8192 if not small else 4096), 4096, 32, 8, 128
+    x = torch.randn(T, W, device="cuda")
+    y1, y2 = (torch.randn(T, W, device="cuda").to(torch.bfloat16) for _ in range(2))
+    w = torch.ones(W, device="cuda")
+    sec = timeit(lambda: ops.layernorm_residual(x, torch.bfloat16, [(y1, 1.0), (y2, 0.5)], w, 1e-5))
+    report("layernorm_residual_kernel", sec, T * W * (8 + 2 + 2 + 2), f"T={T} W={W}, two summands")
+    proj = torch.randn(T, (H + 2 * G) * D, device="cuda").to(torch.bfloat16)
+    cache = torch.zeros(T // 64, 2, G, 64, D, device="cuda", dtype=torch.bfloat16)
+    slots = torch.arange(T, device="cuda")
+    sec = timeit(lambda: ops.qk_unit_norm_cache(proj[:, :H * D], proj[:, H * D:(H + G) * D], proj[:, (H + G) * D:], cache,
+                                                slots, H, G, 1e-5))
+    report("qk_unit_norm_cache_kernel", sec, 2 * T * (H + 2 * G) * D * 2, f"T={T} {H}/{G} heads of {D}")
+    out = torch.empty(T, W, device="cuda", dtype=torch.bfloat16)
+    for n, name in ((W, "whole row"), (D, f"groups of {D}")):
+        sec = timeit(lambda: ops.gated_group_rmsnorm(x, y1, w[:n], 1e-5, out))
+        report("gated_group_rmsnorm_kernel", sec, T * W * 8, f"T={T} W={W}, {name}")
+    ids, pos = torch.randint(0, 32000, (T,), device="cuda"), torch.arange(T, device="cuda")
+    table, turns = torch.randn(32000, W, device="cuda").to(torch.bfloat16), ops.position_turns(W, 10000.0).cuda()
+    sec = timeit(lambda: ops.embed_positions_layernorm(ids, pos, table, turns, w, 1e-5))
+    report("embed_layernorm_kernel", sec, T * W * 8, f"T={T} W={W}")
+
+
 def case_conv(small):
     C, W = 8192, 4
     T = 32768 if not small else 4096
@@ -145,7 +191,7 @@ if __name__ == "__main__":
     ap.add_argument("--case", default="all")
     ap.add_argument("--small", action="store_true")
     a = ap.parse_args()
-    cases = {"sample": case_sample, "gdn": case_gdn, "conv": case_conv, "lora": case_lora}
+    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "conv": case_conv, "lora": case_lora}
     explicit = {"gemm_splits": case_gemm_splits}  # not part of "all"
     with torch.inference_mode():
         for n, fn in cases.items():
