@@ -19,6 +19,11 @@ template <> __device__ __forceinline__ float from_f<float>(float v) { return v; 
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 template <> __device__ __forceinline__ __half from_f<__half>(float v) { return __float2half(v); }
 
+// smallest power of two >= x (x positive and normal), from the bits: exact also when x is a power of two itself
+__device__ __forceinline__ float pow2_ceil(float x) {
+  return __uint_as_float((__float_as_uint(x) + 0x7fffffu) & 0xff800000u);
+}
+
 // 16-byte vector of T
 template <typename T>
 struct alignas(16) Vec16 {

@@ -193,7 +193,7 @@ __global__ void indexer_k_quant_and_cache_kernel(const T* __restrict__ k, uint8_
   for (int j = 0; j < 4; ++j) { v[j] = to_f(k[t * k_stride + lane * 4 + j]); amax = fmaxf(amax, fabsf(v[j])); }
   amax = fmaxf(warp_max(amax), 1e-10f);
   float scale = amax / 448.f;
-  if (ue8m0) scale = exp2f(ceilf(log2f(scale)));
+  if (ue8m0) scale = pow2_ceil(__fdiv_rn(amax, 448.f));
   uint8_t* blk = cache + (slot / block_size) * ((int64_t)block_size * 132);
   const int off = (int)(slot % block_size);
   uint32_t packed = 0;
@@ -248,7 +248,7 @@ __global__ void indexer_prep_kernel(const T* __restrict__ q, const T* __restrict
     float amax = fmaxf(fmaxf(fabsf(v[0]), fabsf(v[1])), fmaxf(fabsf(v[2]), fabsf(v[3])));
     amax = fmaxf(warp_max(amax), 1e-10f);
     scale = amax / 448.f;
-    if (ue8m0) scale = exp2f(ceilf(log2f(scale)));
+    if (ue8m0) scale = pow2_ceil(__fdiv_rn(amax, 448.f));
     uint32_t packed = 0;
 #pragma unroll
     for (int j = 0; j < 4; ++j) packed |= (uint32_t)to_e4m3(v[j] / scale) << (8 * j);

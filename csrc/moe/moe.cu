@@ -312,7 +312,7 @@ __global__ void quant_fp8_group_kernel(uint8_t* __restrict__ q, float* __restric
   for (int j = 0; j < 4; ++j) { v[j] = to_f(src[j]); amax = fmaxf(amax, fabsf(v[j])); }
   amax = fmaxf(warp_max(amax), 1e-10f);
   float scale = amax / 448.f;
-  if (ue8m0) scale = exp2f(ceilf(log2f(scale)));
+  if (ue8m0) scale = pow2_ceil(__fdiv_rn(amax, 448.f));
   const float inv = 1.f / scale;
   uint32_t packed = 0;
 #pragma unroll

@@ -277,6 +277,21 @@ def test_cache_ops():
     _close(ml, rl, 1e-3, 1e-3, "merge lse")
 
 
+def test_indexer_key_scale_at_powers_of_two():
+    """A largest magnitude of 7 x 2^n makes amax / 448 a power of two: the scale is that power, not the next one."""
+    T, bs = 24, 64
+    k = (torch.rand(T, 128, device=DEV) - 0.5).bfloat16()
+    k *= torch.tensor([2.0 ** (n - 12) for n in range(T)], device=DEV, dtype=torch.bfloat16).unsqueeze(1)
+    k[:, 17] = torch.tensor([7 * 2.0 ** (n - 12) for n in range(T)], device=DEV).bfloat16()
+    got = torch.zeros(1, bs, 132, device=DEV, dtype=torch.uint8)
+    want = torch.zeros(1, bs, 132, dtype=torch.uint8)
+    slots = torch.arange(T, device=DEV)
+    ops.indexer_k_quant_and_cache(k, got, slots)
+    ra.indexer_k_quant_and_cache(k.cpu(), want, slots.cpu())
+    (_, sa), (_, sb) = ra.indexer_cache_views(got.cpu()), ra.indexer_cache_views(want)
+    assert torch.equal(sa, sb)
+
+
 @pytest.mark.parametrize("Hq,Hkv,q_len", [(32, 8, 1), (4, 1, 1), (8, 2, 2), (16, 1, 1), (4, 4, 3)])
 @pytest.mark.parametrize("splits", [None, 1, 3, 8])
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float16])
