@@ -33,7 +33,7 @@ def softplus(z):
 
 
 def position_vectors(n, width, start=0):
-    """[n, width]: entry 2i is sin(p / 10000^(2i / width)), entry 2i + 1 the cosine of the same angle."""
+    """[n, width]: column pair i holds (sin, cos) of position / 10000^(2i / width)."""
     out = torch.zeros(n, width, dtype=torch.float64)
     for p in range(n):
         for j in range(width):

@@ -207,7 +207,7 @@ def _paged(device, dtype, q, k, v, scale, window, sink, lens_before, bs=16, eps=
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
-@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 12, 20), (3, 1, 64, 64), (8, 1, 96, 80), (4, 4, 128, 128), (2, 1, 200, 136)])
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 12, 20), (3, 1, 64, 64), (6, 2, 96, 80), (4, 4, 128, 128), (2, 1, 200, 136)])
 def test_windowed_attention_with_sink(device, dtype, H, G, D, Dv):
     """Unequal requests, decode rows beside prompt portions, windows from 1 to longer than everything; the first tokens
     (where the sink weighs most)."""
@@ -341,7 +341,7 @@ def test_fixed_decay_attention(device, dtype, H, D, Dv):
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
-@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 12, 8), (2, 2, 64, 32), (3, 1, 7, 20), (2, 1, 128, 128), (2, 2, 96, 36),
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 12, 8), (2, 2, 64, 40), (3, 1, 7, 20), (2, 1, 128, 128), (2, 2, 96, 36),
                                       (1, 1, 200, 12)])
 def test_channel_delta_rule(device, dtype, H, G, D, Dv):
     """Strong and weak decays side by side (from nearly 1 to below the smallest fp32 number), portions, grouped heads."""
@@ -461,6 +461,22 @@ def test_mixed_batches_and_reuse(checkpoints, device, dtype):
         have, keep = torch.cat(got[k]), [i for i in range(lens[k]) if i % 3 != 1]
         close_rows(have, want[k][keep], dtype, f"request {k}")
     assert pool.num_free == pool.num_blocks and len(r.engine.scheduler.free_state_slots) == 4
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("kind", ["parallel", "channel_delta"])
+def test_models_of_one_kind(device, dtype, kind, tmp_path):
+    """No paged cache at all, or no convolution state at all; grouped heads beyond one decode tile."""
+    mix = parallel(heads=20, kv_heads=1, dim=24, vdim=8, size=50, rheads=2) if kind == "parallel" else delta(conv=1)
+    cfg = config([layer(kind, mix, ff=40)] * 2, width=48)
+    w = oracle.random_weights(cfg, seed=21)
+    save_safetensors({k: v.to(torch.bfloat16) for k, v in w.items()}, str(tmp_path), cfg)
+    t = tokens(90, cfg["vocab"], 3)
+    want, _ = oracle.forward(t, w, cfg)
+    r = replay(str(tmp_path), dtype, device, 128)
+    got = [r.step([{"id": "a", "tokens": t[i:i + n], "want": list(range(n))}]) for i, n in
+           [(0, 50), (50, 2), (52, 1), (53, 1), (54, 30)] + [(i, 1) for i in range(84, 90)]]
+    close_rows(torch.cat(got), want, dtype)
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)

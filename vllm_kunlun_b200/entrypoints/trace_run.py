@@ -4,7 +4,7 @@
 
 Reads one JSON object a line from standard input,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 0, "entries": [{"id": "req-1", "tokens": [11, 4, 90, 2], "want": [3]}], "end": ["req-1"]}
 
 runs the entries as one batch of the engine, writes the logits at the wanted places to ``DIR/<step>.f32`` (little-endian
 fp32 ``[wanted, vocab]``, only when something is wanted) and prints ``done <step>``.  Nothing is sampled."""
