@@ -179,8 +179,8 @@ int b200_decode_attention_umma(void* out, const void* q, const void* tmap, const
 // tokens per request.  `tmap`: the cache as a 2-D [blocks * 64, 576] 16-bit tensor, 64 x 64 boxes, 128-byte swizzle.
 // early_meta as for b200_decode_attention_umma.  Returns 3 for shapes it does not serve.
 int b200_mla_decode_umma(void* out, const void* q, const void* tmap, const int* block_tables, const int* seq_lens,
-                         const int* qsl, float* ws_o, float* ws_lse, int* status, int64_t T, int B, int N,
-                         int block_size, int max_blocks, int64_t num_blocks, int max_query_len, int num_splits,
+                         const int* qsl, const float* sinks, float* ws_o, float* ws_lse, int* status, int64_t T, int B, int N,
+                         int block_size, int max_blocks, int64_t num_blocks, int max_query_len, int num_splits, int window,
                          float scale, int early_meta, int dtype, unsigned long long* trace, cudaStream_t st);
 
 int b200_mla_decode_max_clusters(int R, int S, int dtype);
@@ -189,8 +189,9 @@ int b200_prefill_attention_umma(void* out, float* lse, const void* tmQ, const vo
                                 int D, int block_size, int max_blocks, int64_t num_blocks, int max_query_len, int window,
                                 float scale, int dtype, unsigned long long* trace, cudaStream_t st);
 int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, const void* tmKV, const void* tmKpe, const int* kv_starts,
-                          const int* kv_lens, const int* qsl, int* status, int B, int Hq, int max_query_len, int causal,
-                          float scale, int dtype, unsigned long long* trace, cudaStream_t st);
+                          const int* kv_lens, const int* qsl, const float* sinks, const void* gate, int64_t gate_stride,
+                          int* status, int B, int Hq, int max_query_len, int causal, int window, float scale, int dtype,
+                          unsigned long long* trace, cudaStream_t st);
 int b200_gather_mla_rows(void* out, const void* cache, const int32_t* slots, int64_t M, int64_t total_slots, int fp8,
                          int dtype, cudaStream_t st);
 int b200_quant_int8_token(void* q, float* scale, const void* x, const float* static_scale, int64_t rows, int K,
@@ -291,10 +292,54 @@ int b200_qk_unit_norm_cache(void* q_out, const void* q, const void* k, const voi
 int b200_gemm_f32(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, int64_t ldw, const float* bias,
                   int64_t T, int N, int K, cudaStream_t st);
 
+// ---- latent attention of any size (attention/latent.cu) --------------------------------------------------
+typedef struct LatentPrepArgs {
+  const void *q_down, *kv_down;  // down-projections [T][q_rank], [T][kv_rank | rot_dim], rows `stride` apart
+  const float *q_norm, *kv_norm, *table;  // RMS norm weights; cos / sin pairs [T][pairs][2]
+  const int64_t* slots;
+  void *q_out, *cache;           // [T][q_out_stride] (padded with zeros); latent cache, rows of `row` columns
+  int64_t stride, total_slots;
+  int q_out_stride, q_rank, kv_rank, rot_dim, rot_off, row, pairs, vec;
+  float eps;
+} LatentPrepArgs;
+int b200_latent_prep(const LatentPrepArgs* args, int64_t T, int dtype, cudaStream_t st);
+int b200_rotary_table(float* out, const int64_t* positions, const int64_t* turns, int64_t T, int pairs, cudaStream_t st);
+int b200_rotate_heads(void* q, const float* table, int64_t T, int H, int D, int off, int pairs, int dtype, cudaStream_t st);
+int b200_absorb_query(void* out, const void* q, const void* w, int64_t w_head, const float* table, int64_t T, int H, int D,
+                      int R, int C, int rot_off, int row, int pairs, int dtype, cudaStream_t st);
+int b200_expand_value(void* out, int64_t out_stride, const void* o, const void* w, int64_t w_head, const void* gate,
+                      int64_t gate_stride, int64_t T, int H, int Dv, int C, int dtype, cudaStream_t st);
+int b200_gather_window(void* out, const void* cache, const int* block_tables, const int* seq_lens, const int* starts,
+                       const int* lens, int B, int max_len, int64_t max_blocks, int block_size, int64_t num_blocks,
+                       int64_t row_bytes, int64_t total, cudaStream_t st);
+
+// ---- fp32 stream with one norm per layer, gated summands and token shift (elementwise/gated_stream.cu) ------------
+typedef struct StreamNormArgs {
+  // source of a row: tables (table != null) or stream + gated summands (y1 may be null: the stream as it is)
+  const void *table, *bigram_table;
+  const int64_t *ids, *bigram_rows;
+  int64_t table_rows, bigram_table_rows;
+  const float* x_in;
+  const void *y1, *g1, *y2, *g2;
+  int64_t y1_stride, g1_stride, y2_stride, g2_stride;
+  // results: stream (may be null), norm, norm mixed with the previous token's (may be null)
+  float* x_out;
+  void *h, *shifted;
+  const float *weight, *mix;
+  float* state;              // [slots][ld] norm of the last token of every request
+  const int *req_of_token, *qsl, *slots, *has_init;
+  int64_t T, num_slots;
+  int width, ld, rows_per_cta;
+  float scale, eps;
+} StreamNormArgs;
+int b200_stream_layernorm(const StreamNormArgs* args, int dtype, cudaStream_t st);
+int b200_bigram_rows(int64_t* rows, const int64_t* ids, int64_t* state, const int* qsl, const int* slots, const int* has_init,
+                     int B, int64_t num_slots, int64_t mul_prev, int64_t mul_cur, int64_t buckets, cudaStream_t st);
+
 // ---- paged attention for any head size and for fp32 (attention/paged_generic.cu) -----------------
 int b200_paged_attention_generic(void* out, const void* q, const void* kv_cache, const int* block_tables,
                                  const int* seq_lens, const int* qsl, const float* sinks, int64_t T, int B, int Hq,
-                                 int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks, int max_query_len,
+                                 int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks, int latent_dv,
                                  int window, float scale, int dtype, cudaStream_t st);
 
 // ---- gated delta net / conv / MTP glue --------------------------------------------------------

@@ -4,6 +4,9 @@
 //   kv  [blocks, 64, 576]  = [kv_c (512) | k_pe (64)] per cached token, 16-bit
 //   out [T, N, 512]        = softmax(q . kv^T * scale) . kv[:, :512]
 //
+// Optional sliding window (a token sees the last `window` positions up to itself; pages in front of it are not read) and
+// optional sink per head (exp(sink) joins the softmax denominator once, whatever the number of splits).
+//
 // All heads of a token share ONE latent row, so a request's (heads x query tokens) rows are the small side of both
 // products and the cached tokens the large one.  As in decode_umma.cu the operands are swapped so that the tensor
 // core rows are full:
@@ -52,9 +55,11 @@ struct Params {
   const int* block_tables;
   const int* seq_lens;
   const int* qsl;
+  const float* sinks;       // [N] or null
   int* status;
   unsigned long long* trace;  // optional phase timestamps [CTA][24] (null = off); slots 8-12 follow tile 4 through the pipeline, 13-19 the split merge
   int N, heads_per_cta, max_blocks, num_splits, early_meta;
+  int window;               // 0 = all earlier positions
   int cluster_merge;        // the num_splits CTAs of a (request, head group) form a cluster and merge in shared memory
   int64_t num_blocks, T;
   float scale_log2;
@@ -156,10 +161,12 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
   const int ctx = seq_len - q_len;
   const int kv_end = seq_len;
   const bool served = q_len > 0 && rows_total <= R && nh > 0;
-  const int n_tiles_all = served ? (kv_end + kKeys - 1) / kKeys : 0;
-  const int per_split = (n_tiles_all + p.num_splits - 1) / p.num_splits;
-  const int tile_lo = split * per_split;
-  const int tile_hi = min(n_tiles_all, tile_lo + per_split);
+  // query token i sits at position ctx + i; nobody looks further back than the first token's window
+  const int tile_first = p.window > 0 ? max(0, ctx - p.window + 1) / kKeys : 0;
+  const int tile_end = served ? (kv_end + kKeys - 1) / kKeys : tile_first;
+  const int per_split = (tile_end - tile_first + p.num_splits - 1) / p.num_splits;
+  const int tile_lo = tile_first + split * per_split;
+  const int tile_hi = min(tile_end, tile_lo + per_split);
   const int n_tiles = max(0, tile_hi - tile_lo);
 
   if (warp == 0) {
@@ -327,7 +334,8 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
       if (lane == 0) mbar_arrive(&s_empty[buf]);
       const int key0 = (tile_lo + i) * kKeys;
       const int key = key0 + key_in_tile;
-      const bool full = key0 + kKeys - 1 <= ctx && key0 + kKeys <= kv_end;
+      const bool full = key0 + kKeys - 1 <= ctx && key0 + kKeys <= kv_end &&
+                        (p.window <= 0 || key0 > ctx + q_len - 1 - p.window);
       bool need = fail;   // does any score exceed its row's reference maximum by more than the slack?
       if (full) {  // every key of the page is visible to every query token: no per-row positions needed
 #pragma unroll
@@ -340,7 +348,8 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
         int tok = 0, hh = 0;  // row r = token tok, head hh (walked without divisions)
 #pragma unroll
         for (int r = 0; r < R; ++r) {
-          const bool in = key_thread && r < rows_total && key < kv_end && key <= ctx + tok;
+          const bool in = key_thread && r < rows_total && key < kv_end && key <= ctx + tok &&
+                          (p.window <= 0 || key > ctx + tok - p.window);
           const float v = in ? sc[r] * p.scale_log2 : -INFINITY;
           sc[r] = v;
           need |= v > m_used[r] + kMaxSlack;
@@ -418,6 +427,11 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
       tc_fence_after_sync();
     }
     ok = bar_red_or(1, 128, !ok) == 0;   // one thread's time-out ends the tile for all
+    // share of row r's sink in a denominator whose terms are relative to the maximum M (log2 units)
+    auto sink_term = [&](int r, float M) -> float {
+      return p.sinks != nullptr && r < rows_total && M > -INFINITY
+                 ? exp2f(p.sinks[head0 + r % nh] * 1.4426950408889634f - M) : 0.f;
+    };
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       float v = l_part[r];
@@ -487,6 +501,7 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
           den = fmaf(recv_ml[(s2 * R + r) * 2 + 1], w, den);
           sW[s2 * R + r] = w;
         }
+        den += sink_term(r, M);
         const float inv = den > 0.f ? 1.f / den : 0.f;
         for (int s2 = 0; s2 < S; ++s2) sW[s2 * R + r] *= inv;
         sRow[r] = (r < rows_total && served) ? (long long)(qs + r / nh) * p.N + head0 + r % nh : 0;
@@ -520,7 +535,7 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
         for (int rr = 0; rr < R; ++rr) m_mine = (tid == rr) ? m_used[rr] : m_mine;
         const float L = sSum[r] + sSum[R + r] + sSum[2 * R + r] + sSum[3 * R + r];
         const int64_t orow = r < rows_total ? (int64_t)(qs + r / nh) * p.N + head0 + r % nh : 0;
-        sInv[r] = (ok && L > 0.f) ? 1.f / L : 0.f;
+        sInv[r] = (ok && L > 0.f) ? 1.f / (p.num_splits == 1 ? L + sink_term(r, m_mine) : L) : 0.f;
         sRow[r] = orow;
         if (p.num_splits > 1 && r < rows_total)
           p.ws_lse[(int64_t)split * p.T * p.N + orow] = (ok && L > 0.f) ? m_mine + log2f(L) : -INFINITY;
@@ -590,6 +605,7 @@ mla_decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_co
             den += w;
             sW[s2 * R + r] = w;
           }
+          den += sink_term(r, M);
           const float inv = den > 0.f ? 1.f / den : 0.f;
           for (int s2 = 0; s2 < S; ++s2) sW[s2 * R + r] *= inv;
         }
@@ -704,12 +720,14 @@ extern "C" int b200_mla_decode_max_clusters(int R, int S, int dtype) {
 // 16-bit tensor with 64 x 64 boxes and 128-byte swizzle.  Serves block_size 64 and max_query_len <= 32; heads are
 // processed in groups of R / max_query_len (R = 16 or 32).  Returns 3 for shapes it does not serve.
 extern "C" int b200_mla_decode_umma(void* out, const void* q, const void* tmap, const int* block_tables,
-                                    const int* seq_lens, const int* qsl, float* ws_o, float* ws_lse, int* status,
+                                    const int* seq_lens, const int* qsl, const float* sinks, float* ws_o, float* ws_lse,
+                                    int* status,
                                     int64_t T_, int B, int N, int block_size, int max_blocks, int64_t num_blocks,
-                                    int max_query_len, int num_splits, float scale, int early_meta, int dtype,
+                                    int max_query_len, int num_splits, int window, float scale, int early_meta, int dtype,
                                     unsigned long long* trace, cudaStream_t st) {
   using namespace b200;
   if (B == 0 || T_ == 0) return 0;
+  if (window < 0) return 2;
   if (block_size != mlad::kKeys || max_query_len < 1 || max_query_len > 32 || num_splits < 1 || num_splits > 16) return 3;
   const int R = (N * max_query_len <= 16) ? 16 : 32;
   const int H = R / max_query_len;  // heads per CTA
@@ -721,7 +739,7 @@ extern "C" int b200_mla_decode_umma(void* out, const void* q, const void* tmap, 
   mlad::Params p;
   p.cluster_merge = cluster_merge ? 1 : 0;
   p.q = q; p.out = out; p.ws_o = ws_o; p.ws_lse = ws_lse; p.block_tables = block_tables; p.seq_lens = seq_lens;
-  p.qsl = qsl; p.status = status; p.trace = trace; p.N = N; p.heads_per_cta = H; p.max_blocks = max_blocks; p.num_splits = num_splits;
+  p.qsl = qsl; p.sinks = sinks; p.window = window; p.status = status; p.trace = trace; p.N = N; p.heads_per_cta = H; p.max_blocks = max_blocks; p.num_splits = num_splits;
   p.early_meta = early_meta; p.num_blocks = num_blocks; p.T = T_;
   p.scale_log2 = scale * 1.4426950408889634f;
   const CUtensorMap& tm = *reinterpret_cast<const CUtensorMap*>(tmap);

@@ -1,4 +1,6 @@
-// Paged attention for any head size and for fp32 models: causal, optional sliding window, optional sinks.  The
+// Paged attention for any head size and for fp32 models: causal, optional sliding window, optional sinks; over keys and
+// values [block][2][head][slot][D], or over latent rows [block][slot][D] that all heads share and whose first `latent_dv`
+// columns are the values (absorbed multi-head latent attention).  The
 // tensor-core kernels (prefill_umma.cu, decode_umma.cu, paged_attention.cu, paged_decode.cu) serve 16-bit heads of 64,
 // 128 and 256; this one serves the rest on the CUDA cores, in fp32 throughout.
 // One CTA = one (query token, query head).  Each of its 4 warps walks 32-key tiles of the visible range: scores with a
@@ -15,15 +17,15 @@ namespace {
 
 constexpr int kGenWarps = 4;
 
-template <typename T, int ND>  // ND: value dims per lane, D <= 32 ND
+template <typename T, int ND>  // ND: value dims per lane, Dv <= 32 ND
 __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel(
     T* out, const T* q, const T* cache, const int* block_tables,
     const int* seq_lens, const int* qsl, const float* sinks, int B, int Hq, int Hkv,
-    int D, int block_size, int max_blocks, int64_t num_blocks, int window, float scale) {
+    int D, int Dv, int latent, int block_size, int max_blocks, int64_t num_blocks, int window, float scale) {
   extern __shared__ float sm_gen[];
   float* sq = sm_gen;                       // [D]
-  float* so = sq + D;                       // [kGenWarps][D]
-  float* sml = so + kGenWarps * D;          // [kGenWarps][2]
+  float* so = sq + D;                       // [kGenWarps][Dv]
+  float* sml = so + kGenWarps * Dv;         // [kGenWarps][2]
   griddep_launch();
   griddep_wait();
   const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -40,12 +42,13 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
   for (int i = tid; i < D; i += kGenWarps * 32) sq[i] = to_f(q[((int64_t)t * Hq + h) * D + i]) * scale;
   __syncthreads();
   const int* bt = block_tables + (int64_t)req * max_blocks;
-  const int64_t v_off = (int64_t)Hkv * block_size * D;
+  const int64_t v_off = latent ? 0 : (int64_t)Hkv * block_size * D;
   auto row_of = [&](int key) -> int64_t {
     const int bi = key / block_size;
     const int64_t blk = bi < max_blocks ? bt[bi] : -1;
     if (blk < 0 || blk >= num_blocks) return -1;
-    return (((blk * 2) * Hkv + kvh) * block_size + key % block_size) * (int64_t)D;
+    const int64_t page = latent ? blk : (blk * 2) * Hkv + kvh;
+    return (page * block_size + key % block_size) * (int64_t)D;
   };
   float m = -INFINITY, l = 0.f, acc[ND];
 #pragma unroll
@@ -77,13 +80,13 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
         const int d = i * 32 + lane;
-        if (d < D) acc[i] += pj * to_f(vr[d]);
+        if (d < Dv) acc[i] += pj * to_f(vr[d]);
       }
     }
   }
 #pragma unroll
   for (int i = 0; i < ND; ++i)
-    if (i * 32 + lane < D) so[warp * D + i * 32 + lane] = acc[i];
+    if (i * 32 + lane < Dv) so[warp * Dv + i * 32 + lane] = acc[i];
   if (lane == 0) { sml[warp * 2] = m; sml[warp * 2 + 1] = l; }
   __syncthreads();
   float M = sinks != nullptr ? sinks[h] : -INFINITY;
@@ -93,11 +96,11 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
 #pragma unroll
   for (int w = 0; w < kGenWarps; ++w) { wg[w] = expf(sml[w * 2] - M); den += sml[w * 2 + 1] * wg[w]; }
   const float inv = den > 0.f ? 1.f / den : 0.f;
-  for (int d = tid; d < D; d += kGenWarps * 32) {
+  for (int d = tid; d < Dv; d += kGenWarps * 32) {
     float a = 0.f;
 #pragma unroll
-    for (int w = 0; w < kGenWarps; ++w) a += so[w * D + d] * wg[w];
-    out[((int64_t)t * Hq + h) * D + d] = from_f<T>(a * inv);
+    for (int w = 0; w < kGenWarps; ++w) a += so[w * Dv + d] * wg[w];
+    out[((int64_t)t * Hq + h) * Dv + d] = from_f<T>(a * inv);
   }
 }
 
@@ -107,22 +110,23 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
 extern "C" int b200_paged_attention_generic(void* out, const void* q, const void* kv_cache, const int* block_tables,
                                             const int* seq_lens, const int* qsl, const float* sinks, int64_t T_, int B,
                                             int Hq, int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks,
-                                            int max_query_len, int window, float scale, int dtype, cudaStream_t st) {
+                                            int latent_dv, int window, float scale, int dtype, cudaStream_t st) {
   using namespace b200;
-  (void)max_query_len;
+  const int Dv = latent_dv > 0 ? latent_dv : D;
   if (B == 0 || T_ == 0) return 0;
-  if (Hq % Hkv || Hq > 65535 || window < 0) return 2;
-  const size_t smem = (size_t)(D * (1 + kGenWarps) + 2 * kGenWarps) * sizeof(float);
+  if (Hq % Hkv || Hq > 65535 || window < 0 || Dv > D || (latent_dv > 0 && Hkv != 1)) return 2;
+  const size_t smem = (size_t)(D + kGenWarps * (Dv + 2)) * sizeof(float);
+  if (smem > 48 * 1024) return 3;
   dim3 grid((unsigned)T_, Hq);
 #define B200_GEN_ATTN(ND)                                                                                                \
   B200_DISPATCH_DTYPE(dtype, launch_pdl(paged_attention_generic_kernel<T, ND>, grid, dim3(kGenWarps * 32), smem, st,        \
                                        (T*)out, (const T*)q, (const T*)kv_cache, block_tables, seq_lens, qsl, sinks, B, Hq, \
-                                       Hkv, D, block_size, max_blocks, num_blocks, window, scale))
-  if (D <= 64) { B200_GEN_ATTN(2); }
-  else if (D <= 128) { B200_GEN_ATTN(4); }
-  else if (D <= 256) { B200_GEN_ATTN(8); }
-  else if (D <= 512) { B200_GEN_ATTN(16); }
-  else if (D <= 1024) { B200_GEN_ATTN(32); }
+                                       Hkv, D, Dv, latent_dv > 0, block_size, max_blocks, num_blocks, window, scale))
+  if (Dv <= 64) { B200_GEN_ATTN(2); }
+  else if (Dv <= 128) { B200_GEN_ATTN(4); }
+  else if (Dv <= 256) { B200_GEN_ATTN(8); }
+  else if (Dv <= 512) { B200_GEN_ATTN(16); }
+  else if (Dv <= 1024) { B200_GEN_ATTN(32); }
   else return 3;
 #undef B200_GEN_ATTN
   return (int)cudaGetLastError();

@@ -17,8 +17,9 @@
 // (v1/attention/backends/mla/common.py:1782-1843): 192-dim q / k (128 "nope" dims per head + 64 rotary dims shared
 // by all heads), 128-dim v, keys and values read as contiguous rows of the up-projected `kv_b_proj` output
 // ([rows, heads * 256], k_nope | v per head) plus the rotary key rows ([rows, 64]); each request's keys start at
-// `kv_starts[req]`.  Causal (new tokens) or not (a chunk of cached context); the log-sum-exp output lets the caller
-// merge chunks.  Its K ring has two 48 KB stages and V a single 32 KB one (208 KB of shared memory in all).
+// `kv_starts[req]`.  Causal (new tokens, possibly behind cached ones in front of the same rows; window and sinks as
+// above) or not (a chunk of cached context); the log-sum-exp output lets the caller merge chunks.  Optionally every head's
+// output is multiplied by sigmoid(gate[token, head]).  Its K ring has two 48 KB stages and V a single 32 KB one (208 KB of shared memory in all).
 // TMA loads carry no cluster multicast.  Every wait is bounded; on time-out the status word is set and the CTA unwinds.
 #include <cuda.h>
 #include <cuda_bf16.h>
@@ -55,6 +56,8 @@ struct Params {
   const int* qsl;
   const int* kv_starts;     // MLA form: first key row of each request in the contiguous K / V tensors
   const float* sinks;       // [Hq] or null
+  const void* gate;         // [T, >= Hq] in the output's type, or null
+  int64_t gate_stride;
   int* status;
   unsigned long long* trace;   // optional phase timestamps [CTA][24] (null = off)
   int Hq, Hkv, block_size, max_blocks, window, causal;
@@ -448,7 +451,11 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       float den = l_sum;
       const float ms = (m_used == -INFINITY) ? 0.f : m_used;
       if (p.sinks != nullptr) den += exp2f(p.sinks[head] * 1.4426950408889634f - ms);
-      const float inv = (ok && den > 0.f) ? 1.f / den : 0.f;
+      float inv = (ok && den > 0.f) ? 1.f / den : 0.f;
+      if (p.gate != nullptr && row_ok) {
+        const float g = to_float(reinterpret_cast<const T*>(p.gate)[(int64_t)(qs + row0 + r) * p.gate_stride + head]);
+        inv = inv / (1.f + __expf(-g));
+      }
       T* dst = reinterpret_cast<T*>(p.out) + orow * kD;
       uint32_t o[kD];
 #pragma unroll
@@ -506,7 +513,7 @@ extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tm
   p.out = out; p.lse = lse; p.block_tables = block_tables; p.seq_lens = seq_lens; p.qsl = qsl; p.sinks = sinks;
   p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.max_blocks = max_blocks; p.window = window;
   p.num_blocks = num_blocks; p.scale_log2 = scale * 1.4426950408889634f;
-  p.kv_starts = nullptr; p.causal = 1;
+  p.kv_starts = nullptr; p.causal = 1; p.gate = nullptr; p.gate_stride = 0;
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
   if (dtype == 1) return pattn::launch<__nv_bfloat16, false>(p, q, kv, kv, B, max_query_len, st);
@@ -521,16 +528,18 @@ extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tm
 // kv_starts[r] .. kv_starts[r] + kv_lens[r] and query rows qsl[r] .. qsl[r + 1]; causal: its queries are its last
 // keys.  Rows of requests with no key are not written (the caller presets out = 0, lse = -inf).
 extern "C" int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, const void* tmKV, const void* tmKpe,
-                                     const int* kv_starts, const int* kv_lens, const int* qsl, int* status, int B,
-                                     int Hq, int max_query_len, int causal, float scale, int dtype,
+                                     const int* kv_starts, const int* kv_lens, const int* qsl, const float* sinks,
+                                     const void* gate, int64_t gate_stride, int* status, int B, int Hq,
+                                     int max_query_len, int causal, int window, float scale, int dtype,
                                      unsigned long long* trace, cudaStream_t st) {
   using namespace b200;
   if (B == 0 || max_query_len <= 0) return 0;
   if (B > 65535 || Hq > 65535) return 3;
+  if (window < 0 || (window > 0 && !causal)) return 2;
   pattn::Params p;
   p.out = out; p.lse = lse; p.block_tables = nullptr; p.seq_lens = kv_lens; p.qsl = qsl; p.kv_starts = kv_starts;
-  p.sinks = nullptr; p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hq; p.block_size = pattn::kPage;
-  p.max_blocks = 0; p.window = 0; p.causal = causal ? 1 : 0; p.num_blocks = 0;
+  p.sinks = sinks; p.gate = gate; p.gate_stride = gate_stride; p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hq; p.block_size = pattn::kPage;
+  p.max_blocks = 0; p.window = window; p.causal = causal ? 1 : 0; p.num_blocks = 0;
   p.scale_log2 = scale * 1.4426950408889634f;
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);

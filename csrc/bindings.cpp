@@ -76,7 +76,7 @@ struct GemmState {
 };
 GemmState& gemm_state() { static GemmState s; return s; }
 
-const Tmap& get_tmap(GemmState& gs, const at::Tensor& t, int box_rows, int elem_bytes) {
+Tmap get_tmap(GemmState& gs, const at::Tensor& t, int box_rows, int elem_bytes) {
   TmapKey key{t.data_ptr(), t.size(0), t.size(1), t.stride(0), box_rows, elem_bytes};
   auto it = gs.cache.find(key);
   if (it != gs.cache.end()) return it->second;
@@ -89,7 +89,7 @@ const Tmap& get_tmap(GemmState& gs, const at::Tensor& t, int box_rows, int elem_
 }
 
 // Plain (unswizzled) byte tensor map with a [box_rows, box_bytes] box; cached under elem_bytes = -box_bytes.
-const Tmap& get_tmap_raw(GemmState& gs, const at::Tensor& t, int box_rows, int box_bytes) {
+Tmap get_tmap_raw(GemmState& gs, const at::Tensor& t, int box_rows, int box_bytes) {
   TmapKey key{t.data_ptr(), t.size(0), t.size(1), t.stride(0), box_rows, -box_bytes};
   auto it = gs.cache.find(key);
   if (it != gs.cache.end()) return it->second;
@@ -1018,7 +1018,8 @@ void prefill_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tenso
 // untouched: preset out = 0 and lse = -inf when that can happen.
 void mla_prefill_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv, const at::Tensor& k_pe,
                       const at::Tensor& kv_starts, const at::Tensor& kv_lens, const at::Tensor& qsl,
-                      const c10::optional<at::Tensor>& lse, int64_t max_query_len, bool causal, double scale) {
+                      const c10::optional<at::Tensor>& lse, int64_t max_query_len, bool causal, double scale, int64_t window,
+                      const c10::optional<at::Tensor>& sinks, const c10::optional<at::Tensor>& gate) {
   TORCH_CHECK(q.is_cuda() && q.is_contiguous() && out.is_contiguous() && q.dim() == 3 && q.size(2) == 192);
   TORCH_CHECK(out.dim() == 3 && out.size(0) == q.size(0) && out.size(1) == q.size(1) && out.size(2) == 128);
   TORCH_CHECK(kv.dim() == 2 && kv.stride(1) == 1 && kv.size(1) == q.size(1) * 256 && (kv.stride(0) * 2) % 16 == 0);
@@ -1030,6 +1031,10 @@ void mla_prefill_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv,
   TORCH_CHECK(kv_starts.is_contiguous() && kv_lens.is_contiguous() && qsl.is_contiguous());
   TORCH_CHECK(kv_starts.numel() == kv_lens.numel() && qsl.numel() == kv_lens.numel() + 1);
   if (lse.has_value()) TORCH_CHECK(lse->scalar_type() == at::kFloat && lse->is_contiguous() && lse->numel() == q.size(0) * q.size(1));
+  if (sinks.has_value()) TORCH_CHECK(sinks->scalar_type() == at::kFloat && sinks->is_contiguous() && sinks->numel() == q.size(1));
+  if (gate.has_value())
+    TORCH_CHECK(gate->dim() == 2 && gate->scalar_type() == q.scalar_type() && gate->stride(1) == 1 &&
+                gate->size(0) == q.size(0) && gate->size(1) == q.size(1));
   if (q.size(0) == 0 || kv.size(0) == 0) return;
   c10::cuda::CUDAGuard guard(q.device());
   GemmState& gs = gemm_state();
@@ -1047,8 +1052,9 @@ void mla_prefill_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv,
   const int B = (int)kv_lens.numel();
   check(b200_mla_prefill_umma(out.data_ptr(), lse.has_value() ? lse->data_ptr<float>() : nullptr, tq.b, tk.b, tp.b,
                               kv_starts.data_ptr<int>(), kv_lens.data_ptr<int>(), qsl.data_ptr<int>(),
-                              gs.status.data_ptr<int>(), B, (int)q.size(1), (int)max_query_len, causal ? 1 : 0,
-                              (float)scale, dtype_code(q),
+                              sinks.has_value() ? sinks->data_ptr<float>() : nullptr, opt_ptr(gate),
+                              gate.has_value() ? gate->stride(0) : 0, gs.status.data_ptr<int>(), B, (int)q.size(1),
+                              (int)max_query_len, causal ? 1 : 0, (int)window, (float)scale, dtype_code(q),
                               (g_kernel_trace.defined() &&
                                g_kernel_trace.numel() >= (int64_t)B * q.size(1) * ((max_query_len + 127) / 128) * 24)
                                   ? reinterpret_cast<unsigned long long*>(g_kernel_trace.data_ptr<int64_t>()) : nullptr,
@@ -1071,8 +1077,9 @@ void set_kernel_trace(const c10::optional<at::Tensor>& t) {
 void mla_decode_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv, const at::Tensor& block_tables,
                      const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& ws_o,
                      const c10::optional<at::Tensor>& ws_lse, int64_t max_query_len, int64_t num_splits, double scale,
-                     bool early_meta) {
+                     bool early_meta, int64_t window, const c10::optional<at::Tensor>& sinks) {
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv.is_contiguous() && q.dim() == 3 && kv.dim() == 3);
+  if (sinks.has_value()) TORCH_CHECK(sinks->scalar_type() == at::kFloat && sinks->is_contiguous() && sinks->numel() == q.size(1));
   TORCH_CHECK(q.size(2) == 576 && kv.size(2) == 576 && out.size(2) == 512 && q.scalar_type() == kv.scalar_type());
   TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && qsl.scalar_type() == at::kInt);
   TORCH_CHECK(block_tables.stride(1) == 1);
@@ -1091,10 +1098,11 @@ void mla_decode_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv, 
   const Tmap& tm = get_tmap(gs, flat, 64, 2);
   int B = seq_lens.size(0);
   check(b200_mla_decode_umma(out.data_ptr(), q.data_ptr(), tm.b, block_tables.data_ptr<int>(), seq_lens.data_ptr<int>(),
-                             qsl.data_ptr<int>(), ws_o.has_value() ? ws_o->data_ptr<float>() : nullptr,
+                             qsl.data_ptr<int>(), sinks.has_value() ? sinks->data_ptr<float>() : nullptr,
+                             ws_o.has_value() ? ws_o->data_ptr<float>() : nullptr,
                              ws_lse.has_value() ? ws_lse->data_ptr<float>() : nullptr, gs.status.data_ptr<int>(),
                              q.size(0), B, q.size(1), kv.size(1), block_tables.stride(0), kv.size(0), max_query_len,
-                             num_splits, (float)scale, early_meta ? 1 : 0, dtype_code(q),
+                             num_splits, (int)window, (float)scale, early_meta ? 1 : 0, dtype_code(q),
                              (g_kernel_trace.defined() && g_kernel_trace.numel() >= (int64_t)B * num_splits * 64 * 24)
                                  ? reinterpret_cast<unsigned long long*>(g_kernel_trace.data_ptr<int64_t>()) : nullptr,
                              stream()),
@@ -1477,19 +1485,172 @@ void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c1
                       bias.has_value() ? bias->data_ptr<float>() : nullptr, x.size(0), (int)w.size(0), (int)w.size(1),
                       stream()), "gemm_f32");
 }
+// latent_dv > 0: kv_cache [blocks, block_size, D] holds latent rows shared by all heads, out [T, Hq, latent_dv]
 void paged_attention_generic(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
                              const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
-                             int64_t max_query_len, int64_t window, double scale) {
-  TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && kv_cache.dim() == 5);
-  TORCH_CHECK(q.size(2) == kv_cache.size(4) && out.sizes() == q.sizes() && q.scalar_type() == kv_cache.scalar_type());
+                             int64_t latent_dv, int64_t window, double scale) {
+  const bool latent = latent_dv > 0;
+  TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && out.dim() == 3 &&
+              kv_cache.dim() == (latent ? 3 : 5));
+  TORCH_CHECK(q.size(2) == kv_cache.size(-1) && out.size(0) == q.size(0) && out.size(1) == q.size(1) &&
+              out.size(2) == (latent ? latent_dv : q.size(2)) && q.scalar_type() == kv_cache.scalar_type() &&
+              out.scalar_type() == q.scalar_type());
   TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && qsl.scalar_type() == at::kInt);
   TORCH_CHECK(block_tables.stride(1) == 1);
+  if (sinks.has_value()) TORCH_CHECK(sinks->scalar_type() == at::kFloat && sinks->is_contiguous() && sinks->numel() == q.size(1));
   check(b200_paged_attention_generic(out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(), block_tables.data_ptr<int>(),
                                      seq_lens.data_ptr<int>(), qsl.data_ptr<int>(),
                                      sinks.has_value() ? sinks->data_ptr<float>() : nullptr, q.size(0), (int)seq_lens.size(0),
-                                     (int)q.size(1), (int)kv_cache.size(2), (int)q.size(2), (int)kv_cache.size(3),
-                                     (int)block_tables.stride(0), kv_cache.size(0), (int)max_query_len, (int)window,
-                                     (float)scale, dtype_code(q), stream()), "paged_attention_generic");
+                                     (int)q.size(1), latent ? 1 : (int)kv_cache.size(2), (int)q.size(2),
+                                     (int)kv_cache.size(latent ? 1 : 3), (int)block_tables.stride(0), kv_cache.size(0),
+                                     (int)latent_dv, (int)window, (float)scale, dtype_code(q), stream()),
+        "paged_attention_generic");
+}
+
+// ------------------------------------------------------------------------- latent attention of any size
+void rotary_table(at::Tensor out, const at::Tensor& positions, const at::Tensor& turns) {
+  TORCH_CHECK(out.is_contiguous() && out.scalar_type() == at::kFloat && out.dim() == 3 && out.size(2) == 2);
+  TORCH_CHECK(positions.scalar_type() == at::kLong && turns.scalar_type() == at::kLong && positions.is_contiguous() &&
+              turns.is_contiguous() && turns.is_cuda() && out.size(0) == positions.numel() && out.size(1) == turns.numel());
+  check(b200_rotary_table(out.data_ptr<float>(), positions.data_ptr<int64_t>(), turns.data_ptr<int64_t>(), out.size(0),
+                          (int)out.size(1), stream()), "rotary_table");
+}
+// q_down [T, q_rank], kv_down [T, kv_rank + rot_dim]: column slices of one tensor; cache [blocks, block_size, row]
+void latent_prep(at::Tensor q_out, at::Tensor cache, const at::Tensor& q_down, const at::Tensor& kv_down,
+                 const at::Tensor& q_norm, const at::Tensor& kv_norm, const at::Tensor& table, const at::Tensor& slots,
+                 int64_t rot_off, double eps) {
+  TORCH_CHECK(q_out.is_contiguous() && cache.is_contiguous() && cache.dim() == 3 && q_down.stride(1) == 1 && kv_down.stride(1) == 1);
+  TORCH_CHECK(q_down.stride(0) == kv_down.stride(0) && q_down.size(0) == kv_down.size(0) && q_out.size(0) == q_down.size(0));
+  TORCH_CHECK(q_down.scalar_type() == q_out.scalar_type() && kv_down.scalar_type() == q_out.scalar_type() && cache.scalar_type() == q_out.scalar_type());
+  TORCH_CHECK(q_norm.scalar_type() == at::kFloat && kv_norm.scalar_type() == at::kFloat && q_norm.numel() == q_down.size(1));
+  TORCH_CHECK(table.scalar_type() == at::kFloat && table.is_contiguous() && table.dim() == 3 && table.size(0) == q_down.size(0));
+  TORCH_CHECK(slots.scalar_type() == at::kLong && slots.numel() == q_down.size(0));
+  LatentPrepArgs a;
+  memset(&a, 0, sizeof(a));
+  a.q_down = q_down.data_ptr(); a.kv_down = kv_down.data_ptr(); a.q_norm = q_norm.data_ptr<float>();
+  a.kv_norm = kv_norm.data_ptr<float>(); a.table = table.data_ptr<float>(); a.slots = slots.data_ptr<int64_t>();
+  a.q_out = q_out.data_ptr(); a.cache = cache.data_ptr(); a.stride = q_down.stride(0);
+  a.total_slots = cache.size(0) * cache.size(1); a.q_out_stride = (int)q_out.size(1); a.q_rank = (int)q_down.size(1);
+  a.kv_rank = (int)kv_norm.numel(); a.rot_dim = (int)(kv_down.size(1) - kv_norm.numel()); a.rot_off = (int)rot_off;
+  a.row = (int)cache.size(2); a.pairs = (int)table.size(1); a.eps = (float)eps;
+  check(b200_latent_prep(&a, q_down.size(0), dtype_code(q_out), stream()), "latent_prep");
+}
+void rotate_heads(at::Tensor q, const at::Tensor& table, int64_t off) {
+  TORCH_CHECK(q.is_contiguous() && q.dim() == 3 && table.scalar_type() == at::kFloat && table.is_contiguous() &&
+              table.dim() == 3 && table.size(0) == q.size(0));
+  check(b200_rotate_heads(q.data_ptr(), table.data_ptr<float>(), q.size(0), (int)q.size(1), (int)q.size(2), (int)off,
+                          (int)table.size(1), dtype_code(q), stream()), "rotate_heads");
+}
+// q [T, H, D + R], w [H, D, C] -> out [T, H, row]
+void absorb_query(at::Tensor out, const at::Tensor& q, const at::Tensor& w, const at::Tensor& table, int64_t rot_off) {
+  TORCH_CHECK(out.is_contiguous() && q.is_contiguous() && out.dim() == 3 && q.dim() == 3 && w.dim() == 3);
+  TORCH_CHECK(w.size(0) == q.size(1) && out.size(0) == q.size(0) && out.size(1) == q.size(1) && q.size(2) > w.size(1));
+  TORCH_CHECK(w.stride(2) == 1 && w.stride(1) == w.size(2) && w.scalar_type() == q.scalar_type() && out.scalar_type() == q.scalar_type());
+  TORCH_CHECK(table.scalar_type() == at::kFloat && table.is_contiguous() && table.dim() == 3 && table.size(0) == q.size(0));
+  check(b200_absorb_query(out.data_ptr(), q.data_ptr(), w.data_ptr(), w.stride(0), table.data_ptr<float>(), q.size(0),
+                          (int)q.size(1), (int)w.size(1), (int)(q.size(2) - w.size(1)), (int)w.size(2), (int)rot_off,
+                          (int)out.size(2), (int)table.size(1), dtype_code(q), stream()), "absorb_query");
+}
+// o [T, H, C], w [H, Dv, C], gate [T, H] -> out [T, >= H * Dv]
+void expand_value(at::Tensor out, const at::Tensor& o, const at::Tensor& w, const c10::optional<at::Tensor>& gate) {
+  TORCH_CHECK(out.is_contiguous() && o.is_contiguous() && out.dim() == 2 && o.dim() == 3 && w.dim() == 3);
+  TORCH_CHECK(w.size(0) == o.size(1) && w.size(2) == o.size(2) && out.size(0) == o.size(0) && out.size(1) >= w.size(0) * w.size(1));
+  TORCH_CHECK(w.stride(2) == 1 && w.stride(1) == w.size(2) && w.scalar_type() == o.scalar_type() && out.scalar_type() == o.scalar_type());
+  if (gate.has_value())
+    TORCH_CHECK(gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == o.size(0) && gate->size(1) == o.size(1) &&
+                gate->scalar_type() == o.scalar_type());
+  check(b200_expand_value(out.data_ptr(), out.stride(0), o.data_ptr(), w.data_ptr(), w.stride(0), opt_ptr(gate),
+                          gate.has_value() ? gate->stride(0) : 0, o.size(0), (int)o.size(1), (int)w.size(1), (int)w.size(2),
+                          dtype_code(o), stream()), "expand_value");
+}
+// out [total, row]: the last lens[r] cached rows of every request r from row starts[r] on
+void gather_window(at::Tensor out, const at::Tensor& cache, const at::Tensor& block_tables, const at::Tensor& seq_lens,
+                   const at::Tensor& starts, const at::Tensor& lens, int64_t max_len) {
+  TORCH_CHECK(out.is_contiguous() && cache.is_contiguous() && cache.dim() == 3 && out.dim() == 2 && out.size(1) == cache.size(2) &&
+              out.scalar_type() == cache.scalar_type());
+  TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && starts.scalar_type() == at::kInt &&
+              lens.scalar_type() == at::kInt && block_tables.stride(1) == 1);
+  TORCH_CHECK(seq_lens.numel() == lens.numel() && starts.numel() == lens.numel() && block_tables.size(0) == lens.numel());
+  check(b200_gather_window(out.data_ptr(), cache.data_ptr(), block_tables.data_ptr<int>(), seq_lens.data_ptr<int>(),
+                           starts.data_ptr<int>(), lens.data_ptr<int>(), (int)lens.numel(), (int)max_len,
+                           block_tables.stride(0), (int)cache.size(1), cache.size(0), cache.size(2) * cache.element_size(),
+                           out.size(0), stream()), "gather_window");
+}
+
+// ------------------------------------------------------------------------- fp32 stream, one norm per layer
+void bigram_rows(at::Tensor rows, const at::Tensor& ids, at::Tensor state, const at::Tensor& qsl, const at::Tensor& slots,
+                 const at::Tensor& has_init, int64_t mul_prev, int64_t mul_cur, int64_t buckets) {
+  TORCH_CHECK(rows.scalar_type() == at::kLong && ids.scalar_type() == at::kLong && state.scalar_type() == at::kLong &&
+              rows.numel() == ids.numel() && rows.is_contiguous() && ids.is_contiguous() && state.is_contiguous());
+  TORCH_CHECK(qsl.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && has_init.scalar_type() == at::kInt &&
+              qsl.numel() == slots.numel() + 1 && has_init.numel() == slots.numel());
+  check(b200_bigram_rows(rows.data_ptr<int64_t>(), ids.data_ptr<int64_t>(), state.data_ptr<int64_t>(), qsl.data_ptr<int>(),
+                         slots.data_ptr<int>(), has_init.data_ptr<int>(), (int)slots.numel(), state.numel(), mul_prev, mul_cur,
+                         buckets, stream()), "bigram_rows");
+}
+// mix [ld], state [slots, ld] and the step's metadata belong to the token shift (all or none)
+void fill_stream(StreamNormArgs& a, const at::Tensor& h, const c10::optional<at::Tensor>& x_out, const at::Tensor& weight,
+                 double eps, const c10::optional<at::Tensor>& shifted, const c10::optional<at::Tensor>& mix,
+                 const c10::optional<at::Tensor>& state, const c10::optional<at::Tensor>& req_of_token,
+                 const c10::optional<at::Tensor>& qsl, const c10::optional<at::Tensor>& slots,
+                 const c10::optional<at::Tensor>& has_init) {
+  memset(&a, 0, sizeof(a));
+  TORCH_CHECK(h.dim() == 2 && h.is_contiguous() && weight.scalar_type() == at::kFloat && weight.numel() <= h.size(1));
+  a.T = h.size(0); a.ld = (int)h.size(1); a.width = (int)weight.numel(); a.eps = (float)eps;
+  a.h = h.data_ptr(); a.weight = weight.data_ptr<float>();
+  if (x_out.has_value()) {
+    TORCH_CHECK(x_out->is_contiguous() && x_out->sizes() == h.sizes() && x_out->scalar_type() == at::kFloat);
+    a.x_out = x_out->data_ptr<float>();
+  }
+  if (!shifted.has_value()) return;
+  TORCH_CHECK(shifted->is_contiguous() && shifted->sizes() == h.sizes() && shifted->scalar_type() == h.scalar_type());
+  TORCH_CHECK(mix->scalar_type() == at::kFloat && mix->numel() == h.size(1) && state->scalar_type() == at::kFloat &&
+              state->is_contiguous() && state->dim() == 2 && state->size(1) == h.size(1));
+  TORCH_CHECK(req_of_token->scalar_type() == at::kInt && req_of_token->numel() == h.size(0) && qsl->scalar_type() == at::kInt &&
+              slots->scalar_type() == at::kInt && has_init->scalar_type() == at::kInt && qsl->numel() == slots->numel() + 1);
+  a.shifted = shifted->data_ptr(); a.mix = mix->data_ptr<float>(); a.state = state->data_ptr<float>();
+  a.num_slots = state->size(0); a.req_of_token = req_of_token->data_ptr<int>(); a.qsl = qsl->data_ptr<int>();
+  a.slots = slots->data_ptr<int>(); a.has_init = has_init->data_ptr<int>();
+}
+void embed_stream_layernorm(at::Tensor x_out, at::Tensor h, const at::Tensor& ids, const at::Tensor& table, double scale,
+                            const c10::optional<at::Tensor>& bigram_rows_, const c10::optional<at::Tensor>& bigram_table,
+                            const at::Tensor& weight, double eps, const c10::optional<at::Tensor>& shifted,
+                            const c10::optional<at::Tensor>& mix, const c10::optional<at::Tensor>& state,
+                            const c10::optional<at::Tensor>& req_of_token, const c10::optional<at::Tensor>& qsl,
+                            const c10::optional<at::Tensor>& slots, const c10::optional<at::Tensor>& has_init) {
+  StreamNormArgs a;
+  fill_stream(a, h, x_out, weight, eps, shifted, mix, state, req_of_token, qsl, slots, has_init);
+  TORCH_CHECK(ids.scalar_type() == at::kLong && ids.numel() == h.size(0) && table.is_contiguous() && table.size(1) == h.size(1) &&
+              table.scalar_type() == h.scalar_type());
+  a.table = table.data_ptr(); a.ids = ids.data_ptr<int64_t>(); a.table_rows = table.size(0); a.scale = (float)scale;
+  if (bigram_table.has_value()) {
+    TORCH_CHECK(bigram_table->is_contiguous() && bigram_table->size(1) == h.size(1) && bigram_table->scalar_type() == h.scalar_type());
+    TORCH_CHECK(bigram_rows_->scalar_type() == at::kLong && bigram_rows_->numel() == h.size(0));
+    a.bigram_table = bigram_table->data_ptr(); a.bigram_table_rows = bigram_table->size(0);
+    a.bigram_rows = bigram_rows_->data_ptr<int64_t>();
+  }
+  check(b200_stream_layernorm(&a, dtype_code(h), stream()), "embed_stream_layernorm");
+}
+// x_out = x_in + sigmoid(g1) y1 [+ sigmoid(g2) y2]; h = LayerNorm(x_out); shifted = h + (h_prev - h) mix
+void gated_residual_layernorm(const c10::optional<at::Tensor>& x_out, at::Tensor h, const at::Tensor& x_in,
+                              const c10::optional<at::Tensor>& y1, const c10::optional<at::Tensor>& g1,
+                              const c10::optional<at::Tensor>& y2, const c10::optional<at::Tensor>& g2, const at::Tensor& weight,
+                              double eps, const c10::optional<at::Tensor>& shifted, const c10::optional<at::Tensor>& mix,
+                              const c10::optional<at::Tensor>& state, const c10::optional<at::Tensor>& req_of_token,
+                              const c10::optional<at::Tensor>& qsl, const c10::optional<at::Tensor>& slots,
+                              const c10::optional<at::Tensor>& has_init) {
+  StreamNormArgs a;
+  fill_stream(a, h, x_out, weight, eps, shifted, mix, state, req_of_token, qsl, slots, has_init);
+  TORCH_CHECK(x_in.is_contiguous() && x_in.sizes() == h.sizes() && x_in.scalar_type() == at::kFloat);
+  a.x_in = x_in.data_ptr<float>();
+  auto part = [&](const c10::optional<at::Tensor>& t, const void*& p, int64_t& s) {
+    TORCH_CHECK(t->dim() == 2 && t->sizes() == h.sizes() && t->stride(1) == 1 && t->scalar_type() == h.scalar_type());
+    p = t->data_ptr(); s = t->stride(0);
+  };
+  TORCH_CHECK(y1.has_value() == g1.has_value() && y2.has_value() == g2.has_value() && (y1.has_value() || !y2.has_value()));
+  if (y1.has_value()) { part(y1, a.y1, a.y1_stride); part(g1, a.g1, a.g1_stride); }
+  if (y2.has_value()) { part(y2, a.y2, a.y2_stride); part(g2, a.g2, a.g2_stride); }
+  check(b200_stream_layernorm(&a, dtype_code(h), stream()), "gated_residual_layernorm");
 }
 
 // ------------------------------------------------------------------- expert-parallel dispatch / combine
@@ -1605,6 +1766,15 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("fixed_decay_attention", &fixed_decay_attention);
   m.def("gemm_f32", &gemm_f32);
   m.def("paged_attention_generic", &paged_attention_generic);
+  m.def("rotary_table", &rotary_table);
+  m.def("latent_prep", &latent_prep);
+  m.def("rotate_heads", &rotate_heads);
+  m.def("absorb_query", &absorb_query);
+  m.def("expand_value", &expand_value);
+  m.def("gather_window", &gather_window);
+  m.def("bigram_rows", &bigram_rows);
+  m.def("embed_stream_layernorm", &embed_stream_layernorm);
+  m.def("gated_residual_layernorm", &gated_residual_layernorm);
   m.def("gdn_gating", &gdn_gating);
   m.def("gdn_recurrent", &gdn_recurrent);
   m.def("mtp_concat_norm", &mtp_concat_norm);

@@ -115,7 +115,7 @@ __global__ void act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x,
       float gf = to_f(g.v[j]), uf = to_f(u.v[j]);
       float a;
       if (act == 0) a = gf / (1.f + __expf(-gf));
-      else { float t = 0.7978845608f * (gf + 0.044715f * gf * gf * gf); a = 0.5f * gf * (1.f + tanhf(t)); }
+      else a = gf / (1.f + __expf(-1.5957691216f * (gf + 0.044715f * gf * gf * gf)));  // gelu: (1 + tanh(t)) / 2 = sigmoid(2 t)
       o.v[j] = from_f<T>(a * uf);
     }
   }

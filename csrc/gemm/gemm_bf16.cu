@@ -73,8 +73,8 @@ __device__ __forceinline__ void red_release_sys_add(uint32_t* p, uint32_t v) {
 __device__ __forceinline__ float gated_act(float g, float u, int act) {
   if (act == 1) return g / (1.f + __expf(-g)) * u;
   if (act == 2) {
-    const float t = tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g));
-    return 0.5f * g * (1.f + t) * u;
+    // (1 + tanh(t)) / 2 = sigmoid(2 t): without the cancellation near t = -1
+    return g / (1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
   }
   g = fminf(g, 7.f);
   u = fminf(fmaxf(u, -7.f), 7.f);

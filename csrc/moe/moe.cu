@@ -434,7 +434,7 @@ __global__ void act_mul_quant_fp8_kernel(uint8_t* __restrict__ q, float* __restr
     const float gf = to_f(gp[j]), uf = to_f(gp[I + j]);
     float a;
     if (act == 0) a = gf / (1.f + __expf(-gf));
-    else { float t = 0.7978845608f * (gf + 0.044715f * gf * gf * gf); a = 0.5f * gf * (1.f + tanhf(t)); }
+    else a = gf / (1.f + __expf(-1.5957691216f * (gf + 0.044715f * gf * gf * gf)));  // gelu: (1 + tanh(t)) / 2 = sigmoid(2 t)
     // round through T exactly like the two-kernel path (activation kernel output, then quantiser input)
     v[j] = to_f(from_f<T>(a * uf));
     amax = fmaxf(amax, fabsf(v[j]));

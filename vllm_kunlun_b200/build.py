@@ -26,7 +26,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 
 # Kernels that also serve fp32 models: exp / log / division / square root at full fp32 accuracy.
 PRECISE = {"linear_attn/gdn.cu", "linear_attn/recurrence.cu", "linear_attn/chunk_decay.cu", "elementwise/layernorm.cu", "gemm/gemm_f32.cu",
-           "attention/paged_generic.cu"}
+           "attention/paged_generic.cu", "attention/latent.cu", "elementwise/gated_stream.cu"}
 
 
 def _nvcc() -> str:
@@ -122,7 +122,9 @@ def build(verbose: bool = False, force: bool = False) -> str:
             logs[src] = log
             if verbose and log:
                 print(f"== {os.path.relpath(src, ROOT)}\n{log}")
-    if changed or not os.path.exists(OUT):
+    # an earlier build may have been interrupted between compiling and linking
+    stale = not os.path.exists(OUT) or any(os.path.getmtime(o) > os.path.getmtime(OUT) for o in objs)
+    if changed or stale:
         lib_dirs = ce.library_paths()
         cuda_lib = os.path.join(os.path.dirname(cuda_inc), "lib64")
         cmd = ["g++", "-shared", "-o", OUT, *objs, *[f"-L{d}" for d in lib_dirs], f"-L{cuda_lib}",

@@ -128,7 +128,11 @@ class ModelConfig:
     global_head_dim: Optional[int] = None  # head size of the full-attention layers when it differs (Gemma-4)
     num_global_kv_heads: Optional[int] = None  # their KV head count when values are the keys (attention_k_eq_v)
     attention_k_eq_v: bool = False  # full-attention layers have no v_proj: V is the (un-normalised, un-rotated) K
-    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel); the flat fields above then hold the largest sizes
+    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel, Seturax)
+    embedding_scale: float = 1.0  # factor of the token rows
+    bigram: Optional[dict] = None  # embedding of token pairs: {"buckets", "mul_prev", "mul_cur"}
+    token_shift: bool = False  # the mixers read a blend of this token's and the previous token's norm
+    logit_scale: float = 1.0
     attn_output_gate: bool = False  # q_proj carries a sigmoid output gate (Qwen3-Next full-attention layers)
     # quantization of the checkpoint
     quantization: Optional[str] = None  # None | "fp8" | "int8" | "awq" | "gptq" | "w4a16"
@@ -182,10 +186,20 @@ class ModelConfig:
         """Some layer keeps a per-request state besides (or instead of) the paged cache."""
         if self.linear_attn_pattern > 0:
             return True
+        if self.token_shift or self.bigram:
+            return True
         if not self.layer_specs:
             return False
         from .models.mixers import MIXERS
         return any(MIXERS[spec.type].has_state for spec in self.layer_specs)
+
+    @property
+    def cache_block(self) -> Optional[int]:
+        """Tokens per cache block that the attention kernels of this model need (None = any)."""
+        if self.use_mla:
+            return 64
+        from .models.mixers import MIXERS
+        return next((MIXERS[s.type].cache_block for s in self.layer_specs if MIXERS[s.type].cache_block), None)
 
     def num_params(self) -> int:
         """Rough parameter count (used for memory planning)."""
@@ -464,7 +478,7 @@ class ModelConfig:
     @classmethod
     def _from_layer_list(cls, cfg: dict) -> "ModelConfig":
         """Configurations that list their layers one by one (``architecture``, ``width``, ``vocab``, ``norm.eps``,
-        ``layers: [{type, mixer, mlp}]``)."""
+        ``layers: [{type, mixer, mlp}]``; optionally ``embedding.{scale, bigram}`` and ``logit_scale``)."""
         from .models.mixers import MIXERS
         specs = []
         for i, entry in enumerate(cfg["layers"]):
@@ -475,11 +489,16 @@ class ModelConfig:
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
             specs.append(LayerSpec(entry["type"], dict(entry["mixer"]), None if mlp is None else dict(mlp)))
         arch = cfg["architecture"]
+        emb = cfg.get("embedding") or {}
+        bigram = emb.get("bigram")
         return cls(architecture=arch, name=cfg.get("_name_or_path", arch), vocab_size=int(cfg["vocab"]),
                    hidden_size=int(cfg["width"]), num_layers=len(specs), num_heads=1, num_kv_heads=1, head_dim=1,
                    intermediate_size=max([1] + [int(s.mlp["ff"]) for s in specs if s.mlp]),
                    rms_norm_eps=float(cfg["norm"]["eps"]), max_position=1 << 30, layer_specs=tuple(specs),
-                   dtype=str(cfg.get("torch_dtype", "bfloat16")))
+                   embedding_scale=float(emb.get("scale", 1.0)),
+                   bigram=None if bigram is None else {k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")},
+                   logit_scale=float(cfg.get("logit_scale", 1.0)), dtype=str(cfg.get("torch_dtype", "bfloat16")),
+                   **_LAYER_LIST_TRAITS.get(arch, {}))
 
     def complete_from_shapes(self, shapes: dict) -> "ModelConfig":
         """Sizes that only the checkpoint's tensors tell (``shapes``: name -> shape): the low-rank widths of mixers."""
@@ -498,6 +517,10 @@ class ModelConfig:
             from .models.loader import tensor_shapes
             out.complete_from_shapes(tensor_shapes(path))
         return out
+
+
+# what a design with listed layers fixes without naming it in its configuration
+_LAYER_LIST_TRAITS: dict = {"Seturax": {"hidden_act": "gelu_tanh", "token_shift": True}}
 
 
 def _leading_dense(cfg: dict) -> int:
@@ -587,8 +610,8 @@ class EngineConfig:
         """Apply the platform fix-ups the reference performs in
         ``check_and_update_config`` (``platforms/kunlun.py:147-245``)."""
         m = self.model
-        if m.use_mla and self.cache.block_size not in (64,):
-            self.cache.block_size = 64
+        if m.cache_block:
+            self.cache.block_size = m.cache_block
         if m.index_topk and self.cache.cache_dtype == "auto":
             self.cache.cache_dtype = "bfloat16"
         if self.device == "cpu":

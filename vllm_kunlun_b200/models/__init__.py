@@ -39,6 +39,8 @@ _REGISTRY = {
     "Qwen3_5MoeForCausalLM": "qwen3_next:Qwen3NextForCausalLM",
     # layers listed one by one: windowed attention beside linear attention, channel-wise delta rule
     "Bolopel": "bolopel:BolopelForCausalLM",
+    # windowed latent attention beside the feed-forward, gated residuals, token shift, bigram embedding
+    "Seturax": "seturax:SeturaxForCausalLM",
     # asymmetric V / sliding window with sinks
     "MiMoV2FlashForCausalLM": "mimo_v2_flash:MiMoV2FlashForCausalLM",
     # Gemma family

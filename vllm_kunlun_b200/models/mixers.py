@@ -9,6 +9,7 @@ A mixer reads the residual stream's 16-bit (or fp32) copy ``h [T, ld]`` and retu
 * :class:`LightningAttention` linear attention with a fixed decay per head, jointly normed and gated output
 * :class:`ParallelMixer`     both of them on the same input, one input projection, scaled sum
 * :class:`ChannelDelta`      short convolutions + delta rule with one decay per head and key channel
+* :class:`LatentAttention`   windowed attention over a shared latent row per token, learned sink, output gate per head
 
 Checkpoint rows are padded so that every column slice of a fused projection starts on a 16-byte boundary; padding rows
 and columns are zero.
@@ -168,6 +169,7 @@ class ParallelMixer(nn.Module):
     """Windowed softmax attention and lightning attention on the same input, added with constant scales."""
 
     has_state = True
+    cache_block = None          # any cache block size
     sink_score = 0.0            # one unit in the softmax denominator
 
     @staticmethod
@@ -212,6 +214,9 @@ class ParallelMixer(nn.Module):
     def state_spec(self, dtype):
         return self.right.state_spec()
 
+    def workspace_size(self) -> tuple:
+        return self.left.heads, self.left.cache_dim
+
     def forward(self, h):
         ctx = get_forward_context()
         md = ctx.attn
@@ -229,6 +234,7 @@ class ChannelDelta(nn.Module):
     whose second factors run as one block-diagonal GEMM."""
 
     has_state = True
+    cache_block = None
 
     @staticmethod
     def complete_sizes(sizes: dict, shapes: dict) -> None:
@@ -297,6 +303,9 @@ class ChannelDelta(nn.Module):
         return [((self.taps - 1, self.conv_dim), dtype),
                 ((self.heads, self.vdim, round_up(self.dim, 4)), torch.float32)]
 
+    def workspace_size(self) -> tuple:
+        return 0, 0
+
     def forward(self, h):
         ctx = get_forward_context()
         md = ctx.attn
@@ -321,4 +330,158 @@ class ChannelDelta(nn.Module):
         return [(self.o(z), 1.0)]
 
 
-MIXERS = {"channel_delta": ChannelDelta, "parallel": ParallelMixer}
+class LatentAttention(nn.Module):
+    """Multi-head attention over one latent row per token.  Queries come through their own latent; keys and values are
+    per-head products of the cached latent, plus one rotated key part that all heads share.  Optional sliding ``window``,
+    a learned sink per head, the output of every head times ``sigmoid`` of its gate.
+
+    Single tokens attend in the absorbed form (the query moves into the latent space, ``W_uk`` never meets the cache);
+    prompt portions in the up-projected form: the cached rows that the portion can see and its own ones are gathered
+    contiguously, up-projected by one GEMM and attended by the prefill kernel.  16-bit models up to the kernels' head sizes
+    run both on the tensor cores, with every part zero-padded to them; other sizes and fp32 take the absorbed form on the
+    CUDA cores throughout."""
+
+    has_state = False
+    cache_block = 64                       # tokens per cache block that the decode kernel takes
+    TENSOR_CORE = (128, 64, 128, 512)      # unrotated and rotated query / key dims, value dims, latent
+    KV_BYTES = 512 << 20                   # bound of the up-projected keys and values of one attention call
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        if "dq" in shapes:
+            sizes["q_rank"] = int(shapes["dq"][0])
+
+    @staticmethod
+    def _sizes(m: dict) -> tuple:
+        return m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        super().__init__()
+        H, D, R, V, C, Q = self._sizes(sizes)
+        self.layer_idx, self.eps, self.scale = layer_idx, eps, float(sizes["scale"])
+        self.heads, self.dim, self.rot_dim, self.vdim, self.rank, self.q_rank = H, D, R, V, C, Q
+        rot = sizes["rot"]
+        self.rotary_key = (int(rot.get("dims", R)), float(rot["base"]))
+        if self.rotary_key[0] > R or self.rotary_key[0] % 2:
+            raise ValueError(f"{self.rotary_key[0]} rotated columns in a rotated part of {R}")
+        window = (sizes.get("mask") or {}).get("size")
+        self.window = None if window is None else int(window)
+        self.tensor_cores = (torch.device(device).type == "cuda" and dtype in (torch.bfloat16, torch.float16)
+                             and all(n <= m for n, m in zip((D, R, V, C), self.TENSOR_CORE)))
+        # sizes as the kernels see them, and the place of the rotated key part in a cache row
+        self.D, self.R, self.V, self.C = self.TENSOR_CORE if self.tensor_cores else (D, R, V, align(C))
+        self.row = align(self.C + self.R)
+        self.in_proj = FusedProjection(width, {"dq": Q, "dkv": C + R, "g": H}, dtype, device)
+        self.uq = ReplicatedLinear(align(Q), H * (self.D + self.R), dtype=dtype, device=device)
+        self.up = ReplicatedLinear(self.C, H * (self.D + self.V), dtype=dtype, device=device)      # per head keys | values
+        for lin in (self.uq, self.up):
+            lin.weight.data.zero_()
+        self.o = output_projection(align(H * self.V), width, dtype, device)
+        self.q_norm, self.kv_norm, self.sinks = (param(n, dtype=torch.float32, device=device) for n in (Q, C, H))
+        self.register_buffer("turns", ops.position_turns(*self.rotary_key).to(device))
+
+    @classmethod
+    def tensor_shapes(cls, sizes: dict, width: int) -> dict:
+        H, D, R, V, C, Q = cls._sizes(sizes)
+        return {"dq": (Q, width), "dq.norm": (Q,), "uq": (H * (D + R), Q), "dkv": (C + R, width), "dkv.norm": (C,),
+                "uk": (H * D, C), "uv": (H * V, C), "sink": (H,), "g": (H, width), "o": (width, H * V)}
+
+    def _up(self) -> tuple:
+        """``w_uk [H, D, C]`` and ``w_uv [H, V, C]``, views of the up-projection's weight."""
+        w = self.up.weight.view(self.heads, self.D + self.V, self.C)
+        return w[:, :self.D], w[:, self.D:]
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        H = self.heads
+        if key in ("dq", "dkv", "g"):
+            self.in_proj.load_part(key, w)
+        elif key == "uq":
+            q, g = w.reshape(H, self.dim + self.rot_dim, -1), self.uq.weight.data.view(H, self.D + self.R, -1)
+            g[:, :self.dim, :self.q_rank].copy_(q[:, :self.dim])
+            g[:, self.D:self.D + self.rot_dim, :self.q_rank].copy_(q[:, self.dim:])
+        elif key in ("uk", "uv"):
+            n = self.dim if key == "uk" else self.vdim
+            self._up()[key == "uv"].data[:, :n, :self.rank].copy_(w.reshape(H, n, -1))
+        elif key == "o":
+            g = self.o.weight.data[:, :H * self.V].view(self.o.out_features, H, self.V)
+            g[:w.shape[0], :, :self.vdim].copy_(w.reshape(w.shape[0], H, self.vdim))
+        else:
+            {"dq.norm": self.q_norm, "dkv.norm": self.kv_norm, "sink": self.sinks}[key].data.copy_(w)
+
+    def kv_cache_spec(self, block_size: int, dtype):
+        return ((block_size, self.row), dtype)
+
+    def state_spec(self, dtype):
+        return []
+
+    def workspace_size(self) -> tuple:
+        return 0, 0
+
+    def _portions(self, md, first: int) -> list:
+        """Attention calls of the prompt portions (requests ``first ..``): runs of requests whose visible rows, cached and
+        new, fit the bound on up-projected keys and values.  The same for every layer with this window and row size."""
+        key = ("latent_portions", self.window, self.heads)
+        if key not in md.extras:
+            lens = md.seq_lens_cpu.tolist()
+            qsl = md.query_start_loc_cpu.tolist()
+            limit = max(1, self.KV_BYTES // (self.heads * (self.D + self.V) * 2))
+            calls, lo, rows = [], first, []
+            for b in range(first, md.num_reqs + 1):
+                n = 0
+                if b < md.num_reqs:
+                    q = qsl[b + 1] - qsl[b]
+                    n = lens[b] if self.window is None else min(lens[b], q + self.window - 1)
+                if rows and (b == md.num_reqs or sum(rows) + n > limit):
+                    starts = [sum(rows[:i]) for i in range(len(rows))]
+                    both = torch.tensor([starts, rows], dtype=torch.int32).to(md.seq_lens.device, non_blocking=True)
+                    calls.append((lo, b, both[0], both[1], sum(rows), max(rows),
+                                  max(qsl[i + 1] - qsl[i] for i in range(lo, b))))
+                    lo, rows = b, []
+                rows.append(n)
+            md.extras[key] = calls
+        return md.extras[key]
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md = ctx.attn
+        cache = ctx.kv_caches[self.layer_idx]
+        cache = cache[0] if isinstance(cache, tuple) else cache
+        T, H, p = h.shape[0], self.heads, self.in_proj
+        table = md.extras["rotary"][self.rotary_key]
+        y = p(h)
+        g = p.slice(y, "g")
+        cq = ops.latent_prep(p.slice(y, "dq"), p.slice(y, "dkv"), self.q_norm, self.kv_norm, table, cache, md.slot_mapping,
+                             self.C, self.uq.in_features, self.eps)
+        q = self.uq(cq).view(T, H, self.D + self.R)
+        out = _rows(T, H * self.V, h.dtype, h.device)
+        nd = md.num_decodes if self.tensor_cores else md.num_reqs
+        nt = md.num_decode_tokens if self.tensor_cores else T
+        if nd:
+            w_uk, w_uv = self._up()
+            qa = ops.absorb_query(q[:nt], w_uk, table[:nt], self.C, self.row)
+            cpu = (md.seq_lens_cpu[:nd], md.query_start_loc_cpu[:nd + 1]) if md.seq_lens_cpu is not None else (None, None)
+            o = ops.mla_attention(qa, cache, md.block_tables[:nd], md.seq_lens[:nd], md.query_start_loc[:nd + 1], self.scale,
+                                  self.C, 1 + md.num_spec_tokens if self.tensor_cores else md.max_query_len, md.max_seq_len,
+                                  *cpu, stable_metadata=True, window=self.window, sinks=self.sinks)
+            ops.expand_value(o, w_uv, g[:nt], out[:nt])
+        if nd < md.num_reqs:
+            ops.rotate_heads(q[nt:], table[nt:], self.D)
+            heads = out.view(T, H, self.V)
+            for lo, hi, starts, lens, total, longest, max_q in self._portions(md, nd):
+                rows = ops.gather_window(cache, md.block_tables[lo:hi], md.seq_lens[lo:hi], starts, lens, total, longest)
+                ops.mla_prefill_attention(q, self.up(rows[:, :self.C]), rows[:, self.C:], starts, lens,
+                                          md.query_start_loc[lo:hi + 1], True, self.scale, max_q, out=heads,
+                                          window=self.window, sinks=self.sinks, gate=g, want_lse=False)
+        return [(self.o(out), 1.0)]
+
+
+def rotary_tables(mixers, md) -> None:
+    """cos / sin of the step's positions for every rotation among ``mixers``: made once per step, before the layers."""
+    md.extras["rotary"] = {}
+    for m in mixers:
+        key = getattr(m, "rotary_key", None)
+        if key is not None and key not in md.extras["rotary"]:
+            md.extras["rotary"][key] = ops.rotary_table(md.positions, m.turns)
+
+
+MIXERS = {"channel_delta": ChannelDelta, "latent_attention": LatentAttention, "parallel": ParallelMixer}

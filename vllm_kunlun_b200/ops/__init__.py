@@ -15,6 +15,7 @@ import torch
 from . import _ext
 from .reference import attention as _ra
 from .reference import basic as _rb
+from .reference import latent as _rt
 from .reference import linear_recurrence as _rl
 from .reference import misc as _rx
 from .reference import moe as _rm
@@ -414,36 +415,47 @@ def bmm_heads(x, w):
 
 def mla_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale: float, kv_lora_rank: int,
                   max_query_len: int, max_seq_len: int, seq_lens_cpu=None, query_start_loc_cpu=None, workspace=None,
-                  return_lse: bool = False, stable_metadata: bool = False):
+                  return_lse: bool = False, stable_metadata: bool = False, window: Optional[int] = None, sinks=None):
     """Weight-absorbed MLA attention over the latent cache (decode, spec-verify and causal prefill):
-    ``q [T, N, 576]`` -> ``out [T, N, 512]`` (and the natural-log LSE ``[T, N]`` when asked; rows without any
-    visible key give zeros and ``-inf``)."""
+    ``q [T, N, row]`` -> ``out [T, N, kv_lora_rank]`` (and the natural-log LSE ``[T, N]`` when asked; rows without any
+    visible key give zeros and ``-inf``).  ``window``: a position sees the last ``window`` ones up to itself; ``sinks``:
+    fp32 score per head that joins the denominator.  CUDA: 16-bit models with rows of 512 + 64 run on the tensor cores,
+    other sizes and fp32 on ``csrc/attention/paged_generic.cu``."""
     if q.is_cuda:
         from .mla_cuda import mla_attention_cuda
         return mla_attention_cuda(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, kv_lora_rank,
                                   max_query_len, max_seq_len, workspace, return_lse=return_lse,
-                                  stable_metadata=stable_metadata)
+                                  stable_metadata=stable_metadata, window=window, sinks=sinks)
     sl = seq_lens if seq_lens_cpu is None else seq_lens_cpu
     ql = query_start_loc if query_start_loc_cpu is None else query_start_loc_cpu
-    return _ra.mla_decode(q, kv_cache, block_tables, sl, ql, scale, kv_lora_rank, return_lse=return_lse)
+    return _ra.mla_decode(q, kv_cache, block_tables, sl, ql, scale, kv_lora_rank, return_lse=return_lse, window=window,
+                          sinks=sinks)
 
 
 def mla_prefill_attention(q, kv, k_pe, kv_starts, kv_lens, query_start_loc, causal: bool, scale: float,
-                          max_query_len: int, out=None, lse=None):
+                          max_query_len: int, out=None, lse=None, window: Optional[int] = None, sinks=None, gate=None,
+                          want_lse: bool = True):
     """MLA prefill in the up-projected 192 / 128 form over contiguous keys (the new tokens themselves, causal; or a
     gathered and up-projected chunk of cached context, not causal): ``q [T, N, 192]``, ``kv [rows, N * 256]``,
     ``k_pe [rows, 64]`` -> ``out [T, N, 128]``, natural-log ``lse [T, N]``.  Rows of requests without keys give
-    zeros and ``-inf``.  CUDA: the tcgen05 prefill kernel (``csrc/attention/prefill_umma.cu``, MLA instantiation)."""
+    zeros and ``-inf``.  Causal calls may carry a sliding ``window`` and ``sinks [N]`` (fp32); ``gate [T, N]`` multiplies
+    every head's output by its sigmoid.  CUDA: the tcgen05 prefill kernel (``csrc/attention/prefill_umma.cu``, MLA
+    instantiation)."""
     if q.is_cuda:
         T, N, _ = q.shape
         if out is None:
             out = torch.zeros(T, N, 128, dtype=q.dtype, device=q.device)
-        if lse is None:
+        if lse is None and want_lse:
             lse = torch.full((T, N), float("-inf"), dtype=torch.float32, device=q.device)
         _c().mla_prefill_umma(out, q, kv, k_pe, kv_starts, kv_lens, query_start_loc, lse, int(max_query_len),
-                              bool(causal), float(scale))
+                              bool(causal), float(scale), window or 0, sinks, gate)
         return out, lse
-    return _ra.mla_prefill(q, kv, k_pe, kv_starts, kv_lens, query_start_loc, causal, scale)
+    o, l = _ra.mla_prefill(q, kv, k_pe, kv_starts, kv_lens, query_start_loc, causal, scale, window, sinks, gate)
+    if out is not None:      # rows of other requests stay as they are
+        lo, hi = int(query_start_loc[0]), int(query_start_loc[-1])
+        out[lo:hi] = o[lo:hi]
+        o = out
+    return o, l
 
 
 def sparse_mla_attention(q, kv_cache, indices, scale: float, d_v: int = 512):
@@ -747,6 +759,117 @@ def fixed_decay_attention(q, k, v, decay, states, cu_seqlens, state_indices, has
             _c().fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens[lo:hi + 1], state_indices[lo:hi],
                                        has_initial_state[lo:hi], chunked and not decode, decode)
     return out
+
+
+# ----------------------------------------------------------------- latent attention of any size
+
+def rotary_table(positions, turns):
+    """cos / sin ``[T, pairs, 2]`` (fp32) of every position; ``turns`` as made by :func:`position_turns`."""
+    if positions.is_cuda:
+        out = torch.empty(positions.shape[0], turns.shape[0], 2, dtype=torch.float32, device=positions.device)
+        _c().rotary_table(out, positions, turns)
+        return out
+    return _rt.rotary_table(positions, turns)
+
+
+def latent_prep(q_down, kv_down, q_norm, kv_norm, table, cache, slot_mapping, rot_off: int, q_width: int, eps: float):
+    """RMS norms of both latents and the rotation of the shared key part: returns the query latent ``[T, q_width]``
+    (zero-padded) and writes ``[latent | zeros | key part at rot_off | zeros]`` into the cache ``[blocks, block, row]``."""
+    q = torch.empty(q_down.shape[0], q_width, dtype=q_down.dtype, device=q_down.device)
+    fn = _c().latent_prep if q_down.is_cuda else _rt.latent_prep
+    fn(q, cache, q_down, kv_down, q_norm, kv_norm, table, slot_mapping, rot_off, eps)
+    return q
+
+
+def rotate_heads(q, table, off: int):
+    """Rotate columns ``off ..`` of every head of ``q [T, H, D]`` (in place on CUDA); returns ``q``."""
+    if q.is_cuda:
+        _c().rotate_heads(q, table, off)
+        return q
+    return torch.cat([q[..., :off], _rt.rotate(q[..., off:].float(), table).to(q.dtype)], -1)
+
+
+def absorb_query(q, w_uk, table, rot_off: int, row: int):
+    """``q [T, H, D + R]`` -> ``[q_D . w_uk (H x D x C) | zeros | rotated q_R at rot_off | zeros]``, ``[T, H, row]``."""
+    if q.is_cuda:
+        out = torch.empty(q.shape[0], q.shape[1], row, dtype=q.dtype, device=q.device)
+        _c().absorb_query(out, q, w_uk, table, rot_off)
+        return out
+    return _rt.absorb_query(q, w_uk, table, rot_off, row)
+
+
+def expand_value(o, w_uv, gate, out=None):
+    """``o [T, H, C] . w_uv^T (H x Dv x C)``, each head times ``sigmoid(gate [T, H])``, into ``out [T, >= H * Dv]``."""
+    width = w_uv.shape[0] * w_uv.shape[1] if out is None else out.shape[1]
+    if o.is_cuda:
+        if out is None:
+            out = torch.empty(o.shape[0], width, dtype=o.dtype, device=o.device)
+        _c().expand_value(out, o, w_uv, gate)
+        return out
+    y = _rt.expand_value(o, w_uv, gate, width)
+    return y if out is None else out.copy_(y)
+
+
+def gather_window(cache, block_tables, seq_lens, starts, lens, total: int, max_len: int):
+    """The last ``lens[r]`` cached rows of every request, contiguous from row ``starts[r]``: ``[total, row]``."""
+    if cache.is_cuda:
+        out = torch.empty(total, cache.shape[2], dtype=cache.dtype, device=cache.device)
+        _c().gather_window(out, cache, block_tables, seq_lens, starts, lens, max_len)
+        return out
+    return _rt.gather_window(cache, block_tables, seq_lens, lens)
+
+
+# ----------------------------------------------------- fp32 stream with one norm per layer, gates and token shift
+
+def bigram_rows(ids, state, cu_seqlens, state_indices, has_initial_state, mul_prev: int, mul_cur: int, buckets: int):
+    """``(prev * mul_prev + cur * mul_cur) mod buckets`` per token; a sequence's first token has row ``buckets``.
+    ``state [slots]`` (int64) holds every request's last token between steps."""
+    if ids.is_cuda:
+        rows = torch.empty_like(ids)
+        _c().bigram_rows(rows, ids, state, cu_seqlens, state_indices, has_initial_state, mul_prev, mul_cur, buckets)
+        return rows
+    return _rt.bigram_rows(ids, state, cu_seqlens, state_indices, has_initial_state, mul_prev, mul_cur, buckets)
+
+
+def _shift_args(shift, md):
+    """Arguments of the token shift: ``shift`` is ``(mix [ld], state [slots, ld])`` or None."""
+    if shift is None:
+        return (None,) * 6
+    return shift[0], shift[1], md.req_id_per_token, md.query_start_loc, md.state_indices, md.has_initial_state
+
+
+def embed_stream_layernorm(ids, table, scale: float, bigram, weight, eps: float, shift=None, md=None):
+    """Start of a stream: ``table[id] * scale`` plus, with ``bigram = (rows, bigram_table)``, ``bigram_table[row]``.
+    Returns ``(stream fp32, its LayerNorm in table.dtype, the norm mixed with the previous token's or None)``."""
+    T, ld = ids.shape[0], table.shape[1]
+    x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
+    h = torch.empty(T, ld, dtype=table.dtype, device=table.device)
+    rows, big = (None, None) if bigram is None else bigram
+    if table.is_cuda:
+        hs = None if shift is None else torch.empty_like(h)
+        _c().embed_stream_layernorm(x, h, ids, table, scale, rows, big, weight, eps, hs, *_shift_args(shift, md))
+        return x, h, hs
+    x.copy_(table[ids.long()].float() * scale)
+    if big is not None:
+        x += big[rows.long()].float()
+    return x, h, _rt.stream_layernorm(x, weight, eps, h, None if shift is None else (*shift, *_shift_args(shift, md)[3:]))
+
+
+def gated_residual_layernorm(x, parts, weight, eps: float, dtype, shift=None, md=None, keep_stream: bool = True):
+    """``x' = x + sum of sigmoid(g) * y`` over one or two ``(y, g)`` of ``parts`` (none: the stream as it is) and its
+    LayerNorm: returns ``(x' fp32 in a new buffer or None, norm in dtype, shifted norm or None)``."""
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    if x.is_cuda:
+        new = torch.empty_like(x) if keep_stream else None
+        hs = None if shift is None else torch.empty_like(h)
+        (y1, g1), (y2, g2) = (list(parts) + [(None, None)] * 2)[:2]
+        _c().gated_residual_layernorm(new, h, x, y1, g1, y2, g2, weight, eps, hs, *_shift_args(shift, md))
+        return new, h, hs
+    new = x.clone()
+    for y, g in parts:
+        new += torch.sigmoid(g.float()) * y.float()
+    hs = _rt.stream_layernorm(new, weight, eps, h, None if shift is None else (*shift, *_shift_args(shift, md)[3:]))
+    return new, h, hs
 
 
 # ----------------------------------------------------------------------------- LoRA

@@ -82,7 +82,7 @@ def paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_l
     decode_layout = max_query_len * g <= 16
     if q.dtype == torch.float32 or D not in (64, 128, 256) or (decode_layout and kv_cache.shape[3] % 16):
         # fp32 models, and head sizes (or cache blocks) that the tensor-core kernels do not take
-        _ext.C().paged_attention_generic(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, max_query_len,
+        _ext.C().paged_attention_generic(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, 0,
                                          window or 0, scale)
         return out
     if (decode_layout and UMMA_DECODE[0] and D == 128 and kv_cache.shape[3] % 64 == 0

@@ -68,7 +68,7 @@ def plan_mla_splits(units: int, tiles: int, R: int, dtype, device):
 
 
 def mla_decode_umma(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, max_query_len, max_seq_len,
-                    num_splits=None, stable_metadata: bool = False):
+                    num_splits=None, stable_metadata: bool = False, window=None, sinks=None):
     """Dense paged MLA decode on tcgen05: every request has at most ``max_query_len`` (<= 4) query tokens."""
     T, N, _ = q.shape
     B = seq_lens.shape[0]
@@ -76,25 +76,37 @@ def mla_decode_umma(q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
     R = 16 if N * max_query_len <= 16 else 32
     groups = -(-N // (R // max_query_len))
     if num_splits is None:
-        num_splits, cluster = plan_mla_splits(groups * B, max(1, -(-max_seq_len // 64)), R, q.dtype, q.device)
+        pages = max(1, -(-max_seq_len // 64))
+        if window is not None:      # pages that the window of max_query_len consecutive tokens can touch
+            pages = min(pages, (window + max_query_len + 61) // 64 + 1)
+        num_splits, cluster = plan_mla_splits(groups * B, pages, R, q.dtype, q.device)
     else:
         cluster = num_splits in (2, 4, 8) and groups * B <= _max_clusters(R, num_splits, q.dtype, q.device)
     cluster = cluster and not _FORCE_WORKSPACE[0]
     ws_o, ws_lse = _ws(T, N, num_splits, q.device) if num_splits > 1 and not cluster else (None, None)
     _ext.C().mla_decode_umma(out, q, kv_cache, block_tables, seq_lens, query_start_loc, ws_o, ws_lse, max_query_len,
-                             num_splits, scale, bool(stable_metadata))
+                             num_splits, scale, bool(stable_metadata), window or 0, sinks)
     return out
 
 
 def mla_attention_cuda(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, kv_lora_rank, max_query_len,
                        max_seq_len, workspace=None, req_of_token=None, return_lse: bool = False,
-                       stable_metadata: bool = False):
-    assert kv_lora_rank == 512 and q.shape[-1] == 576 and kv_cache.dtype == q.dtype
+                       stable_metadata: bool = False, window=None, sinks=None):
+    assert kv_cache.dtype == q.dtype
     T, N, _ = q.shape
+    full = kv_lora_rank == 512 and q.shape[-1] == 576 and q.dtype != torch.float32
+    if not full or ((window is not None or sinks is not None) and (max_query_len > _UMMA_MAX_QLEN or not UMMA_DECODE[0])):
+        # fp32 models, other row sizes, windows over more query tokens than the decode kernel takes
+        assert not return_lse, "the log-sum-exp is returned for 16-bit rows of 512 + 64 without a window"
+        out = torch.empty(T, N, kv_lora_rank, dtype=q.dtype, device=q.device)
+        _ext.C().paged_attention_generic(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, kv_lora_rank,
+                                         window or 0, scale)
+        return out
     if (UMMA_DECODE[0] and not return_lse and 1 <= max_query_len <= _UMMA_MAX_QLEN and kv_cache.dim() == 3
             and kv_cache.shape[1] == 64 and q.is_contiguous() and kv_cache.is_contiguous()):
         return mla_decode_umma(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, max_query_len, max_seq_len,
-                               stable_metadata=stable_metadata)
+                               stable_metadata=stable_metadata, window=window, sinks=sinks)
+    assert window is None and sinks is None, "windows and sinks need 64-token cache blocks and contiguous tensors"
     if req_of_token is None:
         lens = (query_start_loc[1:] - query_start_loc[:-1]).long()
         req_of_token = torch.repeat_interleave(torch.arange(lens.shape[0], device=q.device, dtype=torch.int32), lens,

@@ -254,7 +254,8 @@ def merge_attn_states(o1, lse1, o2, lse2):
 
 # ----------------------------------------------------------------------------- MLA
 
-def mla_prefill(q, kv, k_pe, kv_starts, kv_lens, query_start_loc, causal: bool, scale: float):
+def mla_prefill(q, kv, k_pe, kv_starts, kv_lens, query_start_loc, causal: bool, scale: float, window=None, sinks=None,
+                gate=None):
     """Multi-head latent attention in the up-projected ("compute-friendly") form used for prefill
     (``v1/attention/backends/mla/common.py:1782-1843``): ``q [T, N, 192]`` (q_nope | rotated q_pe),
     ``kv [rows, N * 256]`` (k_nope | v per head: the ``kv_b_proj`` output), ``k_pe [rows, 64]`` (one rotary key per
@@ -278,16 +279,23 @@ def mla_prefill(q, kv, k_pe, kv_starts, kv_lens, query_start_loc, causal: bool, 
         s = torch.einsum("qnd,knd->nqk", q[qs:qe].float(), k) * scale
         if causal:
             pos = (L - (qe - qs)) + torch.arange(qe - qs)
-            s = s.masked_fill(torch.arange(L)[None, None, :] > pos[None, :, None], float("-inf"))
+            key = torch.arange(L)[None, None, :]
+            s = s.masked_fill(key > pos[None, :, None], float("-inf"))
+            if window is not None:
+                s = s.masked_fill(key <= pos[None, :, None] - window, float("-inf"))
         l = torch.logsumexp(s, -1)                                   # [N, q]
+        if sinks is not None:
+            l = torch.logaddexp(l, sinks.float().unsqueeze(-1))
         p = torch.exp(s - l.unsqueeze(-1))
         out[qs:qe] = torch.einsum("nqk,knd->qnd", p, v).to(q.dtype)
         lse[qs:qe] = l.t()
+    if gate is not None:
+        out = (out.float() * torch.sigmoid(gate.float()).unsqueeze(-1)).to(out.dtype)
     return out, lse
 
 
 def mla_decode(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, kv_lora_rank: int = 512,
-               return_lse: bool = False):
+               return_lse: bool = False, window=None, sinks=None):
     """Weight-absorbed MQA decode (``flash_mla_with_kvcache``, ``ops/attention/flashmla.py:61-128``).
     ``q [T, N, 576]`` (``[q_nope . W_UK | q_pe]``), cache ``[blocks, bs, 576]`` (or 656-byte fp8).
     Output ``[T, N, 512]``; the ``q_len`` rows of a request are its last positions (causal)."""
@@ -307,7 +315,7 @@ def mla_decode(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, kv_l
         rows = dequant_mla_fp8_rows(rows) if kv_cache.dtype == torch.uint8 else rows.float()
         k = rows.unsqueeze(1)  # [L,1,576]
         v = rows[:, :kv_lora_rank].unsqueeze(1)
-        o, l = _attend(q[qs:qe], k, v, scale, L - (qe - qs), None, None, return_lse=True)
+        o, l = _attend(q[qs:qe], k, v, scale, L - (qe - qs), window, sinks, return_lse=True)
         out[qs:qe], lse[qs:qe] = o.to(q.dtype), l
     return (out, lse) if return_lse else out
 
