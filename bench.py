@@ -78,10 +78,10 @@ def parse():
     ap.add_argument("--layers", type=int, default=0,
                     help="debugging only: run with this many layers (the JSON line then says so and is not a result)")
     ap.add_argument("--layer-bench", nargs="?", const="all", default=None, metavar="SIZE",
-                    help="instead of the headline run: prefill and decode throughput of Bolopel layers beside the "
-                         "closest existing hybrid (Qwen3-Next with dense feed-forwards) at equal sizes; one JSON line "
-                         "per size and model (SIZE: small | large | all)")
-    ap.add_argument("--layer-bench-model", default="both", choices=["both", "bolopel", "qwen3-next"])
+                    help="instead of the headline run: prefill and decode throughput of Bolopel and Seturax layers, each "
+                         "beside the closest other model (Qwen3-Next and DeepSeek, both with dense feed-forwards) at equal "
+                         "sizes; one JSON line per size and model (SIZE: small | large | all)")
+    ap.add_argument("--layer-bench-model", default="all", choices=["all", "bolopel", "qwen3-next", "seturax", "deepseek"])
     a = ap.parse_args()
     c = CONFIGS[a.config]
     a.model = a.model or c["model"]
@@ -164,17 +164,19 @@ def reference_arm(args):
 
 
 # Sizes of the layer benchmark: width, feed-forward, query / key-value heads of the softmax attention, heads of the
-# recurrent layers (head size 128 throughout), layers (every 4th one differs in kind).
+# recurrent layers (head size 128 throughout), layers (every 4th one of the hybrids differs in kind), window, query latent
+# of the latent-attention models (their key / value latent is 512, their rotated part 64).
 LAYER_SIZES = {
-    "small": dict(width=2048, ff=6144, heads=16, kv_heads=4, lin_heads=16, layers=8, window=1024),
-    "large": dict(width=4096, ff=12288, heads=32, kv_heads=8, lin_heads=32, layers=8, window=1024),
+    "small": dict(width=2048, ff=6144, heads=16, kv_heads=4, lin_heads=16, layers=8, window=1024, q_rank=768),
+    "large": dict(width=4096, ff=12288, heads=32, kv_heads=8, lin_heads=32, layers=8, window=1024, q_rank=1536),
 }
 LAYER_VOCAB = 32000
 
 
 def layer_models(size):
-    """The two models of one size: Bolopel (3 of 4 layers 'parallel', 1 'channel_delta') and the existing hybrid (3 of
-    4 layers gated delta net, 1 gated full attention), both with dense feed-forwards of the same width."""
+    """The models of one size, all with dense feed-forwards of the same width: Bolopel (3 of 4 layers 'parallel', 1
+    'channel_delta') and Qwen3-Next (3 of 4 layers gated delta net, 1 gated full attention); Seturax (windowed latent
+    attention) and DeepSeek (latent attention over all positions)."""
     from vllm_kunlun_b200.config import LayerSpec, ModelConfig
     z = LAYER_SIZES[size]
     H = z["lin_heads"]
@@ -193,7 +195,20 @@ def layer_models(size):
                        head_dim=128, intermediate_size=z["ff"], rms_norm_eps=1e-6, qk_norm=True, gemma_norm=True,
                        attn_output_gate=True, max_position=1 << 16, linear_attn_pattern=4, gdn_num_k_heads=H,
                        gdn_num_v_heads=H, gdn_head_k_dim=128, gdn_head_v_dim=128, gdn_conv_kernel=4)
-    return {"bolopel": own, "qwen3-next": like}
+    latent = dict(heads=z["heads"], dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=z["q_rank"], scale=192 ** -0.5,
+                  mask=dict(size=z["window"]), rot=dict(base=10000.0, dims=64))
+    seturax = ModelConfig(architecture="Seturax", name=f"seturax-{size}", vocab_size=LAYER_VOCAB, hidden_size=z["width"],
+                          num_layers=z["layers"], num_heads=1, num_kv_heads=1, head_dim=1, intermediate_size=z["ff"],
+                          rms_norm_eps=1e-6, max_position=1 << 30, hidden_act="gelu_tanh", token_shift=True,
+                          embedding_scale=z["width"] ** 0.5, bigram=dict(buckets=65521, mul_prev=31337, mul_cur=271),
+                          layer_specs=tuple(LayerSpec("latent_attention", dict(latent), dict(kind="dense", ff=z["ff"]))
+                                            for _ in range(z["layers"])))
+    deepseek = ModelConfig(architecture="DeepseekV3ForCausalLM", name=f"deepseek-dense-{size}", vocab_size=LAYER_VOCAB,
+                           hidden_size=z["width"], num_layers=z["layers"], num_heads=z["heads"], num_kv_heads=z["heads"],
+                           head_dim=192, v_head_dim=128, intermediate_size=z["ff"], rms_norm_eps=1e-6, max_position=1 << 16,
+                           rope_neox=False, use_mla=True, q_lora_rank=z["q_rank"], kv_lora_rank=512, qk_nope_head_dim=128,
+                           qk_rope_head_dim=64)
+    return {"bolopel": own, "qwen3-next": like, "seturax": seturax, "deepseek": deepseek}
 
 
 def layer_bench(args):
@@ -208,7 +223,7 @@ def layer_bench(args):
     W, K, IN, DEC = max(3, args.warmup), max(1, args.steps), 2048, 32
     for size in sizes:
         for name, cfg in layer_models(size).items():
-            if args.layer_bench_model not in ("both", name):
+            if args.layer_bench_model not in ("all", name):
                 continue
             llm = LLM(cfg, device="cuda", block_size=64, max_model_len=IN + 2 * DEC + 64, max_num_seqs=64,
                       max_num_batched_tokens=4 * IN, gpu_memory_utilization=0.5)

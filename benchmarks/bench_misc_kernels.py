@@ -1,7 +1,7 @@
 """Device timings of the sampling, gated-delta-net, conv, LoRA and MTP-glue kernels (CUDA events, L2 flushed
 between iterations, 3 warm-ups), reported against the algorithmic bytes and the measured copy bandwidth.
 
-    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|conv|lora|all] [--small]
+    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|latent|conv|lora|all] [--small]
 
 ``--small`` shrinks every case to a few hundred MB so that a profiler capture of one launch ends quickly."""
 import argparse
@@ -133,6 +133,73 @@ def case_stream(small):
     report("embed_layernorm_kernel", sec, T * W * 8, f"T={T} W={W}")
 
 
+def case_latent(small):
+    """Kernels around latent attention (32 heads, 128 + 64 / 128, latents of 1536 and 512) and the gated fp32 stream of
+    width 4096: 4 prompts of 2048 tokens, and 16 single tokens behind a context of 2080."""
+    from types import SimpleNamespace
+    W, H, Q, C, R, win = (4096, 32, 1536, 512, 64, 1024) if not small else (4096, 32, 1536, 512, 64, 256)
+    dev, bf = "cuda", torch.bfloat16
+
+    def rnd(*shape):
+        return torch.randn(*shape, device=dev).to(bf)
+
+    w, mix = torch.randn(W, device=dev), torch.rand(W, device=dev)
+    table, bigram = rnd(32000, W), rnd(65522, W)
+    up = rnd(H * 256, C)
+    w_uk, w_uv = up.view(H, 256, C)[:, :128], up.view(H, 256, C)[:, 128:]
+    qn, kn, sinks = torch.randn(Q, device=dev), torch.randn(C, device=dev), torch.randn(H, device=dev)
+    turns = ops.position_turns(R, 10000.0).to(dev)
+    for tag, B, n, ctx in (("prompts", 4, 2048 if not small else 512, 0), ("single tokens", 16, 1, 2080)):
+        T, blocks = B * n, -(-(ctx + n) // 64)
+        lens = torch.full((B,), ctx + n, dtype=torch.int32, device=dev)
+        qsl = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
+        md = SimpleNamespace(req_id_per_token=torch.arange(B, device=dev).repeat_interleave(n).int(), query_start_loc=qsl,
+                             state_indices=torch.arange(B, dtype=torch.int32, device=dev),
+                             has_initial_state=torch.full((B,), int(ctx > 0), dtype=torch.int32, device=dev))
+        shift = (mix, torch.randn(B, W, device=dev))
+        x, y1, y2, g = torch.randn(T, W, device=dev), rnd(T, W), rnd(T, W), rnd(T, 2 * W)
+        parts = [(y1, g[:, :W]), (y2, g[:, W:])]
+        sec = timeit(lambda: ops.gated_residual_layernorm(x, parts, w, 1e-6, bf, shift, md))
+        report("stream_layernorm (gated sum)", sec, T * W * 20, tag)
+        ids = torch.randint(0, 32000, (T,), device=dev)
+        rows = torch.randint(0, 65521, (T,), device=dev)
+        sec = timeit(lambda: ops.embed_stream_layernorm(ids, table, 64.0, (rows, bigram), w, 1e-6, shift, md))
+        report("stream_layernorm (embedding)", sec, T * W * 12, tag)
+        pos = (torch.arange(T, device=dev) % n) + ctx
+        tab = ops.rotary_table(pos, turns)
+        cache = rnd(B * blocks, 64, C + R)
+        bt = torch.arange(B * blocks, dtype=torch.int32, device=dev).view(B, blocks)
+        slots = torch.cat([bt[b].long()[pos[b * n:(b + 1) * n] // 64] * 64 + pos[b * n:(b + 1) * n] % 64 for b in range(B)])
+        down = rnd(T, Q + C + R + 32)
+        sec = timeit(lambda: ops.latent_prep(down[:, :Q], down[:, Q:Q + C + R], qn, kn, tab, cache, slots, C, Q, 1e-6))
+        report("latent_prep", sec, T * (2 * Q + 2 * C + 2 * R) * 2, tag)
+        q, gate = rnd(T, H, 192), down[:, Q + C + R:]
+        if n > 1:
+            sec = timeit(lambda: ops.rotate_heads(q, tab, 128))
+            report("rotate_heads", sec, T * H * R * 4, tag)
+            starts, klens = qsl[:-1].contiguous(), torch.full((B,), n, dtype=torch.int32, device=dev)
+            sec = timeit(lambda: ops.gather_window(cache, bt, lens, starts, klens, T, n))
+            report("gather_window", sec, T * (C + R) * 4, tag)
+            got = ops.gather_window(cache, bt, lens, starts, klens, T, n)
+            kv, out = rnd(T, H * 256), rnd(T, H, 128)
+            for name, wd, s in (("window and sinks", win, sinks), ("all positions", None, None)):
+                keys = sum(min(i + 1, wd or n) for i in range(n)) * B
+                sec = timeit(lambda: ops.mla_prefill_attention(q, kv, got[:, C:], starts, klens, qsl, True, 0.07, n, out=out,
+                                                               window=wd, sinks=s, want_lse=False))
+                report(f"prefill_umma_kernel (latent, {name})", sec, T * H * 256 * 2,
+                       f"{tag}; {keys * H * 640 / sec / 1e12:.0f} TFLOP/s of visible scores")
+        else:
+            sec = timeit(lambda: ops.absorb_query(q, w_uk, tab, C, C + R))
+            report("absorb_query", sec, H * 128 * C * 2 + T * H * (192 + 576) * 2, tag)
+            qa = ops.absorb_query(q, w_uk, tab, C, C + R)
+            for name, wd, s in (("window and sinks", win, sinks), ("all positions", None, None)):
+                sec = timeit(lambda: ops.mla_attention(qa, cache, bt, lens, qsl, 0.07, C, 1, ctx + 1, window=wd, sinks=s))
+                report(f"mla_decode_umma_kernel ({name})", sec, B * min(ctx + 1, wd or ctx + 1) * 1152, tag)
+            o = rnd(T, H, C)
+            sec = timeit(lambda: ops.expand_value(o, w_uv, gate))
+            report("expand_value", sec, H * 128 * C * 2 + T * H * (512 + 128) * 2, tag)
+
+
 def case_conv(small):
     C, W = 8192, 4
     T = 32768 if not small else 4096
@@ -191,7 +258,7 @@ if __name__ == "__main__":
     ap.add_argument("--case", default="all")
     ap.add_argument("--small", action="store_true")
     a = ap.parse_args()
-    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "conv": case_conv, "lora": case_lora}
+    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "latent": case_latent, "conv": case_conv, "lora": case_lora}
     explicit = {"gemm_splits": case_gemm_splits}  # not part of "all"
     with torch.inference_mode():
         for n, fn in cases.items():

@@ -40,9 +40,18 @@ __device__ __forceinline__ float rotated(int i, int pairs, const float2* cs, F x
   return i < pairs ? x(i) * r.x - x(i + pairs) * r.y : x(i) * r.x + x(i - pairs) * r.y;
 }
 
+template <typename T> struct alignas(4 * sizeof(T)) Quad { T v[4]; };
+template <typename T> __device__ __forceinline__ float4 get4(const T* p) {
+  const Quad<T> r = *reinterpret_cast<const Quad<T>*>(p);
+  return make_float4(to_f(r.v[0]), to_f(r.v[1]), to_f(r.v[2]), to_f(r.v[3]));
+}
+template <typename T> __device__ __forceinline__ void put4(T* p, float a, float b, float c, float d) {
+  *reinterpret_cast<Quad<T>*>(p) = Quad<T>{{from_f<T>(a), from_f<T>(b), from_f<T>(c), from_f<T>(d)}};
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
-  extern __shared__ float sv[];          // [Q query latent | C + R key / value latent and shared key part]
+  extern __shared__ __align__(16) float sv[];          // [Q query latent | C + R key / value latent and shared key part]
   __shared__ float red[2][4];
   griddep_launch();
   griddep_wait();
@@ -52,19 +61,17 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
   const T* kv = reinterpret_cast<const T*>(a.kv_down) + t * a.stride;
   float sq = 0.f, sc = 0.f;
   if (a.vec) {
+#pragma unroll 4
     for (int i = tid * 4; i < Q; i += 512) {
-      alignas(16) T v[4];
-      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(v) = *reinterpret_cast<const uint2*>(q + i);
-      else *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(q + i);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) { const float f = to_f(v[j]); sv[i + j] = f; sq += f * f; }
+      const float4 f = get4(q + i);
+      *reinterpret_cast<float4*>(sv + i) = f;
+      sq += (f.x * f.x + f.y * f.y) + (f.z * f.z + f.w * f.w);
     }
+#pragma unroll 2
     for (int i = tid * 4; i < C + R; i += 512) {
-      alignas(16) T v[4];
-      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(v) = *reinterpret_cast<const uint2*>(kv + i);
-      else *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(kv + i);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) { const float f = to_f(v[j]); sv[Q + i + j] = f; if (i < C) sc += f * f; }
+      const float4 f = get4(kv + i);
+      *reinterpret_cast<float4*>(sv + Q + i) = f;
+      if (i < C) sc += (f.x * f.x + f.y * f.y) + (f.z * f.z + f.w * f.w);
     }
   } else {
     for (int i = tid; i < Q; i += 128) { const float f = to_f(q[i]); sv[i] = f; sq += f * f; }
@@ -88,21 +95,19 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
     const int j = i - a.rot_off;
     return j >= 0 && j < R ? rotated(j, a.pairs, cs, [&](int k) { return sk[k]; }) : 0.f;
   };
-  if (a.vec) {
+  if (a.vec) {   // sizes are multiples of 4: a quad lies inside one part
+    auto scaled = [&](const float* x, float inv, const float* w, T* dst) {
+      const float4 u = *reinterpret_cast<const float4*>(x), v = *reinterpret_cast<const float4*>(w);
+      put4(dst, u.x * inv * v.x, u.y * inv * v.y, u.z * inv * v.z, u.w * inv * v.w);
+    };
     for (int i = tid * 4; i < a.q_out_stride; i += 512) {
-      alignas(16) T v[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) v[j] = from_f<T>(i < Q ? sv[i + j] * iq * a.q_norm[i + j] : 0.f);
-      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(qo + i) = *reinterpret_cast<const uint2*>(v);
-      else *reinterpret_cast<uint4*>(qo + i) = *reinterpret_cast<const uint4*>(v);
+      if (i < Q) scaled(sv + i, iq, a.q_norm + i, qo + i);
+      else put4(qo + i, 0.f, 0.f, 0.f, 0.f);
     }
     if (store)
       for (int i = tid * 4; i < a.row; i += 512) {
-        alignas(16) T v[4];
-#pragma unroll
-        for (int j = 0; j < 4; ++j) v[j] = from_f<T>(cached(i + j));
-        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(co + i) = *reinterpret_cast<const uint2*>(v);
-        else *reinterpret_cast<uint4*>(co + i) = *reinterpret_cast<const uint4*>(v);
+        if (i < C) scaled(sv + Q + i, ic, a.kv_norm + i, co + i);
+        else put4(co + i, cached(i), cached(i + 1), cached(i + 2), cached(i + 3));
       }
   } else {
     for (int i = tid; i < a.q_out_stride; i += 128) qo[i] = from_f<T>(i < Q ? sv[i] * iq * a.q_norm[i] : 0.f);
@@ -385,7 +390,7 @@ extern "C" int b200_latent_prep(const LatentPrepArgs* args, int64_t T_, int dtyp
   const size_t smem = (size_t)(a.q_rank + a.kv_rank + a.rot_dim) * sizeof(float);
   if (smem > 46 * 1024) return 3;
   a.vec = a.q_rank % 4 == 0 && a.kv_rank % 4 == 0 && a.rot_dim % 4 == 0 && a.stride % 4 == 0 && a.q_out_stride % 4 == 0 &&
-          a.row % 4 == 0 && ((uintptr_t)a.q_down | (uintptr_t)a.kv_down | (uintptr_t)a.q_out | (uintptr_t)a.cache) % 16 == 0;
+          a.row % 4 == 0 && a.rot_off % 4 == 0 && ((uintptr_t)a.q_norm | (uintptr_t)a.kv_norm | (uintptr_t)a.q_down | (uintptr_t)a.kv_down | (uintptr_t)a.q_out | (uintptr_t)a.cache) % 16 == 0;
   B200_DISPATCH_DTYPE(dtype, launch_pdl(latent_prep_kernel<T>, dim3((unsigned)T_), dim3(128), smem, st, a));
   return (int)cudaGetLastError();
 }

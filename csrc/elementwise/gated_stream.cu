@@ -15,7 +15,7 @@
 namespace b200 {
 namespace {
 
-constexpr int kThreads = 256;
+constexpr int kThreads = 256;      // of bigram_rows
 
 template <typename T> struct alignas(4 * sizeof(T)) Quad { T v[4]; };
 template <typename T> __device__ __forceinline__ void load4(float (&d)[4], const T* p) {
@@ -28,6 +28,11 @@ template <typename T> __device__ __forceinline__ void store4(T* p, const float (
 #pragma unroll
   for (int j = 0; j < 4; ++j) r.v[j] = from_f<T>(s[j]);
   *reinterpret_cast<Quad<T>*>(p) = r;
+}
+
+template <int N> __device__ __forceinline__ void copy_async(void* smem, const void* gmem) {
+  const uint32_t s = static_cast<uint32_t>(__cvta_generic_to_shared(smem));
+  asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(s), "l"(gmem), "n"(N) : "memory");
 }
 
 // One CTA per request: the state is read before any row is written and replaced at the end.
@@ -50,16 +55,44 @@ __global__ void __launch_bounds__(kThreads) bigram_rows_kernel(int64_t* rows, co
   if (threadIdx.x == 0 && held && t1 > t0) state[slot] = ids[t1 - 1];
 }
 
-// kEmbed: rows come from the tables; otherwise from the stream and up to two gated summands.
-template <typename T, int NV, bool kEmbed>
-__global__ void __launch_bounds__(kThreads) stream_layernorm_kernel(StreamNormArgs a) {
-  __shared__ float red[32];
+// sigmoid with the hardware exponential and reciprocal (a few units in the last place of fp32)
+__device__ __forceinline__ float gate(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
+// kEmbed: rows come from the tables; otherwise from the stream and up to two gated summands.  NT threads hold a row as NV
+// quads each.  kAhead (runs of rows): the next row travels into shared memory while this one is normalised and written;
+// every thread copies and reads its own quads only, so that needs no barrier.
+template <typename T, int NT, int NV, bool kEmbed, bool kAhead>
+__global__ void __launch_bounds__(NT, 1024 / NT) stream_layernorm_kernel(StreamNormArgs a) {
+  extern __shared__ __align__(16) uint8_t ahead[];
+  __shared__ __align__(16) float red[2][NT / 32];
   griddep_launch();
   griddep_wait();
   const int H = a.width, ld = a.ld;
+  const float inv_h = 1.f / H;
   T* hp = reinterpret_cast<T*>(a.h);
   T* sp = reinterpret_cast<T*>(a.shifted);
+  const int c0 = threadIdx.x * 4;
 
+  auto block_total = [&](float v, int buf) -> float {   // buffers alternate: one barrier per sum
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[buf][threadIdx.x >> 5] = v;
+    __syncthreads();
+    if constexpr (NT > 256) return warp_sum((threadIdx.x & 31) < NT / 32 ? red[buf][threadIdx.x & 31] : 0.f);
+    float r = 0.f;
+#pragma unroll
+    for (int w = 0; w < NT / 32; w += 4) {
+      const float4 q = *reinterpret_cast<const float4*>(&red[buf][w]);
+      r += (q.x + q.y) + (q.z + q.w);
+    }
+    return r;
+  };
+  auto clear_tail = [&](float (&q)[4], int c) {         // columns from the width on
+    if (c + 4 > H) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j >= H) q[j] = 0.f;
+    }
+  };
   auto row = [&](int64_t t, float (&y)[NV][4]) {
     [[maybe_unused]] int64_t id = 0, bg = 0;
     [[maybe_unused]] bool id_ok = false, bg_ok = false;
@@ -71,7 +104,7 @@ __global__ void __launch_bounds__(kThreads) stream_layernorm_kernel(StreamNormAr
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kThreads + threadIdx.x) * 4;
+      const int c = c0 + i * NT * 4;
       y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.f;
       if (c >= ld) continue;
       float u[4], g[4];
@@ -92,86 +125,129 @@ __global__ void __launch_bounds__(kThreads) stream_layernorm_kernel(StreamNormAr
           load4(u, reinterpret_cast<const T*>(a.y1) + t * a.y1_stride + c);
           load4(g, reinterpret_cast<const T*>(a.g1) + t * a.g1_stride + c);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) u[j] = u[j] / (1.f + expf(-g[j]));
-          if (a.y2 != nullptr) {
-            float u2[4];
-            load4(u2, reinterpret_cast<const T*>(a.y2) + t * a.y2_stride + c);
-            load4(g, reinterpret_cast<const T*>(a.g2) + t * a.g2_stride + c);
+          for (int j = 0; j < 4; ++j) y[i][j] += u[j] * gate(g[j]);
+        }
+        if (a.y2 != nullptr) {
+          load4(u, reinterpret_cast<const T*>(a.y2) + t * a.y2_stride + c);
+          load4(g, reinterpret_cast<const T*>(a.g2) + t * a.g2_stride + c);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) u[j] += u2[j] / (1.f + expf(-g[j]));
-          }
-#pragma unroll
-          for (int j = 0; j < 4; ++j) y[i][j] += u[j];
+          for (int j = 0; j < 4; ++j) y[i][j] += u[j] * gate(g[j]);
         }
       }
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (c + j >= H) y[i][j] = 0.f;
+      clear_tail(y[i], c);
     }
   };
-  auto norm = [&](float (&y)[NV][4]) {
+  // shared memory of kAhead: NV quads of the stream per thread, then of y1, g1, y2, g2
+  auto own_x = [&](int i) { return reinterpret_cast<float*>(ahead) + (i * NT + threadIdx.x) * 4; };
+  auto own_t = [&](int k, int i) {
+    return reinterpret_cast<T*>(ahead + NV * NT * 16) + ((k * NV + i) * NT + threadIdx.x) * 4;
+  };
+  auto fetch = [&](int64_t t) {
+    if constexpr (kAhead) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * NT * 4;
+        if (c >= ld) continue;
+        copy_async<16>(own_x(i), a.x_in + t * ld + c);
+        if (a.y1 != nullptr) {
+          copy_async<4 * sizeof(T)>(own_t(0, i), reinterpret_cast<const T*>(a.y1) + t * a.y1_stride + c);
+          copy_async<4 * sizeof(T)>(own_t(1, i), reinterpret_cast<const T*>(a.g1) + t * a.g1_stride + c);
+        }
+        if (a.y2 != nullptr) {
+          copy_async<4 * sizeof(T)>(own_t(2, i), reinterpret_cast<const T*>(a.y2) + t * a.y2_stride + c);
+          copy_async<4 * sizeof(T)>(own_t(3, i), reinterpret_cast<const T*>(a.g2) + t * a.g2_stride + c);
+        }
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+  };
+  auto fetched_row = [&](float (&y)[NV][4]) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * NT * 4;
+      y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.f;
+      if (c >= ld) continue;
+      load4(y[i], own_x(i));
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        if ((k == 0 ? a.y1 : a.y2) == nullptr) continue;
+        float u[4], g[4];
+        load4(u, own_t(2 * k, i));
+        load4(g, own_t(2 * k + 1, i));
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[i][j] += u[j] * gate(g[j]);
+      }
+      clear_tail(y[i], c);
+    }
+  };
+  auto norm = [&](float (&y)[NV][4], int64_t next) {    // next >= 0: the row to fetch once this one has been read
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) s += y[i][j];
-    const float mean = block_sum(s, red) / H;
+    for (int i = 0; i < NV; ++i) s += (y[i][0] + y[i][1]) + (y[i][2] + y[i][3]);
+    const float mean = block_total(s, 0) * inv_h;
+    if (next >= 0) fetch(next);
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i)
+    for (int i = 0; i < NV; ++i) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = (i * kThreads + threadIdx.x) * 4 + j;
-        const float d = c < H ? y[i][j] - mean : 0.f;
-        y[i][j] = d;
-        ss += d * d;
+      for (int j = 0; j < 4; ++j) y[i][j] -= mean;
+      clear_tail(y[i], c0 + i * NT * 4);
+      ss += (y[i][0] * y[i][0] + y[i][1] * y[i][1]) + (y[i][2] * y[i][2] + y[i][3] * y[i][3]);
+    }
+    const float inv = 1.f / sqrtf(block_total(ss, 1) * inv_h + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * NT * 4;
+      if (c >= H) continue;
+      float w[4];
+      if (c + 4 <= H) {
+        load4(w, a.weight + c);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j] = c + j < H ? a.weight[c + j] : 0.f;
       }
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / H + a.eps);
 #pragma unroll
-    for (int i = 0; i < NV; ++i)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = (i * kThreads + threadIdx.x) * 4 + j;
-        y[i][j] = c < H ? y[i][j] * inv * a.weight[c] : 0.f;
-      }
+      for (int j = 0; j < 4; ++j) y[i][j] *= inv * w[j];
+    }
   };
 
   const int64_t lo = (int64_t)blockIdx.x * a.rows_per_cta, hi = min(a.T, lo + a.rows_per_cta);
   float y[NV][4], prev[NV][4];
+  if (lo < hi) fetch(lo);
   for (int64_t t = lo; t < hi; ++t) {
     int64_t slot = -1, last = t;
-    bool first = false;
     if (sp != nullptr) {
       const int r = a.req_of_token[t];
-      first = t == a.qsl[r];
-      if (first) {
+      if (t == a.qsl[r]) {                       // first row of a request
         last = a.qsl[r + 1] - 1;
         slot = a.slots[r];
         if (slot >= a.num_slots) slot = -1;
         const bool carried = slot >= 0 && a.has_init[r];
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-          const int c = (i * kThreads + threadIdx.x) * 4;
+          const int c = c0 + i * NT * 4;
           prev[i][0] = prev[i][1] = prev[i][2] = prev[i][3] = 0.f;
           if (carried && c < ld) load4(prev[i], a.state + slot * ld + c);
         }
       } else if (t == lo) {
         row(t - 1, prev);
-        norm(prev);
+        norm(prev, -1);
       }
     }
-    row(t, y);
+    if constexpr (kAhead) fetched_row(y);
+    else row(t, y);
     if (a.x_out != nullptr) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        const int c = (i * kThreads + threadIdx.x) * 4;
+        const int c = c0 + i * NT * 4;
         if (c < ld) store4(a.x_out + t * ld + c, y[i]);
       }
     }
-    norm(y);
+    norm(y, kAhead && t + 1 < hi ? t + 1 : -1);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kThreads + threadIdx.x) * 4;
+      const int c = c0 + i * NT * 4;
       if (c >= ld) continue;
       store4(hp + t * ld + c, y[i]);
       if (sp == nullptr) continue;
@@ -182,14 +258,14 @@ __global__ void __launch_bounds__(kThreads) stream_layernorm_kernel(StreamNormAr
       store4(sp + t * ld + c, o);
     }
     if (sp == nullptr) continue;
-    if (slot >= 0) {          // first row of a request: its last row's norm becomes the state
+    if (slot >= 0) {          // its last row's norm becomes the request's state
       if (last > t) {
         row(last, prev);
-        norm(prev);
+        norm(prev, -1);
       }
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        const int c = (i * kThreads + threadIdx.x) * 4;
+        const int c = c0 + i * NT * 4;
         if (c < ld) store4(a.state + slot * ld + c, last > t ? prev[i] : y[i]);
       }
     }
@@ -200,11 +276,26 @@ __global__ void __launch_bounds__(kThreads) stream_layernorm_kernel(StreamNormAr
   }
 }
 
-template <typename T, int NV>
-void launch_stream(const StreamNormArgs& a, cudaStream_t st) {
+// Runs of rows: one wave of CTAs, each with an equal share.
+template <typename T, int NT, int NV>
+int launch_runs(StreamNormArgs a, cudaStream_t st) {
+  const int per_sm = 1024 / NT;
+  a.rows_per_cta = (int)max((int64_t)4, (a.T + 148 * per_sm - 1) / (148 * per_sm));
   const dim3 grid((unsigned)((a.T + a.rows_per_cta - 1) / a.rows_per_cta));
-  if (a.table != nullptr) launch_pdl(stream_layernorm_kernel<T, NV, true>, grid, dim3(kThreads), 0, st, a);
-  else launch_pdl(stream_layernorm_kernel<T, NV, false>, grid, dim3(kThreads), 0, st, a);
+  if (a.table != nullptr) return (int)launch_pdl(stream_layernorm_kernel<T, NT, NV, true, false>, grid, dim3(NT), 0, st, a);
+  const int smem = NT * NV * (16 + 16 * (int)sizeof(T));
+  const auto kern = stream_layernorm_kernel<T, NT, NV, false, true>;
+  const cudaError_t e = ensure_dynamic_smem((const void*)kern, smem);
+  if (e != cudaSuccess) return (int)e;
+  return (int)launch_pdl(kern, grid, dim3(NT), smem, st, a);
+}
+// A CTA per row.
+template <typename T, int NT, int NV>
+int launch_rows(StreamNormArgs a, cudaStream_t st) {
+  a.rows_per_cta = 1;
+  const dim3 grid((unsigned)a.T);
+  if (a.table != nullptr) return (int)launch_pdl(stream_layernorm_kernel<T, NT, NV, true, false>, grid, dim3(NT), 0, st, a);
+  return (int)launch_pdl(stream_layernorm_kernel<T, NT, NV, false, false>, grid, dim3(NT), 0, st, a);
 }
 
 }  // namespace
@@ -227,16 +318,23 @@ extern "C" int b200_stream_layernorm(const StreamNormArgs* args, int dtype, cuda
   if (a.T == 0) return 0;
   if (a.ld % 4 || a.width > a.ld || a.y1_stride % 4 || a.y2_stride % 4 || a.g1_stride % 4 || a.g2_stride % 4) return 3;
   if (a.x_out != nullptr && a.x_out == a.x_in) return 2;   // rows are read again by the CTA of the next row
-  // decode-sized batches: a CTA per row; long portions: runs of rows, so that few rows are computed twice
-  a.rows_per_cta = a.T <= 1024 ? 1 : 8;
-  const int need = (a.ld / 4 + kThreads - 1) / kThreads;
+  // few rows: a CTA of up to 1024 threads for each; long portions: small CTAs over runs of rows, so that few rows are
+  // computed twice
+  const int quads = a.ld / 4;
+  if (a.T <= 1024 || quads > 1024) {
+    B200_DISPATCH_DTYPE(dtype, {
+      if (quads <= 256) return launch_rows<T, 256, 1>(a, st);
+      if (quads <= 512) return launch_rows<T, 512, 1>(a, st);
+      if (quads <= 1024) return launch_rows<T, 1024, 1>(a, st);
+      if (quads <= 2048) return launch_rows<T, 1024, 2>(a, st);
+      if (quads <= 4096) return launch_rows<T, 1024, 4>(a, st);
+    });
+    return 3;
+  }
   B200_DISPATCH_DTYPE(dtype, {
-    if (need <= 1) launch_stream<T, 1>(a, st);
-    else if (need <= 2) launch_stream<T, 2>(a, st);
-    else if (need <= 4) launch_stream<T, 4>(a, st);
-    else if (need <= 8) launch_stream<T, 8>(a, st);
-    else if (need <= 16) launch_stream<T, 16>(a, st);
-    else return 3;
+    if (quads <= 256) return launch_runs<T, 256, 1>(a, st);
+    if (quads <= 512) return launch_runs<T, 256, 2>(a, st);
+    return launch_runs<T, 512, 2>(a, st);
   });
   return (int)cudaGetLastError();
 }

@@ -49,6 +49,11 @@ class ListedLayer(nn.Module):
             out.update({"mlp.gate": (ff, width), "mlp.up": (ff, width), "mlp.down": (width, ff)})
         return out
 
+    @classmethod
+    def unused_tensors(cls, spec: LayerSpec) -> tuple:
+        """Names that a checkpoint may carry without effect."""
+        return ()
+
     def state_spec(self, dtype) -> list:
         """``(shape per request, dtype)`` of everything the layer keeps per request, the mixer's first."""
         return self.mixer.state_spec(dtype) if self.mixer.has_state else []
@@ -153,11 +158,14 @@ class LayerListForCausalLM(DenseForCausalLM):
 
     def load_weights(self, weights: Iterable[tuple[str, torch.Tensor]]):
         want, outer = self.tensor_shapes(), self.outer_tensor_shapes()
+        unused = {f"l{i}.{k}" for i, spec in enumerate(self.cfg.layer_specs) for k in self.layer_cls.unused_tensors(spec)}
         loaded = set()
         for m in self.modules():
             if isinstance(m, GatedMLP):
                 m.set_act_fused(False)  # checkpoints carry the plain [gate | up] order
         for name, w in weights:
+            if name in unused:
+                continue
             if name not in want:
                 raise ValueError(f"unexpected tensor {name!r} in the checkpoint")
             if tuple(w.shape) != tuple(want[name]):

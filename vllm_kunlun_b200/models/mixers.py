@@ -372,7 +372,7 @@ class LatentAttention(nn.Module):
         self.D, self.R, self.V, self.C = self.TENSOR_CORE if self.tensor_cores else (D, R, V, align(C))
         self.row = align(self.C + self.R)
         self.in_proj = FusedProjection(width, {"dq": Q, "dkv": C + R, "g": H}, dtype, device)
-        self.uq = ReplicatedLinear(align(Q), H * (self.D + self.R), dtype=dtype, device=device)
+        self.uq = ReplicatedLinear(align(Q), align(H * (self.D + self.R)), dtype=dtype, device=device)
         self.up = ReplicatedLinear(self.C, H * (self.D + self.V), dtype=dtype, device=device)      # per head keys | values
         for lin in (self.uq, self.up):
             lin.weight.data.zero_()
@@ -396,7 +396,7 @@ class LatentAttention(nn.Module):
         if key in ("dq", "dkv", "g"):
             self.in_proj.load_part(key, w)
         elif key == "uq":
-            q, g = w.reshape(H, self.dim + self.rot_dim, -1), self.uq.weight.data.view(H, self.D + self.R, -1)
+            q, g = w.reshape(H, self.dim + self.rot_dim, -1), self.uq.weight.data[:H * (self.D + self.R)].view(H, self.D + self.R, -1)
             g[:, :self.dim, :self.q_rank].copy_(q[:, :self.dim])
             g[:, self.D:self.D + self.rot_dim, :self.q_rank].copy_(q[:, self.dim:])
         elif key in ("uk", "uv"):
@@ -452,7 +452,7 @@ class LatentAttention(nn.Module):
         g = p.slice(y, "g")
         cq = ops.latent_prep(p.slice(y, "dq"), p.slice(y, "dkv"), self.q_norm, self.kv_norm, table, cache, md.slot_mapping,
                              self.C, self.uq.in_features, self.eps)
-        q = self.uq(cq).view(T, H, self.D + self.R)
+        q = self.uq(cq)[:, :H * (self.D + self.R)].contiguous().view(T, H, self.D + self.R)
         out = _rows(T, H * self.V, h.dtype, h.device)
         nd = md.num_decodes if self.tensor_cores else md.num_reqs
         nt = md.num_decode_tokens if self.tensor_cores else T

@@ -48,6 +48,10 @@ class SeturaxDecoderLayer(ListedLayer):
             out.update({f"rg{k + 1}": (width, width), f"rg{k + 1}.b": (width,)})
         return out
 
+    @classmethod
+    def unused_tensors(cls, spec: LayerSpec) -> tuple:
+        return ("rg2", "rg2.b") if spec.mlp is None else ()       # the gate of a feed-forward that is not there
+
     def state_spec(self, dtype) -> list:
         return super().state_spec(dtype) + [((self.ld,), torch.float32)]
 
