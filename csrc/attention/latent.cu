@@ -49,10 +49,10 @@ template <typename T> __device__ __forceinline__ void put4(T* p, float a, float 
   *reinterpret_cast<Quad<T>*>(p) = Quad<T>{{from_f<T>(a), from_f<T>(b), from_f<T>(c), from_f<T>(d)}};
 }
 
-template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
+template <typename T, int NT>
+__global__ void __launch_bounds__(NT) latent_prep_kernel(LatentPrepArgs a) {
   extern __shared__ __align__(16) float sv[];          // [Q query latent | C + R key / value latent and shared key part]
-  __shared__ float red[2][4];
+  __shared__ float red[2][NT / 32];
   griddep_launch();
   griddep_wait();
   const int64_t t = blockIdx.x;
@@ -62,27 +62,29 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
   float sq = 0.f, sc = 0.f;
   if (a.vec) {
 #pragma unroll 4
-    for (int i = tid * 4; i < Q; i += 512) {
+    for (int i = tid * 4; i < Q; i += 4 * NT) {
       const float4 f = get4(q + i);
       *reinterpret_cast<float4*>(sv + i) = f;
       sq += (f.x * f.x + f.y * f.y) + (f.z * f.z + f.w * f.w);
     }
 #pragma unroll 2
-    for (int i = tid * 4; i < C + R; i += 512) {
+    for (int i = tid * 4; i < C + R; i += 4 * NT) {
       const float4 f = get4(kv + i);
       *reinterpret_cast<float4*>(sv + Q + i) = f;
       if (i < C) sc += (f.x * f.x + f.y * f.y) + (f.z * f.z + f.w * f.w);
     }
   } else {
-    for (int i = tid; i < Q; i += 128) { const float f = to_f(q[i]); sv[i] = f; sq += f * f; }
-    for (int i = tid; i < C + R; i += 128) { const float f = to_f(kv[i]); sv[Q + i] = f; if (i < C) sc += f * f; }
+    for (int i = tid; i < Q; i += NT) { const float f = to_f(q[i]); sv[i] = f; sq += f * f; }
+    for (int i = tid; i < C + R; i += NT) { const float f = to_f(kv[i]); sv[Q + i] = f; if (i < C) sc += f * f; }
   }
   sq = warp_sum(sq);
   sc = warp_sum(sc);
   if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sc; }
   __syncthreads();
-  const float iq = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / Q + a.eps);
-  const float ic = 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / C + a.eps);
+  sq = sc = 0.f;
+#pragma unroll
+  for (int w = 0; w < NT / 32; ++w) { sq += red[0][w]; sc += red[1][w]; }
+  const float iq = 1.f / sqrtf(sq / Q + a.eps), ic = 1.f / sqrtf(sc / C + a.eps);
   T* qo = reinterpret_cast<T*>(a.q_out) + t * a.q_out_stride;
   const int64_t slot = a.slots[t];
   const bool store = slot >= 0 && slot < a.total_slots;
@@ -100,19 +102,19 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
       const float4 u = *reinterpret_cast<const float4*>(x), v = *reinterpret_cast<const float4*>(w);
       put4(dst, u.x * inv * v.x, u.y * inv * v.y, u.z * inv * v.z, u.w * inv * v.w);
     };
-    for (int i = tid * 4; i < a.q_out_stride; i += 512) {
+    for (int i = tid * 4; i < a.q_out_stride; i += 4 * NT) {
       if (i < Q) scaled(sv + i, iq, a.q_norm + i, qo + i);
       else put4(qo + i, 0.f, 0.f, 0.f, 0.f);
     }
     if (store)
-      for (int i = tid * 4; i < a.row; i += 512) {
+      for (int i = tid * 4; i < a.row; i += 4 * NT) {
         if (i < C) scaled(sv + Q + i, ic, a.kv_norm + i, co + i);
         else put4(co + i, cached(i), cached(i + 1), cached(i + 2), cached(i + 3));
       }
   } else {
-    for (int i = tid; i < a.q_out_stride; i += 128) qo[i] = from_f<T>(i < Q ? sv[i] * iq * a.q_norm[i] : 0.f);
+    for (int i = tid; i < a.q_out_stride; i += NT) qo[i] = from_f<T>(i < Q ? sv[i] * iq * a.q_norm[i] : 0.f);
     if (store)
-      for (int i = tid; i < a.row; i += 128) co[i] = from_f<T>(cached(i));
+      for (int i = tid; i < a.row; i += NT) co[i] = from_f<T>(cached(i));
   }
 }
 
@@ -391,7 +393,11 @@ extern "C" int b200_latent_prep(const LatentPrepArgs* args, int64_t T_, int dtyp
   if (smem > 46 * 1024) return 3;
   a.vec = a.q_rank % 4 == 0 && a.kv_rank % 4 == 0 && a.rot_dim % 4 == 0 && a.stride % 4 == 0 && a.q_out_stride % 4 == 0 &&
           a.row % 4 == 0 && a.rot_off % 4 == 0 && ((uintptr_t)a.q_norm | (uintptr_t)a.kv_norm | (uintptr_t)a.q_down | (uintptr_t)a.kv_down | (uintptr_t)a.q_out | (uintptr_t)a.cache) % 16 == 0;
-  B200_DISPATCH_DTYPE(dtype, launch_pdl(latent_prep_kernel<T>, dim3((unsigned)T_), dim3(128), smem, st, a));
+  // few tokens: more threads each, for a short chain; many tokens: more of them at once
+  B200_DISPATCH_DTYPE(dtype, {
+    if (T_ <= 256) launch_pdl(latent_prep_kernel<T, 512>, dim3((unsigned)T_), dim3(512), smem, st, a);
+    else launch_pdl(latent_prep_kernel<T, 128>, dim3((unsigned)T_), dim3(128), smem, st, a);
+  });
   return (int)cudaGetLastError();
 }
 
