@@ -99,7 +99,7 @@ typedef struct GroupedGemmArgs {
   int M, N, K, E, ldo, a_stride;
   int fp8;               // 1 = e4m3 inputs
   int fmt;               // 16-bit inputs: 1 = bf16, 0 = fp16
-  int out_fmt;           // 1 = bf16, 0 = fp16
+  int out_fmt;           // 1 = bf16, 0 = fp16, 2 = fp32 (16-bit inputs, no bias)
   int bn;                // token tile 16 / 32 / 64 / 128
   int grid;
 } GroupedGemmArgs;
@@ -123,7 +123,7 @@ int b200_rmsnorm(void* out, const void* x, void* residual, const void* w, int64_
                  int64_t x_stride, int64_t out_stride, int dtype, cudaStream_t st);
 int b200_rownorm(void* out, const void* x, const void* z, const void* w, int64_t rows, int D, float eps, int mode,
                  int dtype, cudaStream_t st);
-int b200_act_and_mul(void* out, const void* x, int64_t rows, int d, int act, int dtype, cudaStream_t st);
+int b200_act_and_mul(void* out, const void* x, int64_t rows, int d, int act, float limit, int dtype, cudaStream_t st);
 int b200_quick_gelu(void* out, const void* x, int64_t n, int dtype, cudaStream_t st);
 int b200_embedding(void* out, const int64_t* ids, const void* w, int64_t T, int H, int64_t rows, int64_t vocab_start,
                    int dtype, cudaStream_t st);
@@ -173,7 +173,8 @@ int b200_decode_attention_umma(void* out, const void* q, const void* tmap, const
                                const int* seq_lens, const int* qsl, const float* sinks, float* ws_o, float* ws_lse,
                                int* status, int64_t T, int B, int Hq, int Hkv, int D, int block_size, int max_blocks,
                                int64_t num_blocks, int max_query_len, int num_splits, int window, float scale,
-                               int early_meta, int dtype, cudaStream_t st);
+                               int early_meta, const float* bias, int bias_len, const void* gate, int64_t gate_stride,
+                               int dtype, cudaStream_t st);
 
 // Dense paged MLA decode on tcgen05 (attention/mla_decode_umma.cu): cache blocks of 64 tokens, at most 32 query
 // tokens per request.  `tmap`: the cache as a 2-D [blocks * 64, 576] 16-bit tensor, 64 x 64 boxes, 128-byte swizzle.
@@ -187,7 +188,8 @@ int b200_mla_decode_max_clusters(int R, int S, int dtype);
 int b200_prefill_attention_umma(void* out, float* lse, const void* tmQ, const void* tmKV, const int* block_tables,
                                 const int* seq_lens, const int* qsl, const float* sinks, int* status, int B, int Hq, int Hkv,
                                 int D, int block_size, int max_blocks, int64_t num_blocks, int max_query_len, int window,
-                                float scale, int dtype, unsigned long long* trace, cudaStream_t st);
+                                float scale, const float* bias, int bias_len, const void* gate, int64_t gate_stride,
+                                int dtype, unsigned long long* trace, cudaStream_t st);
 int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, const void* tmKV, const void* tmKpe, const int* kv_starts,
                           const int* kv_lens, const int* qsl, const float* sinks, const void* gate, int64_t gate_stride,
                           int* status, int B, int Hq, int max_query_len, int causal, int window, float scale, int dtype,
@@ -220,8 +222,8 @@ int b200_topk_rows(int* out, const float* logits, const int* row_len, int64_t ro
 int b200_moe_route(float* out_w, int* out_ids, const void* logits, const float* bias, int64_t T, int E, int k, int mode,
                    int renorm, int n_group, int topk_group, float scale, int64_t stride, int dtype, cudaStream_t st);
 int b200_moe_permute(void* x_sorted, int* pos_of_pair, int* lod, int* counts, int* cursor, const void* x, const int* ids,
-                     const int* emap, int64_t T, int k, int H, int E_local, int E_global, int64_t x_stride,
-                     int64_t max_rows, int dtype, cudaStream_t st);
+                     const int* emap, const float* factors, int64_t T, int k, int H, int E_local, int E_global,
+                     int64_t x_stride, int64_t max_rows, int dtype, cudaStream_t st);  // factors [T][k] (or null): times the rows
 int b200_moe_unpermute(void* out, const void* y_sorted, const int* pos_of_pair, const float* w, int64_t T, int k, int H,
                        int dtype, cudaStream_t st);
 int b200_router_gemm_small(float* out, const void* x, int64_t x_stride, const void* w, const void* bias,
@@ -231,8 +233,8 @@ int b200_router_route_small(float* out_w, int* out_ids, const void* x, int64_t x
                             int renorm, int n_group, int topk_group, float scale, int dtype, cudaStream_t st);
 int b200_moe_small_pairs();
 int b200_moe_prepare_small(void* x_sorted, float* scale_t, int64_t s_stride, int* pos_of_pair, int* lod,
-                           const void* x, const int* ids, const int* emap, int64_t T_, int k, int H, int E_local,
-                           int E_global, int64_t x_stride, int quant, int dtype, cudaStream_t st);
+                           const void* x, const int* ids, const int* emap, const float* factors, int64_t T_, int k,
+                           int H, int E_local, int E_global, int64_t x_stride, int quant, int dtype, cudaStream_t st);
 int b200_act_mul_quant_fp8(void* q, float* scale_t, const void* h, int64_t rows, int I, int64_t s_stride, int act,
                            const int* rows_valid_ptr, int dtype, cudaStream_t st);
 int b200_quant_fp8_group(void* q, float* scale_t, const void* x, int64_t rows, int K, int64_t x_stride, int64_t s_stride,
@@ -288,9 +290,24 @@ int b200_qk_unit_norm_cache(void* q_out, const void* q, const void* k, const voi
                             const int64_t* slots, int64_t T, int Hq, int Hkv, int D, int Dv, int Dc, int block_size,
                             int64_t num_blocks, float eps, int dtype, cudaStream_t st);
 
+// ---- norms before and after every sublayer, polynomial activation, value-normed attention split (elementwise/sandwich.cu) ----
+int b200_embed_rmsnorm(float* x, void* h, const int64_t* ids, const void* table, const float* w, int64_t T, int H, int ld,
+                       int64_t rows, float eps, int dtype, cudaStream_t st);
+// pos [T][k] (or null): rows of y that add up to a token's
+int b200_sandwich_rmsnorm(float* x, void* h, const void* y, int64_t y_stride, const int* pos, int k, const float* w_post,
+                          const float* w_pre, int64_t T, int H, int ld, float eps, int dtype, cudaStream_t st);
+int b200_poly_norm(void* out, int64_t ldo, const void* z, int64_t ldz, const float* coeff, int64_t T, int F, int ld, float eps,
+                   int dtype, cudaStream_t st);
+int b200_attn_prep_cache(void* q_out, const void* q, const void* k, const void* v, int64_t stride, void* kv_cache,
+                         const int64_t* slots, const int64_t* positions, void* v_out, const void* v_in, float share,
+                         float temp_coef, int64_t temp_every, int64_t T, int Hq, int Hkv, int D, int Dv, int Dc,
+                         int block_size, int64_t num_blocks, float eps, int dtype, cudaStream_t st);
+
 // ---- fp32 GEMM on the CUDA cores (gemm/gemm_f32.cu): out[T, N] = x[T, K] . w[N, K]^T (+ bias) -----------------
 int b200_gemm_f32(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, int64_t ldw, const float* bias,
                   int64_t T, int N, int K, cudaStream_t st);
+int b200_gemm_f32_grouped(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, const int* lod, int64_t M,
+                          int E, int N, int K, cudaStream_t st);
 
 // ---- latent attention of any size (attention/latent.cu) --------------------------------------------------
 typedef struct LatentPrepArgs {
@@ -340,7 +357,8 @@ int b200_bigram_rows(int64_t* rows, const int64_t* ids, int64_t* state, const in
 int b200_paged_attention_generic(void* out, const void* q, const void* kv_cache, const int* block_tables,
                                  const int* seq_lens, const int* qsl, const float* sinks, int64_t T, int B, int Hq,
                                  int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks, int latent_dv,
-                                 int window, float scale, int dtype, cudaStream_t st);
+                                 int window, float scale, const float* bias, int bias_len, const void* gate,
+                                 int64_t gate_stride, int dtype, cudaStream_t st);
 
 // ---- gated delta net / conv / MTP glue --------------------------------------------------------
 int b200_causal_conv1d_fwd(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w,
@@ -360,9 +378,10 @@ int b200_gdn_recurrent(void* out, int64_t o_stride, const void* q, const void* k
 typedef struct RecurrenceArgs {
   float* out;                // [T][H][Dv], rows out_stride apart
   const void *q, *k, *v;     // raw (kind 1) or convolved (kind 0) projections, rows qkv_stride apart
-  const void *a, *b;         // kind 0: raw decay [T][H][Dk] and step-size [T][H] projections
-  const float *A_log, *dt_bias;  // kind 0: [H], [H][Dk]
+  const void *a, *b;         // kind 0: raw decay [T][H][Dk] and step-size [T][H] projections; kind 2: a = raw forget gates
+  const float *A_log, *dt_bias;  // kind 0: [H], [H][Dk]; kind 2: dt_bias = bias of the forget gates
   const float* decay;        // kind 1: [H]
+  const float* lower;        // kind 2: [H][Dk] lower bound of the forget gates
   float* states;             // [slots][H][Dv][Dks]
   const int *cu, *slots, *has_init;
   int64_t out_stride, qkv_stride, a_stride, b_stride;
@@ -372,6 +391,7 @@ typedef struct RecurrenceArgs {
 } RecurrenceArgs;
 int b200_linear_recurrence(const RecurrenceArgs* a, int dtype, cudaStream_t st);
 int b200_chunk_decay(const RecurrenceArgs* a, int dtype, cudaStream_t st);  // kind 1, prompt portions (linear_attn/chunk_decay.cu)
+int b200_chunk_gated_write(const RecurrenceArgs* a, int dtype, cudaStream_t st);  // kind 2, prompt portions (linear_attn/chunk_gated.cu)
 int b200_sigmoid_gate_mul(void* out, const void* o, const void* gate, int64_t gate_stride, int D, int64_t T_,
                           int dtype, cudaStream_t st);
 int b200_mtp_concat_norm(void* out, const void* embed, const void* hidden, const void* we, const void* wh,

@@ -48,8 +48,12 @@ struct Params {
   const int* seq_lens;
   const int* qsl;
   const float* sinks;
+  const float* bias;        // [Hq][bias_len] score bias by distance (position of the query minus the key's), or null; the last
+                            // entry serves every farther distance
+  const void* gate;         // [T, >= Hq] raw output gates in the output's type, or null
+  int64_t gate_stride;
   int* status;
-  int Hq, Hkv, block_size, max_blocks, num_splits, window, num_stages;
+  int Hq, Hkv, block_size, max_blocks, num_splits, window, num_stages, bias_len;
   int early_meta;           // lengths / block table were written long before this launch: read them, and fetch
                             // old-context tiles, before the programmatic-dependency wait
   int64_t num_blocks, T;
@@ -90,7 +94,7 @@ template <> __device__ __forceinline__ uint16_t to_bits16<__half>(float v) { ret
 // maximum exceeds it by more than kMaxSlack (in log2 units), so p = exp2(s - m_used) stays below 2^kMaxSlack and the
 // result O / l is unchanged; in the common case O^T needs no rescale and the softmax warps never wait for the
 // previous P.V to finish - they run ahead into a second P buffer while the tensor core works.
-template <typename T, int D, int NR>
+template <typename T, int D, int NR, bool kBias>
 __global__ void __launch_bounds__(kThreads)
 decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_constant__ Params p) {
   constexpr int KB = D / 64;                       // 64-dim blocks
@@ -321,7 +325,20 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       l_part[r] = 0.f;
       pos[r] = (r < rows_total) ? ctx + r / g : -1;  // position of the row's query token (-1: padded row)
     }
+    const float* bias[kBias ? NR : 1];
+    float far_bias[kBias ? NR : 1];
+    if constexpr (kBias) {
+#pragma unroll
+      for (int r = 0; r < NR; ++r) {
+        bias[r] = p.bias + (int64_t)(kvh * g + (r < rows_total ? r % g : 0)) * p.bias_len;
+        far_bias[r] = bias[r][p.bias_len - 1] * 1.4426950408889634f;
+      }
+    }
     const int pos_min = ctx, pos_max = ctx + max(q_len, 1) - 1;
+    auto gate_of = [&](int tok, int hh) {
+      const float z = to_float<T>(reinterpret_cast<const T*>(p.gate)[(int64_t)tok * p.gate_stride + hh]);
+      return 1.f / (1.f + __expf(-z));
+    };
     // byte offset of this key's column in a P buffer row
     const int p_off = (lane_id >> 6) * (kRows * 128) + (lane_id & 7) * 2;
     const int p_ch = (lane_id & 63) >> 3;
@@ -347,11 +364,15 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       const int key = key0 + lane_id;
       const bool full = key0 + kTileKeys - 1 <= pos_min && key0 + kTileKeys <= kv_end &&
                         (p.window <= 0 || key0 > pos_max - p.window);
+      // nearest distance of the tile: beyond the table's last entry the bias is one constant per row
+      const bool near_tile = kBias && pos_min - (key0 + kTileKeys - 1) < p.bias_len - 1;
       float sc[NR];
       bool need = fail;   // does any score exceed its row's reference maximum by more than the slack?
 #pragma unroll
       for (int r = 0; r < NR; ++r) {
         float v = __uint_as_float(sr[r]) * p.scale_log2;
+        if constexpr (kBias)
+          v += near_tile ? bias[r][min(max(pos[r] - key, 0), p.bias_len - 1)] * 1.4426950408889634f : far_bias[r];
         if (!full) {
           const bool in = key < kv_end && key <= pos[r] && (p.window <= 0 || key > pos[r] - p.window);
           v = in ? v : -INFINITY;
@@ -450,6 +471,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       float den = L;
       if (p.num_splits == 1 && p.sinks != nullptr && r < rows_total) den += exp2f(p.sinks[hh] * 1.4426950408889634f - Ms);
       sInv[r] = (ok && den > 0.f) ? 1.f / den : 0.f;
+      if (p.num_splits == 1 && p.gate != nullptr && r < rows_total) sInv[r] *= gate_of(qs + r / g, hh);
       sRow[r] = orow;
       if (p.num_splits > 1 && r < rows_total)
         p.ws_lse[(int64_t)split * p.T * p.Hq + orow] = (ok && L > 0.f) ? Ms + log2f(L) : -INFINITY;
@@ -514,7 +536,8 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
             sW[s2 * kRows + r] = w;
           }
           if (p.sinks != nullptr) den += exp2f(p.sinks[kvh * g + r % g] * 1.4426950408889634f - Ms);
-          const float inv = den > 0.f ? 1.f / den : 0.f;
+          float inv = den > 0.f ? 1.f / den : 0.f;
+          if (p.gate != nullptr) inv *= gate_of(qs + r / g, kvh * g + r % g);
           for (int s2 = 0; s2 < S; ++s2) sW[s2 * kRows + r] *= inv;
         }
         named_bar_sync(1, 128);
@@ -554,10 +577,10 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   }
 }
 
-template <typename T, int NR>
+template <typename T, int NR, bool kBias>
 static int launch_nr(const Params& p0, const CUtensorMap& tm, int B, cudaStream_t st) {
   constexpr int D = 128;
-  auto kern = decode_umma_kernel<T, D, NR>;
+  auto kern = decode_umma_kernel<T, D, NR, kBias>;
   Params p = p0;
   constexpr int kStageBytes = 2 * (D / 64) * kTileKeys * 128;
   p.num_stages = 3;
@@ -571,9 +594,14 @@ static int launch_nr(const Params& p0, const CUtensorMap& tm, int B, cudaStream_
 
 template <typename T>
 static int launch(const Params& p, const CUtensorMap& tm, int B, int max_rows, cudaStream_t st) {
-  if (max_rows <= 4) return launch_nr<T, 4>(p, tm, B, st);
-  if (max_rows <= 8) return launch_nr<T, 8>(p, tm, B, st);
-  return launch_nr<T, 16>(p, tm, B, st);
+  if (p.bias != nullptr) {
+    if (max_rows <= 4) return launch_nr<T, 4, true>(p, tm, B, st);
+    if (max_rows <= 8) return launch_nr<T, 8, true>(p, tm, B, st);
+    return launch_nr<T, 16, true>(p, tm, B, st);
+  }
+  if (max_rows <= 4) return launch_nr<T, 4, false>(p, tm, B, st);
+  if (max_rows <= 8) return launch_nr<T, 8, false>(p, tm, B, st);
+  return launch_nr<T, 16, false>(p, tm, B, st);
 }
 
 }  // namespace dattn
@@ -586,7 +614,8 @@ extern "C" int b200_decode_attention_umma(void* out, const void* q, const void* 
                                           const int* seq_lens, const int* qsl, const float* sinks, float* ws_o,
                                           float* ws_lse, int* status, int64_t T_, int B, int Hq, int Hkv, int D,
                                           int block_size, int max_blocks, int64_t num_blocks, int max_query_len,
-                                          int num_splits, int window, float scale, int early_meta, int dtype,
+                                          int num_splits, int window, float scale, int early_meta, const float* bias,
+                                          int bias_len, const void* gate, int64_t gate_stride, int dtype,
                                           cudaStream_t st) {
   using namespace b200;
   if (B == 0 || T_ == 0) return 0;
@@ -601,6 +630,8 @@ extern "C" int b200_decode_attention_umma(void* out, const void* q, const void* 
   p.scale_log2 = scale * 1.4426950408889634f;
   p.num_stages = 3;
   p.early_meta = early_meta;
+  p.bias = bias; p.bias_len = bias_len; p.gate = gate; p.gate_stride = gate_stride;
+  if (bias != nullptr && bias_len < 1) return 2;
   const CUtensorMap& tm = *reinterpret_cast<const CUtensorMap*>(tmap);
   const int max_rows = max_query_len * (Hq / Hkv);
   if (dtype == 1) return dattn::launch<__nv_bfloat16>(p, tm, B, max_rows, st);

@@ -1,4 +1,5 @@
-// Paged attention for any head size and for fp32 models: causal, optional sliding window, optional sinks; over keys and
+// Paged attention for any head size and for fp32 models: causal, optional sliding window, sinks, score
+// bias by distance and output gates; over keys and
 // values [block][2][head][slot][D], or over latent rows [block][slot][D] that all heads share and whose first `latent_dv`
 // columns are the values (absorbed multi-head latent attention).  The
 // tensor-core kernels (prefill_umma.cu, decode_umma.cu, paged_attention.cu, paged_decode.cu) serve 16-bit heads of 64,
@@ -20,8 +21,8 @@ constexpr int kGenWarps = 4;
 template <typename T, int ND>  // ND: value dims per lane, Dv <= 32 ND
 __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel(
     T* out, const T* q, const T* cache, const int* block_tables,
-    const int* seq_lens, const int* qsl, const float* sinks, int B, int Hq, int Hkv,
-    int D, int Dv, int latent, int block_size, int max_blocks, int64_t num_blocks, int window, float scale) {
+    const int* seq_lens, const int* qsl, const float* sinks, const float* bias, int bias_len, const T* gate,
+    int64_t gate_stride, int B, int Hq, int Hkv, int D, int Dv, int latent, int block_size, int max_blocks, int64_t num_blocks, int window, float scale) {
   extern __shared__ float sm_gen[];
   float* sq = sm_gen;                       // [D]
   float* so = sq + D;                       // [kGenWarps][Dv]
@@ -64,6 +65,7 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
       for (; d + 1 < D; d += 2) { a0 += sq[d] * to_f(kr[d]); a1 += sq[d + 1] * to_f(kr[d + 1]); }
       if (d < D) a0 += sq[d] * to_f(kr[d]);
       s = a0 + a1;
+      if (bias != nullptr) s += bias[(int64_t)h * bias_len + min(pos - key, bias_len - 1)];
     }
     const float mn = fmaxf(m, warp_max(s));
     if (mn == -INFINITY) continue;
@@ -95,7 +97,8 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
   float den = sinks != nullptr ? expf(sinks[h] - M) : 0.f, wg[kGenWarps];
 #pragma unroll
   for (int w = 0; w < kGenWarps; ++w) { wg[w] = expf(sml[w * 2] - M); den += sml[w * 2 + 1] * wg[w]; }
-  const float inv = den > 0.f ? 1.f / den : 0.f;
+  float inv = den > 0.f ? 1.f / den : 0.f;
+  if (gate != nullptr) inv /= 1.f + expf(-to_f(gate[(int64_t)t * gate_stride + h]));
   for (int d = tid; d < Dv; d += kGenWarps * 32) {
     float a = 0.f;
 #pragma unroll
@@ -110,18 +113,21 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
 extern "C" int b200_paged_attention_generic(void* out, const void* q, const void* kv_cache, const int* block_tables,
                                             const int* seq_lens, const int* qsl, const float* sinks, int64_t T_, int B,
                                             int Hq, int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks,
-                                            int latent_dv, int window, float scale, int dtype, cudaStream_t st) {
+                                            int latent_dv, int window, float scale, const float* bias, int bias_len,
+                                            const void* gate, int64_t gate_stride, int dtype, cudaStream_t st) {
   using namespace b200;
   const int Dv = latent_dv > 0 ? latent_dv : D;
   if (B == 0 || T_ == 0) return 0;
-  if (Hq % Hkv || Hq > 65535 || window < 0 || Dv > D || (latent_dv > 0 && Hkv != 1)) return 2;
+  if (Hq % Hkv || Hq > 65535 || window < 0 || Dv > D || (latent_dv > 0 && Hkv != 1) ||
+      (bias != nullptr && bias_len < 1))
+    return 2;
   const size_t smem = (size_t)(D + kGenWarps * (Dv + 2)) * sizeof(float);
   if (smem > 48 * 1024) return 3;
   dim3 grid((unsigned)T_, Hq);
 #define B200_GEN_ATTN(ND)                                                                                                \
   B200_DISPATCH_DTYPE(dtype, launch_pdl(paged_attention_generic_kernel<T, ND>, grid, dim3(kGenWarps * 32), smem, st,        \
-                                       (T*)out, (const T*)q, (const T*)kv_cache, block_tables, seq_lens, qsl, sinks, B, Hq, \
-                                       Hkv, D, Dv, latent_dv > 0, block_size, max_blocks, num_blocks, window, scale))
+                                       (T*)out, (const T*)q, (const T*)kv_cache, block_tables, seq_lens, qsl, sinks, bias,  \
+                                       bias_len, (const T*)gate, gate_stride, B, Hq, Hkv, D, Dv, latent_dv > 0, block_size, max_blocks, num_blocks, window, scale))
   if (Dv <= 64) { B200_GEN_ATTN(2); }
   else if (Dv <= 128) { B200_GEN_ATTN(4); }
   else if (Dv <= 256) { B200_GEN_ATTN(8); }

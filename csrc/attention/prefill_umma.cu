@@ -13,13 +13,16 @@
 // current one are issued as they become ready), warps 2-5 softmax + epilogue.  Two S buffers (2 x 128 TMEM columns)
 // + O (128 columns).  Causal masking by position (chunked prefill: row r of the request sits at ctx + r), optional
 // sliding window and attention sinks, optional log-sum-exp output.
+// `kBias`: a score bias per head and distance (query position minus key position) from a table [Hq][bias_len], whose last
+// entry serves every farther distance.  A tile that lies farther away altogether adds that constant inside the exponent; for
+// a nearer one the softmax warps put the 255 entries the tile can meet into shared memory (two buffers, one per tile parity).
 // The MLA instantiation (`kMla`) is the compute-friendly prefill form of multi-head latent attention
 // (v1/attention/backends/mla/common.py:1782-1843): 192-dim q / k (128 "nope" dims per head + 64 rotary dims shared
 // by all heads), 128-dim v, keys and values read as contiguous rows of the up-projected `kv_b_proj` output
 // ([rows, heads * 256], k_nope | v per head) plus the rotary key rows ([rows, 64]); each request's keys start at
 // `kv_starts[req]`.  Causal (new tokens, possibly behind cached ones in front of the same rows; window and sinks as
-// above) or not (a chunk of cached context); the log-sum-exp output lets the caller merge chunks.  Optionally every head's
-// output is multiplied by sigmoid(gate[token, head]).  Its K ring has two 48 KB stages and V a single 32 KB one (208 KB of shared memory in all).
+// above) or not (a chunk of cached context); the log-sum-exp output lets the caller merge chunks.  Its K ring has two 48 KB stages and V a single 32 KB one (208 KB of shared memory in all).
+// In both forms every head's output may be multiplied by sigmoid(gate[token, head]).
 // TMA loads carry no cluster multicast.  Every wait is bounded; on time-out the status word is set and the CTA unwinds.
 #include <cuda.h>
 #include <cuda_bf16.h>
@@ -44,6 +47,7 @@ template <bool kMla> struct Cfg {
   static constexpr int kKBytes = kQBlocks * kHalfBytes;         // Q tile or one K stage
   static constexpr int kVStages = kMla ? 1 : 2;
   static constexpr size_t kSmem = 1024 + (size_t)kStages * kKBytes + (size_t)kVStages * kOpBytes + kKBytes + kOpBytes + 256;
+  static constexpr size_t kBiasSmem = 2 * 256 * sizeof(float);
 };
 constexpr int kTmemCols = 512;                 // 2 x 128 (S) + 128 (O)
 constexpr float kMaxSlack = 8.f;
@@ -56,11 +60,12 @@ struct Params {
   const int* qsl;
   const int* kv_starts;     // MLA form: first key row of each request in the contiguous K / V tensors
   const float* sinks;       // [Hq] or null
+  const float* bias;        // [Hq][bias_len] score bias by distance (kBias)
   const void* gate;         // [T, >= Hq] in the output's type, or null
   int64_t gate_stride;
   int* status;
   unsigned long long* trace;   // optional phase timestamps [CTA][24] (null = off)
-  int Hq, Hkv, block_size, max_blocks, window, causal;
+  int Hq, Hkv, block_size, max_blocks, window, causal, bias_len;
   int64_t num_blocks;
   float scale_log2;
 };
@@ -121,7 +126,7 @@ template <> __device__ __forceinline__ uint32_t pack2<__half>(float a, float b) 
   return (uint32_t)__half_as_ushort(__float2half(a)) | ((uint32_t)__half_as_ushort(__float2half(b)) << 16);
 }
 
-template <typename T, bool kMla>
+template <typename T, bool kMla, bool kBias>
 __global__ void __launch_bounds__(kThreads)
 prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                     const __grid_constant__ CUtensorMap tmKpe, const __grid_constant__ Params p) {
@@ -145,6 +150,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint64_t* v_empty = bars + 15;       // [2] P.V of the tile has been computed
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* sBias = reinterpret_cast<float*>(sP + kOpBytes + 256);   // [2][256] (kBias)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   Abort ab{p.status, abort_flag};
@@ -340,6 +346,9 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     const int pos = ctx + row0 + r;                    // position of this row's token
     float m_used = -INFINITY, l_sum = 0.f;
     bool fail = false;
+    constexpr float kLog2e = 1.4426950408889634f;
+    const float* bias = kBias ? p.bias + (int64_t)head * p.bias_len : nullptr;
+    const float far_bias = kBias ? bias[p.bias_len - 1] * kLog2e : 0.f;
     for (int i = 0; i < n_tiles; ++i) {
       const int buf = i & 1;
       if (!fail && !wait_or_abort(&s_full[buf], (i >> 1) & 1, ab, 805)) fail = true;
@@ -351,6 +360,17 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const int key0 = kv_begin + i * kKTile;
       const bool full_tile = key0 + kKTile - 1 <= pos_first && key0 + kKTile <= kv_end &&
                              (p.window <= 0 || key0 > pos_last - p.window);
+      // nearest distance of the tile: beyond the table's last entry its bias is one constant
+      const bool near_tile = kBias && pos_first - (key0 + kKTile - 1) < p.bias_len - 1;
+      if constexpr (kBias) {
+        if (near_tile) {   // entry d: distance pos_first - key0 - 127 + d
+          float* dst = sBias + (i & 1) * 256;
+          const int tid = threadIdx.x - 64, d0 = pos_first - key0 - (kKTile - 1);
+#pragma unroll
+          for (int d = 0; d < 256; d += 128) dst[tid + d] = bias[min(max(d0 + tid + d, 0), p.bias_len - 1)] * kLog2e;
+          asm volatile("bar.sync 3, 128;" ::: "memory");
+        }
+      }
       // ---- the whole row (128 scores) in one TMEM round trip: a tcgen05.ld + wait pair costs several hundred
       // nanoseconds whatever its width, so all four 32-column loads are issued before the single wait, and the
       // S buffer goes back to the tensor core at once
@@ -365,6 +385,16 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       // One warp per scheduler: nothing hides instruction latency but independent work inside the thread, so the
       // row maximum runs on four partial maxima and the exponentials in chunks of 32 with four partial sums; the
       // raw scores are masked in place and scaled inside the exponent (one FMA + one ex2 per element).
+      float sc = p.scale_log2, off = far_bias;     // exponent = raw score * sc + off - maximum
+      if constexpr (kBias) {
+        if (near_tile) {
+          const float* src = sBias + (i & 1) * 256 + (kKTile - 1) + r;
+#pragma unroll
+          for (int e = 0; e < kKTile; ++e) v[e] = __float_as_uint(fmaf(__uint_as_float(v[e]), p.scale_log2, src[-e]));
+          sc = 1.f;
+          off = 0.f;
+        }
+      }
       if (!full_tile) {
 #pragma unroll
         for (int e = 0; e < kKTile; ++e) {
@@ -379,7 +409,8 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
         for (int u = 0; u < 4; ++u) mx[u] = fmaxf(mx[u], __uint_as_float(v[e + u]));
       }
-      float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.scale_log2;   // scale > 0: max commutes
+      float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * sc;   // scale > 0: max commutes
+      if (kBias) tmax += off;
       if (!row_ok) tmax = -INFINITY;
       if (threadIdx.x == 64 && i == 4) trace_mark(p.trace, cta_id, 3);
       // ---- lazy running maximum; the rescale of O is warp-collective (TMEM access), so the warp decides together
@@ -406,7 +437,8 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
       // ---- exponentials, row sum and the P row (16-bit, K-major over keys, 16-byte chunks swizzled by row; keys
       // 8 q .. 8 q + 7 = chunk q % 8 of key block q / 8), 32 keys at a time
-      const float neg_ms = (m_used == -INFINITY || !row_ok) ? -INFINITY : -m_used;   // invalid rows: P = 0
+      float neg_ms = (m_used == -INFINITY || !row_ok) ? -INFINITY : -m_used;   // invalid rows: P = 0
+      if (kBias) neg_ms += off;
       float ls[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int c = 0; c < kKTile; c += 32) {
@@ -416,7 +448,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           float pe[4];
 #pragma unroll
           for (int u = 0; u < 4; ++u) {
-            pe[u] = ex2_approx(fmaf(__uint_as_float(v[c + e + u]), p.scale_log2, neg_ms));
+            pe[u] = ex2_approx(fmaf(__uint_as_float(v[c + e + u]), sc, neg_ms));
             ls[u] += pe[u];
           }
           pk[e / 2] = pack2<T>(pe[0], pe[1]);
@@ -484,11 +516,11 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
 }
 
-template <typename T, bool kMla>
+template <typename T, bool kMla, bool kBias>
 static int launch(const Params& p, const CUtensorMap& tmQ, const CUtensorMap& tmKV, const CUtensorMap& tmKpe, int B,
                   int max_query_len, cudaStream_t st) {
-  auto kern = prefill_umma_kernel<T, kMla>;
-  const size_t smem = Cfg<kMla>::kSmem;
+  auto kern = prefill_umma_kernel<T, kMla, kBias>;
+  const size_t smem = Cfg<kMla>::kSmem + (kBias ? Cfg<kMla>::kBiasSmem : 0);
   cudaError_t e = ensure_dynamic_smem((const void*)kern, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid((unsigned)((max_query_len + kQTile - 1) / kQTile), (unsigned)p.Hq, (unsigned)B);
@@ -500,24 +532,31 @@ static int launch(const Params& p, const CUtensorMap& tmQ, const CUtensorMap& tm
 
 // Paged GQA prefill attention on tcgen05 (head_dim 128, block_size a multiple of 64).  `tmQ`: q as a 2-D
 // [T, Hq * 128] 16-bit tensor with 64-column x 128-row boxes; `tmKV`: the cache as [rows, 128] with 64 x 64 boxes;
-// both with 128-byte swizzle.  Returns 3 for shapes it does not serve.
+// both with 128-byte swizzle.  `bias` [Hq][bias_len] (or null): score bias by distance, the last entry for all farther ones;
+// `gate` [T][>= Hq] (or null): raw output gates.  Returns 3 for shapes it does not serve.
 extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tmQ, const void* tmKV,
                                            const int* block_tables, const int* seq_lens, const int* qsl,
                                            const float* sinks, int* status, int B, int Hq, int Hkv, int D, int block_size,
                                            int max_blocks, int64_t num_blocks, int max_query_len, int window, float scale,
+                                           const float* bias, int bias_len, const void* gate, int64_t gate_stride,
                                            int dtype, unsigned long long* trace, cudaStream_t st) {
   using namespace b200;
   if (B == 0 || max_query_len <= 0) return 0;
+  if (bias != nullptr && bias_len < 1) return 2;
   if (D != 128 || Hq % Hkv || block_size % pattn::kPage || B > 65535 || Hq > 65535) return 3;
   pattn::Params p;
   p.out = out; p.lse = lse; p.block_tables = block_tables; p.seq_lens = seq_lens; p.qsl = qsl; p.sinks = sinks;
   p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.max_blocks = max_blocks; p.window = window;
   p.num_blocks = num_blocks; p.scale_log2 = scale * 1.4426950408889634f;
-  p.kv_starts = nullptr; p.causal = 1; p.gate = nullptr; p.gate_stride = 0;
+  p.kv_starts = nullptr; p.causal = 1; p.gate = gate; p.gate_stride = gate_stride; p.bias = bias; p.bias_len = bias_len;
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
-  if (dtype == 1) return pattn::launch<__nv_bfloat16, false>(p, q, kv, kv, B, max_query_len, st);
-  if (dtype == 2) return pattn::launch<__half, false>(p, q, kv, kv, B, max_query_len, st);
+  if (dtype == 1)
+    return bias != nullptr ? pattn::launch<__nv_bfloat16, false, true>(p, q, kv, kv, B, max_query_len, st)
+                           : pattn::launch<__nv_bfloat16, false, false>(p, q, kv, kv, B, max_query_len, st);
+  if (dtype == 2)
+    return bias != nullptr ? pattn::launch<__half, false, true>(p, q, kv, kv, B, max_query_len, st)
+                           : pattn::launch<__half, false, false>(p, q, kv, kv, B, max_query_len, st);
   return 3;
 }
 
@@ -538,13 +577,13 @@ extern "C" int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, con
   if (window < 0 || (window > 0 && !causal)) return 2;
   pattn::Params p;
   p.out = out; p.lse = lse; p.block_tables = nullptr; p.seq_lens = kv_lens; p.qsl = qsl; p.kv_starts = kv_starts;
-  p.sinks = sinks; p.gate = gate; p.gate_stride = gate_stride; p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hq; p.block_size = pattn::kPage;
+  p.sinks = sinks; p.bias = nullptr; p.bias_len = 0; p.gate = gate; p.gate_stride = gate_stride; p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hq; p.block_size = pattn::kPage;
   p.max_blocks = 0; p.window = window; p.causal = causal ? 1 : 0; p.num_blocks = 0;
   p.scale_log2 = scale * 1.4426950408889634f;
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
   const CUtensorMap& kpe = *reinterpret_cast<const CUtensorMap*>(tmKpe);
-  if (dtype == 1) return pattn::launch<__nv_bfloat16, true>(p, q, kv, kpe, B, max_query_len, st);
-  if (dtype == 2) return pattn::launch<__half, true>(p, q, kv, kpe, B, max_query_len, st);
+  if (dtype == 1) return pattn::launch<__nv_bfloat16, true, false>(p, q, kv, kpe, B, max_query_len, st);
+  if (dtype == 2) return pattn::launch<__half, true, false>(p, q, kv, kpe, B, max_query_len, st);
   return 3;
 }

@@ -609,7 +609,8 @@ void grouped_gemm(at::Tensor out, const at::Tensor& x, const at::Tensor& w, cons
   a.status = gs.status.data_ptr<int>();
   a.M = M; a.N = N; a.K = K; a.E = E; a.ldo = out.stride(0);
   a.a_stride = fp8 ? a_scale_t->stride(0) : 0;
-  a.fp8 = fp8; a.fmt = x.scalar_type() == at::kBFloat16 ? 1 : 0; a.out_fmt = out.scalar_type() == at::kBFloat16 ? 1 : 0;
+  a.fp8 = fp8; a.fmt = x.scalar_type() == at::kBFloat16 ? 1 : 0; a.out_fmt = out.scalar_type() == at::kBFloat16 ? 1 : out.scalar_type() == at::kFloat ? 2 : 0;
+  if (a.out_fmt == 2) TORCH_CHECK(!fp8 && !bias.has_value(), "fp32 output: 16-bit inputs, no bias");
   int b = (int)bn;
   if (b <= 0) {
     // rows per group decide the token tile: decode batches spread thin over many experts
@@ -640,10 +641,17 @@ std::vector<at::Tensor> moe_route(const at::Tensor& logits, const c10::optional<
   return {w, ids};
 }
 
+const float* factor_ptr(const c10::optional<at::Tensor>& f) { return f.has_value() ? f->data_ptr<float>() : nullptr; }
+void check_factors(const c10::optional<at::Tensor>& f, const at::Tensor& ids) {
+  if (f.has_value()) TORCH_CHECK(f->scalar_type() == at::kFloat && f->is_contiguous() && f->numel() == ids.numel());
+}
+
 // Returns x_sorted [T*k, H], pos_of_pair [T*k], lod [E_local + 1].  `state` = int32 [2 * E_local] zero-initialised
 // scratch (counts | cursor) owned by the caller.
 std::vector<at::Tensor> moe_permute(const at::Tensor& x, const at::Tensor& ids, const c10::optional<at::Tensor>& emap,
-                                    int64_t E_local, int64_t E_global, at::Tensor state, int64_t max_rows) {
+                                    int64_t E_local, int64_t E_global, at::Tensor state, int64_t max_rows,
+                                    const c10::optional<at::Tensor>& factors) {
+  check_factors(factors, ids);
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && ids.is_contiguous() && ids.scalar_type() == at::kInt);
   TORCH_CHECK(state.scalar_type() == at::kInt && state.numel() >= 2 * E_local);
   const int64_t T = x.size(0), k = ids.size(1), H = x.size(1);
@@ -653,8 +661,8 @@ std::vector<at::Tensor> moe_permute(const at::Tensor& x, const at::Tensor& ids, 
   auto lod = at::empty({E_local + 1}, ids.options());
   check(b200_moe_permute(xs.data_ptr(), pos.data_ptr<int>(), lod.data_ptr<int>(), state.data_ptr<int>(),
                          state.data_ptr<int>() + E_local, x.data_ptr(), ids.data_ptr<int>(),
-                         emap.has_value() ? emap->data_ptr<int>() : nullptr, T, k, H, E_local, E_global, x.stride(0),
-                         max_rows, dtype_code(x), stream()),
+                         emap.has_value() ? emap->data_ptr<int>() : nullptr, factor_ptr(factors), T, k, H, E_local, E_global,
+                         x.stride(0), max_rows, dtype_code(x), stream()),
         "moe_permute", 3);
   return {xs, pos, lod};
 }
@@ -687,7 +695,9 @@ at::Tensor router_gemm_small(const at::Tensor& x, const at::Tensor& w, const c10
 // Small-batch permute in one launch; with `quant` the rows are written as fp8 with transposed 1x128 scales.
 // Returns (x_sorted | q_sorted, pos_of_pair, lod, scale_t or empty).
 std::vector<at::Tensor> moe_prepare_small(const at::Tensor& x, const at::Tensor& ids, const c10::optional<at::Tensor>& emap,
-                                          int64_t E_local, int64_t E_global, bool quant) {
+                                          int64_t E_local, int64_t E_global, bool quant,
+                                          const c10::optional<at::Tensor>& factors) {
+  check_factors(factors, ids);
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && ids.is_contiguous() && ids.scalar_type() == at::kInt);
   const int64_t T = x.size(0), k = ids.size(1), H = x.size(1), M = T * k;
   TORCH_CHECK(M <= b200_moe_small_pairs() && M >= 1);
@@ -698,8 +708,8 @@ std::vector<at::Tensor> moe_prepare_small(const at::Tensor& x, const at::Tensor&
   auto st = quant ? at::empty({H / 128, stride}, x.options().dtype(at::kFloat)) : at::empty({0}, x.options().dtype(at::kFloat));
   check(b200_moe_prepare_small(xs.data_ptr(), quant ? st.data_ptr<float>() : nullptr, stride, pos.data_ptr<int>(),
                                lod.data_ptr<int>(), x.data_ptr(), ids.data_ptr<int>(),
-                               emap.has_value() ? emap->data_ptr<int>() : nullptr, T, k, H, E_local, E_global, x.stride(0),
-                               quant, dtype_code(x), stream()), "moe_prepare_small");
+                               emap.has_value() ? emap->data_ptr<int>() : nullptr, factor_ptr(factors), T, k, H, E_local,
+                               E_global, x.stride(0), quant, dtype_code(x), stream()), "moe_prepare_small");
   return {xs, pos, lod, st};
 }
 
@@ -762,11 +772,11 @@ void rownorm(at::Tensor out, const at::Tensor& x, const c10::optional<at::Tensor
   check(b200_rownorm(out.data_ptr(), x.data_ptr(), opt_ptr(z), opt_ptr(w), x.numel() / D, D, (float)eps, (int)mode,
                      dtype_code(x), stream()), "rownorm");
 }
-void act_and_mul(at::Tensor out, const at::Tensor& x, int64_t act) {
+void act_and_mul(at::Tensor out, const at::Tensor& x, int64_t act, double limit) {
   int d = x.size(-1) / 2;
   TORCH_CHECK(x.is_contiguous() && out.is_contiguous());
-  check(b200_act_and_mul(out.data_ptr(), x.data_ptr(), x.numel() / (2 * d), d, (int)act, dtype_code(x), stream()),
-        "act_and_mul");
+  check(b200_act_and_mul(out.data_ptr(), x.data_ptr(), x.numel() / (2 * d), d, (int)act, (float)limit, dtype_code(x),
+                         stream()), "act_and_mul");
 }
 void quick_gelu(at::Tensor out, const at::Tensor& x) {
   TORCH_CHECK(x.is_contiguous());
@@ -940,13 +950,28 @@ void paged_attention(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_c
         "paged_attention", num_splits > 1 ? 2 : 1);
 }
 
+// score bias by distance [Hq, len] fp32 and raw output gates [T, Hq] of an attention call
+void check_bias_gate(const at::Tensor& q, const c10::optional<at::Tensor>& bias, const c10::optional<at::Tensor>& gate) {
+  if (bias.has_value())
+    TORCH_CHECK(bias->dim() == 2 && bias->scalar_type() == at::kFloat && bias->is_contiguous() && bias->size(0) == q.size(1) &&
+                bias->size(1) >= 1);
+  if (gate.has_value())
+    TORCH_CHECK(gate->dim() == 2 && gate->scalar_type() == q.scalar_type() && gate->stride(1) == 1 &&
+                gate->size(0) == q.size(0) && gate->size(1) == q.size(1));
+}
+#define BIAS_GATE_ARGS                                                                                     \
+  (bias.has_value() ? bias->data_ptr<float>() : nullptr), (bias.has_value() ? (int)bias->size(1) : 0),      \
+      opt_ptr(gate), (gate.has_value() ? gate->stride(0) : 0)
+
 // Decode attention on tcgen05 (see api.h); shares the GEMM module's tensor-map cache and status word.
 void decode_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
                            const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
                            const c10::optional<at::Tensor>& ws_o, const c10::optional<at::Tensor>& ws_lse,
                            int64_t max_query_len, int64_t num_splits, int64_t window, double scale,
-                           bool early_meta) {
+                           bool early_meta, const c10::optional<at::Tensor>& bias,
+                           const c10::optional<at::Tensor>& gate) {
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && kv_cache.dim() == 5);
+  check_bias_gate(q, bias, gate);
   TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && qsl.scalar_type() == at::kInt);
   TORCH_CHECK(block_tables.stride(1) == 1 && q.scalar_type() == kv_cache.scalar_type());
   if (num_splits > 1) TORCH_CHECK(ws_o.has_value() && ws_lse.has_value());
@@ -970,7 +995,7 @@ void decode_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tensor
                                    ws_lse.has_value() ? ws_lse->data_ptr<float>() : nullptr, gs.status.data_ptr<int>(),
                                    q.size(0), B, q.size(1), kv_cache.size(2), D, kv_cache.size(3), block_tables.stride(0),
                                    kv_cache.size(0), max_query_len, num_splits, window, (float)scale,
-                                   early_meta ? 1 : 0, dtype_code(q), stream()), "decode_attention_umma");
+                                   early_meta ? 1 : 0, BIAS_GATE_ARGS, dtype_code(q), stream()), "decode_attention_umma");
 }
 
 extern at::Tensor g_kernel_trace;
@@ -978,7 +1003,9 @@ extern at::Tensor g_kernel_trace;
 // optional lse [T, Hq] (natural log).
 void prefill_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
                             const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
-                            const c10::optional<at::Tensor>& lse, int64_t max_query_len, int64_t window, double scale) {
+                            const c10::optional<at::Tensor>& lse, int64_t max_query_len, int64_t window, double scale,
+                            const c10::optional<at::Tensor>& bias, const c10::optional<at::Tensor>& gate) {
+  check_bias_gate(q, bias, gate);
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && kv_cache.dim() == 5);
   TORCH_CHECK(q.size(2) == 128 && kv_cache.size(4) == 128 && kv_cache.size(1) == 2 && out.sizes() == q.sizes());
   TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && qsl.scalar_type() == at::kInt);
@@ -1004,7 +1031,7 @@ void prefill_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tenso
                                     sinks.has_value() ? sinks->data_ptr<float>() : nullptr, gs.status.data_ptr<int>(),
                                     (int)seq_lens.size(0), (int)q.size(1), (int)kv_cache.size(2), 128, (int)kv_cache.size(3),
                                     (int)block_tables.stride(0), kv_cache.size(0), (int)max_query_len, (int)window,
-                                    (float)scale, dtype_code(q),
+                                    (float)scale, BIAS_GATE_ARGS, dtype_code(q),
                                     (g_kernel_trace.defined() &&
                                      g_kernel_trace.numel() >= (int64_t)seq_lens.size(0) * q.size(1) * ((max_query_len + 127) / 128) * 24)
                                         ? reinterpret_cast<unsigned long long*>(g_kernel_trace.data_ptr<int64_t>()) : nullptr,
@@ -1409,13 +1436,16 @@ void layernorm_residual(at::Tensor x, at::Tensor h, const c10::optional<at::Tens
                                 (int)w.numel(), (int)x.size(1), (float)eps, y1.has_value() ? 1 : 0, dtype_code(h), stream()),
         "layernorm_residual");
 }
-// out, gate [T, groups * D] (row-strided), o fp32; w [D]
-void gated_group_rmsnorm(at::Tensor out, const at::Tensor& o, const at::Tensor& gate, const at::Tensor& w, double eps) {
-  TORCH_CHECK(out.dim() == 2 && o.dim() == 2 && gate.dim() == 2 && out.stride(1) == 1 && o.stride(1) == 1 && gate.stride(1) == 1);
-  TORCH_CHECK(o.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && gate.scalar_type() == out.scalar_type());
-  TORCH_CHECK(o.size(1) % w.numel() == 0 && gate.sizes() == o.sizes() && out.size(0) == o.size(0) && out.size(1) >= o.size(1));
-  check(b200_gated_group_rmsnorm(out.data_ptr(), out.stride(0), o.data_ptr<float>(), o.stride(0), gate.data_ptr(),
-                                 gate.stride(0), w.data_ptr<float>(), o.size(0), (int)(o.size(1) / w.numel()), (int)w.numel(),
+// out, gate (optional) [T, groups * D] (row-strided), o fp32; w [D]
+void gated_group_rmsnorm(at::Tensor out, const at::Tensor& o, const c10::optional<at::Tensor>& gate, const at::Tensor& w,
+                         double eps) {
+  TORCH_CHECK(out.dim() == 2 && o.dim() == 2 && out.stride(1) == 1 && o.stride(1) == 1);
+  TORCH_CHECK(o.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat);
+  if (gate.has_value())
+    TORCH_CHECK(gate->dim() == 2 && gate->stride(1) == 1 && gate->scalar_type() == out.scalar_type() && gate->sizes() == o.sizes());
+  TORCH_CHECK(o.size(1) % w.numel() == 0 && out.size(0) == o.size(0) && out.size(1) >= o.size(1));
+  check(b200_gated_group_rmsnorm(out.data_ptr(), out.stride(0), o.data_ptr<float>(), o.stride(0), opt_ptr(gate),
+                                 gate.has_value() ? gate->stride(0) : 0, w.data_ptr<float>(), o.size(0), (int)(o.size(1) / w.numel()), (int)w.numel(),
                                  (float)eps, dtype_code(out), stream()), "gated_group_rmsnorm");
 }
 // q, k, v: column slices [T, heads * head size] of one row-strided tensor; q_out [T, Hq, Dc]
@@ -1476,6 +1506,87 @@ void fixed_decay_attention(at::Tensor out, const at::Tensor& q, const at::Tensor
   if (chunked) check(b200_chunk_decay(&a, dtype_code(q), stream()), "fixed_decay_attention (chunked)");
   else check(b200_linear_recurrence(&a, dtype_code(q), stream()), "fixed_decay_attention");
 }
+// forget gates a_ [T, H * Dk], their bias and lower bound [H * Dk]
+void gated_write_attention(at::Tensor out, const at::Tensor& q, const at::Tensor& v, const at::Tensor& a_,
+                           const at::Tensor& bias, const at::Tensor& lower, at::Tensor states, const at::Tensor& cu,
+                           const at::Tensor& slots, const at::Tensor& has_init, bool chunked, bool decode) {
+  RecurrenceArgs a;
+  fill_recurrence(a, out, q, q, v, states, cu, slots, has_init);
+  TORCH_CHECK(a.Hk == a.H && a_.dim() == 2 && a_.stride(1) == 1 && a_.size(1) == a.H * a.Dk && a_.scalar_type() == q.scalar_type());
+  for (const at::Tensor* t : {&bias, &lower})
+    TORCH_CHECK(t->scalar_type() == at::kFloat && t->is_contiguous() && t->numel() == a.H * a.Dk);
+  a.a = a_.data_ptr(); a.a_stride = a_.stride(0);
+  a.dt_bias = bias.data_ptr<float>(); a.lower = lower.data_ptr<float>();
+  a.kind = 2; a.decode = decode;
+  if (chunked) check(b200_chunk_gated_write(&a, dtype_code(q), stream()), "gated_write_attention (chunked)");
+  else check(b200_linear_recurrence(&a, dtype_code(q), stream()), "gated_write_attention");
+}
+
+// ------------------------------------------------------- norms before and after every sublayer, polynomial activation
+void embed_rmsnorm(at::Tensor x, at::Tensor h, const at::Tensor& ids, const at::Tensor& table, const at::Tensor& w, double eps) {
+  TORCH_CHECK(x.is_contiguous() && h.is_contiguous() && table.is_contiguous() && x.scalar_type() == at::kFloat && x.dim() == 2);
+  TORCH_CHECK(h.sizes() == x.sizes() && table.size(1) == x.size(1) && table.scalar_type() == h.scalar_type());
+  TORCH_CHECK(x.data_ptr() != h.data_ptr() && ids.numel() == x.size(0) && w.scalar_type() == at::kFloat && w.numel() <= x.size(1));
+  check(b200_embed_rmsnorm(x.data_ptr<float>(), h.data_ptr(), ids.data_ptr<int64_t>(), table.data_ptr(), w.data_ptr<float>(),
+                           x.size(0), (int)w.numel(), (int)x.size(1), table.size(0), (float)eps, dtype_code(h), stream()),
+        "embed_rmsnorm");
+}
+// y [T, ld], or rows of which pos [T * k] picks the summands of every token
+void sandwich_rmsnorm(at::Tensor x, at::Tensor h, const at::Tensor& y, const c10::optional<at::Tensor>& pos,
+                      const at::Tensor& w_post, const at::Tensor& w_pre, double eps) {
+  TORCH_CHECK(x.is_contiguous() && h.is_contiguous() && x.scalar_type() == at::kFloat && h.sizes() == x.sizes() && x.dim() == 2);
+  TORCH_CHECK(x.data_ptr() != h.data_ptr() && y.dim() == 2 && y.size(1) == x.size(1) && y.stride(1) == 1 &&
+              y.scalar_type() == h.scalar_type());
+  TORCH_CHECK(w_post.scalar_type() == at::kFloat && w_pre.scalar_type() == at::kFloat && w_post.numel() == w_pre.numel() &&
+              w_pre.numel() <= x.size(1));
+  const int64_t T = x.size(0);
+  if (T == 0) return;
+  if (pos.has_value()) {
+    TORCH_CHECK(pos->scalar_type() == at::kInt && pos->is_contiguous() && pos->numel() % T == 0);
+  } else {
+    TORCH_CHECK(y.size(0) == T);
+  }
+  check(b200_sandwich_rmsnorm(x.data_ptr<float>(), h.data_ptr(), y.data_ptr(), y.stride(0),
+                              pos.has_value() ? pos->data_ptr<int>() : nullptr, pos.has_value() ? (int)(pos->numel() / T) : 1,
+                              w_post.data_ptr<float>(), w_pre.data_ptr<float>(), T, (int)w_pre.numel(), (int)x.size(1),
+                              (float)eps, dtype_code(h), stream()), "sandwich_rmsnorm");
+}
+// out, z [T, ld]; the first `width` columns count
+void poly_norm(at::Tensor out, const at::Tensor& z, const at::Tensor& coeff, int64_t width, double eps) {
+  TORCH_CHECK(z.dim() == 2 && out.sizes() == z.sizes() && z.stride(1) == 1 && out.stride(1) == 1 && z.scalar_type() == out.scalar_type());
+  TORCH_CHECK(coeff.scalar_type() == at::kFloat && coeff.is_contiguous() && coeff.numel() == 4 && width <= z.size(1) && width > 0);
+  check(b200_poly_norm(out.data_ptr(), out.stride(0), z.data_ptr(), z.stride(0), coeff.data_ptr<float>(), z.size(0), (int)width,
+                       (int)z.size(1), (float)eps, dtype_code(z), stream()), "poly_norm");
+}
+// q, k, v: column slices [T, heads * head size] of one row-strided tensor; q_out [T, Hq, Dc]; v_out / v_in [T, Hkv * Dv]
+void attn_prep_cache(at::Tensor q_out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at::Tensor kv_cache,
+                     const at::Tensor& slots, const at::Tensor& positions, int64_t num_heads, int64_t num_kv_heads,
+                     double temp_coef, int64_t temp_every, const c10::optional<at::Tensor>& v_out,
+                     const c10::optional<at::Tensor>& v_in, double share, double eps) {
+  TORCH_CHECK(q_out.is_contiguous() && kv_cache.is_contiguous() && kv_cache.dim() == 5 && kv_cache.size(2) == num_kv_heads);
+  TORCH_CHECK(q.stride(1) == 1 && k.stride(1) == 1 && v.stride(1) == 1 && q.stride(0) == k.stride(0) && q.stride(0) == v.stride(0));
+  TORCH_CHECK(q.scalar_type() == q_out.scalar_type() && q.scalar_type() == kv_cache.scalar_type() && temp_every >= 0);
+  const int64_t D = q.size(1) / num_heads, Dv = v.size(1) / num_kv_heads, Dc = kv_cache.size(4);
+  TORCH_CHECK(k.size(1) == D * num_kv_heads && q_out.numel() == q.size(0) * num_heads * Dc && slots.numel() == q.size(0) &&
+              positions.numel() == q.size(0));
+  for (const auto* t : {&v_out, &v_in})
+    if (t->has_value()) TORCH_CHECK((*t)->is_contiguous() && (*t)->sizes() == v.sizes() && (*t)->scalar_type() == v.scalar_type());
+  check(b200_attn_prep_cache(q_out.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), kv_cache.data_ptr(),
+                             slots.data_ptr<int64_t>(), positions.data_ptr<int64_t>(), const_cast<void*>(opt_ptr(v_out)),
+                             opt_ptr(v_in), (float)share, (float)temp_coef, temp_every, q.size(0), (int)num_heads,
+                             (int)num_kv_heads, (int)D, (int)Dv, (int)Dc, (int)kv_cache.size(3), kv_cache.size(0), (float)eps,
+                             dtype_code(q), stream()), "attn_prep_cache");
+}
+// x [M, K] sorted by expert (lod [E + 1]), w [E, N, K]
+void gemm_f32_grouped(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const at::Tensor& lod) {
+  TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && out.dim() == 2 && x.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1);
+  TORCH_CHECK(x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && out.scalar_type() == at::kFloat);
+  TORCH_CHECK(x.size(1) == w.size(2) && out.size(0) == x.size(0) && out.size(1) == w.size(1) && lod.scalar_type() == at::kInt &&
+              lod.is_contiguous() && lod.numel() == w.size(0) + 1);
+  check(b200_gemm_f32_grouped(out.data_ptr<float>(), out.stride(0), x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(),
+                              lod.data_ptr<int>(), x.size(0), (int)w.size(0), (int)w.size(1), (int)w.size(2), stream()),
+        "gemm_f32_grouped");
+}
 void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& bias) {
   TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1);
   TORCH_CHECK(x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && out.scalar_type() == at::kFloat);
@@ -1488,7 +1599,9 @@ void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c1
 // latent_dv > 0: kv_cache [blocks, block_size, D] holds latent rows shared by all heads, out [T, Hq, latent_dv]
 void paged_attention_generic(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
                              const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
-                             int64_t latent_dv, int64_t window, double scale) {
+                             int64_t latent_dv, int64_t window, double scale, const c10::optional<at::Tensor>& bias,
+                             const c10::optional<at::Tensor>& gate) {
+  check_bias_gate(q, bias, gate);
   const bool latent = latent_dv > 0;
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && out.dim() == 3 &&
               kv_cache.dim() == (latent ? 3 : 5));
@@ -1503,7 +1616,7 @@ void paged_attention_generic(at::Tensor out, const at::Tensor& q, const at::Tens
                                      sinks.has_value() ? sinks->data_ptr<float>() : nullptr, q.size(0), (int)seq_lens.size(0),
                                      (int)q.size(1), latent ? 1 : (int)kv_cache.size(2), (int)q.size(2),
                                      (int)kv_cache.size(latent ? 1 : 3), (int)block_tables.stride(0), kv_cache.size(0),
-                                     (int)latent_dv, (int)window, (float)scale, dtype_code(q), stream()),
+                                     (int)latent_dv, (int)window, (float)scale, BIAS_GATE_ARGS, dtype_code(q), stream()),
         "paged_attention_generic");
 }
 
@@ -1742,11 +1855,12 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("grouped_gemm", &grouped_gemm);
   m.def("moe_route", &moe_route);
   m.def("moe_permute", &moe_permute, py::arg("x"), py::arg("ids"), py::arg("emap"), py::arg("E_local"),
-        py::arg("E_global"), py::arg("state"), py::arg("max_rows") = 0);
+        py::arg("E_global"), py::arg("state"), py::arg("max_rows") = 0, py::arg("factors") = py::none());
   m.def("moe_unpermute", &moe_unpermute);
   m.def("router_gemm_small", &router_gemm_small);
   m.def("router_route_small", &router_route_small);
-  m.def("moe_prepare_small", &moe_prepare_small);
+  m.def("moe_prepare_small", &moe_prepare_small, py::arg("x"), py::arg("ids"), py::arg("emap"), py::arg("E_local"),
+        py::arg("E_global"), py::arg("quant"), py::arg("factors") = py::none());
   m.def("act_mul_quant_fp8", &act_mul_quant_fp8);
   m.def("moe_small_pairs", []() { return (int64_t)b200_moe_small_pairs(); });
   m.def("quant_fp8_group", &quant_fp8_group);
@@ -1765,7 +1879,15 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("channel_delta_rule", &channel_delta_rule);
   m.def("fixed_decay_attention", &fixed_decay_attention);
   m.def("gemm_f32", &gemm_f32);
-  m.def("paged_attention_generic", &paged_attention_generic);
+  m.def("gemm_f32_grouped", &gemm_f32_grouped);
+  m.def("gated_write_attention", &gated_write_attention);
+  m.def("embed_rmsnorm", &embed_rmsnorm);
+  m.def("sandwich_rmsnorm", &sandwich_rmsnorm);
+  m.def("poly_norm", &poly_norm);
+  m.def("attn_prep_cache", &attn_prep_cache);
+  m.def("paged_attention_generic", &paged_attention_generic, py::arg("out"), py::arg("q"), py::arg("kv_cache"),
+        py::arg("block_tables"), py::arg("seq_lens"), py::arg("qsl"), py::arg("sinks"), py::arg("latent_dv"),
+        py::arg("window"), py::arg("scale"), py::arg("bias") = py::none(), py::arg("gate") = py::none());
   m.def("rotary_table", &rotary_table);
   m.def("latent_prep", &latent_prep);
   m.def("rotate_heads", &rotate_heads);
@@ -1782,7 +1904,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("lora_shrink", &lora_shrink);
   m.def("lora_expand", &lora_expand);
   m.def("rownorm", &rownorm);
-  m.def("act_and_mul", &act_and_mul);
+  m.def("act_and_mul", &act_and_mul, py::arg("out"), py::arg("x"), py::arg("act"), py::arg("limit") = 0.0);
   m.def("quick_gelu", &quick_gelu);
   m.def("embedding", &embedding);
   m.def("argmax", &argmax);
@@ -1796,9 +1918,15 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("copy_blocks", &copy_blocks);
   m.def("merge_attn_states", &merge_attn_states);
   m.def("paged_attention", &paged_attention);
-  m.def("decode_attention_umma", &decode_attention_umma);
+  m.def("decode_attention_umma", &decode_attention_umma, py::arg("out"), py::arg("q"), py::arg("kv_cache"),
+        py::arg("block_tables"), py::arg("seq_lens"), py::arg("qsl"), py::arg("sinks"), py::arg("ws_o"),
+        py::arg("ws_lse"), py::arg("max_query_len"), py::arg("num_splits"), py::arg("window"), py::arg("scale"),
+        py::arg("early_meta"), py::arg("bias") = py::none(), py::arg("gate") = py::none());
   m.def("mla_decode_umma", &mla_decode_umma);
-  m.def("prefill_attention_umma", &prefill_attention_umma);
+  m.def("prefill_attention_umma", &prefill_attention_umma, py::arg("out"), py::arg("q"), py::arg("kv_cache"),
+        py::arg("block_tables"), py::arg("seq_lens"), py::arg("qsl"), py::arg("sinks"), py::arg("lse"),
+        py::arg("max_query_len"), py::arg("window"), py::arg("scale"), py::arg("bias") = py::none(),
+        py::arg("gate") = py::none());
   m.def("mla_prefill_umma", &mla_prefill_umma);
   m.def("indexer_prep", &indexer_prep);
   m.def("gather_mla_rows", &gather_mla_rows);

@@ -83,9 +83,11 @@ __global__ void warp_rownorm_kernel(T* __restrict__ out, const T* __restrict__ x
   }
 }
 
-// act: 0 = silu(gate)*up with x = [gate | up]; 1 = gelu_tanh(gate)*up; 2 = swigluoai (interleaved, clamped)
+// act: 0 = silu(gate)*up with x = [gate | up]; 1 = gelu_tanh(gate)*up; 2 = swigluoai (interleaved, clamped); 3 = the same
+// function of x = [gate | up] with a given limit
 template <typename T>
-__global__ void act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t rows, int d, int act) {
+__global__ void act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t rows, int d, int act,
+                                   float limit) {
   constexpr int V = Vec16<T>::N;
   griddep_launch();
   griddep_wait();
@@ -114,7 +116,11 @@ __global__ void act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x,
     for (int j = 0; j < V; ++j) {
       float gf = to_f(g.v[j]), uf = to_f(u.v[j]);
       float a;
-      if (act == 0) a = gf / (1.f + __expf(-gf));
+      if (act == 3) {
+        gf = fminf(gf, limit);
+        uf = fminf(fmaxf(uf, -limit), limit) + 1.f;
+        a = gf / (1.f + __expf(-1.702f * gf));
+      } else if (act == 0) a = gf / (1.f + __expf(-gf));
       else a = gf / (1.f + __expf(-1.5957691216f * (gf + 0.044715f * gf * gf * gf)));  // gelu: (1 + tanh(t)) / 2 = sigmoid(2 t)
       o.v[j] = from_f<T>(a * uf);
     }
@@ -245,13 +251,13 @@ extern "C" int b200_rownorm(void* out, const void* x, const void* z, const void*
   return (int)cudaGetLastError();
 }
 
-extern "C" int b200_act_and_mul(void* out, const void* x, int64_t rows, int d, int act, int dtype, cudaStream_t st) {
+extern "C" int b200_act_and_mul(void* out, const void* x, int64_t rows, int d, int act, float limit, int dtype, cudaStream_t st) {
   if (rows == 0) return 0;
   B200_DISPATCH_DTYPE(dtype, {
     constexpr int V = Vec16<T>::N;
     if (d % V || (act == 2 && d % V)) return 2;
     int64_t total = rows * (d / V);
-    launch_pdl(act_and_mul_kernel<T>, dim3((total + 255) / 256), dim3(256), 0, st, (T*)out, (const T*)x, rows, d, act);
+    launch_pdl(act_and_mul_kernel<T>, dim3((total + 255) / 256), dim3(256), 0, st, (T*)out, (const T*)x, rows, d, act, limit);
   });
   return (int)cudaGetLastError();
 }

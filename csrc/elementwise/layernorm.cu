@@ -1,7 +1,7 @@
 // Kernels of decoders whose residual stream is kept in fp32 and normalised on the sublayers' outputs:
 //   embed_layernorm        token row + sinusoidal position vector -> LayerNorm -> stream (fp32) + 16-bit copy
 //   layernorm_residual     stream += LayerNorm(s1 y1 [+ s2 y2]) (or the final norm of the stream) + 16-bit copy
-//   gated_group_rmsnorm    RMS norm over groups of a mixer's output, times weight and sigmoid(gate)
+//   gated_group_rmsnorm    RMS norm over groups of a mixer's output, times weight and (with a gate) sigmoid(gate)
 //   qk_unit_norm_cache     split a fused projection, scale q / k to unit RMS per head, K / V into the paged cache
 // These kernels are launched with programmatic dependent launch, so they may be resident while the producer of their
 // inputs still runs: the pointers carry no __restrict__, which would let the compiler read them through the
@@ -152,7 +152,7 @@ __global__ void __launch_bounds__(kLnThreads) layernorm_residual_kernel(float* x
   }
 }
 
-// out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) over groups of D columns; RT threads per group.
+// out = o / sqrt(mean(o^2) + eps) * w [* sigmoid(gate)] over groups of D columns; RT threads per group.
 template <typename T, int RT, bool VEC>
 __global__ void __launch_bounds__(256) gated_group_rmsnorm_kernel(T* out, int64_t out_stride,
                                                                   const float* o, int64_t o_stride,
@@ -169,7 +169,7 @@ __global__ void __launch_bounds__(256) gated_group_rmsnorm_kernel(T* out, int64_
   const int64_t t = row / groups;
   const int g = (int)(row % groups);
   const float* orow = o + t * o_stride + (int64_t)g * D;
-  const T* grow = gate + t * gate_stride + (int64_t)g * D;
+  const T* grow = gate == nullptr ? nullptr : gate + t * gate_stride + (int64_t)g * D;
   T* dst = out + t * out_stride + (int64_t)g * D;
   float ss = 0.f;
   for (int i = lane * V; i < D; i += RT * V) {
@@ -187,13 +187,13 @@ __global__ void __launch_bounds__(256) gated_group_rmsnorm_kernel(T* out, int64_
     if constexpr (VEC) {
       float a[4], b[4], ww[4];
       load4(a, orow + i);
-      load4(b, grow + i);
+      if (grow != nullptr) load4(b, grow + i);
       load4(ww, w + i);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) a[j] = a[j] * inv * ww[j] * (1.f / (1.f + expf(-b[j])));
+      for (int j = 0; j < 4; ++j) a[j] = a[j] * inv * ww[j] * (grow != nullptr ? 1.f / (1.f + expf(-b[j])) : 1.f);
       store4(dst + i, a);
     } else {
-      dst[i] = from_f<T>(orow[i] * inv * w[i] * (1.f / (1.f + expf(-to_f(grow[i])))));
+      dst[i] = from_f<T>(orow[i] * inv * w[i] * (grow != nullptr ? 1.f / (1.f + expf(-to_f(grow[i]))) : 1.f));
     }
   }
 }

@@ -1,0 +1,335 @@
+// Kernels of decoders that normalise before and after every sublayer around an fp32 residual stream:
+//   embed_rmsnorm        token row -> stream (fp32), its RMS norm in the model's dtype
+//   sandwich_rmsnorm     stream += rms(y) * w_post;  h = rms(stream) * w_pre        (one sublayer's end, the next one's start;
+//                        y may be given as `k` rows per token in expert order, which are summed on the way in)
+//   poly_norm            a N(z) + b N(z^2) + c N(z^3) + e over a feed-forward row, N = division by the root mean square
+//   attn_prep_cache      split a fused projection: q times a temperature that grows with the position, k as it is, v of
+//                        unit root mean square and mixed with another layer's values; K / V into the paged cache
+// Weights come ready to multiply (a weight stored around zero arrives as 1 + w, a residual factor folded in).
+// These kernels are launched with programmatic dependent launch: pointers carry no __restrict__, which would let the
+// compiler read them through the non-coherent path before the producers have finished.  Statistics are fp32 (this file is
+// compiled without fast-math).  `ld` is the row length of stream and copy: the width rounded up, padding columns zero.
+#include "../api.h"
+#include "../common/launch.cuh"
+#include "../common/utils.cuh"
+
+namespace b200 {
+namespace {
+
+constexpr int kThr = 256;
+
+template <typename T> struct alignas(4 * sizeof(T)) Vec4 { T v[4]; };
+template <typename T> __device__ __forceinline__ void load4(float (&d)[4], const T* p) {
+  const Vec4<T> r = *reinterpret_cast<const Vec4<T>*>(p);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) d[j] = to_f(r.v[j]);
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, const float (&s)[4]) {
+  Vec4<T> r;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) r.v[j] = from_f<T>(s[j]);
+  *reinterpret_cast<Vec4<T>*>(p) = r;
+}
+
+// 1 / root mean square of a row spread over the block (columns beyond H hold zeros)
+template <int NV>
+__device__ __forceinline__ float inv_rms(const float (&y)[NV][4], int H, float eps, float* red) {
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) s += y[i][j] * y[i][j];
+  return 1.f / sqrtf(block_sum(s, red) / H + eps);
+}
+
+template <typename T, int NV>
+__device__ __forceinline__ void store_normed(T* h, const float (&x)[NV][4], const float* w, float inv, int H, int ld) {
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * kThr + threadIdx.x) * 4;
+    if (c >= ld) continue;
+    float o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] = c + j < H ? x[i][j] * inv * w[c + j] : 0.f;
+    store4(h + c, o);
+  }
+}
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(kThr) embed_rmsnorm_kernel(float* x, T* h, const int64_t* ids, const T* table,
+                                                             const float* w, int H, int ld, int64_t rows, float eps) {
+  __shared__ float red[32];
+  griddep_launch();
+  griddep_wait();
+  const int64_t t = blockIdx.x, id = ids[t];
+  const bool ok = id >= 0 && id < rows;
+  float y[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * kThr + threadIdx.x) * 4;
+    y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.f;
+    if (c >= ld) continue;
+    if (ok) load4(y[i], table + id * ld + c);
+    store4(x + t * ld + c, y[i]);
+  }
+  store_normed<T, NV>(h + t * ld, y, w, inv_rms<NV>(y, H, eps, red), H, ld);
+}
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(kThr) sandwich_rmsnorm_kernel(float* x, T* h, const T* y_, int64_t y_stride, const int* pos,
+                                                                int k, const float* w_post, const float* w_pre, int H,
+                                                                int ld, float eps) {
+  __shared__ float red[32];
+  griddep_launch();
+  griddep_wait();
+  const int64_t t = blockIdx.x;
+  float y[NV][4], s[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * kThr + threadIdx.x) * 4;
+    y[i][0] = y[i][1] = y[i][2] = y[i][3] = s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+    if (c >= ld) continue;
+    load4(s[i], x + t * ld + c);
+    if (pos == nullptr) {
+      load4(y[i], y_ + t * y_stride + c);
+    } else {
+      for (int q = 0; q < k; ++q) {
+        const int r = pos[t * k + q];
+        if (r < 0) continue;
+        float z[4];
+        load4(z, y_ + (int64_t)r * y_stride + c);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[i][j] += z[j];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (c + j >= H) y[i][j] = 0.f;
+  }
+  const float inv = inv_rms<NV>(y, H, eps, red);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * kThr + threadIdx.x) * 4;
+    if (c >= ld) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (c + j < H) s[i][j] += y[i][j] * inv * w_post[c + j];
+    store4(x + t * ld + c, s[i]);
+  }
+  store_normed<T, NV>(h + t * ld, s, w_pre, inv_rms<NV>(s, H, eps, red), H, ld);
+}
+
+// Three sums of a row at once, broadcast to the block.
+__device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float (*red)[3]) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  c = warp_sum(c);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
+  if (l == 0) { red[w][0] = a; red[w][1] = b; red[w][2] = c; }
+  __syncthreads();
+  a = b = c = 0.f;
+#pragma unroll
+  for (int i = 0; i < kThr / 32; ++i) { a += red[i][0]; b += red[i][1]; c += red[i][2]; }
+}
+
+// NV vectors of 4 columns per thread; NV = 0: rows of any length, read twice.  Columns F .. ld of the output are zero.
+template <typename T, int NV>
+__global__ void __launch_bounds__(kThr) poly_norm_kernel(T* out, int64_t ldo, const T* z, int64_t ldz, const float* coeff,
+                                                         int F, int ld, float eps) {
+  __shared__ float red[kThr / 32][3];
+  griddep_launch();
+  griddep_wait();
+  const int64_t t = blockIdx.x;
+  const T* zr = z + t * ldz;
+  constexpr int NR = NV > 0 ? NV : 1;
+  float v[NR][4], s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  auto add = [&](const float (&a)[4], int c) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float q = c + j < F ? a[j] * a[j] : 0.f;
+      s1 += q;
+      s2 += q * q;
+      s3 += q * q * q;
+    }
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * kThr + threadIdx.x) * 4;
+      v[i][0] = v[i][1] = v[i][2] = v[i][3] = 0.f;
+      if (c >= ld) continue;
+      load4(v[i], zr + c);
+      add(v[i], c);
+    }
+  } else {
+    for (int c = threadIdx.x * 4; c < ld; c += kThr * 4) {
+      load4(v[0], zr + c);
+      add(v[0], c);
+    }
+  }
+  block_sum3(s1, s2, s3, red);
+  const float a = coeff[0] / sqrtf(s1 / F + eps), b = coeff[1] / sqrtf(s2 / F + eps), c3 = coeff[2] / sqrtf(s3 / F + eps),
+              e = coeff[3];
+  auto put = [&](const float (&x)[4], int c) {
+    float o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] = c + j < F ? x[j] * (a + x[j] * (b + x[j] * c3)) + e : 0.f;
+    store4(out + t * ldo + c, o);
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * kThr + threadIdx.x) * 4;
+      if (c < ld) put(v[i], c);
+    }
+  } else {
+    for (int c = threadIdx.x * 4; c < ld; c += kThr * 4) {
+      load4(v[0], zr + c);
+      put(v[0], c);
+    }
+  }
+}
+
+// One warp per (token, head) of q, k and v; head sizes D (q, k) and Dv (v) are zero-padded to Dc in q_out and in the cache
+// [block][2][Hkv][slot][Dc].  v_out [T][Hkv * Dv]: the normed values (before mixing) for later layers; v_in: such values of
+// an earlier layer, mixed in with the given share.
+template <typename T>
+__global__ void __launch_bounds__(256) attn_prep_cache_kernel(T* q_out, const T* q, const T* k, const T* v, int64_t stride,
+                                                              T* cache, const int64_t* slots, const int64_t* positions,
+                                                              T* v_out, const T* v_in, float share, float temp_coef,
+                                                              int64_t temp_every, int Hq, int Hkv, int D, int Dv, int Dc,
+                                                              int block_size, int64_t num_blocks, float eps, int vec) {
+  griddep_launch();
+  griddep_wait();
+  const int64_t t = blockIdx.x;
+  const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (head >= Hq + 2 * Hkv) return;
+  const bool is_q = head < Hq, is_v = head >= Hq + Hkv;
+  const int n = is_v ? Dv : D;
+  const int kvh = is_v ? head - Hq - Hkv : head - Hq;
+  const T* src;
+  T* dst = nullptr;
+  float f = 1.f;
+  if (is_q) {
+    src = q + t * stride + (int64_t)head * D;
+    dst = q_out + (t * Hq + head) * (int64_t)Dc;
+    if (temp_every > 0) f = 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1));
+  } else {
+    src = (is_v ? v : k) + t * stride + (int64_t)kvh * n;
+    const int64_t slot = slots[t];
+    if (slot >= 0 && slot < num_blocks * block_size)
+      dst = cache + ((((slot / block_size) * 2 + (is_v ? 1 : 0)) * Hkv + kvh) * block_size + slot % block_size) * (int64_t)Dc;
+  }
+  if (is_v) {
+    float ss = 0.f;
+    if (vec) {
+      for (int i = lane * 4; i < n; i += 128) {
+        float a[4];
+        load4(a, src + i);
+        ss += a[0] * a[0] + a[1] * a[1] + a[2] * a[2] + a[3] * a[3];
+      }
+    } else {
+      for (int i = lane; i < n; i += 32) { const float x = to_f(src[i]); ss += x * x; }
+    }
+    f = 1.f / sqrtf(warp_sum(ss) / n + eps);
+  }
+  const int64_t vo = (t * Hkv + kvh) * (int64_t)Dv;
+  const T* mix = is_v && v_in != nullptr ? v_in + vo : nullptr;
+  T* keep = is_v && v_out != nullptr ? v_out + vo : nullptr;
+  if (vec) {
+    for (int i = lane * 4; i < Dc; i += 128) {
+      float a[4] = {0.f, 0.f, 0.f, 0.f};
+      if (i < n) {
+        load4(a, src + i);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) a[j] *= f;
+        if (keep != nullptr) store4(keep + i, a);
+        if (mix != nullptr) {
+          float b[4];
+          load4(b, mix + i);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) a[j] = (1.f - share) * a[j] + share * b[j];
+        }
+      }
+      if (dst != nullptr) store4(dst + i, a);
+    }
+  } else {
+    for (int i = lane; i < Dc; i += 32) {
+      float a = 0.f;
+      if (i < n) {
+        a = to_f(src[i]) * f;
+        if (keep != nullptr) keep[i] = from_f<T>(a);
+        if (mix != nullptr) a = (1.f - share) * a + share * to_f(mix[i]);
+      }
+      if (dst != nullptr) dst[i] = from_f<T>(a);
+    }
+  }
+}
+
+#define B200_SW_NV(NVEC, ...)                                                     \
+  {                                                                               \
+    const int need_ = (ld / 4 + kThr - 1) / kThr;                                 \
+    if (need_ <= 1) { constexpr int NVEC = 1; __VA_ARGS__; }                      \
+    else if (need_ <= 2) { constexpr int NVEC = 2; __VA_ARGS__; }                 \
+    else if (need_ <= 4) { constexpr int NVEC = 4; __VA_ARGS__; }                 \
+    else if (need_ <= 8) { constexpr int NVEC = 8; __VA_ARGS__; }                 \
+    else if (need_ <= 16) { constexpr int NVEC = 16; __VA_ARGS__; }               \
+    else return 3;                                                                \
+  }
+
+}  // namespace
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int b200_embed_rmsnorm(float* x, void* h, const int64_t* ids, const void* table, const float* w, int64_t T_, int H,
+                                  int ld, int64_t rows, float eps, int dtype, cudaStream_t st) {
+  if (T_ == 0) return 0;
+  if (ld % 4 || H > ld) return 3;
+  B200_DISPATCH_DTYPE(dtype, B200_SW_NV(NV, launch_pdl(embed_rmsnorm_kernel<T, NV>, dim3(T_), dim3(kThr), 0, st, x, (T*)h, ids,
+                                                      (const T*)table, w, H, ld, rows, eps)));
+  return (int)cudaGetLastError();
+}
+
+extern "C" int b200_sandwich_rmsnorm(float* x, void* h, const void* y, int64_t y_stride, const int* pos, int k,
+                                     const float* w_post, const float* w_pre, int64_t T_, int H, int ld, float eps, int dtype,
+                                     cudaStream_t st) {
+  if (T_ == 0) return 0;
+  if (ld % 4 || H > ld || y_stride % 4) return 3;
+  B200_DISPATCH_DTYPE(dtype, B200_SW_NV(NV, launch_pdl(sandwich_rmsnorm_kernel<T, NV>, dim3(T_), dim3(kThr), 0, st, x, (T*)h,
+                                                      (const T*)y, y_stride, pos, k, w_post, w_pre, H, ld, eps)));
+  return (int)cudaGetLastError();
+}
+
+extern "C" int b200_poly_norm(void* out, int64_t ldo, const void* z, int64_t ldz, const float* coeff, int64_t T_, int F, int ld,
+                              float eps, int dtype, cudaStream_t st) {
+  if (T_ == 0) return 0;
+  if (ld % 4 || ldo % 4 || ldz % 4 || F > ld) return 3;
+#define B200_PN(NVEC) launch_pdl(poly_norm_kernel<T, NVEC>, dim3(T_), dim3(kThr), 0, st, (T*)out, ldo, (const T*)z, ldz, coeff, F, ld, eps)
+  B200_DISPATCH_DTYPE(dtype, {
+    const int need = (ld / 4 + kThr - 1) / kThr;
+    if (need <= 1) B200_PN(1);
+    else if (need <= 2) B200_PN(2);
+    else if (need <= 4) B200_PN(4);
+    else if (need <= 8) B200_PN(8);
+    else if (need <= 16) B200_PN(16);
+    else B200_PN(0);
+  });
+#undef B200_PN
+  return (int)cudaGetLastError();
+}
+
+extern "C" int b200_attn_prep_cache(void* q_out, const void* q, const void* k, const void* v, int64_t stride, void* kv_cache,
+                                    const int64_t* slots, const int64_t* positions, void* v_out, const void* v_in, float share,
+                                    float temp_coef, int64_t temp_every, int64_t T_, int Hq, int Hkv, int D, int Dv, int Dc,
+                                    int block_size, int64_t num_blocks, float eps, int dtype, cudaStream_t st) {
+  if (T_ == 0) return 0;
+  if (D > Dc || Dv > Dc) return 3;
+  const uintptr_t al = (uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)v_out | (uintptr_t)v_in;
+  const int vec = D % 4 == 0 && Dv % 4 == 0 && Dc % 4 == 0 && stride % 4 == 0 && al % 16 == 0;
+  dim3 grid((unsigned)T_, (Hq + 2 * Hkv + 7) / 8);
+  B200_DISPATCH_DTYPE(dtype, launch_pdl(attn_prep_cache_kernel<T>, grid, dim3(256), 0, st, (T*)q_out, (const T*)q, (const T*)k,
+                                       (const T*)v, stride, (T*)kv_cache, slots, positions, (T*)v_out, (const T*)v_in, share,
+                                       temp_coef, temp_every, Hq, Hkv, D, Dv, Dc, block_size, num_blocks, eps, vec));
+  return (int)cudaGetLastError();
+}

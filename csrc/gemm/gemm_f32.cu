@@ -2,6 +2,8 @@
 // products and sums (the tensor cores have no such format).  Any T, N, K and row strides.
 //   few rows   one warp per output feature, the weight row streamed once for up to kRows tokens
 //   many rows  64 x 64 output tile per CTA, 16-wide K slices through shared memory, 4 x 4 outputs per thread
+//   grouped    rows sorted by expert, w[E, N, K], lod[e] .. lod[e + 1] the rows of expert e: the tile kernel, a tile per
+//              (expert, 64 rows); the tiles are counted off on the device
 #include "../api.h"
 #include "../common/launch.cuh"
 #include "../common/utils.cuh"
@@ -36,13 +38,9 @@ __global__ void __launch_bounds__(256) gemm_f32_rows_kernel(float* out, int64_t 
   }
 }
 
-__global__ void __launch_bounds__(256) gemm_f32_tile_kernel(float* out, int64_t ldo, const float* x,
-                                                            int64_t ldx, const float* w, int64_t ldw,
-                                                            const float* bias, int64_t T_, int N, int K) {
+__device__ __forceinline__ void gemm_f32_tile(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w,
+                                              int64_t ldw, const float* bias, int64_t t0, int64_t T_, int N, int K) {
   __shared__ __align__(16) float sx[16][68], sw[16][68];
-  griddep_launch();
-  griddep_wait();
-  const int64_t t0 = (int64_t)blockIdx.y * 64;
   const int n0 = blockIdx.x * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
@@ -75,6 +73,29 @@ __global__ void __launch_bounds__(256) gemm_f32_tile_kernel(float* out, int64_t 
     }
 }
 
+__global__ void __launch_bounds__(256) gemm_f32_tile_kernel(float* out, int64_t ldo, const float* x,
+                                                            int64_t ldx, const float* w, int64_t ldw,
+                                                            const float* bias, int64_t T_, int N, int K) {
+  griddep_launch();
+  griddep_wait();
+  gemm_f32_tile(out, ldo, x, ldx, w, ldw, bias, (int64_t)blockIdx.y * 64, T_, N, K);
+}
+
+__global__ void __launch_bounds__(256) gemm_f32_grouped_kernel(float* out, int64_t ldo, const float* x, int64_t ldx,
+                                                               const float* w, const int* lod, int E, int N, int K) {
+  griddep_launch();
+  griddep_wait();
+  int tile = blockIdx.y;
+  for (int e = 0; e < E; ++e) {
+    const int lo = lod[e], hi = lod[e + 1], tiles = (hi - lo + 63) / 64;
+    if (tile < tiles) {
+      gemm_f32_tile(out, ldo, x, ldx, w + (int64_t)e * N * K, K, nullptr, lo + (int64_t)tile * 64, hi, N, K);
+      return;
+    }
+    tile -= tiles;
+  }
+}
+
 }  // namespace
 }  // namespace b200
 
@@ -91,5 +112,16 @@ extern "C" int b200_gemm_f32(float* out, int64_t ldo, const float* x, int64_t ld
     launch_pdl(gemm_f32_tile_kernel, dim3((N + 63) / 64, (unsigned)ty), dim3(256), 0, st, out, ldo, x, ldx, w, ldw, bias, T_,
                N, K);
   }
+  return (int)cudaGetLastError();
+}
+
+// M rows of x in expert order; a grid of ceil(M / 64) + E row tiles covers any split of them over the experts
+extern "C" int b200_gemm_f32_grouped(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, const int* lod,
+                                     int64_t M, int E, int N, int K, cudaStream_t st) {
+  using namespace b200;
+  if (M == 0 || N == 0) return 0;
+  const int64_t ty = (M + 63) / 64 + E;
+  if (ty > 65535) return 3;
+  launch_pdl(gemm_f32_grouped_kernel, dim3((N + 63) / 64, (unsigned)ty), dim3(256), 0, st, out, ldo, x, ldx, w, lod, E, N, K);
   return (int)cudaGetLastError();
 }

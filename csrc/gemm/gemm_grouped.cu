@@ -352,6 +352,7 @@ extern "C" int b200_grouped_gemm_launch(const GroupedGemmArgs* a, const void* tm
   case BN_:                                                                                                  \
     if (a->fp8) e = (a->out_fmt == 1) ? launch_grouped<BN_, true, __nv_bfloat16>(*a, w, x, st)               \
                                       : launch_grouped<BN_, true, __half>(*a, w, x, st);                     \
+    else if (a->out_fmt == 2) e = launch_grouped<BN_, false, float>(*a, w, x, st);                           \
     else e = (a->fmt == 1) ? launch_grouped<BN_, false, __nv_bfloat16>(*a, w, x, st)                         \
                            : launch_grouped<BN_, false, __half>(*a, w, x, st);                               \
     break;

@@ -5,6 +5,8 @@
 //                   a_t = exp(-exp(A_log_h) softplus(x_t + dt_bias)) per key channel, beta_t = sigmoid(b_t);
 //                   q, k scaled to unit length per head (and q by `scale`)
 //   kFixedDecay     S <- decay_h S + k_t v_t^T;  o_t = S^T q_t, with SiLU applied to q, k, v on the way in
+//   kGatedWrite     S <- diag(f_t) S + (1 - f_t) v_t^T;  o_t = S^T q_t:  f_t = l + (1 - l) sigmoid(x_t + bias) per key
+//                   channel with a lower bound l, SiLU applied to q
 //
 // Everything that enters the recurrence (gates, decays, unit norms) is computed here in fp32 from the raw projections.
 // One block = 128 threads = 128 / TPR state rows (value channels) x TPR threads that share a row's key channels.
@@ -22,21 +24,22 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
-enum RecurrenceKind : int { kChannelDelta = 0, kFixedDecay = 1 };
+enum RecurrenceKind : int { kChannelDelta = 0, kFixedDecay = 1, kGatedWrite = 2 };
 
 // CH: tokens per staged chunk.  CH = 1 is the decode instance: few registers, so that enough state rows are in flight to
 // stream the states at memory rate.
 template <typename T, int DK, int TPR, int KIND, int CH>
-__global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kChannelDelta ? 4 : 6) : 1) linear_recurrence_kernel(const RecurrenceArgs p) {
+__global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kFixedDecay ? 6 : 4) : 1) linear_recurrence_kernel(const RecurrenceArgs p) {
   constexpr int RB = kThreads / TPR;                 // state rows of a block
   constexpr int QW = DK / TPR;                       // key channels of a thread
   constexpr int QK_PER = (CH * DK + kThreads - 1) / kThreads;
   constexpr int V_PER = (CH * RB + kThreads - 1) / kThreads;
   static_assert(QW % 4 == 0, "tile");
-  constexpr bool kDelta = KIND == kChannelDelta;
+  constexpr bool kDelta = KIND == kChannelDelta, kGated = KIND == kGatedWrite;
+  constexpr bool kHasA = kDelta || kGated;            // a per-channel projection beside q, k, v
   __shared__ __align__(16) float sk[CH][DK];
   __shared__ __align__(16) float sq[CH][DK];
-  __shared__ __align__(16) float sg[kDelta ? CH : 1][kDelta ? DK : 4];
+  __shared__ __align__(16) float sg[kHasA ? CH : 1][kHasA ? DK : 4];
   __shared__ float sv[CH][RB];
   __shared__ float sb[CH], srk[CH], srq[CH];
   griddep_launch();
@@ -49,7 +52,7 @@ __global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kCha
   const T* q = reinterpret_cast<const T*>(p.q) + hk * p.Dk;
   const T* k = reinterpret_cast<const T*>(p.k) + hk * p.Dk;
   const T* v = reinterpret_cast<const T*>(p.v) + h * p.Dv;
-  const T* a = reinterpret_cast<const T*>(p.a) + (kDelta ? h * p.Dk : 0);
+  const T* a = reinterpret_cast<const T*>(p.a) + (kHasA ? h * p.Dk : 0);
   const T* b = reinterpret_cast<const T*>(p.b) + (kDelta ? h : 0);
   const bool row_ok = row < p.Dv;
   // registers S[4i .. 4i+3] of lane qd hold key channels 4 (TPR i + qd) .. + 3: the TPR lanes of a row read
@@ -63,17 +66,17 @@ __global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kCha
     S[j] = x.x; S[j + 1] = x.y; S[j + 2] = x.z; S[j + 3] = x.w;
   }
   const float rate = kDelta ? -expf(p.A_log[h]) : 0.f;
-  const float decay = kDelta ? 0.f : p.decay[h];
-  float rq_[QK_PER], rk_[QK_PER], ra_[kDelta ? QK_PER : 1], rv_[V_PER], rb = 0.f;
+  const float decay = KIND == kFixedDecay ? p.decay[h] : 0.f;
+  float rq_[QK_PER], rk_[QK_PER], ra_[kHasA ? QK_PER : 1], rv_[V_PER], rb = 0.f;
   auto fetch = [&](int c0) {
 #pragma unroll
     for (int i = 0; i < QK_PER; ++i) {
       const int e = i * kThreads + tid, t = e / DK, d = e % DK;
       const bool ok = t < CH && c0 + t < L && d < p.Dk;
       const int64_t tok = s + c0 + t;
-      rk_[i] = ok ? to_f(k[tok * p.qkv_stride + d]) : 0.f;
+      if constexpr (!kGated) rk_[i] = ok ? to_f(k[tok * p.qkv_stride + d]) : 0.f;
       rq_[i] = ok ? to_f(q[tok * p.qkv_stride + d]) : 0.f;
-      if constexpr (kDelta) ra_[i] = ok ? to_f(a[tok * p.a_stride + d]) : 0.f;
+      if constexpr (kHasA) ra_[i] = ok ? to_f(a[tok * p.a_stride + d]) : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < V_PER; ++i) {
@@ -94,6 +97,17 @@ __global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kCha
           sk[t][d] = rk_[i];
           sq[t][d] = rq_[i];
           sg[t][d] = d < p.Dk ? expf(rate * softplus_f(ra_[i] + p.dt_bias[h * p.Dk + d])) : 0.f;
+        } else if constexpr (kGated) {
+          float f = 0.f, w = 0.f;     // kept and written share; padding channels stay zero
+          if (d < p.Dk) {
+            const float z = ra_[i] + p.dt_bias[h * p.Dk + d], low = p.lower[h * p.Dk + d];
+            const float e = expf(-fabsf(z)), big = 1.f / (1.f + e), small = e * big;   // sigmoid of |z| and of -|z|
+            f = low + (1.f - low) * (z >= 0.f ? big : small);
+            w = (1.f - low) * (z >= 0.f ? small : big);
+          }
+          sg[t][d] = f;
+          sk[t][d] = w;
+          sq[t][d] = silu_f(rq_[i]);
         } else {
           sk[t][d] = silu_f(rk_[i]);
           sq[t][d] = silu_f(rq_[i]);
@@ -103,7 +117,7 @@ __global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kCha
 #pragma unroll
     for (int i = 0; i < V_PER; ++i) {
       const int e = i * kThreads + tid, t = e / RB, d = e % RB;
-      if (t < n) sv[t][d] = kDelta ? rv_[i] : silu_f(rv_[i]);
+      if (t < n) sv[t][d] = KIND == kFixedDecay ? silu_f(rv_[i]) : rv_[i];
     }
     if (kDelta && tid < n) sb[tid] = sigmoid_f(rb);
     __syncthreads();
@@ -150,6 +164,18 @@ __global__ void __launch_bounds__(kThreads, CH == 1 && DK <= 128 ? (KIND == kCha
           o += S[j] * q4.x + S[j + 1] * q4.y;
           o2 += S[j + 2] * q4.z + S[j + 3] * q4.w;
         }
+      } else if constexpr (kGated) {
+        const float* gg = &sg[t][qd * 4];
+#pragma unroll
+        for (int j = 0; j < QW; j += 4) {
+          const float4 k4 = *reinterpret_cast<const float4*>(kk + j * TPR);
+          const float4 q4 = *reinterpret_cast<const float4*>(qq + j * TPR);
+          const float4 g4 = *reinterpret_cast<const float4*>(gg + j * TPR);
+          S[j] = S[j] * g4.x + vt * k4.x; S[j + 1] = S[j + 1] * g4.y + vt * k4.y;
+          S[j + 2] = S[j + 2] * g4.z + vt * k4.z; S[j + 3] = S[j + 3] * g4.w + vt * k4.w;
+          o += S[j] * q4.x + S[j + 1] * q4.y;
+          o2 += S[j + 2] * q4.z + S[j + 3] * q4.w;
+        }
       } else {
 #pragma unroll
         for (int j = 0; j < QW; j += 4) {
@@ -177,6 +203,8 @@ template <typename T, int DK, int TPR, int CH>
 void launch_ch(const RecurrenceArgs& a, dim3 grid, cudaStream_t st) {
   if (a.kind == kChannelDelta)
     launch_pdl(linear_recurrence_kernel<T, DK, TPR, kChannelDelta, CH>, grid, dim3(kThreads), 0, st, a);
+  else if (a.kind == kGatedWrite)
+    launch_pdl(linear_recurrence_kernel<T, DK, TPR, kGatedWrite, CH>, grid, dim3(kThreads), 0, st, a);
   else
     launch_pdl(linear_recurrence_kernel<T, DK, TPR, kFixedDecay, CH>, grid, dim3(kThreads), 0, st, a);
 }

@@ -237,13 +237,30 @@ __global__ void moe_scan_kernel(int* __restrict__ lod, int* __restrict__ cursor,
   if (lane == 0) lod[E_local] = run;
 }
 
-// One warp per (token, slot) pair: claim a row of the expert's segment and copy the token row there.
+// row copy, optionally times a factor
+template <typename T>
+__device__ __forceinline__ void copy_row(T* dst, const T* src, int H, int lane, const float* factor) {
+  constexpr int V = Vec16<T>::N;
+  if (factor == nullptr) {
+    for (int i = lane; i < H / V; i += 32) st_vec(dst + i * V, ld_vec(src + i * V));
+    return;
+  }
+  const float f = *factor;
+  for (int i = lane; i < H / V; i += 32) {
+    Vec16<T> a = ld_vec(src + i * V);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a.v[j] = from_f<T>(to_f(a.v[j]) * f);
+    st_vec(dst + i * V, a);
+  }
+}
+
+// One warp per (token, slot) pair: claim a row of the expert's segment and copy the token row there (times the pair's factor,
+// when the routing weights act on the experts' inputs).
 template <typename T>
 __global__ void moe_scatter_kernel(T* __restrict__ x_sorted, int* __restrict__ pos_of_pair, int* __restrict__ cursor,
                                    const T* __restrict__ x, const int* __restrict__ ids, const int* __restrict__ emap,
-                                   int64_t pairs, int k, int H, int E_local, int E_global, int64_t x_stride,
-                                   int64_t max_rows) {
-  constexpr int V = Vec16<T>::N;
+                                   const float* factors, int64_t pairs, int k, int H, int E_local, int E_global,
+                                   int64_t x_stride, int64_t max_rows) {
   griddep_launch();
   griddep_wait();
   const int64_t pair = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -260,8 +277,7 @@ __global__ void moe_scatter_kernel(T* __restrict__ x_sorted, int* __restrict__ p
   if (lane == 0) pos_of_pair[pair] = pos;
   if (pos < 0) return;
   const T* src = x + (pair / k) * x_stride;
-  T* dst = x_sorted + (int64_t)pos * H;
-  for (int i = lane; i < H / V; i += 32) st_vec(dst + i * V, ld_vec(src + i * V));
+  copy_row(x_sorted + (int64_t)pos * H, src, H, lane, factors == nullptr ? nullptr : factors + pair);
 }
 
 template <typename T>
@@ -334,8 +350,8 @@ constexpr int kSmallPairs = 1024;
 template <typename T, bool kQuant>
 __global__ void __launch_bounds__(256) moe_prepare_small_kernel(
     void* __restrict__ x_sorted, float* __restrict__ scale_t, int64_t s_stride, int* __restrict__ pos_of_pair,
-    int* __restrict__ lod, const T* __restrict__ x, const int* __restrict__ ids, const int* __restrict__ emap, int pairs,
-    int k, int H, int E_local, int E_global, int64_t x_stride) {
+    int* __restrict__ lod, const T* __restrict__ x, const int* __restrict__ ids, const int* __restrict__ emap,
+    const float* factors, int pairs, int k, int H, int E_local, int E_global, int64_t x_stride) {
   extern __shared__ int sh[];          // [E_local + 1] lod | [pairs] expert of pair | [pairs] position
   int* s_lod = sh;
   int* s_e = sh + E_local + 1;
@@ -406,9 +422,7 @@ __global__ void __launch_bounds__(256) moe_prepare_small_kernel(
         if (lane == 0) scale_t[(int64_t)g * s_stride + pos] = scale;
       }
     } else {
-      constexpr int V = Vec16<T>::N;
-      T* dst = reinterpret_cast<T*>(x_sorted) + (int64_t)pos * H;
-      for (int i = lane; i < H / V; i += 32) st_vec(dst + i * V, ld_vec(src + i * V));
+      copy_row(reinterpret_cast<T*>(x_sorted) + (int64_t)pos * H, src, H, lane, factors == nullptr ? nullptr : factors + p);
     }
   }
 }
@@ -502,8 +516,8 @@ extern "C" int b200_moe_route(float* out_w, int* out_ids, const void* logits, co
 }
 
 extern "C" int b200_moe_permute(void* x_sorted, int* pos_of_pair, int* lod, int* counts, int* cursor, const void* x,
-                                const int* ids, const int* emap, int64_t T_, int k, int H, int E_local, int E_global,
-                                int64_t x_stride, int64_t max_rows, int dtype, cudaStream_t st) {
+                                const int* ids, const int* emap, const float* factors, int64_t T_, int k, int H,
+                                int E_local, int E_global, int64_t x_stride, int64_t max_rows, int dtype, cudaStream_t st) {
   const int64_t pairs = T_ * k;
   int blocks = (int)((pairs + 255) / 256);
   if (blocks > 256) blocks = 256;
@@ -515,7 +529,7 @@ extern "C" int b200_moe_permute(void* x_sorted, int* pos_of_pair, int* lod, int*
     B200_DISPATCH_DTYPE(dtype, {
       if (H % Vec16<T>::N) return 2;
       launch_pdl(moe_scatter_kernel<T>, dim3((pairs + 7) / 8), dim3(256), 0, st, (T*)x_sorted, pos_of_pair, cursor,
-                 (const T*)x, ids, emap, pairs, k, H, E_local, E_global, x_stride, max_rows);
+                 (const T*)x, ids, emap, factors, pairs, k, H, E_local, E_global, x_stride, max_rows);
     });
   }
   return (int)cudaGetLastError();
@@ -582,10 +596,10 @@ extern "C" int b200_quant_fp8_group(void* q, float* scale_t, const void* x, int6
 extern "C" int b200_moe_small_pairs() { return kSmallPairs; }
 
 extern "C" int b200_moe_prepare_small(void* x_sorted, float* scale_t, int64_t s_stride, int* pos_of_pair, int* lod,
-                                      const void* x, const int* ids, const int* emap, int64_t T_, int k, int H, int E_local,
-                                      int E_global, int64_t x_stride, int quant, int dtype, cudaStream_t st) {
+                                      const void* x, const int* ids, const int* emap, const float* factors, int64_t T_,
+                                      int k, int H, int E_local, int E_global, int64_t x_stride, int quant, int dtype, cudaStream_t st) {
   const int pairs = (int)(T_ * k);
-  if (pairs > kSmallPairs || pairs < 1 || (quant && H % 128)) return 2;
+  if (pairs > kSmallPairs || pairs < 1 || (quant && (H % 128 || factors != nullptr))) return 2;
   const size_t smem = (size_t)(E_local + 1 + 2 * pairs) * sizeof(int);
   int grid = (pairs + 7) / 8;
   if (grid > 64) grid = 64;
@@ -593,10 +607,10 @@ extern "C" int b200_moe_prepare_small(void* x_sorted, float* scale_t, int64_t s_
     if (H % Vec16<T>::N) return 2;
     if (quant)
       launch_pdl(moe_prepare_small_kernel<T, true>, dim3(grid), dim3(256), smem, st, x_sorted, scale_t, s_stride, pos_of_pair,
-                 lod, (const T*)x, ids, emap, pairs, k, H, E_local, E_global, x_stride);
+                 lod, (const T*)x, ids, emap, factors, pairs, k, H, E_local, E_global, x_stride);
     else
       launch_pdl(moe_prepare_small_kernel<T, false>, dim3(grid), dim3(256), smem, st, x_sorted, scale_t, s_stride,
-                 pos_of_pair, lod, (const T*)x, ids, emap, pairs, k, H, E_local, E_global, x_stride);
+                 pos_of_pair, lod, (const T*)x, ids, emap, factors, pairs, k, H, E_local, E_global, x_stride);
   });
   return (int)cudaGetLastError();
 }

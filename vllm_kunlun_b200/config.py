@@ -40,7 +40,8 @@ class LayerSpec:
 
     type: str                   # name of the mixer (``models/mixers.py``)
     mixer: dict                 # its sizes and constants
-    mlp: Optional[dict] = None  # {"kind": "dense", "ff": width}, or None: the layer has no feed-forward
+    mlp: Optional[dict] = None  # {"kind": "dense", "ff": width} or {"kind": "moe", "expert": {"ff", "limit"}, "router":
+    # {"experts", "top"}} (``models/feed_forward.py``), or None: the layer has no feed-forward
 
 
 @dataclass
@@ -67,7 +68,7 @@ class ModelConfig:
     o_bias: bool = False
     mlp_bias: bool = False
     qk_norm: bool = False  # per-head q/k RMSNorm (Qwen3)
-    hidden_act: str = "silu"  # "silu" | "swigluoai" | "gelu_tanh"
+    hidden_act: str = "silu"  # "silu" | "swigluoai" | "gelu_tanh" | "poly_norm" (listed layers: no gate matrix)
     gemma_norm: bool = False  # (1 + w) RMSNorm
     # sliding window / sinks (GPT-OSS, MiMo-V2, Gemma)
     sliding_window: Optional[int] = None
@@ -128,11 +129,12 @@ class ModelConfig:
     global_head_dim: Optional[int] = None  # head size of the full-attention layers when it differs (Gemma-4)
     num_global_kv_heads: Optional[int] = None  # their KV head count when values are the keys (attention_k_eq_v)
     attention_k_eq_v: bool = False  # full-attention layers have no v_proj: V is the (un-normalised, un-rotated) K
-    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel, Seturax)
+    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel, Seturax, Petipel)
     embedding_scale: float = 1.0  # factor of the token rows
     bigram: Optional[dict] = None  # embedding of token pairs: {"buckets", "mul_prev", "mul_cur"}
     token_shift: bool = False  # the mixers read a blend of this token's and the previous token's norm
     logit_scale: float = 1.0
+    residual_multiplier: float = 1.0  # factor of every sublayer's contribution to the stream
     attn_output_gate: bool = False  # q_proj carries a sigmoid output gate (Qwen3-Next full-attention layers)
     # quantization of the checkpoint
     quantization: Optional[str] = None  # None | "fp8" | "int8" | "awq" | "gptq" | "w4a16"
@@ -478,14 +480,16 @@ class ModelConfig:
     @classmethod
     def _from_layer_list(cls, cfg: dict) -> "ModelConfig":
         """Configurations that list their layers one by one (``architecture``, ``width``, ``vocab``, ``norm.eps``,
-        ``layers: [{type, mixer, mlp}]``; optionally ``embedding.{scale, bigram}`` and ``logit_scale``)."""
+        ``layers: [{type, mixer, mlp}]``; optionally ``embedding.{scale, bigram}``, ``logit_scale`` and
+        ``residual_mult``)."""
+        from .models.feed_forward import FEED_FORWARDS
         from .models.mixers import MIXERS
         specs = []
         for i, entry in enumerate(cfg["layers"]):
             if entry["type"] not in MIXERS:
                 raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}; known: {sorted(MIXERS)}")
             mlp = entry.get("mlp")
-            if mlp is not None and mlp.get("kind", "dense") != "dense":
+            if mlp is not None and mlp.get("kind", "dense") not in FEED_FORWARDS:
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
             specs.append(LayerSpec(entry["type"], dict(entry["mixer"]), None if mlp is None else dict(mlp)))
         arch = cfg["architecture"]
@@ -493,11 +497,12 @@ class ModelConfig:
         bigram = emb.get("bigram")
         return cls(architecture=arch, name=cfg.get("_name_or_path", arch), vocab_size=int(cfg["vocab"]),
                    hidden_size=int(cfg["width"]), num_layers=len(specs), num_heads=1, num_kv_heads=1, head_dim=1,
-                   intermediate_size=max([1] + [int(s.mlp["ff"]) for s in specs if s.mlp]),
+                   intermediate_size=max([1] + [int((s.mlp.get("expert") or s.mlp)["ff"]) for s in specs if s.mlp]),
                    rms_norm_eps=float(cfg["norm"]["eps"]), max_position=1 << 30, layer_specs=tuple(specs),
                    embedding_scale=float(emb.get("scale", 1.0)),
                    bigram=None if bigram is None else {k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")},
-                   logit_scale=float(cfg.get("logit_scale", 1.0)), dtype=str(cfg.get("torch_dtype", "bfloat16")),
+                   logit_scale=float(cfg.get("logit_scale", 1.0)),
+                   residual_multiplier=float(cfg.get("residual_mult", 1.0)), dtype=str(cfg.get("torch_dtype", "bfloat16")),
                    **_LAYER_LIST_TRAITS.get(arch, {}))
 
     def complete_from_shapes(self, shapes: dict) -> "ModelConfig":
@@ -520,7 +525,8 @@ class ModelConfig:
 
 
 # what a design with listed layers fixes without naming it in its configuration
-_LAYER_LIST_TRAITS: dict = {"Seturax": {"hidden_act": "gelu_tanh", "token_shift": True}}
+_LAYER_LIST_TRAITS: dict = {"Seturax": {"hidden_act": "gelu_tanh", "token_shift": True},
+                            "Petipel": {"hidden_act": "poly_norm"}}
 
 
 def _leading_dense(cfg: dict) -> int:

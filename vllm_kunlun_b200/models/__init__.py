@@ -41,6 +41,8 @@ _REGISTRY = {
     "Bolopel": "bolopel:BolopelForCausalLM",
     # windowed latent attention beside the feed-forward, gated residuals, token shift, bigram embedding
     "Seturax": "seturax:SeturaxForCausalLM",
+    # attention with a bias by distance and mixed values beside HGRN2, norms around every sublayer, experts on weighted inputs
+    "Petipel": "petipel:PetipelForCausalLM",
     # asymmetric V / sliding window with sinks
     "MiMoV2FlashForCausalLM": "mimo_v2_flash:MiMoV2FlashForCausalLM",
     # Gemma family

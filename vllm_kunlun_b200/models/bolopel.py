@@ -31,9 +31,9 @@ class BolopelDecoderLayer(ListedLayer):
         self.mlp_norm = None if self.mlp is None else NormWeight(cfg.hidden_size, device)
 
     @classmethod
-    def tensor_shapes(cls, spec: LayerSpec, width: int) -> dict:
+    def tensor_shapes(cls, spec: LayerSpec, width: int, act: str) -> dict:
         norms = ("norm1",) if spec.mlp is None else ("norm1", "norm2")
-        return {**{n: (width,) for n in norms}, **super().tensor_shapes(spec, width)}
+        return {**{n: (width,) for n in norms}, **super().tensor_shapes(spec, width, act)}
 
     def forward(self, x, h):
         h = ops.layernorm_residual(x, self.dtype, self.mixer(h), self.mixer_norm.weight, self.eps)

@@ -3,8 +3,8 @@ per-request state, strict checkpoint loading, random initialisation.  A design a
 the tensors outside the layers.
 
 The residual stream and every norm are fp32; the GEMMs read copies in the model's dtype.  Rows are padded to a multiple of 8
-columns (zeros) and feed-forward widths to a multiple of 64 (the fused gate / up epilogue), so any width runs through the
-tensor-core GEMMs.  Checkpoint tensors of layer i are named ``l<i>.*``, its mixer's ``l<i>.mix.*``.
+columns (zeros), so any width runs through the tensor-core GEMMs.  Checkpoint tensors of layer i are named ``l<i>.*``, its
+mixer's ``l<i>.mix.*``, its feed-forward's (``models/feed_forward.py``) ``l<i>.mlp.*``.
 """
 from __future__ import annotations
 
@@ -13,13 +13,12 @@ from typing import Iterable, Optional
 import torch
 import torch.nn as nn
 
-from ..config import LayerSpec, ModelConfig, round_up
+from ..config import LayerSpec, ModelConfig
 from ..parallel.state import get_state
 from .dense import DenseForCausalLM, GatedMLP
+from .feed_forward import feed_forward_cls
 from .layers import DTYPES, ParallelLMHead, VocabParallelEmbedding, param
 from .mixers import MIXERS, align, padded
-
-MLP_TILE = 64
 
 
 class NormWeight(nn.Module):
@@ -38,33 +37,31 @@ class ListedLayer(nn.Module):
         self.mixer = MIXERS[spec.type](self.ld, spec.mixer, layer_idx, cfg.rms_norm_eps, dtype, device)
         self.mlp = None
         if spec.mlp is not None:
-            self.mlp = GatedMLP(self.ld, round_up(int(spec.mlp["ff"]), MLP_TILE), dtype, device, act=cfg.hidden_act)
+            self.mlp = feed_forward_cls(spec.mlp, cfg.hidden_act)(self.ld, spec.mlp, cfg.hidden_act, cfg.rms_norm_eps, dtype,
+                                                                  device)
 
     @classmethod
-    def tensor_shapes(cls, spec: LayerSpec, width: int) -> dict:
+    def tensor_shapes(cls, spec: LayerSpec, width: int, act: str) -> dict:
         """Name (behind ``l<i>.``) -> shape of the mixer's and the feed-forward's tensors."""
         out = {f"mix.{k}": s for k, s in MIXERS[spec.type].tensor_shapes(spec.mixer, width).items()}
         if spec.mlp is not None:
-            ff = int(spec.mlp["ff"])
-            out.update({"mlp.gate": (ff, width), "mlp.up": (ff, width), "mlp.down": (width, ff)})
+            shapes = feed_forward_cls(spec.mlp, act).tensor_shapes(spec.mlp, width)
+            out.update({f"mlp.{k}": s for k, s in shapes.items()})
         return out
 
     @classmethod
     def unused_tensors(cls, spec: LayerSpec) -> tuple:
         """Names that a checkpoint may carry without effect."""
-        return ()
+        unused = getattr(MIXERS[spec.type], "unused_tensors", None)
+        return () if unused is None else tuple(f"mix.{k}" for k in unused(spec.mixer))
 
     def state_spec(self, dtype) -> list:
         """``(shape per request, dtype)`` of everything the layer keeps per request, the mixer's first."""
         return self.mixer.state_spec(dtype) if self.mixer.has_state else []
 
     def load_tensor(self, key: str, w: torch.Tensor):
-        if key in ("mlp.gate", "mlp.up"):
-            gu = self.mlp.gate_up_proj
-            gu.load("weight", padded(w, gu.output_sizes[0], gu.in_features), 0 if key == "mlp.gate" else 1)
-        elif key == "mlp.down":
-            dn = self.mlp.down_proj
-            dn.load("weight", padded(w, dn.out_features, dn.in_features))
+        if key.startswith("mlp."):
+            self.mlp.load_tensor(key.removeprefix("mlp."), w)
         elif key.startswith("mix."):
             self.mixer.load_tensor(key.removeprefix("mix."), w)
         else:
@@ -73,6 +70,7 @@ class ListedLayer(nn.Module):
 
 class LayerListForCausalLM(DenseForCausalLM):
     layer_cls = ListedLayer
+    unit_norm_init = 1.0        # what a norm weight of a freshly initialised model is stored as
 
     def __init__(self, cfg: ModelConfig, device="cpu", dtype: Optional[torch.dtype] = None):
         nn.Module.__init__(self)
@@ -129,7 +127,7 @@ class LayerListForCausalLM(DenseForCausalLM):
         """Name -> shape of every tensor of a checkpoint with this configuration."""
         out = dict(self.outer_tensor_shapes())
         for i, spec in enumerate(self.cfg.layer_specs):
-            out.update({f"l{i}.{k}": s for k, s in self.layer_cls.tensor_shapes(spec, self.width).items()})
+            out.update({f"l{i}.{k}": s for k, s in self.layer_cls.tensor_shapes(spec, self.width, self.cfg.hidden_act).items()})
         return out
 
     def init_random(self, seed: int = 0, std: float = 0.02):
@@ -142,15 +140,18 @@ class LayerListForCausalLM(DenseForCausalLM):
                 t = torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
                 leaf = name.rsplit(".", 1)[-1]
                 if "norm" in leaf:
-                    t = torch.ones_like(t)
+                    # norms inside a mixer have plain weights
+                    t = torch.full_like(t, 1.0 if ".mix." in name else self.unit_norm_init)
                 elif leaf == "A_log":
                     t = t.clamp(-1.0, 1.0)
                 elif leaf == "dt_bias":
                     t = t.clamp(-1.0, 1.0) - 3.0
                 elif leaf == "conv":
                     t = t * (10.0 * std)
-                elif leaf == "shift":
+                elif leaf in ("shift", "lower", "vmix"):
                     t = torch.sigmoid(t)
+                elif leaf in ("rel", "act"):
+                    t = t.clamp(-1.0, 1.0)
                 else:
                     t = t * std
                 yield name, t.to(self.dtype)

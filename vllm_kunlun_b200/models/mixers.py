@@ -9,6 +9,9 @@ A mixer reads the residual stream's 16-bit (or fp32) copy ``h [T, ld]`` and retu
 * :class:`LightningAttention` linear attention with a fixed decay per head, jointly normed and gated output
 * :class:`ParallelMixer`     both of them on the same input, one input projection, scaled sum
 * :class:`ChannelDelta`      short convolutions + delta rule with one decay per head and key channel
+* :class:`DistanceBiasAttention` softmax attention with a learned score bias by distance, a query temperature, unit-RMS values
+  that layers may share, output gate per head
+* :class:`GatedWriteAttention` linear attention whose forget gate decides what is written (HGRN2)
 * :class:`LatentAttention`   windowed attention over a shared latent row per token, learned sink, output gate per head
 
 Checkpoint rows are padded so that every column slice of a fused projection starts on a 16-byte boundary; padding rows
@@ -35,12 +38,12 @@ def align(n: int) -> int:
     return round_up(n, ALIGN)
 
 
-def cache_head_dim(dim: int, vdim: int, dtype: torch.dtype) -> int:
+def cache_head_dim(dim: int, vdim: int, dtype: torch.dtype, served=_TENSOR_CORE_HEADS) -> int:
     """Head size of the paged cache: keys and values share it, zero-padded to one the attention kernels serve."""
     n = max(dim, vdim)
     if dtype == torch.float32:
         return round_up(n, 4)
-    return next((d for d in _TENSOR_CORE_HEADS if d >= n), align(n))
+    return next((d for d in served if d >= n), align(n))
 
 
 def padded(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
@@ -90,6 +93,8 @@ class WindowAttention(nn.Module):
     square.  ``window``: position i sees the last ``window`` positions up to itself (None = all of them).  ``sink``: a
     constant score without a value that joins the softmax denominator (None = no sink)."""
 
+    served_heads = _TENSOR_CORE_HEADS       # cache head sizes of the tensor-core kernels that this attention can use
+
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: Optional[int],
                  sink: Optional[float], eps: float, dtype, device):
         super().__init__()
@@ -97,7 +102,7 @@ class WindowAttention(nn.Module):
             raise ValueError(f"{heads} query heads do not divide over {kv_heads} key / value heads")
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
         self.scale, self.window, self.eps = float(scale), window, eps
-        self.cache_dim = cache_head_dim(dim, vdim, dtype)
+        self.cache_dim = cache_head_dim(dim, vdim, dtype, self.served_heads)
         self.sinks = None if sink is None else param(heads, dtype=torch.float32, device=device)
         if sink is not None:
             self.sinks.data.fill_(sink)
@@ -124,6 +129,111 @@ class WindowAttention(nn.Module):
             num_decodes=md.num_decodes, decode_query_len=1 + md.num_spec_tokens,
             num_decode_tokens=md.num_decode_tokens, stable_metadata=True)
         return self.o(o.reshape(T, self.heads * self.cache_dim))
+
+
+def distance_buckets(rows: int, far: int) -> list:
+    """Row of a distance table per distance 0, 1, ... up to the first one from which on all share the last row.  The first
+    half of the rows serve one distance each; row ``h + m`` (``h = rows // 2``) starts at ``h (far / h)^(m / (rows - h))``,
+    decided in integers, so that no rounding moves a boundary."""
+    h = rows // 2
+    log_rows = rows - h
+    if not 0 < h < far:
+        raise ValueError(f"a distance table of {rows} rows that ends at {far}")
+    out, n, m = list(range(h)), h, 0
+    while h + m < rows - 1:
+        while h + m < rows - 1 and n ** log_rows * h ** (m + 1) >= far ** (m + 1) * h ** log_rows:
+            m += 1
+        out.append(h + m)
+        n += 1
+    return out
+
+
+class DistanceBiasAttention(WindowAttention):
+    """Causal softmax attention without rotation: positions enter through a learned bias per head and distance (added to the
+    scaled scores) and through a temperature ``1 + coef ln(floor((p + 1) / every) + 1)`` of the query at position p.  Every
+    value head is divided by its root mean square; layers that share values (``v_mix``) blend them with those of the first
+    such layer (same token), and the cache holds the blend.  Every head's output is multiplied by ``sigmoid`` of its gate."""
+
+    has_state = False
+    cache_block = 64                        # tokens per cache block that the tensor-core kernels take
+    served_heads = (128,)
+    VALUES = "first_values"                 # where the first sharing layer leaves its values for the step's later layers
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        if "rel" in shapes:
+            sizes["bias_rows"] = int(shapes["rel"][0])
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        m = sizes
+        super().__init__(width, m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], None, None, eps, dtype, device)
+        self.layer_idx = layer_idx
+        temp = m.get("q_temp")
+        self.temperature = None if temp is None else (float(temp["coef"]), int(temp["every"]))
+        self.shares_values, self.first_of_sharing, self.value_share = bool(m.get("v_mix")), False, 0.0
+        self.buckets = torch.tensor(distance_buckets(self._bias_rows(m), int(m["bias_max"])), device=device)
+        self.bias = param(self.heads, self.buckets.numel(), dtype=torch.float32, device=device)
+        self.in_proj = FusedProjection(width, {**self.proj_sizes(), "g": self.heads}, dtype, device)
+
+    @staticmethod
+    def _bias_rows(sizes: dict) -> int:
+        return int(sizes.get("bias_rows", 32))
+
+    @classmethod
+    def tensor_shapes(cls, sizes: dict, width: int) -> dict:
+        H, G, D, V = (sizes[k] for k in ("heads", "kv_heads", "dim", "vdim"))
+        out = {"q": (H * D, width), "k": (G * D, width), "v": (G * V, width), "rel": (cls._bias_rows(sizes), H),
+               "g": (H, width), "o": (width, H * V)}
+        return {**out, "vmix": ()} if sizes.get("v_mix") else out
+
+    @staticmethod
+    def unused_tensors(sizes: dict) -> tuple:
+        return () if sizes.get("v_mix") else ("vmix",)
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        if key == "o":
+            self.load_o(w)
+        elif key == "rel":
+            self.bias.data.copy_(w.to(self.bias.device).float()[self.buckets].T)
+        elif key == "vmix":
+            self.value_share = float(w)
+        else:
+            self.in_proj.load_part(key, w)
+
+    def state_spec(self, dtype):
+        return []
+
+    def workspace_size(self) -> tuple:
+        return self.heads, self.cache_dim
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md, p, T = ctx.attn, self.in_proj, h.shape[0]
+        kv_cache = ctx.kv_caches[self.layer_idx]
+        y = p(h)
+        v_out = v_in = None
+        if self.shares_values:
+            if self.first_of_sharing:
+                v_out = md.extras[self.VALUES] = torch.empty(T, self.kv_heads * self.vdim, dtype=h.dtype, device=h.device)
+            else:
+                v_in = md.extras[self.VALUES]
+        q = ops.attn_prep_cache(p.slice(y, "q"), p.slice(y, "k"), p.slice(y, "v"), kv_cache, md.slot_mapping, md.positions,
+                                self.heads, self.kv_heads, self.eps, self.temperature, v_out, v_in, self.value_share)
+        o = ops.paged_attention(
+            q, kv_cache, md.block_tables, md.seq_lens, md.query_start_loc, self.scale, md.max_query_len, md.max_seq_len,
+            None, None, md.seq_lens_cpu, md.query_start_loc_cpu, workspace=md.workspace, num_decodes=md.num_decodes,
+            decode_query_len=1 + md.num_spec_tokens, num_decode_tokens=md.num_decode_tokens, stable_metadata=True,
+            bias=self.bias, gate=p.slice(y, "g"))
+        return [(self.o(o.reshape(T, self.heads * self.cache_dim)), 1.0)]
+
+
+def link_shared_values(mixers) -> None:
+    """The first of the layers that share values is their source; the others need values of the same shape."""
+    sharing = [m for m in mixers if getattr(m, "shares_values", False)]
+    for i, m in enumerate(sharing):
+        m.first_of_sharing = i == 0
+        if m.kv_heads * m.vdim != sharing[0].kv_heads * sharing[0].vdim:
+            raise ValueError("layers that share values have different numbers or sizes of value heads")
 
 
 class LightningAttention(nn.Module):
@@ -330,6 +440,64 @@ class ChannelDelta(nn.Module):
         return [(self.o(z), 1.0)]
 
 
+class GatedWriteAttention(nn.Module):
+    """HGRN2: ``S <- diag(f) S + (1 - f) v^T``, ``o = S^T silu(q)``; the forget gate ``f = l + (1 - l) sigmoid(W_f h + b)`` per
+    head and channel has a lower bound l.  Every head's output is RMS-normed with a weight that the heads share."""
+
+    has_state = True
+    cache_block = None
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        pass
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        super().__init__()
+        self.layer_idx, self.eps = layer_idx, eps
+        self.heads, self.dim, self.vdim = sizes["heads"], sizes["dim"], sizes["vdim"]
+        n, nv = self.heads * self.dim, self.heads * self.vdim
+        self.in_proj = FusedProjection(width, {"q": n, "f": n, "v": nv}, dtype, device)
+        self.f_bias, self.lower = (param(n, dtype=torch.float32, device=device) for _ in range(2))
+        self.norm = nn.Module()
+        self.norm.weight = param(self.vdim, dtype=torch.float32, device=device)
+        self.o = output_projection(align(nv), width, dtype, device)
+
+    @staticmethod
+    def tensor_shapes(sizes: dict, width: int) -> dict:
+        n, nv = sizes["heads"] * sizes["dim"], sizes["heads"] * sizes["vdim"]
+        return {"q": (n, width), "f": (n, width), "f.b": (n,), "lower": (n,), "v": (nv, width), "norm": (sizes["vdim"],),
+                "o": (width, nv)}
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        if key == "o":
+            self.o.weight.data[:w.shape[0], :w.shape[1]].copy_(w)
+        elif key in ("f.b", "lower", "norm"):
+            {"f.b": self.f_bias, "lower": self.lower, "norm": self.norm.weight}[key].data.copy_(w)
+        else:
+            self.in_proj.load_part(key, w)
+
+    def kv_cache_spec(self, block_size: int, dtype):
+        return None
+
+    def state_spec(self, dtype):
+        return [((self.heads, self.vdim, round_up(self.dim, 4)), torch.float32)]
+
+    def workspace_size(self) -> tuple:
+        return 0, 0
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md, p, T, H = ctx.attn, self.in_proj, h.shape[0], self.heads
+        state, = ctx.kv_caches[self.layer_idx]
+        y = p(h)
+        o = ops.gated_write_attention(_heads(p.slice(y, "q"), H, self.dim), _heads(p.slice(y, "v"), H, self.vdim),
+                                      p.slice(y, "f"), self.f_bias, self.lower, state, md.query_start_loc, md.state_indices,
+                                      md.has_initial_state, md.max_query_len, md.num_decodes)
+        n = H * self.vdim
+        z = ops.gated_group_rmsnorm(o.reshape(T, n), None, self.norm.weight, self.eps, _rows(T, n, h.dtype, h.device))
+        return [(self.o(z), 1.0)]
+
+
 class LatentAttention(nn.Module):
     """Multi-head attention over one latent row per token.  Queries come through their own latent; keys and values are
     per-head products of the cached latent, plus one rotated key part that all heads share.  Optional sliding ``window``,
@@ -484,4 +652,5 @@ def rotary_tables(mixers, md) -> None:
             md.extras["rotary"][key] = ops.rotary_table(md.positions, m.turns)
 
 
-MIXERS = {"channel_delta": ChannelDelta, "latent_attention": LatentAttention, "parallel": ParallelMixer}
+MIXERS = {"attention": DistanceBiasAttention, "channel_delta": ChannelDelta, "hgrn2": GatedWriteAttention,
+          "latent_attention": LatentAttention, "parallel": ParallelMixer}

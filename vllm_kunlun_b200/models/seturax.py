@@ -42,8 +42,8 @@ class SeturaxDecoderLayer(ListedLayer):
         self.gates.bias.data.zero_()
 
     @classmethod
-    def tensor_shapes(cls, spec: LayerSpec, width: int) -> dict:
-        out = {"norm1": (width,), "shift": (width,), **super().tensor_shapes(spec, width)}
+    def tensor_shapes(cls, spec: LayerSpec, width: int, act: str) -> dict:
+        out = {"norm1": (width,), "shift": (width,), **super().tensor_shapes(spec, width, act)}
         for k in range(1 if spec.mlp is None else 2):
             out.update({f"rg{k + 1}": (width, width), f"rg{k + 1}.b": (width,)})
         return out

@@ -19,6 +19,7 @@ from .reference import latent as _rt
 from .reference import linear_recurrence as _rl
 from .reference import misc as _rx
 from .reference import moe as _rm
+from .reference import sandwich as _rs
 
 reference_basic = _rb
 reference_attention = _ra
@@ -70,15 +71,19 @@ def l2norm(x, eps: float = 1e-6):
     return _rb.l2norm(x, eps)
 
 
-_ACT_CODES = {"silu": 0, "gelu_tanh": 1, "swigluoai": 2}
+_ACT_CODES = {"silu": 0, "gelu_tanh": 1, "swigluoai": 2, "swiglu_limit": 3}
 
 
-def act_and_mul(x, act: str = "silu"):
+def act_and_mul(x, act: str = "silu", limit: float = 0.0):
+    """``swiglu_limit``: ``g sigmoid(1.702 g) (u + 1)`` with ``g`` capped at ``limit`` and ``u`` clamped to ``+-limit``
+    (``x = [gate | up]``; ``swigluoai`` is the same function with a limit of 7 over interleaved columns)."""
     if x.is_cuda:
         d = x.shape[-1] // 2
         out = torch.empty(*x.shape[:-1], d, dtype=x.dtype, device=x.device)
-        _c().act_and_mul(out, x, _ACT_CODES[act])
+        _c().act_and_mul(out, x, _ACT_CODES[act], limit)
         return out
+    if act == "swiglu_limit":
+        return _rs.swiglu_limit_and_mul(x, limit)
     if act == "silu":
         return _rb.silu_and_mul(x)
     if act == "swigluoai":
@@ -191,8 +196,11 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale:
                     max_query_len: int, max_seq_len: int, window: Optional[int] = None, sinks=None,
                     seq_lens_cpu=None, query_start_loc_cpu=None, out=None, workspace=None,
                     num_decodes: int = 0, decode_query_len: int = 1, num_decode_tokens: int = 0,
-                    stable_metadata: bool = False):
+                    stable_metadata: bool = False, bias=None, gate=None):
     """Unified varlen paged GQA attention (prefill with prefix, decode, spec-verify).
+
+    ``bias [Hq, n]`` (fp32): added to the scaled scores by distance (position of the query minus the key's), the last entry
+    for every distance from ``n - 1`` on.  ``gate [T, Hq]``: every head's output is multiplied by its sigmoid.
 
     The batch is decode-first: the first ``num_decodes`` requests have at most ``decode_query_len``
     query tokens each.  On CUDA a mixed batch is served by two launches (decode layout with
@@ -206,17 +214,18 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale:
             ndt = num_decode_tokens or num_decodes * decode_query_len
             paged_attention_cuda(out[:ndt], q[:ndt], kv_cache, block_tables[:num_decodes], seq_lens[:num_decodes],
                                  query_start_loc[:num_decodes + 1], scale, decode_query_len, max_seq_len,
-                                 window, sinks, workspace, stable_metadata=stable_metadata)
+                                 window, sinks, workspace, stable_metadata=stable_metadata, bias=bias,
+                                 gate=None if gate is None else gate[:ndt])
             paged_attention_cuda(out, q, kv_cache, block_tables[num_decodes:], seq_lens[num_decodes:],
                                  query_start_loc[num_decodes:], scale, max_query_len, max_seq_len,
-                                 window, sinks, workspace)
+                                 window, sinks, workspace, bias=bias, gate=gate)
             return out
         return paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
                                     max_query_len, max_seq_len, window, sinks, workspace,
-                                    stable_metadata=stable_metadata)
+                                    stable_metadata=stable_metadata, bias=bias, gate=gate)
     sl = seq_lens if seq_lens_cpu is None else seq_lens_cpu
     ql = query_start_loc if query_start_loc_cpu is None else query_start_loc_cpu
-    return _ra.paged_attention(q, kv_cache, block_tables, sl, ql, scale, window, sinks)
+    return _ra.paged_attention(q, kv_cache, block_tables, sl, ql, scale, window, sinks, bias=bias, gate=gate)
 
 
 def merge_attn_states(o1, lse1, o2, lse2):
@@ -349,17 +358,25 @@ def int8_linear(x, w_q, w_scale, bias=None, input_scale=None, out_dtype=torch.bf
 
 # ----------------------------------------------------------------------------- MoE
 
-def router_gemm(x, weight, bias=None):
+def router_gemm(x, weight, bias=None, fp32: bool = False):
     """Router logits ``x @ W.T (+ b)``.  CUDA, decode-sized batches: a CUDA-core kernel with fp32 output (the
-    tensor-core GEMM's fixed cost dominates at this size); otherwise the ordinary linear."""
+    tensor-core GEMM's fixed cost dominates at this size); otherwise the ordinary linear, or with ``fp32`` (no bias) the
+    grouped tensor-core GEMM with its fp32 output."""
     if x.is_cuda and x.dim() == 2 and x.shape[0] <= 64 and weight.shape[0] <= 1024 and weight.dtype == x.dtype:
         return _c().router_gemm_small(x if x.stride(-1) == 1 else x.contiguous(), weight, bias)
+    if fp32 and x.dtype != torch.float32:
+        assert bias is None
+        if x.is_cuda:
+            out = torch.empty(x.shape[0], weight.shape[0], dtype=torch.float32, device=x.device)
+            _c().grouped_gemm(out, x, weight, None, None, None, None, 0)
+            return out
+        return _rb.linear(x.float(), weight.float())
     return linear(x, weight, bias)
 
 
 def router_and_route(x, weight, wbias, k: int, scoring: str = "softmax", renormalize: bool = True, bias=None,
-                     n_group: int = 1, topk_group: int = 1, scale: float = 1.0):
-    """Router logits and top-k routing from the hidden states.  CUDA, decode-sized batches with a SMALL router
+                     n_group: int = 1, topk_group: int = 1, scale: float = 1.0, fp32: bool = False):
+    """Router logits (``fp32``: as in :func:`router_gemm`) and top-k routing from the hidden states.  CUDA, decode-sized batches with a SMALL router
     (at most 64 K weights): one launch, logits stay in shared memory.  Larger routers keep two kernels: one CTA per
     token cannot pull a 128 x 2048 router through a single SM fast enough (measured: Qwen3-30B-A3B decode step
     8.69 ms with two kernels, 9.79 ms fused), while the GEMM kernel spreads a token over E / 32 CTAs."""
@@ -370,7 +387,7 @@ def router_and_route(x, weight, wbias, k: int, scoring: str = "softmax", renorma
                                          None if bias is None else bias.float(), k, _MODES[scoring], renormalize,
                                          n_group, topk_group, scale)
         return w, ids
-    return moe_route(router_gemm(x, weight, wbias), k, scoring, renormalize, bias, n_group, topk_group, scale)
+    return moe_route(router_gemm(x, weight, wbias, fp32), k, scoring, renormalize, bias, n_group, topk_group, scale)
 
 
 def moe_route(logits, k: int, scoring: str = "softmax", renormalize: bool = True, bias=None, n_group: int = 1,
@@ -400,6 +417,16 @@ def fused_moe(x, w13, w2, topk_weights, topk_ids, act: str = "silu", b13=None, b
         return fused_moe_cuda(x, w13, w2, topk_weights, topk_ids, act, b13, b2, w13_scale, w2_scale, block,
                               expert_map)
     return _rm.fused_moe(x, w13, w2, topk_weights, topk_ids, act, b13, b2, w13_scale, w2_scale, block, expert_map)
+
+
+def experts_on_weighted_input(x, w13, w2, topk_weights, topk_ids, act: str, limit: float = 0.0):
+    """Routed experts whose weight multiplies their input: rows of ``expert(w * x)`` in expert order and, per (token, choice),
+    the row's place ``[T * k]`` (int32); a token's result is the sum of its rows.  16-bit weights run on the tensor-core
+    grouped GEMM, fp32 ones on the CUDA-core one."""
+    if x.is_cuda:
+        from .moe_cuda import experts_on_weighted_input_cuda
+        return experts_on_weighted_input_cuda(x, w13, w2, topk_weights, topk_ids, act, limit)
+    return _rs.experts_on_weighted_input(x, w13, w2, topk_weights, topk_ids, lambda h: act_and_mul(h, act, limit))
 
 
 # ----------------------------------------------------------------------------- MLA / sparse MLA / indexer
@@ -700,7 +727,7 @@ def layernorm_residual(x, dtype, parts, weight, eps: float):
 
 def gated_group_rmsnorm(o, gate, weight, eps: float, out):
     """``o / rms(o) * weight * sigmoid(gate)`` over groups of ``weight.numel()`` columns into ``out``; ``o`` fp32
-    ``[T, n]``, ``gate [T, n]`` (may be a column slice), ``out [T, >= n]``."""
+    ``[T, n]``, ``gate [T, n]`` (may be a column slice; None: no gate), ``out [T, >= n]``."""
     if o.is_cuda:
         _c().gated_group_rmsnorm(out, o, gate, weight, eps)
     else:
@@ -758,6 +785,70 @@ def fixed_decay_attention(q, k, v, decay, states, cu_seqlens, state_indices, has
         if lo < hi:
             _c().fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens[lo:hi + 1], state_indices[lo:hi],
                                        has_initial_state[lo:hi], chunked and not decode, decode)
+    return out
+
+
+def gated_write_attention(q, v, f, f_bias, lower, states, cu_seqlens, state_indices, has_initial_state,
+                          max_query_len: int = 0, num_decodes: int = 0):
+    """Varlen linear attention whose forget gate decides what is written: ``S <- diag(f) S + (1 - f) v^T``,
+    ``o = S^T silu(q)`` with ``f = lower + (1 - lower) sigmoid(f + f_bias)`` over a state cache ``[slots, H, Dv, >= D]`` (fp32,
+    in place).  ``q [T, H, D]``, ``v [T, H, Dv]``, ``f [T, H * D]`` raw projections; ``f_bias``, ``lower`` fp32.  Returns fp32
+    ``[T, H, Dv]``.  bf16 prompt portions run chunk by chunk on the tensor cores (``csrc/linear_attn/chunk_gated.cu``); the
+    ``num_decodes`` single-token requests at the front, fp32 models and other head sizes take the token-by-token kernel."""
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    if not q.is_cuda:
+        return _rl.gated_write_attention(out, q, v, f, f_bias, lower, states, cu_seqlens, state_indices, has_initial_state)
+    D, Dv = q.shape[2], v.shape[2]
+    chunked = (max_query_len >= LINEAR_CHUNK_MIN and q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128
+               and q.stride(0) % 8 == 0 and f.stride(0) % 8 == 0 and not any(t.data_ptr() % 16 for t in (q, v, f)))
+    R = state_indices.shape[0]
+    nd = R if max_query_len == 1 else num_decodes
+    for lo, hi, decode in ((0, nd, True), (nd, R, False)):
+        if lo < hi:
+            _c().gated_write_attention(out, q, v, f, f_bias, lower, states, cu_seqlens[lo:hi + 1], state_indices[lo:hi],
+                                       has_initial_state[lo:hi], chunked and not decode, decode)
+    return out
+
+
+# ----------------------------------------------------- norms before and after every sublayer, polynomial activation
+
+def embed_rmsnorm(ids, table, weight, eps: float):
+    """Start of a stream: ``(table rows in fp32, their RMS norm times weight in table.dtype)``, both ``[T, ld]``."""
+    T, ld = ids.shape[0], table.shape[1]
+    x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
+    h = torch.empty(T, ld, dtype=table.dtype, device=table.device)
+    (_c() if table.is_cuda else _rs).embed_rmsnorm(x, h, ids, table, weight, eps)
+    return x, h
+
+
+def sandwich_rmsnorm(x, y, w_post, w_pre, eps: float):
+    """End of a sublayer and start of the next one: ``x += rms(y) * w_post`` in place on the fp32 stream, returns
+    ``rms(x) * w_pre`` in ``y``'s dtype.  ``y``: ``[T, ld]``, or ``(rows, places)`` as :func:`experts_on_weighted_input`
+    returns them (a token's rows are summed)."""
+    y, pos = y if isinstance(y, tuple) else (y, None)
+    h = torch.empty(x.shape, dtype=y.dtype, device=x.device)
+    (_c() if x.is_cuda else _rs).sandwich_rmsnorm(x, h, y, pos, w_post, w_pre, eps)
+    return h
+
+
+def poly_norm(z, coeff, width: int, eps: float):
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` per row, ``coeff = (a, b, c, e)`` (fp32), ``N`` = division by the root mean
+    square over the first ``width`` columns; the columns behind them become zero."""
+    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    (_c() if z.is_cuda else _rs).poly_norm(out, z, coeff, width, eps)
+    return out
+
+
+def attn_prep_cache(q, k, v, kv_cache, slot_mapping, positions, num_heads: int, num_kv_heads: int, eps: float,
+                    temperature=None, v_out=None, v_in=None, share: float = 0.0):
+    """Split of an attention projection: K as it is and V divided by its root mean square per head go into the paged cache;
+    returns ``q [T, Hq, Dc]`` times ``1 + coef ln(floor((position + 1) / every) + 1)`` for ``temperature = (coef, every)``.
+    Heads are zero-padded to the cache's head size.  ``v_out [T, Hkv * Dv]`` receives the normed values; ``v_in`` (such values
+    of another layer) is mixed in before caching: ``(1 - share) v + share v_in``."""
+    coef, every = (0.0, 0) if temperature is None else temperature
+    out = torch.empty(q.shape[0], num_heads, kv_cache.shape[-1], dtype=q.dtype, device=q.device)
+    (_c() if q.is_cuda else _rs).attn_prep_cache(out, q, k, v, kv_cache, slot_mapping, positions, num_heads, num_kv_heads,
+                                                 coef, every, v_out, v_in, share, eps)
     return out
 
 

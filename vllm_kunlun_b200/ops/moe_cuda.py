@@ -72,3 +72,26 @@ def fused_moe_cuda(x, w13, w2, topk_weights, topk_ids, act="silu", b13=None, b2=
     out = torch.empty(T, H, dtype=x.dtype, device=x.device)
     C.moe_unpermute(out, y, pos, topk_weights.contiguous())
     return out
+
+
+def experts_on_weighted_input_cuda(x, w13, w2, topk_weights, topk_ids, act, limit):
+    """Rows of ``expert(weight * x)`` in expert order and the row of every (token, choice) pair."""
+    from . import act_and_mul
+    C = _ext.C()
+    T, k = topk_ids.shape
+    E = w13.shape[0]
+    ids, w = topk_ids.contiguous(), topk_weights.contiguous()
+    if 0 < T * k <= _small_pairs() and SMALL_BATCH_FUSION[0]:
+        xs, pos, lod, _ = C.moe_prepare_small(x, ids, None, E, E, False, w)
+    else:
+        xs, pos, lod = C.moe_permute(x, ids, None, E, E, _state(x.device, E), 0, w)
+
+    def gemm(a, weight):
+        out = torch.empty(a.shape[0], weight.shape[1], dtype=a.dtype, device=a.device)
+        if a.dtype == torch.float32:
+            C.gemm_f32_grouped(out, a, weight, lod)
+        else:
+            C.grouped_gemm(out, a, weight, lod, None, None, None, 0)
+        return out
+
+    return gemm(act_and_mul(gemm(xs, w13), act, limit), w2), pos

@@ -160,9 +160,10 @@ def copy_blocks(caches, mapping):
 # ----------------------------------------------------------------------------- GQA attention
 
 def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int], sinks, return_lse=False,
-            softcap: float = 0.0):
+            softcap: float = 0.0, bias=None):
     """q [Lq, Hq, D], k/v [Lk, Hkv, D(v)].  Query row i sits at absolute position
-    ``causal_offset + i`` and sees keys ``<=`` that position (None = no mask)."""
+    ``causal_offset + i`` and sees keys ``<=`` that position (None = no mask).  ``bias [Hq, n]``: added to the scores by
+    distance, the last entry for every distance from ``n - 1`` on."""
     Lq, Hq, D = q.shape
     Lk, Hkv = k.shape[0], k.shape[1]
     g = Hq // Hkv
@@ -176,6 +177,8 @@ def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int],
         qpos = torch.arange(Lq).unsqueeze(1) + causal_offset
         kpos = torch.arange(Lk).unsqueeze(0)
         mask = kpos <= qpos
+        if bias is not None:
+            s = s + bias.float()[:, (qpos - kpos).clamp(0, bias.shape[1] - 1)].reshape(Hkv, g, Lq, Lk)
         if window is not None:
             mask &= kpos > qpos - window
         s = s.masked_fill(~mask, float("-inf"))
@@ -206,7 +209,7 @@ def gather_paged_kv(kv_cache, block_table_row, seq_len: int):
 
 
 def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
-                    window: Optional[int] = None, sinks=None, softcap: float = 0.0):
+                    window: Optional[int] = None, sinks=None, softcap: float = 0.0, bias=None, gate=None):
     """Unified varlen paged attention: covers ``kunlun_ops.prefill_attention`` (with prefix cache,
     ``kunlun_attn.py:849-891``) and ``kunlun_ops.speculative_attention`` (decode with
     ``q_len >= 1``, ``kunlun_attn.py:926-947``).  K/V for all ``seq_lens[r]`` positions are read
@@ -218,7 +221,10 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
             continue
         L = int(seq_lens[r])
         k, v = gather_paged_kv(kv_cache, block_tables[r], L)
-        out[qs:qe] = _attend(q[qs:qe], k, v, scale, L - (qe - qs), window, sinks, softcap=softcap).to(q.dtype)
+        o = _attend(q[qs:qe], k, v, scale, L - (qe - qs), window, sinks, softcap=softcap, bias=bias)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[qs:qe].float()).unsqueeze(-1)
+        out[qs:qe] = o.to(q.dtype)
     return out
 
 

@@ -43,7 +43,8 @@ def gated_group_rmsnorm(out, o, gate, weight, eps):
     T, n = o.shape
     y = o.float().reshape(T, -1, weight.numel())
     y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
-    out[:, :n] = (y.reshape(T, n) * torch.sigmoid(gate.float())).to(out.dtype)
+    y = y.reshape(T, n)
+    out[:, :n] = (y if gate is None else y * torch.sigmoid(gate.float())).to(out.dtype)
 
 
 def qk_unit_norm_cache(q, k, v, kv_cache, slot_mapping, num_heads, num_kv_heads, eps):
@@ -104,6 +105,22 @@ def fixed_decay_attention(out, q, k, v, decay, states, cu_seqlens, state_indices
         S = states[slot, :, :, :D].clone() if init else torch.zeros_like(states[slot, :, :, :D])
         for t in range(s, e):
             S = S * d + torch.einsum("hv,hk->hvk", vf[t], kf[t])
+            out[t] = torch.einsum("hvk,hk->hv", S, qf[t])
+        states[slot].zero_()
+        states[slot, :, :, :D] = S
+    return out
+
+
+def gated_write_attention(out, q, v, f, f_bias, lower, states, cu_seqlens, state_indices, has_initial_state):
+    T, H, D = q.shape
+    z = f.float() + f_bias
+    keep = (lower + (1 - lower) * torch.sigmoid(z)).reshape(T, H, D)
+    write = ((1 - lower) * torch.sigmoid(-z)).reshape(T, H, D)
+    qf, vf = F.silu(q.float()), v.float()
+    for s, e, slot, init in _segments(cu_seqlens, state_indices, has_initial_state):
+        S = states[slot, :, :, :D].clone() if init else torch.zeros_like(states[slot, :, :, :D])          # [H, Dv, D]
+        for t in range(s, e):
+            S = S * keep[t].unsqueeze(1) + torch.einsum("hv,hk->hvk", vf[t], write[t])
             out[t] = torch.einsum("hvk,hk->hv", S, qf[t])
         states[slot].zero_()
         states[slot, :, :, :D] = S
