@@ -36,7 +36,7 @@ def query_temperature(pos, coef, every):
 def distance_bucket(n, rows, far):
     """Row of a distance table with ``rows`` rows: one row per distance below rows / 2, then logarithmically wider ones that
     reach the end at ``far``; farther distances share the last row."""
-    half = rows / 2
+    half = rows // 2
     if n < half:
         return n
     x = half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half) + 1e-9)
@@ -165,3 +165,67 @@ def forward(tokens, w, cfg, layers_out=None):
         if layers_out is not None:
             layers_out.append(x)
     return norm(x, w["final.norm"], eps) @ w["head"].T
+
+
+def tensor_shapes(cfg):
+    W, V = cfg["width"], cfg["vocab"]
+    out = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer.get("mlp")
+        H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        out.update({p + "norm1": (W,), p + "norm1b": (W,)})
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            mix = {"q": (H * D, W), "k": (G * D, W), "v": (G * Dv, W), "rel": (m["bias_rows"], H), "g": (H, W), "o": (W, H * Dv)}
+            if m.get("v_mix"):
+                mix["vmix"] = ()
+        else:
+            mix = {"q": (H * D, W), "f": (H * D, W), "f.b": (H * D,), "lower": (H * D,), "v": (H * Dv, W), "norm": (Dv,),
+                   "o": (W, H * Dv)}
+        out.update({p + "mix." + k: s for k, s in mix.items()})
+        if f is None:
+            continue
+        out.update({p + "norm2": (W,), p + "norm2b": (W,)})
+        if f["kind"] == "dense":
+            mlp = {"up": (f["ff"], W), "down": (W, f["ff"]), "act": (4,)}
+        else:
+            n, E = f["expert"]["ff"], f["router"]["experts"]
+            mlp = {"router": (E, W)}
+            for e in range(E):
+                mlp.update({f"e{e}.gate": (n, W), f"e{e}.up": (n, W), f"e{e}.down": (W, n)})
+        out.update({p + "mlp." + k: s for k, s in mlp.items()})
+    return out
+
+
+def random_weights(cfg, seed=0, dtype=torch.float64):
+    """Seeded weights, already rounded to bfloat16 (what a checkpoint stores).  Queries are scaled up so that the attention
+    is peaked; half of the forget gates hardly forget, so that early tokens still show late."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in sorted(tensor_shapes(cfg).items()):
+        z = torch.randn(shape, generator=g)
+        leaf = name.rsplit(".", 1)[-1]
+        if name.endswith(".mix.norm"):
+            t = 1.0 + 0.1 * z
+        elif leaf.startswith("norm"):
+            t = 0.15 * z
+        elif leaf == "rel":
+            t = 1.5 * z
+        elif leaf == "vmix":
+            t = 0.2 + 0.5 * torch.sigmoid(z)
+        elif leaf == "lower":
+            t = torch.sigmoid(z) * (torch.arange(shape[0]) % 3 > 0)
+        elif leaf == "b":
+            t = torch.where(torch.arange(shape[0]) % 2 == 0, z + 6.0, z)
+        elif leaf == "act":
+            t = 0.5 + 0.3 * z
+        elif leaf == "embed":
+            t = z
+        elif name.endswith(".mix.q"):
+            t = z * 2.0 / math.sqrt(shape[-1])
+        elif leaf == "router":
+            t = z * 3.0 / math.sqrt(shape[-1])
+        else:
+            t = z * 1.3 / math.sqrt(shape[-1])
+        out[name] = t.to(torch.bfloat16).to(dtype)
+    return out

@@ -135,17 +135,23 @@ def distance_buckets(rows: int, far: int) -> list:
     """Row of a distance table per distance 0, 1, ... up to the first one from which on all share the last row.  The first
     half of the rows serve one distance each; row ``h + m`` (``h = rows // 2``) starts at ``h (far / h)^(m / (rows - h))``,
     decided in integers, so that no rounding moves a boundary."""
-    h = rows // 2
-    log_rows = rows - h
+    h, n_log = rows // 2, rows - rows // 2
     if not 0 < h < far:
         raise ValueError(f"a distance table of {rows} rows that ends at {far}")
-    out, n, m = list(range(h)), h, 0
-    while h + m < rows - 1:
-        while h + m < rows - 1 and n ** log_rows * h ** (m + 1) >= far ** (m + 1) * h ** log_rows:
-            m += 1
-        out.append(h + m)
-        n += 1
-    return out
+
+    def start(m: int) -> int:       # first distance of row h + m
+        want, unit = far ** m * h ** n_log, h ** m
+        lo, hi = h, far             # the last row starts at or before ``far``
+        while lo < hi:
+            mid = (lo + hi) // 2
+            lo, hi = (lo, mid) if mid ** n_log * unit >= want else (mid + 1, hi)
+        return lo
+
+    starts = [start(m) for m in range(n_log)]
+    out = list(range(h))
+    for m in range(n_log - 1):
+        out += [h + m] * (starts[m + 1] - starts[m])
+    return out + [rows - 1]
 
 
 class DistanceBiasAttention(WindowAttention):
@@ -232,7 +238,7 @@ def link_shared_values(mixers) -> None:
     sharing = [m for m in mixers if getattr(m, "shares_values", False)]
     for i, m in enumerate(sharing):
         m.first_of_sharing = i == 0
-        if m.kv_heads * m.vdim != sharing[0].kv_heads * sharing[0].vdim:
+        if (m.kv_heads, m.vdim) != (sharing[0].kv_heads, sharing[0].vdim):
             raise ValueError("layers that share values have different numbers or sizes of value heads")
 
 
