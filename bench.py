@@ -78,10 +78,11 @@ def parse():
     ap.add_argument("--layers", type=int, default=0,
                     help="debugging only: run with this many layers (the JSON line then says so and is not a result)")
     ap.add_argument("--layer-bench", nargs="?", const="all", default=None, metavar="SIZE",
-                    help="instead of the headline run: prefill and decode throughput of Bolopel and Seturax layers, each "
-                         "beside the closest other model (Qwen3-Next and DeepSeek, both with dense feed-forwards) at equal "
-                         "sizes; one JSON line per size and model (SIZE: small | large | all)")
-    ap.add_argument("--layer-bench-model", default="all", choices=["all", "bolopel", "qwen3-next", "seturax", "deepseek"])
+                    help="instead of the headline run: prefill and decode throughput of Bolopel, Seturax and Petipel layers, "
+                         "each beside the closest other model (Qwen3-Next and DeepSeek with dense feed-forwards, Qwen3-Next "
+                         "with experts in every other layer) at equal sizes; one JSON line per size and model (SIZE: small | large | all)")
+    ap.add_argument("--layer-bench-model", default="all",
+                    choices=["all", "bolopel", "qwen3-next", "seturax", "deepseek", "petipel", "qwen3-next-moe"])
     a = ap.parse_args()
     c = CONFIGS[a.config]
     a.model = a.model or c["model"]
@@ -165,10 +166,13 @@ def reference_arm(args):
 
 # Sizes of the layer benchmark: width, feed-forward, query / key-value heads of the softmax attention, heads of the
 # recurrent layers (head size 128 throughout), layers (every 4th one of the hybrids differs in kind), window, query latent
-# of the latent-attention models (their key / value latent is 512, their rotated part 64).
+# of the latent-attention models (their key / value latent is 512, their rotated part 64), experts of every other layer of
+# Petipel and its neighbour, experts per token and their width.
 LAYER_SIZES = {
-    "small": dict(width=2048, ff=6144, heads=16, kv_heads=4, lin_heads=16, layers=8, window=1024, q_rank=768),
-    "large": dict(width=4096, ff=12288, heads=32, kv_heads=8, lin_heads=32, layers=8, window=1024, q_rank=1536),
+    "small": dict(width=2048, ff=6144, heads=16, kv_heads=4, lin_heads=16, layers=8, window=1024, q_rank=768,
+                  experts=32, top=4, expert_ff=768),
+    "large": dict(width=4096, ff=12288, heads=32, kv_heads=8, lin_heads=32, layers=8, window=1024, q_rank=1536,
+                  experts=32, top=4, expert_ff=1536),
 }
 LAYER_VOCAB = 32000
 
@@ -176,7 +180,10 @@ LAYER_VOCAB = 32000
 def layer_models(size):
     """The models of one size, all with dense feed-forwards of the same width: Bolopel (3 of 4 layers 'parallel', 1
     'channel_delta') and Qwen3-Next (3 of 4 layers gated delta net, 1 gated full attention); Seturax (windowed latent
-    attention) and DeepSeek (latent attention over all positions)."""
+    attention) and DeepSeek (latent attention over all positions).  Petipel (HGRN2 with experts and attention with a dense
+    feed-forward in turn) and Qwen3-Next with the same order of layers (gated delta net with experts, gated full attention)."""
+    import dataclasses
+
     from vllm_kunlun_b200.config import LayerSpec, ModelConfig
     z = LAYER_SIZES[size]
     H = z["lin_heads"]
@@ -208,7 +215,17 @@ def layer_models(size):
                            head_dim=192, v_head_dim=128, intermediate_size=z["ff"], rms_norm_eps=1e-6, max_position=1 << 16,
                            rope_neox=False, use_mla=True, q_lora_rank=z["q_rank"], kv_lora_rank=512, qk_nope_head_dim=128,
                            qk_rope_head_dim=64)
-    return {"bolopel": own, "qwen3-next": like, "seturax": seturax, "deepseek": deepseek}
+    routed = dict(kind="moe", expert=dict(ff=z["expert_ff"], limit=7.0), router=dict(experts=z["experts"], top=z["top"]))
+    full = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, bias_max=512, v_mix=True,
+                q_temp=dict(coef=0.1, every=1024))
+    petipel = dataclasses.replace(
+        own, architecture="Petipel", name=f"petipel-{size}", hidden_act="poly_norm", residual_multiplier=0.5,
+        layer_specs=tuple(LayerSpec("attention", dict(full), dict(kind="dense", ff=z["ff"])) if i % 2 else
+                          LayerSpec("hgrn2", dict(heads=H, dim=128, vdim=128), dict(routed)) for i in range(z["layers"])))
+    qwen_moe = dataclasses.replace(like, name=f"qwen3-next-moe-{size}", linear_attn_pattern=2, moe_layer_freq=2,
+                                   num_experts=z["experts"], num_experts_per_tok=z["top"], moe_intermediate_size=z["expert_ff"])
+    return {"bolopel": own, "qwen3-next": like, "seturax": seturax, "deepseek": deepseek, "petipel": petipel,
+            "qwen3-next-moe": qwen_moe}
 
 
 def layer_bench(args):

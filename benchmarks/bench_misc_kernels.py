@@ -1,7 +1,7 @@
 """Device timings of the sampling, gated-delta-net, conv, LoRA and MTP-glue kernels (CUDA events, L2 flushed
 between iterations, 3 warm-ups), reported against the algorithmic bytes and the measured copy bandwidth.
 
-    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|latent|conv|lora|all] [--small]
+    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|sandwich|latent|conv|lora|all] [--small]
 
 ``--small`` shrinks every case to a few hundred MB so that a profiler capture of one launch ends quickly."""
 import argparse
@@ -105,6 +105,10 @@ def case_recurrence(small):
         a = torch.randn(T, H * D, device="cuda").to(torch.bfloat16)
         b = torch.randn(T, H, device="cuda").to(torch.bfloat16)
         A_log, dt = torch.zeros(H, device="cuda"), torch.full((H * D,), -3.0, device="cuda")
+        f, bias, low = torch.randn(T, H * D, device="cuda").to(torch.bfloat16), torch.full((H * D,), 3.0, device="cuda"), \
+            torch.rand(H * D, device="cuda")
+        sec = timeit(lambda: ops.gated_write_attention(q, v, f, bias, low, states, cu, idx, init, L, nd))
+        report(f"gated_write_attention({name})", sec, nbytes, f"R={R} L={L}")
         sec = timeit(lambda: ops.channel_delta_rule(q, k, v, a, b, A_log, dt, states, cu, idx, init, D ** -0.5, 1e-6, L, nd))
         report(f"channel_delta_rule({name})", sec, nbytes + T * H * D * 2, f"R={R} L={L}")
 
@@ -131,6 +135,62 @@ def case_stream(small):
     table, turns = torch.randn(32000, W, device="cuda").to(torch.bfloat16), ops.position_turns(W, 10000.0).cuda()
     sec = timeit(lambda: ops.embed_positions_layernorm(ids, pos, table, turns, w, 1e-5))
     report("embed_layernorm_kernel", sec, T * W * 8, f"T={T} W={W}")
+
+
+def case_sandwich(small):
+    """Norms around every sublayer, polynomial activation, attention with a bias by distance and output gates (32 / 8 heads
+    of 128) beside the same kernels without, experts on weighted inputs: 4 prompts of 2048 tokens, 16 tokens behind 2080."""
+    W, F, H, G, D, E, k, ff = 4096, 12288, 32, 8, 128, 32, 4, 1536
+    dev, bf = "cuda", torch.bfloat16
+
+    def rnd(*shape):
+        return torch.randn(*shape, device=dev).to(bf)
+
+    w, coeff, bias = torch.rand(W, device=dev), torch.rand(4, device=dev), torch.randn(H, 400, device=dev)
+    w13, w2, router = rnd(E, 2 * ff, W) * 0.02, rnd(E, W, ff) * 0.02, rnd(E, W) * 0.02
+    for tag, B, n, ctx in (("prompts", 4, 2048 if not small else 512, 0), ("single tokens", 16, 1, 2080)):
+        T, blocks = B * n, -(-(ctx + n) // 64)
+        x, y, z = torch.randn(T, W, device=dev), rnd(T, W), rnd(T, F)
+        sec = timeit(lambda: ops.sandwich_rmsnorm(x, y, w, w, 1e-5))
+        report("sandwich_rmsnorm_kernel", sec, T * W * 12, tag)
+        rows, pos = rnd(T * k, W), torch.randperm(T * k, device=dev).int()
+        sec = timeit(lambda: ops.sandwich_rmsnorm(x, (rows, pos), w, w, 1e-5))
+        report("sandwich_rmsnorm_kernel (experts' rows)", sec, T * W * (10 + 2 * k), tag)
+        res, yy = rnd(T, W), y.clone()
+        sec = timeit(lambda: ops.add_rmsnorm(yy, res, w.to(bf), 1e-5))
+        report("rmsnorm_kernel (with residual add)", sec, T * W * 8, tag)
+        sec = timeit(lambda: ops.poly_norm(z, coeff, F, 1e-5))
+        report("poly_norm_kernel", sec, T * F * 4, tag)
+        z2 = rnd(T, 2 * F)
+        sec = timeit(lambda: ops.act_and_mul(z2, "silu"))
+        report("act_and_mul_kernel", sec, T * F * 6, tag)
+        proj, gate = rnd(T, (H + 2 * G) * D), rnd(T, H)
+        cache = rnd(B * blocks, 2, G, 64, D)
+        bt = torch.arange(B * blocks, dtype=torch.int32, device=dev).view(B, blocks)
+        p = (torch.arange(T, device=dev) % n) + ctx
+        slots = torch.cat([bt[b].long()[p[b * n:(b + 1) * n] // 64] * 64 + p[b * n:(b + 1) * n] % 64 for b in range(B)])
+        keep = rnd(T, G * D)
+        sec = timeit(lambda: ops.attn_prep_cache(proj[:, :H * D], proj[:, H * D:(H + G) * D], proj[:, (H + G) * D:], cache,
+                                                 slots, p, H, G, 1e-5, (0.1, 1024), None, keep, 0.4))
+        report("attn_prep_cache_kernel", sec, T * (2 * (H + 2 * G) + G) * D * 2, tag)
+        lens = torch.full((B,), ctx + n, dtype=torch.int32, device=dev)
+        qsl = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
+        q, nd = rnd(T, H, D), B if n == 1 else 0
+        flops = sum(min(i + 1, ctx + n) for i in range(ctx, ctx + n)) * B * H * D * 4
+        for name, b, gt in (("bias and gate", bias, gate), ("neither", None, None)):
+            sec = timeit(lambda: ops.paged_attention(q, cache, bt, lens, qsl, 0.09, n, ctx + n, num_decodes=nd,
+                                                     num_decode_tokens=nd, bias=b, gate=gt))
+            report(f"attention ({name})", sec, B * (ctx + n) * G * D * 4 + T * H * D * 4,
+                   f"{tag}; {flops / sec / 1e12:.0f} TFLOP/s of visible scores")
+        h = rnd(T, W)
+        wt, ids = ops.router_and_route(h, router, None, k, "sigmoid", False, fp32=True)
+        sec = timeit(lambda: ops.router_and_route(h, router, None, k, "sigmoid", False, fp32=True))
+        report("router + route", sec, T * W * 2 + E * W * 2, tag)
+        touched = min(E, T * k) * 3 * ff * W * 2
+        for name, fn in (("weighted inputs", lambda: ops.experts_on_weighted_input(h, w13, w2, wt, ids, "swiglu_limit", 7.0)),
+                         ("weighted outputs", lambda: ops.fused_moe(h, w13, w2, wt, ids))):
+            sec = timeit(fn)
+            report(f"experts ({name})", sec, touched + T * W * 4, f"{tag}; {T * k * 6 * ff * W / sec / 1e12:.0f} TFLOP/s")
 
 
 def case_latent(small):
@@ -258,7 +318,7 @@ if __name__ == "__main__":
     ap.add_argument("--case", default="all")
     ap.add_argument("--small", action="store_true")
     a = ap.parse_args()
-    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "latent": case_latent, "conv": case_conv, "lora": case_lora}
+    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "sandwich": case_sandwich, "latent": case_latent, "conv": case_conv, "lora": case_lora}
     explicit = {"gemm_splits": case_gemm_splits}  # not part of "all"
     with torch.inference_mode():
         for n, fn in cases.items():

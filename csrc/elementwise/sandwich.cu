@@ -120,6 +120,7 @@ __global__ void __launch_bounds__(kThr) sandwich_rmsnorm_kernel(float* x, T* h, 
 }
 
 // Three sums of a row at once, broadcast to the block.
+template <int THR>
 __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float (*red)[3]) {
   a = warp_sum(a);
   b = warp_sum(b);
@@ -127,66 +128,67 @@ __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float (
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
   if (l == 0) { red[w][0] = a; red[w][1] = b; red[w][2] = c; }
   __syncthreads();
-  a = b = c = 0.f;
-#pragma unroll
-  for (int i = 0; i < kThr / 32; ++i) { a += red[i][0]; b += red[i][1]; c += red[i][2]; }
+  const bool on = l < THR / 32;
+  a = warp_sum(on ? red[l][0] : 0.f);
+  b = warp_sum(on ? red[l][1] : 0.f);
+  c = warp_sum(on ? red[l][2] : 0.f);
 }
 
-// NV vectors of 4 columns per thread; NV = 0: rows of any length, read twice.  Columns F .. ld of the output are zero.
-template <typename T, int NV>
-__global__ void __launch_bounds__(kThr) poly_norm_kernel(T* out, int64_t ldo, const T* z, int64_t ldz, const float* coeff,
-                                                         int F, int ld, float eps) {
-  __shared__ float red[kThr / 32][3];
+// NV 16-byte vectors per thread stay in registers as they were read; NV = 0: rows of any length, read twice.  Columns F .. ld
+// of the output are zero.
+template <typename T, int THR, int NV>
+__global__ void __launch_bounds__(THR) poly_norm_kernel(T* out, int64_t ldo, const T* z, int64_t ldz, const float* coeff,
+                                                        int F, int ld, float eps) {
+  constexpr int V = Vec16<T>::N, NR = NV > 0 ? NV : 1;
+  __shared__ float red[THR / 32][3];
   griddep_launch();
   griddep_wait();
   const int64_t t = blockIdx.x;
   const T* zr = z + t * ldz;
-  constexpr int NR = NV > 0 ? NV : 1;
-  float v[NR][4], s1 = 0.f, s2 = 0.f, s3 = 0.f;
-  auto add = [&](const float (&a)[4], int c) {
+  Vec16<T> v[NR];
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  auto add = [&](const Vec16<T>& a, int c) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float q = c + j < F ? a[j] * a[j] : 0.f;
+    for (int j = 0; j < V; ++j) {
+      const float x = to_f(a.v[j]), q = c + j < F ? x * x : 0.f, q2 = q * q;
       s1 += q;
-      s2 += q * q;
-      s3 += q * q * q;
+      s2 += q2;
+      s3 = fmaf(q2, q, s3);
     }
   };
   if constexpr (NV > 0) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kThr + threadIdx.x) * 4;
-      v[i][0] = v[i][1] = v[i][2] = v[i][3] = 0.f;
-      if (c >= ld) continue;
-      load4(v[i], zr + c);
-      add(v[i], c);
+      const int c = (i * THR + threadIdx.x) * V;
+      if (c < ld) v[i] = ld_vec(zr + c);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * THR + threadIdx.x) * V;
+      if (c < ld) add(v[i], c);
     }
   } else {
-    for (int c = threadIdx.x * 4; c < ld; c += kThr * 4) {
-      load4(v[0], zr + c);
-      add(v[0], c);
-    }
+    for (int c = threadIdx.x * V; c < ld; c += THR * V) add(ld_vec(zr + c), c);
   }
-  block_sum3(s1, s2, s3, red);
-  const float a = coeff[0] / sqrtf(s1 / F + eps), b = coeff[1] / sqrtf(s2 / F + eps), c3 = coeff[2] / sqrtf(s3 / F + eps),
-              e = coeff[3];
-  auto put = [&](const float (&x)[4], int c) {
-    float o[4];
+  block_sum3<THR>(s1, s2, s3, red);
+  const float k1 = coeff[0] / sqrtf(s1 / F + eps), k2 = coeff[1] / sqrtf(s2 / F + eps), k3 = coeff[2] / sqrtf(s3 / F + eps),
+              k0 = coeff[3];
+  auto put = [&](Vec16<T> a, int c) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) o[j] = c + j < F ? x[j] * (a + x[j] * (b + x[j] * c3)) + e : 0.f;
-    store4(out + t * ldo + c, o);
+    for (int j = 0; j < V; ++j) {
+      const float x = to_f(a.v[j]);
+      a.v[j] = from_f<T>(c + j < F ? fmaf(x, fmaf(x, fmaf(x, k3, k2), k1), k0) : 0.f);
+    }
+    st_vec(out + t * ldo + c, a);
   };
   if constexpr (NV > 0) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kThr + threadIdx.x) * 4;
+      const int c = (i * THR + threadIdx.x) * V;
       if (c < ld) put(v[i], c);
     }
   } else {
-    for (int c = threadIdx.x * 4; c < ld; c += kThr * 4) {
-      load4(v[0], zr + c);
-      put(v[0], c);
-    }
+    for (int c = threadIdx.x * V; c < ld; c += THR * V) put(ld_vec(zr + c), c);
   }
 }
 
@@ -304,16 +306,20 @@ extern "C" int b200_sandwich_rmsnorm(float* x, void* h, const void* y, int64_t y
 extern "C" int b200_poly_norm(void* out, int64_t ldo, const void* z, int64_t ldz, const float* coeff, int64_t T_, int F, int ld,
                               float eps, int dtype, cudaStream_t st) {
   if (T_ == 0) return 0;
-  if (ld % 4 || ldo % 4 || ldz % 4 || F > ld) return 3;
-#define B200_PN(NVEC) launch_pdl(poly_norm_kernel<T, NVEC>, dim3(T_), dim3(kThr), 0, st, (T*)out, ldo, (const T*)z, ldz, coeff, F, ld, eps)
+  if (F > ld || ((uintptr_t)out | (uintptr_t)z) % 16) return 3;
+#define B200_PN(THR, NVEC)                                                                                          \
+  launch_pdl(poly_norm_kernel<T, THR, NVEC>, dim3(T_), dim3(THR), 0, st, (T*)out, ldo, (const T*)z, ldz, coeff, F, ld, eps)
   B200_DISPATCH_DTYPE(dtype, {
-    const int need = (ld / 4 + kThr - 1) / kThr;
-    if (need <= 1) B200_PN(1);
-    else if (need <= 2) B200_PN(2);
-    else if (need <= 4) B200_PN(4);
-    else if (need <= 8) B200_PN(8);
-    else if (need <= 16) B200_PN(16);
-    else B200_PN(0);
+    constexpr int V = Vec16<T>::N;
+    if (ld % V || ldo % V || ldz % V) return 3;
+    const int need = ld / V;
+    if (need <= 256) B200_PN(256, 1);
+    else if (need <= 512) B200_PN(256, 2);
+    else if (need <= 1024) B200_PN(512, 2);
+    else if (need <= 1536) B200_PN(512, 3);
+    else if (need <= 2048) B200_PN(512, 4);
+    else if (need <= 4096) B200_PN(1024, 4);
+    else B200_PN(512, 0);
   });
 #undef B200_PN
   return (int)cudaGetLastError();
