@@ -186,6 +186,9 @@ def case_sandwich(small):
         wt, ids = ops.router_and_route(h, router, None, k, "sigmoid", False, fp32=True)
         sec = timeit(lambda: ops.router_and_route(h, router, None, k, "sigmoid", False, fp32=True))
         report("router + route", sec, T * W * 2 + E * W * 2, tag)
+        if n > 1:
+            for name, fn in (("fp32 output", lambda: ops.router_gemm(h, router, fp32=True)), ("16-bit output", lambda: ops.linear(h, router))):
+                report(f"router GEMM ({name})", timeit(fn), T * W * 2 + E * W * 2, tag)
         touched = min(E, T * k) * 3 * ff * W * 2
         for name, fn in (("weighted inputs", lambda: ops.experts_on_weighted_input(h, w13, w2, wt, ids, "swiglu_limit", 7.0)),
                          ("weighted outputs", lambda: ops.fused_moe(h, w13, w2, wt, ids))):
