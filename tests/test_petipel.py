@@ -203,7 +203,7 @@ def spread(table, far):
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
-@pytest.mark.parametrize("H,G,D,V", [(4, 1, 64, 32), (3, 3, 10, 14), (8, 2, 128, 128), (20, 1, 24, 72), (2, 1, 140, 30)])
+@pytest.mark.parametrize("H,G,D,V", [(6, 2, 64, 40), (3, 3, 10, 14), (8, 2, 128, 128), (20, 1, 24, 72), (2, 1, 140, 30)])
 def test_attention_with_a_distance_bias(device, dtype, H, G, D, V):
     """Unequal requests, single tokens beside portions; tables that end inside a page, inside a tile and behind everything."""
     g = torch.Generator().manual_seed(D)
