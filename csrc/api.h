@@ -29,7 +29,8 @@ typedef struct GemmArgs {
   int num_sms;
   int stages;         // 0 = choose from the shared-memory budget
   int ctas_per_sm;    // 0 = choose (2 for small token tiles)
-  int act;            // 0 = plain; 1 silu, 2 gelu-tanh, 3 swigluoai on [64 gate | 64 up] interleaved weight tiles
+  int act;            // 0 = plain; 1 silu, 2 gelu-tanh, 3 swigluoai on [64 gate | 64 up] interleaved weight tiles; 4 = square
+                      // of relu on every output
   // collective fusion over peer memory (all zero / null = plain GEMM)
   void* rs_stage[8];  // reduce-scatter: staging area of every rank (peer mappings)
   void* rs_flags[8];  // reduce-scatter: per-(source, token tile) arrival counters on every rank
@@ -102,6 +103,7 @@ typedef struct GroupedGemmArgs {
   int out_fmt;           // 1 = bf16, 0 = fp16, 2 = fp32 (16-bit inputs, no bias)
   int bn;                // token tile 16 / 32 / 64 / 128
   int grid;
+  int act;               // 0, or 4 = square of relu (16-bit inputs)
 } GroupedGemmArgs;
 int b200_grouped_gemm_launch(const GroupedGemmArgs* a, const void* tmapW, const void* tmapX, cudaStream_t st);
 
@@ -174,7 +176,7 @@ int b200_decode_attention_umma(void* out, const void* q, const void* tmap, const
                                int* status, int64_t T, int B, int Hq, int Hkv, int D, int block_size, int max_blocks,
                                int64_t num_blocks, int max_query_len, int num_splits, int window, float scale,
                                int early_meta, const float* bias, int bias_len, const void* gate, int64_t gate_stride,
-                               int dtype, cudaStream_t st);
+                               int keep_first, int sigmoid, int dtype, cudaStream_t st);
 
 // Dense paged MLA decode on tcgen05 (attention/mla_decode_umma.cu): cache blocks of 64 tokens, at most 32 query
 // tokens per request.  `tmap`: the cache as a 2-D [blocks * 64, 576] 16-bit tensor, 64 x 64 boxes, 128-byte swizzle.
@@ -189,7 +191,7 @@ int b200_prefill_attention_umma(void* out, float* lse, const void* tmQ, const vo
                                 const int* seq_lens, const int* qsl, const float* sinks, int* status, int B, int Hq, int Hkv,
                                 int D, int block_size, int max_blocks, int64_t num_blocks, int max_query_len, int window,
                                 float scale, const float* bias, int bias_len, const void* gate, int64_t gate_stride,
-                                int dtype, unsigned long long* trace, cudaStream_t st);
+                                int keep_first, int sigmoid, int dtype, unsigned long long* trace, cudaStream_t st);
 int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, const void* tmKV, const void* tmKpe, const int* kv_starts,
                           const int* kv_lens, const int* qsl, const float* sinks, const void* gate, int64_t gate_stride,
                           int* status, int B, int Hq, int max_query_len, int causal, int window, float scale, int dtype,
@@ -220,7 +222,8 @@ int b200_topk_rows(int* out, const float* logits, const int* row_len, int64_t ro
 
 // ---- MoE / fp8 activation quantisation --------------------------------------------------------
 int b200_moe_route(float* out_w, int* out_ids, const void* logits, const float* bias, int64_t T, int E, int k, int mode,
-                   int renorm, int n_group, int topk_group, float scale, int64_t stride, int dtype, cudaStream_t st);
+                   int renorm, int n_group, int topk_group, int group_top, float scale, int64_t stride, int dtype,
+                   cudaStream_t st);
 int b200_moe_permute(void* x_sorted, int* pos_of_pair, int* lod, int* counts, int* cursor, const void* x, const int* ids,
                      const int* emap, const float* factors, int64_t T, int k, int H, int E_local, int E_global,
                      int64_t x_stride, int64_t max_rows, int dtype, cudaStream_t st);  // factors [T][k] (or null): times the rows
@@ -230,7 +233,7 @@ int b200_router_gemm_small(float* out, const void* x, int64_t x_stride, const vo
                            int64_t T_, int N, int K, int dtype, cudaStream_t st);
 int b200_router_route_small(float* out_w, int* out_ids, const void* x, int64_t x_stride, const void* w,
                             const void* wbias, const float* bias, int64_t T_, int E, int K, int k, int mode,
-                            int renorm, int n_group, int topk_group, float scale, int dtype, cudaStream_t st);
+                            int renorm, int n_group, int topk_group, int group_top, float scale, int dtype, cudaStream_t st);
 int b200_moe_small_pairs();
 int b200_moe_prepare_small(void* x_sorted, float* scale_t, int64_t s_stride, int* pos_of_pair, int* lod,
                            const void* x, const int* ids, const int* emap, const float* factors, int64_t T_, int k,
@@ -298,16 +301,48 @@ int b200_sandwich_rmsnorm(float* x, void* h, const void* y, int64_t y_stride, co
                           const float* w_pre, int64_t T, int H, int ld, float eps, int dtype, cudaStream_t st);
 int b200_poly_norm(void* out, int64_t ldo, const void* z, int64_t ldz, const float* coeff, int64_t T, int F, int ld, float eps,
                    int dtype, cudaStream_t st);
-int b200_attn_prep_cache(void* q_out, const void* q, const void* k, const void* v, int64_t stride, void* kv_cache,
-                         const int64_t* slots, const int64_t* positions, void* v_out, const void* v_in, float share,
-                         float temp_coef, int64_t temp_every, int64_t T, int Hq, int Hkv, int D, int Dv, int Dc,
-                         int block_size, int64_t num_blocks, float eps, int dtype, cudaStream_t st);
+typedef struct AttnPrepArgs {
+  const void *q, *k, *v;     // [T][heads][head size] column slices of one projection, rows `stride` apart
+  void *q_out, *cache;       // [T][Hq][Dc]; [block][2][Hkv][slot][Dc]
+  const int64_t *slots, *positions;
+  const float *q_norm, *k_norm;  // [D] weights of an RMS norm per head (null: none)
+  const float* table;        // cos / sin pairs [T][pairs][2] of the first 2 pairs columns of q and k (null: no rotation)
+  void* v_out;               // [T][Hkv * Dv] the values (before mixing) for later layers, or null
+  const void* v_in;          // such values of an earlier layer, mixed in with `share`, or null
+  int64_t stride, num_blocks, temp_every;  // temp_every 0: no temperature
+  int Hq, Hkv, D, Dv, Dc, block_size, pairs, v_norm;  // v_norm: values are divided by their root mean square
+  float share, temp_coef, eps;
+} AttnPrepArgs;
+int b200_attn_prep_cache(const AttnPrepArgs* args, int64_t T, int dtype, cudaStream_t st);
+
+// ---- fp32 stream normalised on the sublayers' outputs, short convolution of their inputs (elementwise/postnorm.cu) ------
+typedef struct PostNormArgs {
+  float* x;                  // [T][ld] the stream, updated in place
+  const void* table;         // start of a stream: x = table[ids[t]] * scale; null: x += LayerNorm(y) * weight
+  const int64_t* ids;
+  int64_t table_rows;
+  // y = its row (or null: 0) + sum over k choices of weights[t][q] * (rows[places[t][q]], or pass[t] where the place is < 0)
+  const void *y, *rows, *pass;
+  const int* places;
+  const float* weights;
+  int64_t y_stride, rows_stride, pass_stride;
+  const float* weight;       // [width]
+  void* h;                   // [T][ld] x + conv(x) (taps > 0), or LayerNorm(x) * final_weight (if any), in the model's type
+  const float *conv, *final_weight;  // [taps][ld]; [width]
+  float* state;              // [slots][taps - 1][ld] the stream's last rows of every request
+  const int *qsl, *slots, *has_init;
+  int64_t T, num_slots;
+  int k, taps, width, ld, num_reqs, max_query_len;
+  float scale, eps;
+} PostNormArgs;
+int b200_postnorm(const PostNormArgs* args, int dtype, cudaStream_t st);    // taps > 0: requests of a few tokens
+int b200_input_conv(const PostNormArgs* args, int dtype, cudaStream_t st);  // h = x + conv(x)
 
 // ---- fp32 GEMM on the CUDA cores (gemm/gemm_f32.cu): out[T, N] = x[T, K] . w[N, K]^T (+ bias) -----------------
 int b200_gemm_f32(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, int64_t ldw, const float* bias,
-                  int64_t T, int N, int K, cudaStream_t st);
+                  int64_t T, int N, int K, int relu2, cudaStream_t st);  // relu2: outputs pass the square of relu
 int b200_gemm_f32_grouped(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w, const int* lod, int64_t M,
-                          int E, int N, int K, cudaStream_t st);
+                          int E, int N, int K, int relu2, cudaStream_t st);
 
 // ---- latent attention of any size (attention/latent.cu) --------------------------------------------------
 typedef struct LatentPrepArgs {
@@ -358,7 +393,7 @@ int b200_paged_attention_generic(void* out, const void* q, const void* kv_cache,
                                  const int* seq_lens, const int* qsl, const float* sinks, int64_t T, int B, int Hq,
                                  int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks, int latent_dv,
                                  int window, float scale, const float* bias, int bias_len, const void* gate,
-                                 int64_t gate_stride, int dtype, cudaStream_t st);
+                                 int64_t gate_stride, int keep_first, int sigmoid, int dtype, cudaStream_t st);
 
 // ---- gated delta net / conv / MTP glue --------------------------------------------------------
 int b200_causal_conv1d_fwd(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w,
@@ -392,6 +427,18 @@ typedef struct RecurrenceArgs {
 int b200_linear_recurrence(const RecurrenceArgs* a, int dtype, cudaStream_t st);
 int b200_chunk_decay(const RecurrenceArgs* a, int dtype, cudaStream_t st);  // kind 1, prompt portions (linear_attn/chunk_decay.cu)
 int b200_chunk_gated_write(const RecurrenceArgs* a, int dtype, cudaStream_t st);  // kind 2, prompt portions (linear_attn/chunk_gated.cu)
+// Element-wise gated recurrence with gates of the current token (linear_attn/blend.cu)
+typedef struct BlendArgs {
+  void* out;                 // [T][width] state * silu(g)
+  const void *z, *x, *g;     // raw projections, rows `stride` apart
+  const float *z_bias, *x_bias;
+  float* state;              // [slots][width]
+  const int *qsl, *slots, *has_init;
+  int64_t stride, out_stride, num_slots;
+  int R, width;
+  int steps;                 // the requests have one token each (any number is correct, few are fast)
+} BlendArgs;
+int b200_gated_blend(const BlendArgs* args, int dtype, cudaStream_t st);
 int b200_sigmoid_gate_mul(void* out, const void* o, const void* gate, int64_t gate_stride, int D, int64_t T_,
                           int dtype, cudaStream_t st);
 int b200_mtp_concat_norm(void* out, const void* embed, const void* hidden, const void* we, const void* wh,

@@ -16,6 +16,8 @@
 //   warps 2-5  softmax: thread t owns key t of the tile (TMEM lane t): mask, tile max per row (redux + a
 //              shared-memory exchange between the four warps), exp2, P^T to one of two shared-memory buffers
 //              (16-bit, K-major, swizzled) for the second MMA; the same threads own output dim t in the epilogue
+// `kSigmoid` (with `kBias`): a visible key counts with sigmoid(score + bias), not normalised - no maxima, no row sums, splits add
+// up.  `keep_first`: with a window, the first keys stay visible; their tiles come first in the tile list.
 // Split-KV partials go through the fp32 workspace and are merged by the last CTA of a (request, head) to arrive.
 // Every wait is bounded: on time-out the status word is set, the CTA drains its copies, frees TMEM and returns.
 #include <cuda.h>
@@ -53,7 +55,7 @@ struct Params {
   const void* gate;         // [T, >= Hq] raw output gates in the output's type, or null
   int64_t gate_stride;
   int* status;
-  int Hq, Hkv, block_size, max_blocks, num_splits, window, num_stages, bias_len;
+  int Hq, Hkv, block_size, max_blocks, num_splits, window, keep_first, num_stages, bias_len;
   int early_meta;           // lengths / block table were written long before this launch: read them, and fetch
                             // old-context tiles, before the programmatic-dependency wait
   int64_t num_blocks, T;
@@ -94,7 +96,7 @@ template <> __device__ __forceinline__ uint16_t to_bits16<__half>(float v) { ret
 // maximum exceeds it by more than kMaxSlack (in log2 units), so p = exp2(s - m_used) stays below 2^kMaxSlack and the
 // result O / l is unchanged; in the common case O^T needs no rescale and the softmax warps never wait for the
 // previous P.V to finish - they run ahead into a second P buffer while the tensor core works.
-template <typename T, int D, int NR, bool kBias>
+template <typename T, int D, int NR, bool kBias, bool kSigmoid>
 __global__ void __launch_bounds__(kThreads)
 decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_constant__ Params p) {
   constexpr int KB = D / 64;                       // 64-dim blocks
@@ -106,6 +108,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   constexpr int kTmemCols = 64;                    // S^T x 2 buffers (16 cols each) + O^T (16 cols)
   constexpr float kMaxSlack = 8.f;
   static_assert(D == 128, "one 128-lane O^T tile");
+  static_assert(!kSigmoid || kBias);
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int num_stages = p.num_stages;
@@ -171,11 +174,18 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, ctx - p.window + 1) / kTileKeys * kTileKeys;
   const bool served = q_len > 0 && rows_total <= NR;
-  const int n_tiles_all = served ? (kv_end - kv_begin + kTileKeys - 1) / kTileKeys : 0;
+  // tiles of the kept first keys that lie in front of the window's first tile
+  const int kept = p.window > 0 ? p.keep_first : 0;
+  const int n_head = min((kept + kTileKeys - 1) / kTileKeys, kv_begin / kTileKeys);
+  const int n_tiles_all = served ? n_head + (kv_end - kv_begin + kTileKeys - 1) / kTileKeys : 0;
   const int per_split = (n_tiles_all + p.num_splits - 1) / p.num_splits;
   const int tile_lo = split * per_split;
   const int tile_hi = min(n_tiles_all, tile_lo + per_split);
   const int n_tiles = max(0, tile_hi - tile_lo);
+  auto tile_key = [&](int i) {   // first key of this CTA's tile i
+    i += tile_lo;
+    return i < n_head ? i * kTileKeys : kv_begin + (i - n_head) * kTileKeys;
+  };
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer (does not need Q)
@@ -187,7 +197,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       int issued = 0;
       bool waited = false;
       for (int i = 0; i < n_tiles; ++i) {
-        const bool old_ctx = kv_begin + (tile_lo + i + 1) * kTileKeys <= ctx;  // no key of this step in the tile
+        const bool old_ctx = tile_key(i) + kTileKeys <= ctx;  // no key of this step in the tile
         if (!waited && (i >= num_stages || !old_ctx)) {
           griddep_wait();
           waited = true;
@@ -196,7 +206,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
         mbar_expect_tx(&kv_full[stage], kStageBytes);
         uint8_t* sK = smem + stage * kStageBytes;
         uint8_t* sV = sK + kOpBytes;
-        const int key0 = kv_begin + (tile_lo + i) * kTileKeys;
+        const int key0 = tile_key(i);
 #pragma unroll
         for (int pg = 0; pg < kTileKeys / kPage; ++pg) {
           const int key = key0 + pg * kPage;
@@ -360,12 +370,12 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[buf]);
       // ---- mask (only on tiles that touch the causal / length / window edge)
-      const int key0 = kv_begin + (tile_lo + i) * kTileKeys;
+      const int key0 = tile_key(i);
       const int key = key0 + lane_id;
       const bool full = key0 + kTileKeys - 1 <= pos_min && key0 + kTileKeys <= kv_end &&
-                        (p.window <= 0 || key0 > pos_max - p.window);
+                        (p.window <= 0 || key0 > pos_max - p.window || key0 + kTileKeys <= kept);
       // nearest distance of the tile: beyond the table's last entry the bias is one constant per row
-      const bool near_tile = kBias && pos_min - (key0 + kTileKeys - 1) < p.bias_len - 1;
+      const bool near_tile = kBias && p.bias_len > 1 && pos_min - (key0 + kTileKeys - 1) < p.bias_len - 1;
       float sc[NR];
       bool need = fail;   // does any score exceed its row's reference maximum by more than the slack?
 #pragma unroll
@@ -374,15 +384,15 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
         if constexpr (kBias)
           v += near_tile ? bias[r][min(max(pos[r] - key, 0), p.bias_len - 1)] * 1.4426950408889634f : far_bias[r];
         if (!full) {
-          const bool in = key < kv_end && key <= pos[r] && (p.window <= 0 || key > pos[r] - p.window);
+          const bool in = key < kv_end && key <= pos[r] && (p.window <= 0 || key > pos[r] - p.window || key < kept);
           v = in ? v : -INFINITY;
         } else if (NR > 4 && pos[r] < 0) {
           v = -INFINITY;
         }
         sc[r] = v;
-        need |= v > m_used[r] + kMaxSlack;
+        if constexpr (!kSigmoid) need |= v > m_used[r] + kMaxSlack;
       }
-      if (bar_red_or(1, 128, need)) {
+      if (!kSigmoid && bar_red_or(1, 128, need)) {
         // ---- rare after the first tiles: exchange the per-warp maxima, move the reference maxima, rescale O^T
 #pragma unroll
         for (int r = 0; r < NR; ++r) {
@@ -421,9 +431,13 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       }
 #pragma unroll
       for (int r = 0; r < NR; ++r) {
-        const float ms = (m_used[r] == -INFINITY) ? 0.f : m_used[r];
-        sc[r] = exp2f(sc[r] - ms);
-        l_part[r] += sc[r];
+        if constexpr (kSigmoid) {
+          sc[r] = __fdividef(1.f, 1.f + exp2f(fminf(-sc[r], 60.f))) * (sc[r] == -INFINITY ? 0.f : 1.f);
+        } else {
+          const float ms = (m_used[r] == -INFINITY) ? 0.f : m_used[r];
+          sc[r] = exp2f(sc[r] - ms);
+          l_part[r] += sc[r];
+        }
       }
       // ---- P^T (B operand, K-major): element (row r, this thread's key)
       if (!fail) {
@@ -471,10 +485,12 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       float den = L;
       if (p.num_splits == 1 && p.sinks != nullptr && r < rows_total) den += exp2f(p.sinks[hh] * 1.4426950408889634f - Ms);
       sInv[r] = (ok && den > 0.f) ? 1.f / den : 0.f;
+      if (kSigmoid) sInv[r] = ok ? 1.f : 0.f;
       if (p.num_splits == 1 && p.gate != nullptr && r < rows_total) sInv[r] *= gate_of(qs + r / g, hh);
       sRow[r] = orow;
       if (p.num_splits > 1 && r < rows_total)
-        p.ws_lse[(int64_t)split * p.T * p.Hq + orow] = (ok && L > 0.f) ? Ms + log2f(L) : -INFINITY;
+        p.ws_lse[(int64_t)split * p.T * p.Hq + orow] =
+            kSigmoid ? (ok && n_tiles > 0 ? 0.f : -INFINITY) : (ok && L > 0.f) ? Ms + log2f(L) : -INFINITY;
     }
     named_bar_sync(1, 128);
     if (served) {
@@ -537,6 +553,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
           }
           if (p.sinks != nullptr) den += exp2f(p.sinks[kvh * g + r % g] * 1.4426950408889634f - Ms);
           float inv = den > 0.f ? 1.f / den : 0.f;
+          if (kSigmoid) inv = 1.f;      // every split that saw keys has weight one
           if (p.gate != nullptr) inv *= gate_of(qs + r / g, kvh * g + r % g);
           for (int s2 = 0; s2 < S; ++s2) sW[s2 * kRows + r] *= inv;
         }
@@ -577,10 +594,10 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   }
 }
 
-template <typename T, int NR, bool kBias>
+template <typename T, int NR, bool kBias, bool kSigmoid>
 static int launch_nr(const Params& p0, const CUtensorMap& tm, int B, cudaStream_t st) {
   constexpr int D = 128;
-  auto kern = decode_umma_kernel<T, D, NR, kBias>;
+  auto kern = decode_umma_kernel<T, D, NR, kBias, kSigmoid>;
   Params p = p0;
   constexpr int kStageBytes = 2 * (D / 64) * kTileKeys * 128;
   p.num_stages = 3;
@@ -593,15 +610,15 @@ static int launch_nr(const Params& p0, const CUtensorMap& tm, int B, cudaStream_
 }
 
 template <typename T>
-static int launch(const Params& p, const CUtensorMap& tm, int B, int max_rows, cudaStream_t st) {
-  if (p.bias != nullptr) {
-    if (max_rows <= 4) return launch_nr<T, 4, true>(p, tm, B, st);
-    if (max_rows <= 8) return launch_nr<T, 8, true>(p, tm, B, st);
-    return launch_nr<T, 16, true>(p, tm, B, st);
-  }
-  if (max_rows <= 4) return launch_nr<T, 4, false>(p, tm, B, st);
-  if (max_rows <= 8) return launch_nr<T, 8, false>(p, tm, B, st);
-  return launch_nr<T, 16, false>(p, tm, B, st);
+static int launch(const Params& p, const CUtensorMap& tm, int B, int max_rows, bool sigmoid, cudaStream_t st) {
+#define B200_DA_LAUNCH(BIAS, SIGMOID)                                              \
+  if (max_rows <= 4) return launch_nr<T, 4, BIAS, SIGMOID>(p, tm, B, st);           \
+  if (max_rows <= 8) return launch_nr<T, 8, BIAS, SIGMOID>(p, tm, B, st);           \
+  return launch_nr<T, 16, BIAS, SIGMOID>(p, tm, B, st);
+  if (sigmoid) { B200_DA_LAUNCH(true, true) }
+  if (p.bias != nullptr) { B200_DA_LAUNCH(true, false) }
+  B200_DA_LAUNCH(false, false)
+#undef B200_DA_LAUNCH
 }
 
 }  // namespace dattn
@@ -615,8 +632,8 @@ extern "C" int b200_decode_attention_umma(void* out, const void* q, const void* 
                                           float* ws_lse, int* status, int64_t T_, int B, int Hq, int Hkv, int D,
                                           int block_size, int max_blocks, int64_t num_blocks, int max_query_len,
                                           int num_splits, int window, float scale, int early_meta, const float* bias,
-                                          int bias_len, const void* gate, int64_t gate_stride, int dtype,
-                                          cudaStream_t st) {
+                                          int bias_len, const void* gate, int64_t gate_stride, int keep_first,
+                                          int sigmoid, int dtype, cudaStream_t st) {
   using namespace b200;
   if (B == 0 || T_ == 0) return 0;
   if (D != 128 || Hq % Hkv || max_query_len * (Hq / Hkv) > dattn::kRows || block_size % dattn::kPage) return 3;
@@ -631,10 +648,11 @@ extern "C" int b200_decode_attention_umma(void* out, const void* q, const void* 
   p.num_stages = 3;
   p.early_meta = early_meta;
   p.bias = bias; p.bias_len = bias_len; p.gate = gate; p.gate_stride = gate_stride;
-  if (bias != nullptr && bias_len < 1) return 2;
+  if ((bias != nullptr && bias_len < 1) || keep_first < 0 || (sigmoid && (bias == nullptr || sinks != nullptr))) return 2;
+  p.keep_first = keep_first;
   const CUtensorMap& tm = *reinterpret_cast<const CUtensorMap*>(tmap);
   const int max_rows = max_query_len * (Hq / Hkv);
-  if (dtype == 1) return dattn::launch<__nv_bfloat16>(p, tm, B, max_rows, st);
-  if (dtype == 2) return dattn::launch<__half>(p, tm, B, max_rows, st);
+  if (dtype == 1) return dattn::launch<__nv_bfloat16>(p, tm, B, max_rows, sigmoid != 0, st);
+  if (dtype == 2) return dattn::launch<__half>(p, tm, B, max_rows, sigmoid != 0, st);
   return 3;
 }

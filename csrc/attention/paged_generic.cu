@@ -1,11 +1,11 @@
-// Paged attention for any head size and for fp32 models: causal, optional sliding window, sinks, score
-// bias by distance and output gates; over keys and
+// Paged attention for any head size and for fp32 models: causal, optional sliding window (with first keys that stay visible),
+// sinks, score bias by distance, output gates, sigmoid weights instead of a softmax; over keys and
 // values [block][2][head][slot][D], or over latent rows [block][slot][D] that all heads share and whose first `latent_dv`
 // columns are the values (absorbed multi-head latent attention).  The
 // tensor-core kernels (prefill_umma.cu, decode_umma.cu, paged_attention.cu, paged_decode.cu) serve 16-bit heads of 64,
 // 128 and 256; this one serves the rest on the CUDA cores, in fp32 throughout.
 // One CTA = one (query token, query head).  Each of its 4 warps walks 32-key tiles of the visible range: scores with a
-// lane per key, an online softmax per warp, then P.V with the lanes over the value dims; the warps' states meet at the
+// lane per key, an online softmax (or plain sigmoids) per warp, then P.V with the lanes over the value dims; the warps' states meet at the
 // end.
 #include <math.h>
 
@@ -22,7 +22,8 @@ template <typename T, int ND>  // ND: value dims per lane, Dv <= 32 ND
 __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel(
     T* out, const T* q, const T* cache, const int* block_tables,
     const int* seq_lens, const int* qsl, const float* sinks, const float* bias, int bias_len, const T* gate,
-    int64_t gate_stride, int B, int Hq, int Hkv, int D, int Dv, int latent, int block_size, int max_blocks, int64_t num_blocks, int window, float scale) {
+    int64_t gate_stride, int B, int Hq, int Hkv, int D, int Dv, int latent, int block_size, int max_blocks, int64_t num_blocks, int window, int keep_first,
+    int sigmoid, float scale) {
   extern __shared__ float sm_gen[];
   float* sq = sm_gen;                       // [D]
   float* so = sq + D;                       // [kGenWarps][Dv]
@@ -40,6 +41,7 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
   const int pos = seq_lens[req] - (qsl[req + 1] - t);
   if (pos < 0) return;
   const int first = window > 0 ? max(0, pos - window + 1) : 0;
+  const int kept = min(keep_first, first), visible = kept + pos + 1 - first;   // kept keys, then the window
   for (int i = tid; i < D; i += kGenWarps * 32) sq[i] = to_f(q[((int64_t)t * Hq + h) * D + i]) * scale;
   __syncthreads();
   const int* bt = block_tables + (int64_t)req * max_blocks;
@@ -54,9 +56,9 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
   float m = -INFINITY, l = 0.f, acc[ND];
 #pragma unroll
   for (int i = 0; i < ND; ++i) acc[i] = 0.f;
-  for (int k0 = first + warp * 32; k0 <= pos; k0 += kGenWarps * 32) {
-    const int key = k0 + lane;
-    const int64_t off = key <= pos ? row_of(key) : -1;
+  for (int k0 = warp * 32; k0 < visible; k0 += kGenWarps * 32) {
+    const int i = k0 + lane, key = i < kept ? i : first + i - kept;
+    const int64_t off = i < visible ? row_of(key) : -1;
     float s = -INFINITY;
     if (off >= 0) {
       const T* kr = cache + off;
@@ -67,13 +69,21 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
       s = a0 + a1;
       if (bias != nullptr) s += bias[(int64_t)h * bias_len + min(pos - key, bias_len - 1)];
     }
-    const float mn = fmaxf(m, warp_max(s));
-    if (mn == -INFINITY) continue;
-    const float corr = expf(m - mn), pr = expf(s - mn);
-    m = mn;
-    l = l * corr + warp_sum(pr);
+    float pr;
+    if (sigmoid) {
+      pr = off >= 0 ? 1.f / (1.f + expf(-s)) : 0.f;
+      m = 0.f;
+      l = 1.f;
+    } else {
+      const float mn = fmaxf(m, warp_max(s));
+      if (mn == -INFINITY) continue;
+      const float corr = expf(m - mn);
+      pr = expf(s - mn);
+      m = mn;
+      l = l * corr + warp_sum(pr);
 #pragma unroll
-    for (int i = 0; i < ND; ++i) acc[i] *= corr;
+      for (int j = 0; j < ND; ++j) acc[j] *= corr;
+    }
     for (int j = 0; j < 32; ++j) {
       const float pj = __shfl_sync(0xffffffff, pr, j);
       const int64_t oj = __shfl_sync(0xffffffff, off, j);
@@ -97,7 +107,7 @@ __global__ void __launch_bounds__(kGenWarps * 32) paged_attention_generic_kernel
   float den = sinks != nullptr ? expf(sinks[h] - M) : 0.f, wg[kGenWarps];
 #pragma unroll
   for (int w = 0; w < kGenWarps; ++w) { wg[w] = expf(sml[w * 2] - M); den += sml[w * 2 + 1] * wg[w]; }
-  float inv = den > 0.f ? 1.f / den : 0.f;
+  float inv = sigmoid ? 1.f : den > 0.f ? 1.f / den : 0.f;
   if (gate != nullptr) inv /= 1.f + expf(-to_f(gate[(int64_t)t * gate_stride + h]));
   for (int d = tid; d < Dv; d += kGenWarps * 32) {
     float a = 0.f;
@@ -114,12 +124,13 @@ extern "C" int b200_paged_attention_generic(void* out, const void* q, const void
                                             const int* seq_lens, const int* qsl, const float* sinks, int64_t T_, int B,
                                             int Hq, int Hkv, int D, int block_size, int max_blocks, int64_t num_blocks,
                                             int latent_dv, int window, float scale, const float* bias, int bias_len,
-                                            const void* gate, int64_t gate_stride, int dtype, cudaStream_t st) {
+                                            const void* gate, int64_t gate_stride, int keep_first, int sigmoid, int dtype,
+                                            cudaStream_t st) {
   using namespace b200;
   const int Dv = latent_dv > 0 ? latent_dv : D;
   if (B == 0 || T_ == 0) return 0;
   if (Hq % Hkv || Hq > 65535 || window < 0 || Dv > D || (latent_dv > 0 && Hkv != 1) ||
-      (bias != nullptr && bias_len < 1))
+      (bias != nullptr && bias_len < 1) || keep_first < 0 || (sigmoid && sinks != nullptr))
     return 2;
   const size_t smem = (size_t)(D + kGenWarps * (Dv + 2)) * sizeof(float);
   if (smem > 48 * 1024) return 3;
@@ -127,7 +138,7 @@ extern "C" int b200_paged_attention_generic(void* out, const void* q, const void
 #define B200_GEN_ATTN(ND)                                                                                                \
   B200_DISPATCH_DTYPE(dtype, launch_pdl(paged_attention_generic_kernel<T, ND>, grid, dim3(kGenWarps * 32), smem, st,        \
                                        (T*)out, (const T*)q, (const T*)kv_cache, block_tables, seq_lens, qsl, sinks, bias,  \
-                                       bias_len, (const T*)gate, gate_stride, B, Hq, Hkv, D, Dv, latent_dv > 0, block_size, max_blocks, num_blocks, window, scale))
+                                       bias_len, (const T*)gate, gate_stride, B, Hq, Hkv, D, Dv, latent_dv > 0, block_size, max_blocks, num_blocks, window, keep_first, sigmoid, scale))
   if (Dv <= 64) { B200_GEN_ATTN(2); }
   else if (Dv <= 128) { B200_GEN_ATTN(4); }
   else if (Dv <= 256) { B200_GEN_ATTN(8); }

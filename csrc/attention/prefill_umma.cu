@@ -16,6 +16,10 @@
 // `kBias`: a score bias per head and distance (query position minus key position) from a table [Hq][bias_len], whose last
 // entry serves every farther distance.  A tile that lies farther away altogether adds that constant inside the exponent; for
 // a nearer one the softmax warps put the 255 entries the tile can meet into shared memory (two buffers, one per tile parity).
+// `kSigmoid` (with `kBias`): a visible key counts with sigmoid(score + bias), not normalised - no maximum, no row sum and no
+// rescale; P.V accumulates as it is.
+// `keep_first`: with a window, the first keys of a request stay visible.  Their tiles come first in the tile list, which then
+// jumps to the window's first tile.
 // The MLA instantiation (`kMla`) is the compute-friendly prefill form of multi-head latent attention
 // (v1/attention/backends/mla/common.py:1782-1843): 192-dim q / k (128 "nope" dims per head + 64 rotary dims shared
 // by all heads), 128-dim v, keys and values read as contiguous rows of the up-projected `kv_b_proj` output
@@ -65,7 +69,7 @@ struct Params {
   int64_t gate_stride;
   int* status;
   unsigned long long* trace;   // optional phase timestamps [CTA][24] (null = off)
-  int Hq, Hkv, block_size, max_blocks, window, causal, bias_len;
+  int Hq, Hkv, block_size, max_blocks, window, keep_first, causal, bias_len;
   int64_t num_blocks;
   float scale_log2;
 };
@@ -115,6 +119,15 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
+// sigmoid of x given in log2 units, for two scores at once with one reciprocal: 1 / a and 1 / b from 1 / (a b).  Arguments below
+// -60 count as -60 (a weight of 2^-60), so that the product stays finite.
+__device__ __forceinline__ void sigmoid2_log2(float x0, float x1, float& y0, float& y1) {
+  const float a = 1.f + ex2_approx(fminf(-x0, 60.f)), b = 1.f + ex2_approx(fminf(-x1, 60.f));
+  const float r = __fdividef(1.f, a * b);
+  y0 = r * b;
+  y1 = r * a;
+}
+
 template <typename T> struct FmtOf;
 template <> struct FmtOf<__nv_bfloat16> { static constexpr uint32_t v = 1; };
 template <> struct FmtOf<__half> { static constexpr uint32_t v = 0; };
@@ -126,10 +139,11 @@ template <> __device__ __forceinline__ uint32_t pack2<__half>(float a, float b) 
   return (uint32_t)__half_as_ushort(__float2half(a)) | ((uint32_t)__half_as_ushort(__float2half(b)) << 16);
 }
 
-template <typename T, bool kMla, bool kBias>
+template <typename T, bool kMla, bool kBias, bool kSigmoid>
 __global__ void __launch_bounds__(kThreads)
 prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                     const __grid_constant__ CUtensorMap tmKpe, const __grid_constant__ Params p) {
+  static_assert(!kSigmoid || (kBias && !kMla));
   constexpr int kQBlocks = Cfg<kMla>::kQBlocks, kKBytes = Cfg<kMla>::kKBytes, kVStages = Cfg<kMla>::kVStages;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -194,7 +208,11 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const int kv_end = n_rows > 0 ? min(seq_len, pos_last + 1) : 0;
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, pos_first - p.window + 1) / kKTile * kKTile;
-  const int n_tiles = n_rows > 0 ? (kv_end - kv_begin + kKTile - 1) / kKTile : 0;
+  // tiles of the kept first keys that lie in front of the window's first tile
+  const int kept = p.window > 0 ? p.keep_first : 0;
+  const int n_head = min((kept + kKTile - 1) / kKTile, kv_begin / kKTile);
+  const int n_tiles = n_rows > 0 ? n_head + (kv_end - kv_begin + kKTile - 1) / kKTile : 0;
+  auto tile_key = [&](int i) { return i < n_head ? i * kKTile : kv_begin + (i - n_head) * kKTile; };
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
@@ -219,7 +237,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         uint8_t* sK = smem + stage * kKBytes;
 #pragma unroll
         for (int pg = 0; pg < kKTile / kPage; ++pg) {
-          const int key = kv_begin + i * kKTile + pg * kPage;
+          const int key = tile_key(i) + pg * kPage;
           uint8_t* dst = sK + pg * (kPage * 128);
           if constexpr (kMla) {
             // rows past the request's keys belong to the next request or lie outside the tensor (zero fill): masked
@@ -241,7 +259,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         uint8_t* sV = sVr + stage * kOpBytes;
 #pragma unroll
         for (int pg = 0; pg < kKTile / kPage; ++pg) {
-          const int key = kv_begin + i * kKTile + pg * kPage;
+          const int key = tile_key(i) + pg * kPage;
           uint8_t* dst = sV + pg * (kPage * 128);
           if constexpr (kMla) {
 #pragma unroll
@@ -357,11 +375,11 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (threadIdx.x == 64 && i == 4) trace_mark(p.trace, cta_id, 2);
       if (threadIdx.x == 64 && i == 5) trace_mark(p.trace, cta_id, 7);
       if (threadIdx.x == 64 && i == 20) trace_mark(p.trace, cta_id, 8);
-      const int key0 = kv_begin + i * kKTile;
+      const int key0 = tile_key(i);
       const bool full_tile = key0 + kKTile - 1 <= pos_first && key0 + kKTile <= kv_end &&
-                             (p.window <= 0 || key0 > pos_last - p.window);
+                             (p.window <= 0 || key0 > pos_last - p.window || key0 + kKTile <= kept);
       // nearest distance of the tile: beyond the table's last entry its bias is one constant
-      const bool near_tile = kBias && pos_first - (key0 + kKTile - 1) < p.bias_len - 1;
+      const bool near_tile = kBias && p.bias_len > 1 && pos_first - (key0 + kKTile - 1) < p.bias_len - 1;
       if constexpr (kBias) {
         if (near_tile) {   // entry d: distance pos_first - key0 - 127 + d
           float* dst = sBias + (i & 1) * 256;
@@ -399,9 +417,41 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
         for (int e = 0; e < kKTile; ++e) {
           const int key = key0 + e;
-          const bool in = key < kv_end && key <= pos && (p.window <= 0 || key > pos - p.window);
+          const bool in = key < kv_end && key <= pos && (p.window <= 0 || key > pos - p.window || key < kept);
           v[e] = in ? v[e] : 0xff800000u;   // -inf
         }
+      }
+      if constexpr (kSigmoid) {
+        // P (one buffer): the previous P.V must have read it
+        if (i >= 1 && !fail && !wait_or_abort(p_free, (i - 1) & 1, ab, 806)) fail = true;
+#pragma unroll
+        for (int c = 0; c < kKTile; c += 32) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int e = 0; e < 32; e += 2) {
+            float y0, y1;
+            sigmoid2_log2(fmaf(__uint_as_float(v[c + e]), sc, off), fmaf(__uint_as_float(v[c + e + 1]), sc, off), y0, y1);
+            if (!full_tile) {   // masked scores are -inf
+              if (v[c + e] == 0xff800000u) y0 = 0.f;
+              if (v[c + e + 1] == 0xff800000u) y1 = 0.f;
+            }
+            pk[e / 2] = pack2<T>(y0, y1);
+          }
+          if (!fail) {
+#pragma unroll
+            for (int q4 = 0; q4 < 4; ++q4) {
+              const int q = c / 8 + q4;
+              *reinterpret_cast<uint4*>(sP + (q >> 3) * kHalfBytes + r * 128 + (((q & 7) ^ (r & 7)) << 4)) =
+                  make_uint4(pk[q4 * 4], pk[q4 * 4 + 1], pk[q4 * 4 + 2], pk[q4 * 4 + 3]);
+            }
+          }
+        }
+        fence_proxy_async_smem();
+        tc_fence_before_sync();
+        const bool warp_failed = __any_sync(0xffffffffu, fail);
+        __syncwarp();
+        if (lane == 0 && !warp_failed) mbar_arrive(p_ready);
+        continue;
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -484,6 +534,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const float ms = (m_used == -INFINITY) ? 0.f : m_used;
       if (p.sinks != nullptr) den += exp2f(p.sinks[head] * 1.4426950408889634f - ms);
       float inv = (ok && den > 0.f) ? 1.f / den : 0.f;
+      if (kSigmoid) inv = ok ? 1.f : 0.f;
       if (p.gate != nullptr && row_ok) {
         const float g = to_float(reinterpret_cast<const T*>(p.gate)[(int64_t)(qs + row0 + r) * p.gate_stride + head]);
         inv = inv / (1.f + __expf(-g));
@@ -516,10 +567,10 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
 }
 
-template <typename T, bool kMla, bool kBias>
+template <typename T, bool kMla, bool kBias, bool kSigmoid>
 static int launch(const Params& p, const CUtensorMap& tmQ, const CUtensorMap& tmKV, const CUtensorMap& tmKpe, int B,
                   int max_query_len, cudaStream_t st) {
-  auto kern = prefill_umma_kernel<T, kMla, kBias>;
+  auto kern = prefill_umma_kernel<T, kMla, kBias, kSigmoid>;
   const size_t smem = Cfg<kMla>::kSmem + (kBias ? Cfg<kMla>::kBiasSmem : 0);
   cudaError_t e = ensure_dynamic_smem((const void*)kern, (int)smem);
   if (e != cudaSuccess) return (int)e;
@@ -533,30 +584,34 @@ static int launch(const Params& p, const CUtensorMap& tmQ, const CUtensorMap& tm
 // Paged GQA prefill attention on tcgen05 (head_dim 128, block_size a multiple of 64).  `tmQ`: q as a 2-D
 // [T, Hq * 128] 16-bit tensor with 64-column x 128-row boxes; `tmKV`: the cache as [rows, 128] with 64 x 64 boxes;
 // both with 128-byte swizzle.  `bias` [Hq][bias_len] (or null): score bias by distance, the last entry for all farther ones;
-// `gate` [T][>= Hq] (or null): raw output gates.  Returns 3 for shapes it does not serve.
+// `gate` [T][>= Hq] (or null): raw output gates; `sigmoid`: weights without a softmax (needs a bias; no sinks, no lse);
+// `keep_first`: keys that a window never hides.  Returns 3 for shapes it does not serve.
 extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tmQ, const void* tmKV,
                                            const int* block_tables, const int* seq_lens, const int* qsl,
                                            const float* sinks, int* status, int B, int Hq, int Hkv, int D, int block_size,
                                            int max_blocks, int64_t num_blocks, int max_query_len, int window, float scale,
                                            const float* bias, int bias_len, const void* gate, int64_t gate_stride,
-                                           int dtype, unsigned long long* trace, cudaStream_t st) {
+                                           int keep_first, int sigmoid, int dtype, unsigned long long* trace,
+                                           cudaStream_t st) {
   using namespace b200;
   if (B == 0 || max_query_len <= 0) return 0;
-  if (bias != nullptr && bias_len < 1) return 2;
+  if ((bias != nullptr && bias_len < 1) || keep_first < 0) return 2;
+  if (sigmoid && (bias == nullptr || sinks != nullptr || lse != nullptr)) return 2;
   if (D != 128 || Hq % Hkv || block_size % pattn::kPage || B > 65535 || Hq > 65535) return 3;
   pattn::Params p;
   p.out = out; p.lse = lse; p.block_tables = block_tables; p.seq_lens = seq_lens; p.qsl = qsl; p.sinks = sinks;
-  p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.max_blocks = max_blocks; p.window = window;
+  p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.max_blocks = max_blocks; p.window = window; p.keep_first = keep_first;
   p.num_blocks = num_blocks; p.scale_log2 = scale * 1.4426950408889634f;
   p.kv_starts = nullptr; p.causal = 1; p.gate = gate; p.gate_stride = gate_stride; p.bias = bias; p.bias_len = bias_len;
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
-  if (dtype == 1)
-    return bias != nullptr ? pattn::launch<__nv_bfloat16, false, true>(p, q, kv, kv, B, max_query_len, st)
-                           : pattn::launch<__nv_bfloat16, false, false>(p, q, kv, kv, B, max_query_len, st);
-  if (dtype == 2)
-    return bias != nullptr ? pattn::launch<__half, false, true>(p, q, kv, kv, B, max_query_len, st)
-                           : pattn::launch<__half, false, false>(p, q, kv, kv, B, max_query_len, st);
+#define B200_PA_LAUNCH(T)                                                                            \
+  (sigmoid           ? pattn::launch<T, false, true, true>(p, q, kv, kv, B, max_query_len, st)        \
+   : bias != nullptr ? pattn::launch<T, false, true, false>(p, q, kv, kv, B, max_query_len, st)       \
+                     : pattn::launch<T, false, false, false>(p, q, kv, kv, B, max_query_len, st))
+  if (dtype == 1) return B200_PA_LAUNCH(__nv_bfloat16);
+  if (dtype == 2) return B200_PA_LAUNCH(__half);
+#undef B200_PA_LAUNCH
   return 3;
 }
 
@@ -578,12 +633,12 @@ extern "C" int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, con
   pattn::Params p;
   p.out = out; p.lse = lse; p.block_tables = nullptr; p.seq_lens = kv_lens; p.qsl = qsl; p.kv_starts = kv_starts;
   p.sinks = sinks; p.bias = nullptr; p.bias_len = 0; p.gate = gate; p.gate_stride = gate_stride; p.status = status; p.trace = trace; p.Hq = Hq; p.Hkv = Hq; p.block_size = pattn::kPage;
-  p.max_blocks = 0; p.window = window; p.causal = causal ? 1 : 0; p.num_blocks = 0;
+  p.max_blocks = 0; p.window = window; p.keep_first = 0; p.causal = causal ? 1 : 0; p.num_blocks = 0;
   p.scale_log2 = scale * 1.4426950408889634f;
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
   const CUtensorMap& kpe = *reinterpret_cast<const CUtensorMap*>(tmKpe);
-  if (dtype == 1) return pattn::launch<__nv_bfloat16, true, false>(p, q, kv, kpe, B, max_query_len, st);
-  if (dtype == 2) return pattn::launch<__half, true, false>(p, q, kv, kpe, B, max_query_len, st);
+  if (dtype == 1) return pattn::launch<__nv_bfloat16, true, false, false>(p, q, kv, kpe, B, max_query_len, st);
+  if (dtype == 2) return pattn::launch<__half, true, false, false>(p, q, kv, kpe, B, max_query_len, st);
   return 3;
 }

@@ -131,8 +131,9 @@ void gemm(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::o
   TORCH_CHECK(x.scalar_type() == at::kBFloat16 || x.scalar_type() == at::kHalf, "gemm: bf16/fp16 only");
   TORCH_CHECK(x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1);
   const int T = x.size(0), K = x.size(1), N = w.size(0);
-  TORCH_CHECK(w.size(1) == K && out.size(0) == T && out.size(1) == (act ? N / 2 : N));
-  if (act) {
+  const bool gated = act && act != 4;   // 4: square of relu on every output
+  TORCH_CHECK(w.size(1) == K && out.size(0) == T && out.size(1) == (gated ? N / 2 : N));
+  if (gated) {
     TORCH_CHECK(N % 128 == 0 && out.stride(0) % 8 == 0, "fused gate/up activation needs whole [64 | 64] weight tiles");
     splits = 1;  // whole tiles only: both halves of a feature pair must meet in one epilogue
   }
@@ -324,8 +325,9 @@ void gemm_decode(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const
   TORCH_CHECK(x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1);
   const int T = x.size(0), K = x.size(1), N = w.size(0);
   TORCH_CHECK(T <= 32, "gemm_decode: at most 32 rows");
-  TORCH_CHECK(w.size(1) == K && out.size(0) == T && out.size(1) == (act ? N / 2 : N));
-  if (act) TORCH_CHECK(N % 128 == 0 && out.stride(0) % 8 == 0, "fused gate/up activation needs whole [64 | 64] weight tiles");
+  const bool gated = act && act != 4;   // 4: square of relu on every output
+  TORCH_CHECK(w.size(1) == K && out.size(0) == T && out.size(1) == (gated ? N / 2 : N));
+  if (gated) TORCH_CHECK(N % 128 == 0 && out.stride(0) % 8 == 0, "fused gate/up activation needs whole [64 | 64] weight tiles");
   TORCH_CHECK(K % 8 == 0 && x.stride(0) % 8 == 0 && w.stride(0) % 8 == 0, "gemm_decode: K and row strides must be multiples of 8");
   if (T == 0 || N == 0) return;
   c10::cuda::CUDAGuard guard(x.device());
@@ -581,7 +583,7 @@ void gemm_clear_tmap_cache() { gemm_state().cache.clear(); }
 // fp8: x / w are uint8 views of e4m3 data, a_scale_t [K/128, stride], w_scale [E, N/128, K/128].
 void grouped_gemm(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& lod,
                   const c10::optional<at::Tensor>& bias, const c10::optional<at::Tensor>& a_scale_t,
-                  const c10::optional<at::Tensor>& w_scale, int64_t bn) {
+                  const c10::optional<at::Tensor>& w_scale, int64_t bn, int64_t act) {
   TORCH_CHECK(x.is_cuda() && w.is_cuda() && x.dim() == 2 && (w.dim() == 3 || w.dim() == 2));
   TORCH_CHECK(x.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1);
   const bool fp8 = x.element_size() == 1;
@@ -618,6 +620,7 @@ void grouped_gemm(at::Tensor out, const at::Tensor& x, const at::Tensor& w, cons
     b = per_group <= 16 ? 16 : per_group <= 32 ? 32 : per_group <= 64 ? 64 : 128;
   }
   a.bn = b;
+  a.act = (int)act;
   int64_t n_tiles = (N + 127) / 128;
   int64_t max_tiles = n_tiles * ((M + b - 1) / b + (lod.has_value() ? E : 0));
   a.grid = (int)std::min<int64_t>(max_tiles, (int64_t)gs.num_sms * (b <= 64 ? 2 : 1));
@@ -629,14 +632,15 @@ void grouped_gemm(at::Tensor out, const at::Tensor& x, const at::Tensor& w, cons
 }
 
 std::vector<at::Tensor> moe_route(const at::Tensor& logits, const c10::optional<at::Tensor>& bias, int64_t k,
-                                  int64_t mode, bool renorm, int64_t n_group, int64_t topk_group, double scale) {
+                                  int64_t mode, bool renorm, int64_t n_group, int64_t topk_group, double scale,
+                                  int64_t group_top) {
   TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1);
   auto w = at::empty({logits.size(0), k}, logits.options().dtype(at::kFloat));
   auto ids = at::empty({logits.size(0), k}, logits.options().dtype(at::kInt));
   if (bias.has_value()) TORCH_CHECK(bias->scalar_type() == at::kFloat && bias->is_contiguous());
   check(b200_moe_route(w.data_ptr<float>(), ids.data_ptr<int>(), logits.data_ptr(),
                        bias.has_value() ? bias->data_ptr<float>() : nullptr, logits.size(0), logits.size(1), k, mode,
-                       renorm, n_group, topk_group, (float)scale, logits.stride(0), dtype_code(logits), stream()),
+                       renorm, n_group, topk_group, (int)group_top, (float)scale, logits.stride(0), dtype_code(logits), stream()),
         "moe_route");
   return {w, ids};
 }
@@ -670,7 +674,7 @@ std::vector<at::Tensor> moe_permute(const at::Tensor& x, const at::Tensor& ids, 
 // (weights [T, k] fp32, ids [T, k] int32) straight from the hidden states: router GEMM + routing in one launch
 std::vector<at::Tensor> router_route_small(const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& wbias,
                                            const c10::optional<at::Tensor>& bias, int64_t k, int64_t mode, bool renorm,
-                                           int64_t n_group, int64_t topk_group, double scale) {
+                                           int64_t n_group, int64_t topk_group, double scale, int64_t group_top) {
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && w.dim() == 2 && w.is_contiguous() && w.scalar_type() == x.scalar_type());
   TORCH_CHECK(w.size(1) == x.size(1));
   if (bias.has_value()) TORCH_CHECK(bias->scalar_type() == at::kFloat && bias->is_contiguous());
@@ -679,7 +683,7 @@ std::vector<at::Tensor> router_route_small(const at::Tensor& x, const at::Tensor
   check(b200_router_route_small(ow.data_ptr<float>(), oi.data_ptr<int>(), x.data_ptr(), x.stride(0), w.data_ptr(),
                                 opt_ptr(wbias), bias.has_value() ? bias->data_ptr<float>() : nullptr, x.size(0),
                                 (int)w.size(0), (int)w.size(1), (int)k, (int)mode, renorm, (int)n_group, (int)topk_group,
-                                (float)scale, dtype_code(x), stream()), "router_route_small");
+                                (int)group_top, (float)scale, dtype_code(x), stream()), "router_route_small");
   return {ow, oi};
 }
 
@@ -969,7 +973,7 @@ void decode_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tensor
                            const c10::optional<at::Tensor>& ws_o, const c10::optional<at::Tensor>& ws_lse,
                            int64_t max_query_len, int64_t num_splits, int64_t window, double scale,
                            bool early_meta, const c10::optional<at::Tensor>& bias,
-                           const c10::optional<at::Tensor>& gate) {
+                           const c10::optional<at::Tensor>& gate, int64_t keep_first, bool sigmoid) {
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && kv_cache.dim() == 5);
   check_bias_gate(q, bias, gate);
   TORCH_CHECK(block_tables.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt && qsl.scalar_type() == at::kInt);
@@ -995,7 +999,7 @@ void decode_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tensor
                                    ws_lse.has_value() ? ws_lse->data_ptr<float>() : nullptr, gs.status.data_ptr<int>(),
                                    q.size(0), B, q.size(1), kv_cache.size(2), D, kv_cache.size(3), block_tables.stride(0),
                                    kv_cache.size(0), max_query_len, num_splits, window, (float)scale,
-                                   early_meta ? 1 : 0, BIAS_GATE_ARGS, dtype_code(q), stream()), "decode_attention_umma");
+                                   early_meta ? 1 : 0, BIAS_GATE_ARGS, (int)keep_first, sigmoid, dtype_code(q), stream()), "decode_attention_umma");
 }
 
 extern at::Tensor g_kernel_trace;
@@ -1004,7 +1008,8 @@ extern at::Tensor g_kernel_trace;
 void prefill_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
                             const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
                             const c10::optional<at::Tensor>& lse, int64_t max_query_len, int64_t window, double scale,
-                            const c10::optional<at::Tensor>& bias, const c10::optional<at::Tensor>& gate) {
+                            const c10::optional<at::Tensor>& bias, const c10::optional<at::Tensor>& gate,
+                            int64_t keep_first, bool sigmoid) {
   check_bias_gate(q, bias, gate);
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && kv_cache.dim() == 5);
   TORCH_CHECK(q.size(2) == 128 && kv_cache.size(4) == 128 && kv_cache.size(1) == 2 && out.sizes() == q.sizes());
@@ -1031,7 +1036,7 @@ void prefill_attention_umma(at::Tensor out, const at::Tensor& q, const at::Tenso
                                     sinks.has_value() ? sinks->data_ptr<float>() : nullptr, gs.status.data_ptr<int>(),
                                     (int)seq_lens.size(0), (int)q.size(1), (int)kv_cache.size(2), 128, (int)kv_cache.size(3),
                                     (int)block_tables.stride(0), kv_cache.size(0), (int)max_query_len, (int)window,
-                                    (float)scale, BIAS_GATE_ARGS, dtype_code(q),
+                                    (float)scale, BIAS_GATE_ARGS, (int)keep_first, sigmoid, dtype_code(q),
                                     (g_kernel_trace.defined() &&
                                      g_kernel_trace.numel() >= (int64_t)seq_lens.size(0) * q.size(1) * ((max_query_len + 127) / 128) * 24)
                                         ? reinterpret_cast<unsigned long long*>(g_kernel_trace.data_ptr<int64_t>()) : nullptr,
@@ -1558,49 +1563,173 @@ void poly_norm(at::Tensor out, const at::Tensor& z, const at::Tensor& coeff, int
   check(b200_poly_norm(out.data_ptr(), out.stride(0), z.data_ptr(), z.stride(0), coeff.data_ptr<float>(), z.size(0), (int)width,
                        (int)z.size(1), (float)eps, dtype_code(z), stream()), "poly_norm");
 }
-// q, k, v: column slices [T, heads * head size] of one row-strided tensor; q_out [T, Hq, Dc]; v_out / v_in [T, Hkv * Dv]
+// q, k, v: column slices [T, heads * head size] of one row-strided tensor; q_out [T, Hq, Dc]; v_out / v_in [T, Hkv * Dv];
+// q_norm, k_norm [D] fp32; table [T, pairs, 2] fp32
 void attn_prep_cache(at::Tensor q_out, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at::Tensor kv_cache,
                      const at::Tensor& slots, const at::Tensor& positions, int64_t num_heads, int64_t num_kv_heads,
                      double temp_coef, int64_t temp_every, const c10::optional<at::Tensor>& v_out,
-                     const c10::optional<at::Tensor>& v_in, double share, double eps) {
+                     const c10::optional<at::Tensor>& v_in, double share, double eps, bool v_norm,
+                     const c10::optional<at::Tensor>& q_norm, const c10::optional<at::Tensor>& k_norm,
+                     const c10::optional<at::Tensor>& table) {
   TORCH_CHECK(q_out.is_contiguous() && kv_cache.is_contiguous() && kv_cache.dim() == 5 && kv_cache.size(2) == num_kv_heads);
   TORCH_CHECK(q.stride(1) == 1 && k.stride(1) == 1 && v.stride(1) == 1 && q.stride(0) == k.stride(0) && q.stride(0) == v.stride(0));
   TORCH_CHECK(q.scalar_type() == q_out.scalar_type() && q.scalar_type() == kv_cache.scalar_type() && temp_every >= 0);
-  const int64_t D = q.size(1) / num_heads, Dv = v.size(1) / num_kv_heads, Dc = kv_cache.size(4);
-  TORCH_CHECK(k.size(1) == D * num_kv_heads && q_out.numel() == q.size(0) * num_heads * Dc && slots.numel() == q.size(0) &&
+  AttnPrepArgs a;
+  memset(&a, 0, sizeof(a));
+  a.Hq = (int)num_heads; a.Hkv = (int)num_kv_heads;
+  a.D = (int)(q.size(1) / num_heads); a.Dv = (int)(v.size(1) / num_kv_heads); a.Dc = (int)kv_cache.size(4);
+  TORCH_CHECK(k.size(1) == a.D * num_kv_heads && q_out.numel() == q.size(0) * num_heads * a.Dc && slots.numel() == q.size(0) &&
               positions.numel() == q.size(0));
   for (const auto* t : {&v_out, &v_in})
     if (t->has_value()) TORCH_CHECK((*t)->is_contiguous() && (*t)->sizes() == v.sizes() && (*t)->scalar_type() == v.scalar_type());
-  check(b200_attn_prep_cache(q_out.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), kv_cache.data_ptr(),
-                             slots.data_ptr<int64_t>(), positions.data_ptr<int64_t>(), const_cast<void*>(opt_ptr(v_out)),
-                             opt_ptr(v_in), (float)share, (float)temp_coef, temp_every, q.size(0), (int)num_heads,
-                             (int)num_kv_heads, (int)D, (int)Dv, (int)Dc, (int)kv_cache.size(3), kv_cache.size(0), (float)eps,
-                             dtype_code(q), stream()), "attn_prep_cache");
+  TORCH_CHECK(q_norm.has_value() == k_norm.has_value());
+  for (const auto* t : {&q_norm, &k_norm})
+    if (t->has_value()) TORCH_CHECK((*t)->is_contiguous() && (*t)->scalar_type() == at::kFloat && (*t)->numel() == a.D);
+  if (table.has_value()) {
+    TORCH_CHECK(table->is_contiguous() && table->scalar_type() == at::kFloat && table->dim() == 3 && table->size(0) == q.size(0) &&
+                table->size(2) == 2);
+    a.table = table->data_ptr<float>(); a.pairs = (int)table->size(1);
+  }
+  a.q = q.data_ptr(); a.k = k.data_ptr(); a.v = v.data_ptr(); a.q_out = q_out.data_ptr(); a.cache = kv_cache.data_ptr();
+  a.slots = slots.data_ptr<int64_t>(); a.positions = positions.data_ptr<int64_t>();
+  a.q_norm = q_norm.has_value() ? q_norm->data_ptr<float>() : nullptr;
+  a.k_norm = k_norm.has_value() ? k_norm->data_ptr<float>() : nullptr;
+  a.v_out = const_cast<void*>(opt_ptr(v_out)); a.v_in = opt_ptr(v_in);
+  a.stride = q.stride(0); a.num_blocks = kv_cache.size(0); a.block_size = (int)kv_cache.size(3);
+  a.temp_every = temp_every; a.v_norm = v_norm; a.share = (float)share; a.temp_coef = (float)temp_coef; a.eps = (float)eps;
+  check(b200_attn_prep_cache(&a, q.size(0), dtype_code(q), stream()), "attn_prep_cache");
+}
+// ------------------------------------------- stream normalised on the sublayers' outputs, convolution of their inputs
+// conv [taps, ld], state [slots, taps - 1, ld] (absent for one tap) and the step's metadata
+void fill_conv(PostNormArgs& a, const at::Tensor& x, const at::Tensor& conv, const c10::optional<at::Tensor>& state,
+               const at::Tensor& qsl, const at::Tensor& slots, const at::Tensor& has_init) {
+  TORCH_CHECK(conv.dim() == 2 && conv.is_contiguous() && conv.scalar_type() == at::kFloat && conv.size(1) == x.size(1));
+  a.taps = (int)conv.size(0); a.conv = conv.data_ptr<float>();
+  TORCH_CHECK(a.taps == 1 || state.has_value());
+  if (state.has_value()) {
+    TORCH_CHECK(state->is_contiguous() && state->scalar_type() == at::kFloat && state->dim() == 3 &&
+                state->size(1) == a.taps - 1 && state->size(2) == x.size(1));
+    a.state = state->data_ptr<float>(); a.num_slots = state->size(0);
+  }
+  TORCH_CHECK(qsl.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && has_init.scalar_type() == at::kInt &&
+              qsl.numel() == slots.numel() + 1);
+  a.qsl = qsl.data_ptr<int>(); a.slots = slots.data_ptr<int>(); a.has_init = has_init.data_ptr<int>();
+  a.num_reqs = (int)slots.numel();
+}
+void fill_postnorm(PostNormArgs& a, at::Tensor& x, const c10::optional<at::Tensor>& h, const c10::optional<at::Tensor>& conv,
+                   const c10::optional<at::Tensor>& state, const c10::optional<at::Tensor>& qsl,
+                   const c10::optional<at::Tensor>& slots, const c10::optional<at::Tensor>& has_init) {
+  memset(&a, 0, sizeof(a));
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && x.scalar_type() == at::kFloat);
+  a.x = x.data_ptr<float>(); a.T = x.size(0); a.ld = (int)x.size(1);
+  if (h.has_value()) {
+    TORCH_CHECK(h->is_contiguous() && h->sizes() == x.sizes() && h->data_ptr() != x.data_ptr());
+    a.h = h->data_ptr();
+  }
+  TORCH_CHECK(!conv.has_value() || h.has_value());
+  if (conv.has_value()) fill_conv(a, x, *conv, state, *qsl, *slots, *has_init);
+}
+// x = table[ids] * scale, and with conv h = x + conv(x)
+void embed_postnorm(at::Tensor x, const c10::optional<at::Tensor>& h, const at::Tensor& ids, const at::Tensor& table, double scale,
+                    const c10::optional<at::Tensor>& conv, const c10::optional<at::Tensor>& state,
+                    const c10::optional<at::Tensor>& qsl, const c10::optional<at::Tensor>& slots,
+                    const c10::optional<at::Tensor>& has_init) {
+  PostNormArgs a;
+  fill_postnorm(a, x, h, conv, state, qsl, slots, has_init);
+  TORCH_CHECK(table.is_contiguous() && table.dim() == 2 && table.size(1) == x.size(1) && ids.scalar_type() == at::kLong &&
+              ids.numel() == x.size(0));
+  if (h.has_value()) TORCH_CHECK(h->scalar_type() == table.scalar_type());
+  a.table = table.data_ptr(); a.table_rows = table.size(0); a.ids = ids.data_ptr<int64_t>(); a.scale = (float)scale;
+  a.width = a.ld;
+  check(b200_postnorm(&a, dtype_code(table), stream()), "embed_postnorm");
+}
+// x += LayerNorm(y + sum of weights * (rows[places] | pass)) * weight; h: x + conv(x), or LayerNorm(x) * final_weight
+void postnorm(at::Tensor x, const c10::optional<at::Tensor>& h, const c10::optional<at::Tensor>& y,
+              const c10::optional<at::Tensor>& rows, const c10::optional<at::Tensor>& places,
+              const c10::optional<at::Tensor>& weights, const c10::optional<at::Tensor>& pass, const at::Tensor& weight, double eps,
+              const c10::optional<at::Tensor>& final_weight, const c10::optional<at::Tensor>& conv,
+              const c10::optional<at::Tensor>& state, const c10::optional<at::Tensor>& qsl, const c10::optional<at::Tensor>& slots,
+              const c10::optional<at::Tensor>& has_init) {
+  PostNormArgs a;
+  fill_postnorm(a, x, h, conv, state, qsl, slots, has_init);
+  TORCH_CHECK((y.has_value() || rows.has_value()) && !(conv.has_value() && final_weight.has_value()) &&
+              (h.has_value() == (conv.has_value() || final_weight.has_value())));
+  const int dt = dtype_code(y.has_value() ? *y : *rows);
+  if (h.has_value()) TORCH_CHECK(dtype_code(*h) == dt);
+  TORCH_CHECK(weight.scalar_type() == at::kFloat && weight.is_contiguous() && weight.numel() <= x.size(1));
+  a.width = (int)weight.numel(); a.weight = weight.data_ptr<float>(); a.eps = (float)eps;
+  if (y.has_value()) {
+    TORCH_CHECK(y->dim() == 2 && y->sizes() == x.sizes() && y->stride(1) == 1);
+    a.y = y->data_ptr(); a.y_stride = y->stride(0);
+  }
+  if (rows.has_value() && x.size(0) > 0) {
+    TORCH_CHECK(rows->dim() == 2 && rows->size(1) == x.size(1) && rows->stride(1) == 1 && dtype_code(*rows) == dt);
+    TORCH_CHECK(pass->dim() == 2 && pass->sizes() == x.sizes() && pass->stride(1) == 1 && dtype_code(*pass) == dt);
+    TORCH_CHECK(places->scalar_type() == at::kInt && places->is_contiguous() && weights->scalar_type() == at::kFloat &&
+                weights->is_contiguous() && places->numel() == weights->numel() && places->numel() % x.size(0) == 0);
+    a.rows = rows->data_ptr(); a.rows_stride = rows->stride(0); a.pass = pass->data_ptr(); a.pass_stride = pass->stride(0);
+    a.places = places->data_ptr<int>(); a.weights = weights->data_ptr<float>(); a.k = (int)(places->numel() / x.size(0));
+  }
+  if (final_weight.has_value()) {
+    TORCH_CHECK(final_weight->scalar_type() == at::kFloat && final_weight->is_contiguous() && final_weight->numel() == a.width);
+    a.final_weight = final_weight->data_ptr<float>();
+  }
+  check(b200_postnorm(&a, dt, stream()), "postnorm");
+}
+void input_conv(const at::Tensor& x, at::Tensor h, const at::Tensor& conv, const c10::optional<at::Tensor>& state,
+                const at::Tensor& qsl, const at::Tensor& slots, const at::Tensor& has_init, int64_t max_query_len) {
+  PostNormArgs a;
+  at::Tensor xs = x;
+  fill_postnorm(a, xs, h, conv, state, qsl, slots, has_init);
+  a.max_query_len = (int)max_query_len;
+  check(b200_input_conv(&a, dtype_code(h), stream()), "input_conv");
+}
+// z, x, g: column slices [T, width] of one projection; out [T, >= width]
+void gated_blend(at::Tensor out, const at::Tensor& z, const at::Tensor& x, const at::Tensor& g, const at::Tensor& z_bias,
+                 const at::Tensor& x_bias, at::Tensor state, const at::Tensor& qsl, const at::Tensor& slots,
+                 const at::Tensor& has_init, bool steps) {
+  BlendArgs a;
+  memset(&a, 0, sizeof(a));
+  a.width = (int)z.size(1); a.stride = z.stride(0); a.out_stride = out.stride(0);
+  TORCH_CHECK(out.dim() == 2 && out.stride(1) == 1 && out.size(1) >= a.width && out.scalar_type() == z.scalar_type());
+  for (const at::Tensor* t : {&z, &x, &g})
+    TORCH_CHECK(t->dim() == 2 && t->sizes() == z.sizes() && t->stride(1) == 1 && t->stride(0) == a.stride &&
+                t->scalar_type() == z.scalar_type() && t->size(0) == out.size(0));
+  for (const at::Tensor* t : {&z_bias, &x_bias})
+    TORCH_CHECK(t->scalar_type() == at::kFloat && t->is_contiguous() && t->numel() == a.width);
+  TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() == 2 && state.size(1) == a.width);
+  TORCH_CHECK(qsl.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && has_init.scalar_type() == at::kInt &&
+              qsl.numel() == slots.numel() + 1);
+  a.out = out.data_ptr(); a.z = z.data_ptr(); a.x = x.data_ptr(); a.g = g.data_ptr();
+  a.z_bias = z_bias.data_ptr<float>(); a.x_bias = x_bias.data_ptr<float>(); a.state = state.data_ptr<float>();
+  a.num_slots = state.size(0); a.qsl = qsl.data_ptr<int>(); a.slots = slots.data_ptr<int>();
+  a.has_init = has_init.data_ptr<int>(); a.R = (int)slots.numel(); a.steps = steps;
+  check(b200_gated_blend(&a, dtype_code(z), stream()), "gated_blend");
 }
 // x [M, K] sorted by expert (lod [E + 1]), w [E, N, K]
-void gemm_f32_grouped(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const at::Tensor& lod) {
+void gemm_f32_grouped(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const at::Tensor& lod, bool relu2) {
   TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && out.dim() == 2 && x.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1);
   TORCH_CHECK(x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && out.scalar_type() == at::kFloat);
   TORCH_CHECK(x.size(1) == w.size(2) && out.size(0) == x.size(0) && out.size(1) == w.size(1) && lod.scalar_type() == at::kInt &&
               lod.is_contiguous() && lod.numel() == w.size(0) + 1);
   check(b200_gemm_f32_grouped(out.data_ptr<float>(), out.stride(0), x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(),
-                              lod.data_ptr<int>(), x.size(0), (int)w.size(0), (int)w.size(1), (int)w.size(2), stream()),
+                              lod.data_ptr<int>(), x.size(0), (int)w.size(0), (int)w.size(1), (int)w.size(2), relu2, stream()),
         "gemm_f32_grouped");
 }
-void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& bias) {
+void gemm_f32(at::Tensor out, const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& bias, bool relu2) {
   TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1);
   TORCH_CHECK(x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && out.scalar_type() == at::kFloat);
   TORCH_CHECK(x.size(1) == w.size(1) && out.size(0) == x.size(0) && out.size(1) == w.size(0));
   if (bias.has_value()) TORCH_CHECK(bias->scalar_type() == at::kFloat && bias->numel() == w.size(0));
   check(b200_gemm_f32(out.data_ptr<float>(), out.stride(0), x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(), w.stride(0),
                       bias.has_value() ? bias->data_ptr<float>() : nullptr, x.size(0), (int)w.size(0), (int)w.size(1),
-                      stream()), "gemm_f32");
+                      relu2, stream()), "gemm_f32");
 }
 // latent_dv > 0: kv_cache [blocks, block_size, D] holds latent rows shared by all heads, out [T, Hq, latent_dv]
 void paged_attention_generic(at::Tensor out, const at::Tensor& q, const at::Tensor& kv_cache, const at::Tensor& block_tables,
                              const at::Tensor& seq_lens, const at::Tensor& qsl, const c10::optional<at::Tensor>& sinks,
                              int64_t latent_dv, int64_t window, double scale, const c10::optional<at::Tensor>& bias,
-                             const c10::optional<at::Tensor>& gate) {
+                             const c10::optional<at::Tensor>& gate, int64_t keep_first, bool sigmoid) {
   check_bias_gate(q, bias, gate);
   const bool latent = latent_dv > 0;
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && kv_cache.is_contiguous() && q.dim() == 3 && out.dim() == 3 &&
@@ -1616,7 +1745,8 @@ void paged_attention_generic(at::Tensor out, const at::Tensor& q, const at::Tens
                                      sinks.has_value() ? sinks->data_ptr<float>() : nullptr, q.size(0), (int)seq_lens.size(0),
                                      (int)q.size(1), latent ? 1 : (int)kv_cache.size(2), (int)q.size(2),
                                      (int)kv_cache.size(latent ? 1 : 3), (int)block_tables.stride(0), kv_cache.size(0),
-                                     (int)latent_dv, (int)window, (float)scale, BIAS_GATE_ARGS, dtype_code(q), stream()),
+                                     (int)latent_dv, (int)window, (float)scale, BIAS_GATE_ARGS, (int)keep_first, sigmoid,
+                                     dtype_code(q), stream()),
         "paged_attention_generic");
 }
 
@@ -1852,13 +1982,16 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_int8", &gemm_int8);
   m.def("quant_int8_token", &quant_int8_token);
   m.def("set_gemm_decode_comm", &set_gemm_decode_comm);
-  m.def("grouped_gemm", &grouped_gemm);
-  m.def("moe_route", &moe_route);
+  m.def("grouped_gemm", &grouped_gemm, py::arg("out"), py::arg("x"), py::arg("w"), py::arg("lod"), py::arg("bias"),
+        py::arg("a_scale_t"), py::arg("w_scale"), py::arg("bn"), py::arg("act") = 0);
+  m.def("moe_route", &moe_route, py::arg("logits"), py::arg("bias"), py::arg("k"), py::arg("mode"), py::arg("renorm"),
+        py::arg("n_group"), py::arg("topk_group"), py::arg("scale"), py::arg("group_top") = 2);
   m.def("moe_permute", &moe_permute, py::arg("x"), py::arg("ids"), py::arg("emap"), py::arg("E_local"),
         py::arg("E_global"), py::arg("state"), py::arg("max_rows") = 0, py::arg("factors") = py::none());
   m.def("moe_unpermute", &moe_unpermute);
   m.def("router_gemm_small", &router_gemm_small);
-  m.def("router_route_small", &router_route_small);
+  m.def("router_route_small", &router_route_small, py::arg("x"), py::arg("w"), py::arg("wbias"), py::arg("bias"), py::arg("k"),
+        py::arg("mode"), py::arg("renorm"), py::arg("n_group"), py::arg("topk_group"), py::arg("scale"), py::arg("group_top") = 2);
   m.def("moe_prepare_small", &moe_prepare_small, py::arg("x"), py::arg("ids"), py::arg("emap"), py::arg("E_local"),
         py::arg("E_global"), py::arg("quant"), py::arg("factors") = py::none());
   m.def("act_mul_quant_fp8", &act_mul_quant_fp8);
@@ -1878,16 +2011,25 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("qk_unit_norm_cache", &qk_unit_norm_cache);
   m.def("channel_delta_rule", &channel_delta_rule);
   m.def("fixed_decay_attention", &fixed_decay_attention);
-  m.def("gemm_f32", &gemm_f32);
-  m.def("gemm_f32_grouped", &gemm_f32_grouped);
+  m.def("gemm_f32", &gemm_f32, py::arg("out"), py::arg("x"), py::arg("w"), py::arg("bias"), py::arg("relu2") = false);
+  m.def("gemm_f32_grouped", &gemm_f32_grouped, py::arg("out"), py::arg("x"), py::arg("w"), py::arg("lod"),
+        py::arg("relu2") = false);
   m.def("gated_write_attention", &gated_write_attention);
   m.def("embed_rmsnorm", &embed_rmsnorm);
   m.def("sandwich_rmsnorm", &sandwich_rmsnorm);
   m.def("poly_norm", &poly_norm);
-  m.def("attn_prep_cache", &attn_prep_cache);
+  m.def("embed_postnorm", &embed_postnorm);
+  m.def("postnorm", &postnorm);
+  m.def("input_conv", &input_conv);
+  m.def("gated_blend", &gated_blend);
+  m.def("attn_prep_cache", &attn_prep_cache, py::arg("q_out"), py::arg("q"), py::arg("k"), py::arg("v"), py::arg("kv_cache"),
+        py::arg("slots"), py::arg("positions"), py::arg("num_heads"), py::arg("num_kv_heads"), py::arg("temp_coef"),
+        py::arg("temp_every"), py::arg("v_out"), py::arg("v_in"), py::arg("share"), py::arg("eps"), py::arg("v_norm") = true,
+        py::arg("q_norm") = py::none(), py::arg("k_norm") = py::none(), py::arg("table") = py::none());
   m.def("paged_attention_generic", &paged_attention_generic, py::arg("out"), py::arg("q"), py::arg("kv_cache"),
         py::arg("block_tables"), py::arg("seq_lens"), py::arg("qsl"), py::arg("sinks"), py::arg("latent_dv"),
-        py::arg("window"), py::arg("scale"), py::arg("bias") = py::none(), py::arg("gate") = py::none());
+        py::arg("window"), py::arg("scale"), py::arg("bias") = py::none(), py::arg("gate") = py::none(),
+        py::arg("keep_first") = 0, py::arg("sigmoid") = false);
   m.def("rotary_table", &rotary_table);
   m.def("latent_prep", &latent_prep);
   m.def("rotate_heads", &rotate_heads);
@@ -1921,12 +2063,13 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("decode_attention_umma", &decode_attention_umma, py::arg("out"), py::arg("q"), py::arg("kv_cache"),
         py::arg("block_tables"), py::arg("seq_lens"), py::arg("qsl"), py::arg("sinks"), py::arg("ws_o"),
         py::arg("ws_lse"), py::arg("max_query_len"), py::arg("num_splits"), py::arg("window"), py::arg("scale"),
-        py::arg("early_meta"), py::arg("bias") = py::none(), py::arg("gate") = py::none());
+        py::arg("early_meta"), py::arg("bias") = py::none(), py::arg("gate") = py::none(), py::arg("keep_first") = 0,
+        py::arg("sigmoid") = false);
   m.def("mla_decode_umma", &mla_decode_umma);
   m.def("prefill_attention_umma", &prefill_attention_umma, py::arg("out"), py::arg("q"), py::arg("kv_cache"),
         py::arg("block_tables"), py::arg("seq_lens"), py::arg("qsl"), py::arg("sinks"), py::arg("lse"),
         py::arg("max_query_len"), py::arg("window"), py::arg("scale"), py::arg("bias") = py::none(),
-        py::arg("gate") = py::none());
+        py::arg("gate") = py::none(), py::arg("keep_first") = 0, py::arg("sigmoid") = false);
   m.def("mla_prefill_umma", &mla_prefill_umma);
   m.def("indexer_prep", &indexer_prep);
   m.def("gather_mla_rows", &gather_mla_rows);

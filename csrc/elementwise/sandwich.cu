@@ -3,8 +3,9 @@
 //   sandwich_rmsnorm     stream += rms(y) * w_post;  h = rms(stream) * w_pre        (one sublayer's end, the next one's start;
 //                        y may be given as `k` rows per token in expert order, which are summed on the way in)
 //   poly_norm            a N(z) + b N(z^2) + c N(z^3) + e over a feed-forward row, N = division by the root mean square
-//   attn_prep_cache      split a fused projection: q times a temperature that grows with the position, k as it is, v of
-//                        unit root mean square and mixed with another layer's values; K / V into the paged cache
+//   attn_prep_cache      split a fused projection: q and k heads normed and rotated (or as they are), q times a temperature that
+//                        grows with the position, v as it is or of unit root mean square and mixed with another layer's
+//                        values; K / V into the paged cache
 // Weights come ready to multiply (a weight stored around zero arrives as 1 + w, a residual factor folded in).
 // These kernels are launched with programmatic dependent launch: pointers carry no __restrict__, which would let the
 // compiler read them through the non-coherent path before the producers have finished.  Statistics are fp32 (this file is
@@ -193,77 +194,95 @@ __global__ void __launch_bounds__(THR) poly_norm_kernel(T* out, int64_t ldo, con
 }
 
 // One warp per (token, head) of q, k and v; head sizes D (q, k) and Dv (v) are zero-padded to Dc in q_out and in the cache
-// [block][2][Hkv][slot][Dc].  v_out [T][Hkv * Dv]: the normed values (before mixing) for later layers; v_in: such values of
-// an earlier layer, mixed in with the given share.
+// [block][2][Hkv][slot][Dc].  See AttnPrepArgs for what happens to a head on the way.
 template <typename T>
-__global__ void __launch_bounds__(256) attn_prep_cache_kernel(T* q_out, const T* q, const T* k, const T* v, int64_t stride,
-                                                              T* cache, const int64_t* slots, const int64_t* positions,
-                                                              T* v_out, const T* v_in, float share, float temp_coef,
-                                                              int64_t temp_every, int Hq, int Hkv, int D, int Dv, int Dc,
-                                                              int block_size, int64_t num_blocks, float eps, int vec) {
+__global__ void __launch_bounds__(256) attn_prep_cache_kernel(AttnPrepArgs a, int vec) {
   griddep_launch();
   griddep_wait();
   const int64_t t = blockIdx.x;
+  const int Hq = a.Hq, Hkv = a.Hkv, Dc = a.Dc;
   const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (head >= Hq + 2 * Hkv) return;
   const bool is_q = head < Hq, is_v = head >= Hq + Hkv;
-  const int n = is_v ? Dv : D;
+  const int n = is_v ? a.Dv : a.D;
   const int kvh = is_v ? head - Hq - Hkv : head - Hq;
   const T* src;
   T* dst = nullptr;
   float f = 1.f;
   if (is_q) {
-    src = q + t * stride + (int64_t)head * D;
-    dst = q_out + (t * Hq + head) * (int64_t)Dc;
-    if (temp_every > 0) f = 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1));
+    src = reinterpret_cast<const T*>(a.q) + t * a.stride + (int64_t)head * n;
+    dst = reinterpret_cast<T*>(a.q_out) + (t * Hq + head) * (int64_t)Dc;
+    if (a.temp_every > 0) f = 1.f + a.temp_coef * logf((float)((a.positions[t] + 1) / a.temp_every + 1));
   } else {
-    src = (is_v ? v : k) + t * stride + (int64_t)kvh * n;
-    const int64_t slot = slots[t];
-    if (slot >= 0 && slot < num_blocks * block_size)
-      dst = cache + ((((slot / block_size) * 2 + (is_v ? 1 : 0)) * Hkv + kvh) * block_size + slot % block_size) * (int64_t)Dc;
+    src = reinterpret_cast<const T*>(is_v ? a.v : a.k) + t * a.stride + (int64_t)kvh * n;
+    const int64_t slot = a.slots[t];
+    if (slot >= 0 && slot < a.num_blocks * a.block_size)
+      dst = reinterpret_cast<T*>(a.cache) +
+            ((((slot / a.block_size) * 2 + (is_v ? 1 : 0)) * Hkv + kvh) * a.block_size + slot % a.block_size) * (int64_t)Dc;
   }
-  if (is_v) {
+  const float* w = is_v ? nullptr : is_q ? a.q_norm : a.k_norm;
+  if (is_v ? a.v_norm != 0 : w != nullptr) {
     float ss = 0.f;
     if (vec) {
       for (int i = lane * 4; i < n; i += 128) {
-        float a[4];
-        load4(a, src + i);
-        ss += a[0] * a[0] + a[1] * a[1] + a[2] * a[2] + a[3] * a[3];
+        float x[4];
+        load4(x, src + i);
+        ss += x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3];
       }
     } else {
       for (int i = lane; i < n; i += 32) { const float x = to_f(src[i]); ss += x * x; }
     }
-    f = 1.f / sqrtf(warp_sum(ss) / n + eps);
+    f *= 1.f / sqrtf(warp_sum(ss) / n + a.eps);
   }
-  const int64_t vo = (t * Hkv + kvh) * (int64_t)Dv;
-  const T* mix = is_v && v_in != nullptr ? v_in + vo : nullptr;
-  T* keep = is_v && v_out != nullptr ? v_out + vo : nullptr;
+  const int pairs = is_v || a.table == nullptr ? 0 : a.pairs;   // column i < pairs turns with column i + pairs
+  const float* turn = a.table == nullptr ? nullptr : a.table + t * a.pairs * 2;
+  const int64_t vo = (t * Hkv + kvh) * (int64_t)a.Dv;
+  const T* mix = is_v && a.v_in != nullptr ? reinterpret_cast<const T*>(a.v_in) + vo : nullptr;
+  T* keep = is_v && a.v_out != nullptr ? reinterpret_cast<T*>(a.v_out) + vo : nullptr;
   if (vec) {
-    for (int i = lane * 4; i < Dc; i += 128) {
-      float a[4] = {0.f, 0.f, 0.f, 0.f};
-      if (i < n) {
-        load4(a, src + i);
+    auto scaled = [&](float (&x)[4], int i) {
+      load4(x, src + i);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) a[j] *= f;
-        if (keep != nullptr) store4(keep + i, a);
+      for (int j = 0; j < 4; ++j) x[j] *= w == nullptr ? f : f * w[i + j];
+    };
+    for (int i = lane * 4; i < Dc; i += 128) {
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (i < n) {
+        scaled(x, i);
+        if (i < 2 * pairs) {
+          const bool lower = i < pairs;
+          float o[4];
+          scaled(o, lower ? i + pairs : i - pairs);
+          const float* cs = turn + 2 * (lower ? i : i - pairs);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) x[j] = x[j] * cs[2 * j] + (lower ? -o[j] : o[j]) * cs[2 * j + 1];
+        }
+        if (keep != nullptr) store4(keep + i, x);
         if (mix != nullptr) {
           float b[4];
           load4(b, mix + i);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) a[j] = (1.f - share) * a[j] + share * b[j];
+          for (int j = 0; j < 4; ++j) x[j] = (1.f - a.share) * x[j] + a.share * b[j];
         }
       }
-      if (dst != nullptr) store4(dst + i, a);
+      if (dst != nullptr) store4(dst + i, x);
     }
   } else {
+    auto scaled = [&](int i) { return to_f(src[i]) * (w == nullptr ? f : f * w[i]); };
     for (int i = lane; i < Dc; i += 32) {
-      float a = 0.f;
+      float x = 0.f;
       if (i < n) {
-        a = to_f(src[i]) * f;
-        if (keep != nullptr) keep[i] = from_f<T>(a);
-        if (mix != nullptr) a = (1.f - share) * a + share * to_f(mix[i]);
+        x = scaled(i);
+        if (i < 2 * pairs) {
+          const bool lower = i < pairs;
+          const float o = scaled(lower ? i + pairs : i - pairs);
+          const float* cs = turn + 2 * (lower ? i : i - pairs);
+          x = x * cs[0] + (lower ? -o : o) * cs[1];
+        }
+        if (keep != nullptr) keep[i] = from_f<T>(x);
+        if (mix != nullptr) x = (1.f - a.share) * x + a.share * to_f(mix[i]);
       }
-      if (dst != nullptr) dst[i] = from_f<T>(a);
+      if (dst != nullptr) dst[i] = from_f<T>(x);
     }
   }
 }
@@ -325,17 +344,14 @@ extern "C" int b200_poly_norm(void* out, int64_t ldo, const void* z, int64_t ldz
   return (int)cudaGetLastError();
 }
 
-extern "C" int b200_attn_prep_cache(void* q_out, const void* q, const void* k, const void* v, int64_t stride, void* kv_cache,
-                                    const int64_t* slots, const int64_t* positions, void* v_out, const void* v_in, float share,
-                                    float temp_coef, int64_t temp_every, int64_t T_, int Hq, int Hkv, int D, int Dv, int Dc,
-                                    int block_size, int64_t num_blocks, float eps, int dtype, cudaStream_t st) {
+extern "C" int b200_attn_prep_cache(const AttnPrepArgs* args, int64_t T_, int dtype, cudaStream_t st) {
+  const AttnPrepArgs& a = *args;
   if (T_ == 0) return 0;
-  if (D > Dc || Dv > Dc) return 3;
-  const uintptr_t al = (uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)v_out | (uintptr_t)v_in;
-  const int vec = D % 4 == 0 && Dv % 4 == 0 && Dc % 4 == 0 && stride % 4 == 0 && al % 16 == 0;
-  dim3 grid((unsigned)T_, (Hq + 2 * Hkv + 7) / 8);
-  B200_DISPATCH_DTYPE(dtype, launch_pdl(attn_prep_cache_kernel<T>, grid, dim3(256), 0, st, (T*)q_out, (const T*)q, (const T*)k,
-                                       (const T*)v, stride, (T*)kv_cache, slots, positions, (T*)v_out, (const T*)v_in, share,
-                                       temp_coef, temp_every, Hq, Hkv, D, Dv, Dc, block_size, num_blocks, eps, vec));
+  if (a.D > a.Dc || a.Dv > a.Dc || (a.table != nullptr && 2 * a.pairs > a.D)) return 3;
+  const uintptr_t al = (uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.v_out | (uintptr_t)a.v_in;
+  const int vec = a.D % 4 == 0 && a.Dv % 4 == 0 && a.Dc % 4 == 0 && a.stride % 4 == 0 && al % 16 == 0 &&
+                  (a.table == nullptr || a.pairs % 4 == 0);
+  dim3 grid((unsigned)T_, (a.Hq + 2 * a.Hkv + 7) / 8);
+  B200_DISPATCH_DTYPE(dtype, launch_pdl(attn_prep_cache_kernel<T>, grid, dim3(256), 0, st, a, vec));
   return (int)cudaGetLastError();
 }

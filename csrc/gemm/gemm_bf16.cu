@@ -69,7 +69,8 @@ __device__ __forceinline__ void red_release_sys_add(uint32_t* p, uint32_t v) {
 }
 
 // Gated activations fused into the epilogue of a gate/up projection whose weight rows are interleaved per tile as
-// [64 gate rows | 64 up rows]: act = 1 SiLU, 2 GELU (tanh), 3 clamped SwiGLU of GPT-OSS.
+// [64 gate rows | 64 up rows]: act = 1 SiLU, 2 GELU (tanh), 3 clamped SwiGLU of GPT-OSS.  act = kRelu2 (gemm_common.cuh) is
+// no gate: it applies to every output of a plain projection.
 __device__ __forceinline__ float gated_act(float g, float u, int act) {
   if (act == 1) return g / (1.f + __expf(-g)) * u;
   if (act == 2) {
@@ -335,7 +336,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         // accumulator word of token t -> real value (+ bias)
         auto val = [&](uint32_t r, int t) -> float {
           if (i8) return (float)(int)r * wsc * (t < T ? a_scale[t] : 0.f) + bv;
-          return __uint_as_float(r) + bv;
+          return unary_act(__uint_as_float(r) + bv, act);
         };
         // destination row of token t: the local output, or the owner rank's staging area
         auto row_ptr = [&](int t) -> OutT* {
@@ -346,7 +347,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           }
           return out + (size_t)t * ldo;
         };
-        if (act != 0) {
+        if (act != 0 && act != kRelu2) {
           // gate / up tile: stage [token][128] in shared memory (rounded to OutT, as an unfused projection would hand
           // it to the activation kernel), then every thread combines 8 gate features with their 8 up features and
           // writes 16 bytes of the half-width output row
@@ -515,7 +516,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
               for (int j = 0; j < 16; ++j) {
                 int t = t0 + c0 + j;
-                if (t < T) out[(size_t)t * ldo + n] = from_float<OutT>(acc[j]);
+                if (t < T) out[(size_t)t * ldo + n] = from_float<OutT>(unary_act(acc[j], act));
               }
             }
           }

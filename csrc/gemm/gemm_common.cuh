@@ -29,6 +29,16 @@ __device__ __forceinline__ bool wait_or_abort(uint64_t* bar, uint32_t parity, Ab
   return false;
 }
 
+// Activation code of a plain (ungated) projection's outputs: the square of relu.
+constexpr int kRelu2 = 4;
+__device__ __forceinline__ float unary_act(float v, int act) {
+  if (act == kRelu2) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  }
+  return v;
+}
+
 template <typename OutT>
 __device__ __forceinline__ OutT from_float(float v);
 template <>

@@ -492,7 +492,7 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
           for (int c = 0; c < BN; ++c) acc[c] *= ws * (c < T ? a_scale[c] : 0.f);
         }
 #pragma unroll
-        for (int c = 0; c < BN; ++c) tile[c * kTileStride + n_local] = from_float<OutT>(acc[c] + bv);
+        for (int c = 0; c < BN; ++c) tile[c * kTileStride + n_local] = from_float<OutT>(unary_act(acc[c] + bv, act));
         asm volatile("bar.sync 1, 128;" ::: "memory");
         if (qk.on) {
           // ---- head nt of the fused qkv row: warp = token (round-robin), lane = features l, l + 32, l + 64, l + 96 -
@@ -561,7 +561,7 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
               for (int j = 0; j < 4; ++j) dst[lane + 32 * j] = from_float<OutT>(v[j]);
             }
           }
-        } else if (act != 0) {
+        } else if (act != 0 && act != kRelu2) {
           const int n0 = nt * (BM / 2);
           const int seg = ep_tid & 7;  // 8 segments of 8 output features
           for (int rr = ep_tid >> 3; rr < BN; rr += 16) {

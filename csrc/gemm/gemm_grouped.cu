@@ -53,7 +53,7 @@ struct GParams {
   const float* a_scale; // fp8: [K/128, a_stride] (transposed activation scales)
   const float* w_scale; // fp8: [E, ceil(N/128), ceil(K/128)]
   int* status;
-  int M, N, K, E, ldo, a_stride, fmt, num_stages, bn_rows_per_expert_hint;
+  int M, N, K, E, ldo, a_stride, fmt, num_stages, act;
 };
 
 template <int BN, bool kFp8, typename OutT>
@@ -289,7 +289,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               for (int j = 0; j < 16; ++j) {
                 int row = row0 + c + j;
                 if (row < row_end)
-                  reinterpret_cast<OutT*>(p.out)[(size_t)row * p.ldo + n] = from_float<OutT>(__uint_as_float(r[j]) + bv);
+                  reinterpret_cast<OutT*>(p.out)[(size_t)row * p.ldo + n] = from_float<OutT>(unary_act(__uint_as_float(r[j]) + bv, p.act));
               }
             }
           }
@@ -336,7 +336,7 @@ static cudaError_t launch_grouped(const GroupedGemmArgs& a, const CUtensorMap& t
   GParams p;
   p.out = a.out; p.bias = a.bias; p.lod = a.lod; p.a_scale = a.a_scale; p.w_scale = a.w_scale; p.status = a.status;
   p.M = a.M; p.N = a.N; p.K = a.K; p.E = a.E; p.ldo = a.ldo; p.a_stride = a.a_stride; p.fmt = a.fmt;
-  p.num_stages = stages; p.bn_rows_per_expert_hint = 0;
+  p.num_stages = stages; p.act = a.act;
   return launch_pdl(kern, dim3(a.grid), dim3(kGThreads), (size_t)smem, st, tmW, tmX, p);
 }
 
@@ -344,7 +344,7 @@ static cudaError_t launch_grouped(const GroupedGemmArgs& a, const CUtensorMap& t
 
 extern "C" int b200_grouped_gemm_launch(const GroupedGemmArgs* a, const void* tmW, const void* tmX, cudaStream_t st) {
   using namespace b200;
-  if (a->E > kGMaxExperts) return 2;
+  if (a->E > kGMaxExperts || (a->act != 0 && (a->act != kRelu2 || a->fp8))) return 2;
   const CUtensorMap& w = *reinterpret_cast<const CUtensorMap*>(tmW);
   const CUtensorMap& x = *reinterpret_cast<const CUtensorMap*>(tmX);
   cudaError_t e = cudaErrorInvalidValue;

@@ -1,6 +1,6 @@
 // MoE routing, permutation and fp8 activation quantisation kernels.
 //
-// route:     one warp per token over E <= 512 experts: softmax / sigmoid(+bias, group-limited) /
+// route:     one warp per token over E <= 512 experts: softmax / sigmoid scores (+ selection bias, group-limited) /
 //            top-k-then-softmax, k <= 16 rounds of warp arg-max (ties -> lowest expert id).
 // permute:   histogram of (token, slot) pairs per local expert -> exclusive scan (lod) -> scatter of
 //            token rows into expert-sorted order; pairs routed to non-local experts are dropped.
@@ -18,12 +18,13 @@ namespace b200 {
 constexpr int kMaxEPerLane = 16;  // E <= 512
 constexpr int kMaxTopK = 16;
 
-// mode: 0 softmax->topk, 1 sigmoid group-limited, 2 topk->softmax
+// mode: 0 softmax->topk, 1 sigmoid->topk, 2 topk->softmax.  Modes 0 and 1 choose by score + bias.  group_top: how many of a
+// group's best selection scores add up to the group's score (1 or 2); 0 = choose without groups
 // One warp routes one token; `row` holds the token's E router logits (global or shared memory).
 template <typename T>
 __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __restrict__ out_ids, const T* row,
                                           const float* __restrict__ bias, int64_t t, int lane, int E, int k, int mode,
-                                          int renorm, int n_group, int topk_group, float scale) {
+                                          int renorm, int n_group, int topk_group, int group_top, float scale) {
   const int per = (E + 31) / 32;
   float score[kMaxEPerLane];  // unbiased weight source
   float sel[kMaxEPerLane];    // selection score
@@ -50,7 +51,7 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
     for (int s = 0; s < kMaxEPerLane; ++s) {
       int e = s * 32 + lane;
       score[s] = (s < per && e < E) ? score[s] / sum : -INFINITY;
-      sel[s] = score[s];
+      sel[s] = (bias && s < per && e < E) ? score[s] + bias[e] : score[s];
     }
   } else if (mode == 1) {
 #pragma unroll
@@ -61,53 +62,53 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
       score[s] = sg;
       sel[s] = ok ? sg + (bias ? bias[e] : 0.f) : -INFINITY;
     }
-    if (n_group > 1) {
-      // group score = sum of the two best selection scores in the group; keep the best topk_group groups
-      const int gsz = E / n_group;
-      float gscore_mine = -INFINITY;  // lane g holds the score of group g (n_group <= 32)
-      for (int g = 0; g < n_group; ++g) {
-        float b1 = -INFINITY, b2 = -INFINITY;
-#pragma unroll
-        for (int s = 0; s < kMaxEPerLane; ++s) {
-          int e = s * 32 + lane;
-          if (s < per && e < E && e / gsz == g) {
-            float v = sel[s];
-            if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
-          }
-        }
-        // merge (b1, b2) pairs across lanes
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          float o1 = __shfl_xor_sync(0xffffffff, b1, o), o2 = __shfl_xor_sync(0xffffffff, b2, o);
-          float n1 = fmaxf(b1, o1);
-          float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
-          b1 = n1; b2 = n2;
-        }
-        float gs = (gsz >= 2) ? b1 + b2 : b1;
-        if (lane == g) gscore_mine = gs;
-      }
-      uint32_t keep = 0;
-      for (int r = 0; r < topk_group; ++r) {
-        float v = gscore_mine;
-        int idx = lane;
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          float ov = __shfl_xor_sync(0xffffffff, v, o);
-          int oi = __shfl_xor_sync(0xffffffff, idx, o);
-          if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
-        }
-        keep |= 1u << idx;
-        if (lane == idx) gscore_mine = -INFINITY;
-      }
-#pragma unroll
-      for (int s = 0; s < kMaxEPerLane; ++s) {
-        int e = s * 32 + lane;
-        if (s < per && e < E && !((keep >> (e / gsz)) & 1u)) sel[s] = -INFINITY;
-      }
-    }
   } else {
 #pragma unroll
     for (int s = 0; s < kMaxEPerLane; ++s) sel[s] = score[s];
+  }
+  if (mode != 2 && n_group > 1 && group_top > 0) {
+    // group score = sum of the group_top best selection scores in the group; keep the best topk_group groups
+    const int gsz = E / n_group;
+    float gscore_mine = -INFINITY;  // lane g holds the score of group g (n_group <= 32)
+    for (int g = 0; g < n_group; ++g) {
+      float b1 = -INFINITY, b2 = -INFINITY;
+#pragma unroll
+      for (int s = 0; s < kMaxEPerLane; ++s) {
+        int e = s * 32 + lane;
+        if (s < per && e < E && e / gsz == g) {
+          float v = sel[s];
+          if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
+        }
+      }
+      // merge (b1, b2) pairs across lanes
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        float o1 = __shfl_xor_sync(0xffffffff, b1, o), o2 = __shfl_xor_sync(0xffffffff, b2, o);
+        float n1 = fmaxf(b1, o1);
+        float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
+        b1 = n1; b2 = n2;
+      }
+      float gs = (gsz >= 2 && group_top == 2) ? b1 + b2 : b1;
+      if (lane == g) gscore_mine = gs;
+    }
+    uint32_t keep = 0;
+    for (int r = 0; r < topk_group; ++r) {
+      float v = gscore_mine;
+      int idx = lane;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        float ov = __shfl_xor_sync(0xffffffff, v, o);
+        int oi = __shfl_xor_sync(0xffffffff, idx, o);
+        if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
+      }
+      keep |= 1u << idx;
+      if (lane == idx) gscore_mine = -INFINITY;
+    }
+#pragma unroll
+    for (int s = 0; s < kMaxEPerLane; ++s) {
+      int e = s * 32 + lane;
+      if (s < per && e < E && !((keep >> (e / gsz)) & 1u)) sel[s] = -INFINITY;
+    }
   }
   // k rounds of warp arg-max over sel
   float wsel[kMaxTopK];
@@ -156,13 +157,13 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
 template <typename T>
 __global__ void moe_route_kernel(float* __restrict__ out_w, int* __restrict__ out_ids, const T* __restrict__ logits,
                                  const float* __restrict__ bias, int64_t T_, int E, int k, int mode, int renorm,
-                                 int n_group, int topk_group, float scale, int64_t stride) {
+                                 int n_group, int topk_group, int group_top, float scale, int64_t stride) {
   griddep_launch();
   griddep_wait();
   const int64_t t = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T_) return;
   route_row<T>(out_w, out_ids, logits + t * stride, bias, t, threadIdx.x & 31, E, k, mode, renorm, n_group, topk_group,
-               scale);
+               group_top, scale);
 }
 
 // Router GEMM and routing in one launch for decode-sized batches: one CTA per token computes its E logits into
@@ -171,7 +172,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) router_route_small_kernel(
     float* __restrict__ out_w, int* __restrict__ out_ids, const T* __restrict__ x, int64_t x_stride,
     const T* __restrict__ w, const T* __restrict__ wbias, const float* __restrict__ bias, int E, int K, int k, int mode,
-    int renorm, int n_group, int topk_group, float scale) {
+    int renorm, int n_group, int topk_group, int group_top, float scale) {
   constexpr int V = Vec16<T>::N;
   extern __shared__ __align__(16) unsigned char smem_rr[];
   T* sx = reinterpret_cast<T*>(smem_rr);
@@ -194,7 +195,8 @@ __global__ void __launch_bounds__(256) router_route_small_kernel(
     if (lane == 0) slog[n] = acc + (wbias ? to_f(wbias[n]) : 0.f);
   }
   __syncthreads();
-  if (warp == 0) route_row<float>(out_w, out_ids, slog, bias, t, lane, E, k, mode, renorm, n_group, topk_group, scale);
+  if (warp == 0) route_row<float>(out_w, out_ids, slog, bias, t, lane, E, k, mode, renorm, n_group, topk_group, group_top,
+                                  scale);
 }
 
 // counts[e] += number of pairs routed to local expert e  (counts zeroed by the caller kernel chain)
@@ -503,14 +505,14 @@ __global__ void __launch_bounds__(256) router_gemm_small_kernel(float* __restric
 using namespace b200;
 
 extern "C" int b200_moe_route(float* out_w, int* out_ids, const void* logits, const float* bias, int64_t T_, int E,
-                              int k, int mode, int renorm, int n_group, int topk_group, float scale, int64_t stride,
+                              int k, int mode, int renorm, int n_group, int topk_group, int group_top, float scale, int64_t stride,
                               int dtype, cudaStream_t st) {
   if (T_ == 0) return 0;
   if (E > 32 * kMaxEPerLane || k > kMaxTopK || n_group > 32 || (n_group > 1 && E % n_group)) return 2;
   const int wpb = 4;
   B200_DISPATCH_DTYPE(dtype, {
     launch_pdl(moe_route_kernel<T>, dim3((T_ + wpb - 1) / wpb), dim3(wpb * 32), 0, st, out_w, out_ids,
-               (const T*)logits, bias, T_, E, k, mode, renorm, n_group, topk_group, scale, stride);
+               (const T*)logits, bias, T_, E, k, mode, renorm, n_group, topk_group, group_top, scale, stride);
   });
   return (int)cudaGetLastError();
 }
@@ -642,7 +644,8 @@ extern "C" int b200_router_gemm_small(float* out, const void* x, int64_t x_strid
 
 extern "C" int b200_router_route_small(float* out_w, int* out_ids, const void* x, int64_t x_stride, const void* w,
                                        const void* wbias, const float* bias, int64_t T_, int E, int K, int k, int mode,
-                                       int renorm, int n_group, int topk_group, float scale, int dtype, cudaStream_t st) {
+                                       int renorm, int n_group, int topk_group, int group_top, float scale, int dtype,
+                                       cudaStream_t st) {
   if (T_ == 0) return 0;
   if (E > 32 * kMaxEPerLane || k > kMaxTopK || n_group > 32 || (n_group > 1 && E % n_group)) return 2;
   const int esz = dtype == 0 ? 4 : 2;
@@ -652,7 +655,7 @@ extern "C" int b200_router_route_small(float* out_w, int* out_ids, const void* x
   B200_DISPATCH_DTYPE(dtype, {
     if (smem > 48 * 1024) ensure_dynamic_smem((const void*)router_route_small_kernel<T>, 96 * 1024);
     launch_pdl(router_route_small_kernel<T>, dim3((unsigned)T_), dim3(256), smem, st, out_w, out_ids, (const T*)x,
-               x_stride, (const T*)w, (const T*)wbias, bias, E, K, k, mode, renorm, n_group, topk_group, scale);
+               x_stride, (const T*)w, (const T*)wbias, bias, E, K, k, mode, renorm, n_group, topk_group, group_top, scale);
   });
   return (int)cudaGetLastError();
 }

@@ -27,7 +27,8 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 # Kernels that also serve fp32 models: exp / log / division / square root at full fp32 accuracy.
 PRECISE = {"linear_attn/gdn.cu", "linear_attn/recurrence.cu", "linear_attn/chunk_decay.cu", "elementwise/layernorm.cu", "gemm/gemm_f32.cu",
            "attention/paged_generic.cu", "attention/latent.cu", "elementwise/gated_stream.cu",
-           "elementwise/sandwich.cu", "linear_attn/chunk_gated.cu"}
+           "elementwise/sandwich.cu", "linear_attn/chunk_gated.cu",
+           "elementwise/postnorm.cu", "linear_attn/blend.cu"}
 
 
 def _nvcc() -> str:

@@ -40,8 +40,8 @@ class LayerSpec:
 
     type: str                   # name of the mixer (``models/mixers.py``)
     mixer: dict                 # its sizes and constants
-    mlp: Optional[dict] = None  # {"kind": "dense", "ff": width} or {"kind": "moe", "expert": {"ff", "limit"}, "router":
-    # {"experts", "top"}} (``models/feed_forward.py``), or None: the layer has no feed-forward
+    mlp: Optional[dict] = None  # {"kind": "dense", "ff": width} or {"kind": "moe", "expert": {"ff", ...}, "router":
+    # {"experts", "top", ...}, ...} (``models/feed_forward.py``), or None: the layer has no feed-forward
 
 
 @dataclass
@@ -68,7 +68,7 @@ class ModelConfig:
     o_bias: bool = False
     mlp_bias: bool = False
     qk_norm: bool = False  # per-head q/k RMSNorm (Qwen3)
-    hidden_act: str = "silu"  # "silu" | "swigluoai" | "gelu_tanh" | "poly_norm" (listed layers: no gate matrix)
+    hidden_act: str = "silu"  # "silu" | "swigluoai" | "gelu_tanh" | "poly_norm" | "relu2" (listed layers: no gate matrix)
     gemma_norm: bool = False  # (1 + w) RMSNorm
     # sliding window / sinks (GPT-OSS, MiMo-V2, Gemma)
     sliding_window: Optional[int] = None
@@ -129,7 +129,8 @@ class ModelConfig:
     global_head_dim: Optional[int] = None  # head size of the full-attention layers when it differs (Gemma-4)
     num_global_kv_heads: Optional[int] = None  # their KV head count when values are the keys (attention_k_eq_v)
     attention_k_eq_v: bool = False  # full-attention layers have no v_proj: V is the (un-normalised, un-rotated) K
-    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel, Seturax, Petipel)
+    layer_specs: tuple = ()  # one LayerSpec per layer (Bolopel, Seturax, Petipel, Kefesun)
+    input_conv_taps: int = 0  # taps of the causal convolution in front of every sublayer (listed layers)
     embedding_scale: float = 1.0  # factor of the token rows
     bigram: Optional[dict] = None  # embedding of token pairs: {"buckets", "mul_prev", "mul_cur"}
     token_shift: bool = False  # the mixers read a blend of this token's and the previous token's norm
@@ -188,7 +189,7 @@ class ModelConfig:
         """Some layer keeps a per-request state besides (or instead of) the paged cache."""
         if self.linear_attn_pattern > 0:
             return True
-        if self.token_shift or self.bigram:
+        if self.token_shift or self.bigram or self.input_conv_taps > 1:
             return True
         if not self.layer_specs:
             return False
@@ -480,19 +481,19 @@ class ModelConfig:
     @classmethod
     def _from_layer_list(cls, cfg: dict) -> "ModelConfig":
         """Configurations that list their layers one by one (``architecture``, ``width``, ``vocab``, ``norm.eps``,
-        ``layers: [{type, mixer, mlp}]``; optionally ``embedding.{scale, bigram}``, ``logit_scale`` and
-        ``residual_mult``)."""
+        ``layers: [{type, mixer, mlp}]``; optionally ``embedding.{scale, bigram}``, ``logit_scale``,
+        ``residual_mult`` and ``canon.taps``)."""
         from .models.feed_forward import FEED_FORWARDS
         from .models.mixers import MIXERS
-        specs = []
+        specs, arch = [], cfg["architecture"]
         for i, entry in enumerate(cfg["layers"]):
-            if entry["type"] not in MIXERS:
+            kind = _LAYER_LIST_MIXERS.get((arch, entry["type"]), entry["type"])
+            if kind not in MIXERS:
                 raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}; known: {sorted(MIXERS)}")
             mlp = entry.get("mlp")
             if mlp is not None and mlp.get("kind", "dense") not in FEED_FORWARDS:
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
-            specs.append(LayerSpec(entry["type"], dict(entry["mixer"]), None if mlp is None else dict(mlp)))
-        arch = cfg["architecture"]
+            specs.append(LayerSpec(kind, dict(entry["mixer"]), None if mlp is None else dict(mlp)))
         emb = cfg.get("embedding") or {}
         bigram = emb.get("bigram")
         return cls(architecture=arch, name=cfg.get("_name_or_path", arch), vocab_size=int(cfg["vocab"]),
@@ -502,7 +503,8 @@ class ModelConfig:
                    embedding_scale=float(emb.get("scale", 1.0)),
                    bigram=None if bigram is None else {k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")},
                    logit_scale=float(cfg.get("logit_scale", 1.0)),
-                   residual_multiplier=float(cfg.get("residual_mult", 1.0)), dtype=str(cfg.get("torch_dtype", "bfloat16")),
+                   residual_multiplier=float(cfg.get("residual_mult", 1.0)),
+                   input_conv_taps=int((cfg.get("canon") or {}).get("taps", 0)), dtype=str(cfg.get("torch_dtype", "bfloat16")),
                    **_LAYER_LIST_TRAITS.get(arch, {}))
 
     def complete_from_shapes(self, shapes: dict) -> "ModelConfig":
@@ -526,7 +528,10 @@ class ModelConfig:
 
 # what a design with listed layers fixes without naming it in its configuration
 _LAYER_LIST_TRAITS: dict = {"Seturax": {"hidden_act": "gelu_tanh", "token_shift": True},
-                            "Petipel": {"hidden_act": "poly_norm"}}
+                            "Petipel": {"hidden_act": "poly_norm"},
+                            "Kefesun": {"hidden_act": "relu2", "tie_word_embeddings": True}}
+# mixers that a design's configuration names by a word which other designs use for another one
+_LAYER_LIST_MIXERS: dict = {("Kefesun", "attention"): "sigmoid_attention"}
 
 
 def _leading_dense(cfg: dict) -> int:

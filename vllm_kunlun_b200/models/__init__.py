@@ -43,6 +43,8 @@ _REGISTRY = {
     "Seturax": "seturax:SeturaxForCausalLM",
     # attention with a bias by distance and mixed values beside HGRN2, norms around every sublayer, experts on weighted inputs
     "Petipel": "petipel:PetipelForCausalLM",
+    # sigmoid attention beside minGRU, short convolutions of the sublayers' inputs, norms on their outputs, corrected routing
+    "Kefesun": "kefesun:KefesunForCausalLM",
     # asymmetric V / sliding window with sinks
     "MiMoV2FlashForCausalLM": "mimo_v2_flash:MiMoV2FlashForCausalLM",
     # Gemma family

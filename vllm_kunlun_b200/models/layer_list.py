@@ -88,6 +88,8 @@ class LayerListForCausalLM(DenseForCausalLM):
         self.layers = nn.ModuleDict({str(i): self.layer_cls(cfg, i, self.dtype, device) for i in range(cfg.num_layers)})
         self.norm = NormWeight(self.width, device)
         self.lm_head = ParallelLMHead(cfg.vocab_size, self.ld, self.dtype, device)
+        if cfg.tie_word_embeddings:
+            self.lm_head.weight = self.embed_tokens.weight
 
     # ---- caches
     def kv_cache_spec(self, block_size: int):
@@ -111,7 +113,8 @@ class LayerListForCausalLM(DenseForCausalLM):
     def outer_tensor_shapes(self) -> dict:
         """Name -> shape of the tensors outside the layers."""
         W, V = self.width, self.cfg.vocab_size
-        return {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+        out = {"embed": (V, W), "final.norm": (W,)}
+        return out if self.cfg.tie_word_embeddings else {**out, "head": (V, W)}
 
     def load_outer_tensor(self, name: str, w: torch.Tensor):
         if name == "embed":
@@ -146,7 +149,7 @@ class LayerListForCausalLM(DenseForCausalLM):
                     t = t.clamp(-1.0, 1.0)
                 elif leaf == "dt_bias":
                     t = t.clamp(-1.0, 1.0) - 3.0
-                elif leaf == "conv":
+                elif leaf == "conv" or leaf.startswith("canon"):
                     t = t * (10.0 * std)
                 elif leaf in ("shift", "lower", "vmix"):
                     t = torch.sigmoid(t)

@@ -11,6 +11,8 @@ A mixer reads the residual stream's 16-bit (or fp32) copy ``h [T, ld]`` and retu
 * :class:`ChannelDelta`      short convolutions + delta rule with one decay per head and key channel
 * :class:`DistanceBiasAttention` softmax attention with a learned score bias by distance, a query temperature, unit-RMS values
   that layers may share, output gate per head
+* :class:`SigmoidAttention` sigmoid weights without normalisation, rotated and normed q / k, window with kept first tokens
+* :class:`MinGRU`            element-wise recurrence whose gates read only the current token
 * :class:`GatedWriteAttention` linear attention whose forget gate decides what is written (HGRN2)
 * :class:`LatentAttention`   windowed attention over a shared latent row per token, learned sink, output gate per head
 
@@ -57,19 +59,25 @@ def padded(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
 class FusedProjection(ReplicatedLinear):
     """Several projections of the same input in one GEMM; part ``i`` is a column slice starting at a multiple of 8."""
 
-    def __init__(self, in_features: int, sizes: dict, dtype, device):
+    def __init__(self, in_features: int, sizes: dict, dtype, device, bias: bool = False):
         self.parts, off = {}, 0
         for name, n in sizes.items():
             self.parts[name] = (off, n)
             off += align(n)
-        super().__init__(in_features, off, dtype=dtype, device=device)
+        super().__init__(in_features, off, bias, dtype=dtype, device=device)
         self.weight.data.zero_()
+        if bias:
+            self.bias.data.zero_()
 
     def load_part(self, name: str, w: torch.Tensor):
         off, n = self.parts[name]
         if w.shape[0] != n or w.shape[1] > self.in_features:
             raise ValueError(f"projection {name}: checkpoint shape {tuple(w.shape)}, expected [{n}, <= {self.in_features}]")
         self.weight.data[off:off + n, :w.shape[1]].copy_(w)
+
+    def load_bias(self, name: str, b: torch.Tensor):
+        off, n = self.parts[name]
+        self.bias.data[off:off + n].copy_(b)
 
     def slice(self, y: torch.Tensor, name: str) -> torch.Tensor:
         off, n = self.parts[name]
@@ -230,6 +238,78 @@ class DistanceBiasAttention(WindowAttention):
             None, None, md.seq_lens_cpu, md.query_start_loc_cpu, workspace=md.workspace, num_decodes=md.num_decodes,
             decode_query_len=1 + md.num_spec_tokens, num_decode_tokens=md.num_decode_tokens, stable_metadata=True,
             bias=self.bias, gate=p.slice(y, "g"))
+        return [(self.o(o.reshape(T, self.heads * self.cache_dim)), 1.0)]
+
+
+class SigmoidAttention(WindowAttention):
+    """Causal attention without a softmax: a visible key counts with ``sigmoid(score + b)`` (a learned ``b`` per head), not
+    normalised over the keys.  q, k and v have biases; q and k heads are RMS-normed with a weight that the heads share, then
+    rotated on their first columns.  ``mask``: a position sees the last ``size`` ones up to itself and the first ``keep_first``."""
+
+    has_state = False
+    cache_block = 64                        # tokens per cache block that the tensor-core kernels take
+    served_heads = (128,)
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        pass
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        m, mask, rot = sizes, sizes.get("mask") or {}, sizes.get("rot")
+        window = mask.get("size")
+        super().__init__(width, m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"],
+                         None if window is None else int(window), None, eps, dtype, device)
+        self.layer_idx, self.keep_first = layer_idx, int(mask.get("keep_first") or 0)
+        self.in_proj = FusedProjection(width, self.proj_sizes(), dtype, device, bias=True)
+        self.q_norm, self.k_norm = (param(self.dim, dtype=torch.float32, device=device) for _ in range(2))
+        self.bias = param(self.heads, 1, dtype=torch.float32, device=device)
+        self.rotary_key = None
+        if rot is not None:
+            self.rotary_key = (int(rot.get("dims", self.dim)), float(rot["base"]))
+            if self.rotary_key[0] > self.dim or self.rotary_key[0] % 2:
+                raise ValueError(f"{self.rotary_key[0]} rotated columns in heads of {self.dim}")
+            self.register_buffer("turns", ops.position_turns(*self.rotary_key).to(device))
+
+    @staticmethod
+    def tensor_shapes(sizes: dict, width: int) -> dict:
+        H, G, D, V = (sizes[k] for k in ("heads", "kv_heads", "dim", "vdim"))
+        return {"q": (H * D, width), "q.b": (H * D,), "k": (G * D, width), "k.b": (G * D,), "v": (G * V, width), "v.b": (G * V,),
+                "q.norm": (D,), "k.norm": (D,), "pb": (H,), "o": (width, H * V)}
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        if key == "o":
+            self.load_o(w)
+        elif key == "pb":
+            self.bias.data[:, 0].copy_(w)
+        elif key.endswith(".norm"):
+            (self.q_norm if key == "q.norm" else self.k_norm).data.copy_(w)
+        elif key.endswith(".b"):
+            self.in_proj.load_bias(key.removesuffix(".b"), w)
+        else:
+            self.in_proj.load_part(key, w)
+
+    def state_spec(self, dtype):
+        return []
+
+    def workspace_size(self) -> tuple:
+        return self.heads, self.cache_dim
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md, p, T = ctx.attn, self.in_proj, h.shape[0]
+        kv_cache = ctx.kv_caches[self.layer_idx]
+        kv_cache = kv_cache[0] if isinstance(kv_cache, tuple) else kv_cache
+        table = None if self.rotary_key is None else md.extras["rotary"][self.rotary_key]
+        y = p(h)
+        q = ops.attn_prep_cache(p.slice(y, "q"), p.slice(y, "k"), p.slice(y, "v"), kv_cache, md.slot_mapping, md.positions,
+                                self.heads, self.kv_heads, self.eps, v_norm=False, qk_norm=(self.q_norm, self.k_norm),
+                                table=table)
+        span = md.max_seq_len if self.window is None else min(md.max_seq_len, self.window + self.keep_first + 127)
+        o = ops.paged_attention(
+            q, kv_cache, md.block_tables, md.seq_lens, md.query_start_loc, self.scale, md.max_query_len, span, self.window,
+            None, md.seq_lens_cpu, md.query_start_loc_cpu, workspace=md.workspace, num_decodes=md.num_decodes,
+            decode_query_len=1 + md.num_spec_tokens, num_decode_tokens=md.num_decode_tokens, stable_metadata=True,
+            bias=self.bias, keep_first=self.keep_first, sigmoid=True)
         return [(self.o(o.reshape(T, self.heads * self.cache_dim)), 1.0)]
 
 
@@ -504,6 +584,56 @@ class GatedWriteAttention(nn.Module):
         return [(self.o(z), 1.0)]
 
 
+class MinGRU(nn.Module):
+    """``S <- (1 - z) S + z c`` element by element with ``z = sigmoid(W_z h + b_z)`` and, for ``u = W_x h + b_x``, the candidate
+    ``c = u + 1/2`` where ``u >= 0`` and ``sigmoid(u)`` elsewhere; output ``W_o (S * silu(W_g h))``."""
+
+    has_state = True
+    cache_block = None
+
+    @staticmethod
+    def complete_sizes(sizes: dict, shapes: dict) -> None:
+        pass
+
+    def __init__(self, width: int, sizes: dict, layer_idx: int, eps: float, dtype, device):
+        super().__init__()
+        self.layer_idx, self.size = layer_idx, int(sizes["width"])
+        self.in_proj = FusedProjection(width, {"z": self.size, "x": self.size, "g": self.size}, dtype, device)
+        self.z_bias, self.x_bias = (param(self.size, dtype=torch.float32, device=device) for _ in range(2))
+        self.o = output_projection(align(self.size), width, dtype, device)
+
+    @staticmethod
+    def tensor_shapes(sizes: dict, width: int) -> dict:
+        n = int(sizes["width"])
+        return {"z": (n, width), "z.b": (n,), "x": (n, width), "x.b": (n,), "g": (n, width), "o": (width, n)}
+
+    def load_tensor(self, key: str, w: torch.Tensor):
+        if key == "o":
+            self.o.weight.data[:w.shape[0], :w.shape[1]].copy_(w)
+        elif key in ("z.b", "x.b"):
+            (self.z_bias if key == "z.b" else self.x_bias).data.copy_(w)
+        else:
+            self.in_proj.load_part(key, w)
+
+    def kv_cache_spec(self, block_size: int, dtype):
+        return None
+
+    def state_spec(self, dtype):
+        return [((self.size,), torch.float32)]
+
+    def workspace_size(self) -> tuple:
+        return 0, 0
+
+    def forward(self, h):
+        ctx = get_forward_context()
+        md, p = ctx.attn, self.in_proj
+        y = p(h)
+        out = ops.gated_blend(p.slice(y, "z"), p.slice(y, "x"), p.slice(y, "g"), self.z_bias, self.x_bias,
+                              ctx.kv_caches[self.layer_idx][0], md.query_start_loc, md.state_indices, md.has_initial_state,
+                              _rows(h.shape[0], self.size, h.dtype, h.device), md.max_query_len, md.num_decodes)
+        return [(self.o(out), 1.0)]
+
+
 class LatentAttention(nn.Module):
     """Multi-head attention over one latent row per token.  Queries come through their own latent; keys and values are
     per-head products of the cached latent, plus one rotated key part that all heads share.  Optional sliding ``window``,
@@ -659,4 +789,4 @@ def rotary_tables(mixers, md) -> None:
 
 
 MIXERS = {"attention": DistanceBiasAttention, "channel_delta": ChannelDelta, "hgrn2": GatedWriteAttention,
-          "latent_attention": LatentAttention, "parallel": ParallelMixer}
+          "latent_attention": LatentAttention, "mingru": MinGRU, "parallel": ParallelMixer, "sigmoid_attention": SigmoidAttention}

@@ -8,7 +8,7 @@ layers (``vllm_kunlun/ops/_custom_ops.py`` - 54 ``torch.library.custom_op`` shim
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -19,6 +19,7 @@ from .reference import latent as _rt
 from .reference import linear_recurrence as _rl
 from .reference import misc as _rx
 from .reference import moe as _rm
+from .reference import postnorm as _rp
 from .reference import sandwich as _rs
 
 reference_basic = _rb
@@ -196,11 +197,13 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale:
                     max_query_len: int, max_seq_len: int, window: Optional[int] = None, sinks=None,
                     seq_lens_cpu=None, query_start_loc_cpu=None, out=None, workspace=None,
                     num_decodes: int = 0, decode_query_len: int = 1, num_decode_tokens: int = 0,
-                    stable_metadata: bool = False, bias=None, gate=None):
+                    stable_metadata: bool = False, bias=None, gate=None, keep_first: int = 0, sigmoid: bool = False):
     """Unified varlen paged GQA attention (prefill with prefix, decode, spec-verify).
 
     ``bias [Hq, n]`` (fp32): added to the scaled scores by distance (position of the query minus the key's), the last entry
-    for every distance from ``n - 1`` on.  ``gate [T, Hq]``: every head's output is multiplied by its sigmoid.
+    for every distance from ``n - 1`` on.  ``gate [T, Hq]``: every head's output is multiplied by its sigmoid.  ``keep_first``:
+    positions below it stay visible outside the window.  ``sigmoid``: a visible key counts with ``sigmoid(score + bias)``, not
+    normalised over the keys (a ``bias`` is required, one entry per head will do; no sinks).
 
     The batch is decode-first: the first ``num_decodes`` requests have at most ``decode_query_len``
     query tokens each.  On CUDA a mixed batch is served by two launches (decode layout with
@@ -215,17 +218,19 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale:
             paged_attention_cuda(out[:ndt], q[:ndt], kv_cache, block_tables[:num_decodes], seq_lens[:num_decodes],
                                  query_start_loc[:num_decodes + 1], scale, decode_query_len, max_seq_len,
                                  window, sinks, workspace, stable_metadata=stable_metadata, bias=bias,
-                                 gate=None if gate is None else gate[:ndt])
+                                 gate=None if gate is None else gate[:ndt], keep_first=keep_first, sigmoid=sigmoid)
             paged_attention_cuda(out, q, kv_cache, block_tables[num_decodes:], seq_lens[num_decodes:],
                                  query_start_loc[num_decodes:], scale, max_query_len, max_seq_len,
-                                 window, sinks, workspace, bias=bias, gate=gate)
+                                 window, sinks, workspace, bias=bias, gate=gate, keep_first=keep_first, sigmoid=sigmoid)
             return out
         return paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
                                     max_query_len, max_seq_len, window, sinks, workspace,
-                                    stable_metadata=stable_metadata, bias=bias, gate=gate)
+                                    stable_metadata=stable_metadata, bias=bias, gate=gate, keep_first=keep_first,
+                                    sigmoid=sigmoid)
     sl = seq_lens if seq_lens_cpu is None else seq_lens_cpu
     ql = query_start_loc if query_start_loc_cpu is None else query_start_loc_cpu
-    return _ra.paged_attention(q, kv_cache, block_tables, sl, ql, scale, window, sinks, bias=bias, gate=gate)
+    return _ra.paged_attention(q, kv_cache, block_tables, sl, ql, scale, window, sinks, bias=bias, gate=gate, keep_first=keep_first,
+                               sigmoid=sigmoid)
 
 
 def merge_attn_states(o1, lse1, o2, lse2):
@@ -239,20 +244,22 @@ def merge_attn_states(o1, lse1, o2, lse2):
 
 # ----------------------------------------------------------------------------- GEMM
 
-def linear(x, weight, bias=None, out=None):
-    """``y = x @ W.T (+ b)``, ``W [N, K]`` as stored in checkpoints.  CUDA: the tcgen05 GEMM; fp32 models run on the
-    CUDA-core GEMM with true 32-bit products."""
+def linear(x, weight, bias=None, out=None, act: Optional[str] = None):
+    """``y = act(x @ W.T (+ b))``, ``W [N, K]`` as stored in checkpoints, ``act`` None or ``"relu2"`` (square of relu).  CUDA: the
+    tcgen05 GEMM; fp32 models run on the CUDA-core GEMM with true 32-bit products."""
+    assert act in (None, "relu2")
     if x.is_cuda:
         if x.dtype == torch.float32:
             x2 = x.reshape(-1, x.shape[-1])
             if x2.stride(-1) != 1:
                 x2 = x2.contiguous()
             y = torch.empty(x2.shape[0], weight.shape[0], dtype=x.dtype, device=x.device) if out is None else out
-            _c().gemm_f32(y, x2, weight, bias)
+            _c().gemm_f32(y, x2, weight, bias, act is not None)
             return y.reshape(*x.shape[:-1], weight.shape[0])
         from .gemm_cuda import gemm_bf16
-        return gemm_bf16(x, weight, bias, out)
-    return _rb.linear(x, weight, bias)
+        return gemm_bf16(x, weight, bias, out, act=act)
+    y = _rb.linear(x, weight, bias)
+    return y if act is None else _rb.relu2(y)
 
 
 def linear_gated_act(x, weight_interleaved, bias_interleaved=None, act: str = "silu"):
@@ -375,7 +382,8 @@ def router_gemm(x, weight, bias=None, fp32: bool = False):
 
 
 def router_and_route(x, weight, wbias, k: int, scoring: str = "softmax", renormalize: bool = True, bias=None,
-                     n_group: int = 1, topk_group: int = 1, scale: float = 1.0, fp32: bool = False):
+                     n_group: int = 1, topk_group: int = 1, scale: float = 1.0, fp32: bool = False,
+                     group_top: Optional[int] = None):
     """Router logits (``fp32``: as in :func:`router_gemm`) and top-k routing from the hidden states.  CUDA, decode-sized batches with a SMALL router
     (at most 64 K weights): one launch, logits stay in shared memory.  Larger routers keep two kernels: one CTA per
     token cannot pull a 128 x 2048 router through a single SM fast enough (measured: Qwen3-30B-A3B decode step
@@ -385,27 +393,36 @@ def router_and_route(x, weight, wbias, k: int, scoring: str = "softmax", renorma
         from .moe_cuda import _MODES
         w, ids = _c().router_route_small(x if x.stride(-1) == 1 else x.contiguous(), weight, wbias,
                                          None if bias is None else bias.float(), k, _MODES[scoring], renormalize,
-                                         n_group, topk_group, scale)
+                                         n_group, topk_group, scale, _group_top(scoring, group_top))
         return w, ids
-    return moe_route(router_gemm(x, weight, wbias, fp32), k, scoring, renormalize, bias, n_group, topk_group, scale)
+    return moe_route(router_gemm(x, weight, wbias, fp32), k, scoring, renormalize, bias, n_group, topk_group, scale,
+                     group_top)
+
+
+def _group_top(scoring: str, group_top: Optional[int]) -> int:
+    """Members that make up a group's score: given, or two for sigmoid scores and no groups for softmax scores."""
+    return group_top if group_top is not None else 2 if scoring == "sigmoid" else 0
 
 
 def moe_route(logits, k: int, scoring: str = "softmax", renormalize: bool = True, bias=None, n_group: int = 1,
-              topk_group: int = 1, scale: float = 1.0):
+              topk_group: int = 1, scale: float = 1.0, group_top: Optional[int] = None):
     """Router: ``(weights [T, k] fp32, ids [T, k] int32)``.
 
     ``softmax`` = softmax -> top-k (-> renormalise) (``_C::moe_softmax_topk(_norm)``);
     ``sigmoid`` = DeepSeek-V3 group-limited routing with a selection bias
-    (``_C::moe_sigmoid_group_topk_norm``); ``softmax_after_topk`` = GPT-OSS."""
+    (``_C::moe_sigmoid_group_topk_norm``); ``softmax_after_topk`` = GPT-OSS.  ``bias``: added to the scores for the choice only.
+    ``group_top``: a group's score is the sum of that many of its best choice scores (1 or 2; 0: no groups); by default 2 for
+    ``sigmoid`` and 0 for ``softmax``."""
     if logits.is_cuda:
         from .moe_cuda import moe_route_cuda
-        return moe_route_cuda(logits, k, scoring, renormalize, bias, n_group, topk_group, scale)
-    if scoring == "softmax":
+        return moe_route_cuda(logits, k, scoring, renormalize, bias, n_group, topk_group, scale, _group_top(scoring, group_top))
+    if scoring == "softmax" and bias is None and not group_top:
         w, ids = _rm.route_softmax_topk(logits, k, renormalize)
         return w * scale, ids
     if scoring == "softmax_after_topk":
         return _rm.route_topk_then_softmax(logits, k)
-    return _rm.route_sigmoid_group_topk(logits, bias, k, n_group, topk_group, renormalize, scale)
+    scores = (torch.sigmoid if scoring == "sigmoid" else lambda z: torch.softmax(z, -1))(logits.float())
+    return _rm.route_group_topk(scores, bias, k, n_group, topk_group, renormalize, scale, _group_top(scoring, group_top))
 
 
 def fused_moe(x, w13, w2, topk_weights, topk_ids, act: str = "silu", b13=None, b2=None, w13_scale=None,
@@ -419,14 +436,23 @@ def fused_moe(x, w13, w2, topk_weights, topk_ids, act: str = "silu", b13=None, b
     return _rm.fused_moe(x, w13, w2, topk_weights, topk_ids, act, b13, b2, w13_scale, w2_scale, block, expert_map)
 
 
-def experts_on_weighted_input(x, w13, w2, topk_weights, topk_ids, act: str, limit: float = 0.0):
-    """Routed experts whose weight multiplies their input: rows of ``expert(w * x)`` in expert order and, per (token, choice),
-    the row's place ``[T * k]`` (int32); a token's result is the sum of its rows.  16-bit weights run on the tensor-core
-    grouped GEMM, fp32 ones on the CUDA-core one."""
+def expert_rows(x, w_in, w_out, topk_ids, act: str, limit: float = 0.0, factors=None, choices: Optional[int] = None):
+    """Routed experts without the sum: rows of ``W_out act(W_in x)`` in expert order and, per (token, choice), the row's place
+    ``[T * k]`` (int32).  ``factors [T, k]`` (fp32) multiply the experts' inputs.  ``act``: ``"relu2"`` (square of relu, no gate) or a
+    gated activation of :func:`act_and_mul`.  The router may have more outputs (``choices``) than there are experts: a choice
+    without an expert has place -1.  16-bit weights run on the tensor-core grouped GEMM, fp32 ones on the CUDA-core one."""
+    choices = choices or w_in.shape[0]
     if x.is_cuda:
-        from .moe_cuda import experts_on_weighted_input_cuda
-        return experts_on_weighted_input_cuda(x, w13, w2, topk_weights, topk_ids, act, limit)
-    return _rs.experts_on_weighted_input(x, w13, w2, topk_weights, topk_ids, lambda h: act_and_mul(h, act, limit))
+        from .moe_cuda import expert_rows_cuda
+        return expert_rows_cuda(x, w_in, w_out, topk_ids, act, limit, factors, choices)
+    fn = _rb.relu2 if act == "relu2" else lambda h: act_and_mul(h, act, limit)
+    return _rs.expert_rows(x, w_in, w_out, topk_ids, fn, factors, choices)
+
+
+def experts_on_weighted_input(x, w13, w2, topk_weights, topk_ids, act: str, limit: float = 0.0):
+    """Routed experts whose weight multiplies their input: rows of ``expert(w * x)`` and their places; a token's result is the
+    sum of its rows."""
+    return expert_rows(x, w13, w2, topk_ids, act, limit, topk_weights)
 
 
 # ----------------------------------------------------------------------------- MLA / sparse MLA / indexer
@@ -840,15 +866,98 @@ def poly_norm(z, coeff, width: int, eps: float):
 
 
 def attn_prep_cache(q, k, v, kv_cache, slot_mapping, positions, num_heads: int, num_kv_heads: int, eps: float,
-                    temperature=None, v_out=None, v_in=None, share: float = 0.0):
-    """Split of an attention projection: K as it is and V divided by its root mean square per head go into the paged cache;
+                    temperature=None, v_out=None, v_in=None, share: float = 0.0, v_norm: bool = True, qk_norm=None, table=None):
+    """Split of an attention projection: K and V (``v_norm``: divided by its root mean square per head) go into the paged cache;
     returns ``q [T, Hq, Dc]`` times ``1 + coef ln(floor((position + 1) / every) + 1)`` for ``temperature = (coef, every)``.
-    Heads are zero-padded to the cache's head size.  ``v_out [T, Hkv * Dv]`` receives the normed values; ``v_in`` (such values
-    of another layer) is mixed in before caching: ``(1 - share) v + share v_in``."""
+    Heads are zero-padded to the cache's head size.  ``qk_norm = (q weight, k weight)`` (fp32 ``[D]``): RMS norm of every q / k
+    head; ``table`` (:func:`rotary_table`) then rotates their first ``2 * pairs`` columns, column i with i + pairs.
+    ``v_out [T, Hkv * Dv]`` receives the normed values; ``v_in`` (such values of another layer) is mixed in before caching:
+    ``(1 - share) v + share v_in``."""
     coef, every = (0.0, 0) if temperature is None else temperature
     out = torch.empty(q.shape[0], num_heads, kv_cache.shape[-1], dtype=q.dtype, device=q.device)
     (_c() if q.is_cuda else _rs).attn_prep_cache(out, q, k, v, kv_cache, slot_mapping, positions, num_heads, num_kv_heads,
-                                                 coef, every, v_out, v_in, share, eps)
+                                                 coef, every, v_out, v_in, share, eps, v_norm, *(qk_norm or (None, None)),
+                                                 table)
+    return out
+
+
+# ----------------------------------------------------------------- norms on outputs, short convolutions of the sublayers' inputs
+
+class ChoicesSum(NamedTuple):
+    """A sublayer's result that is still apart: ``y`` (or None) plus, per token, ``weights [T, k]`` times the ``rows`` at
+    ``places [T * k]``, or times ``through`` where a place is below zero."""
+    y: Optional[torch.Tensor]
+    rows: torch.Tensor
+    places: torch.Tensor
+    weights: torch.Tensor
+    through: torch.Tensor
+
+
+FUSED_CONV_ROWS = 4        # up to this many tokens per request the convolution runs inside the norm's kernel
+
+
+def _conv_args(conv, md) -> tuple:
+    """``conv = (taps [n, ld], state [slots, n - 1, ld] or None)`` and the step's metadata for the kernels."""
+    if conv is None:
+        return (None,) * 5
+    return (*conv, md.query_start_loc, md.state_indices, md.has_initial_state)
+
+
+def input_conv(x, dtype, conv, md):
+    """What a sublayer reads: ``x + conv(x)`` in ``dtype``, conv being causal over time and separate per channel."""
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    taps, state, *meta = _conv_args(conv, md)
+    if x.is_cuda:
+        _c().input_conv(x, h, taps, state, *meta, md.max_query_len)
+    else:
+        _rp.input_conv(x, h, taps, state, *meta)
+    return h
+
+
+def embed_input_conv(ids, table, scale: float, conv, md):
+    """Start of a stream: ``(x = table[id] * scale in fp32, x + conv(x) in table.dtype)``."""
+    T, ld = ids.shape[0], table.shape[1]
+    x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
+    if not table.is_cuda:
+        x.copy_(table[ids.long()].float() * scale)
+        return x, input_conv(x, table.dtype, conv, md)
+    fused = md.max_query_len <= FUSED_CONV_ROWS
+    h = torch.empty(T, ld, dtype=table.dtype, device=table.device) if fused else None
+    _c().embed_postnorm(x, h, ids, table, scale, *_conv_args(conv if fused else None, md))
+    return x, h if fused else input_conv(x, table.dtype, conv, md)
+
+
+def postnorm_input_conv(x, y, weight, eps: float, dtype, conv=None, md=None, final_weight=None):
+    """End of a sublayer and start of the next one: ``x += LayerNorm(y) * weight`` in place on the fp32 stream (``y [T, ld]`` or a
+    :class:`ChoicesSum`), then ``x + conv(x)``, or ``LayerNorm(x) * final_weight`` behind the last sublayer, in ``dtype``."""
+    parts = y if isinstance(y, ChoicesSum) else ChoicesSum(y, None, None, None, None)
+    if not x.is_cuda:
+        s = parts.y.float() if parts.rows is None else _rp.choices_sum(*parts)
+        x += _rp.layer_norm(s, weight, eps)
+        return _rp.layer_norm(x, final_weight, eps).to(dtype) if conv is None else input_conv(x, dtype, conv, md)
+    fused = conv is None or md.max_query_len <= FUSED_CONV_ROWS
+    h = torch.empty(x.shape, dtype=dtype, device=x.device) if fused else None
+    _c().postnorm(x, h, *parts, weight, eps, final_weight, *_conv_args(conv if fused else None, md))
+    return h if fused else input_conv(x, dtype, conv, md)
+
+
+BLEND_SCAN_MIN = 16        # longest portion of a step from which its prompt portions take the scan over token blocks
+
+
+def gated_blend(z, x, g, z_bias, x_bias, state, cu_seqlens, state_indices, has_initial_state, out, max_query_len: int = 0,
+                num_decodes: int = 0):
+    """Element-wise recurrence ``S <- (1 - s) S + s c`` with ``s = sigmoid(z + z_bias)`` and, for ``u = x + x_bias``, ``c = u + 1/2``
+    where ``u >= 0`` and ``sigmoid(u)`` elsewhere (minGRU); ``out [T, >= width] = S * silu(g)``.  ``z, x, g [T, width]``: column
+    slices of one raw projection; ``state [slots, width]`` fp32, in place."""
+    if not z.is_cuda:
+        _rp.gated_blend(out, z, x, g, z_bias, x_bias, state, cu_seqlens, state_indices, has_initial_state)
+        return out
+    R = state_indices.shape[0]
+    nd = R if max_query_len < BLEND_SCAN_MIN else num_decodes
+    for lo, hi, steps in ((0, nd, True), (nd, R, False)):
+        if lo < hi:
+            _c().gated_blend(out, z, x, g, z_bias, x_bias, state, cu_seqlens[lo:hi + 1], state_indices[lo:hi],
+                             has_initial_state[lo:hi], steps)
     return out
 
 

@@ -70,9 +70,9 @@ def plan_splits_umma(num_reqs: int, num_kv_heads: int, max_seq_len: int, device,
 def paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_loc, scale: float,
                          max_query_len: int, max_seq_len: int, window: Optional[int] = None, sinks=None,
                          workspace: Optional[AttnWorkspace] = None, num_splits: Optional[int] = None,
-                         stable_metadata: bool = False, bias=None, gate=None):
-    """``bias`` / ``gate`` (score bias by distance, output gates: see :func:`ops.paged_attention`) are served by the tcgen05
-    kernels and the generic one.  ``stable_metadata``: the caller promises that ``block_tables`` / ``seq_lens`` / ``query_start_loc`` were
+                         stable_metadata: bool = False, bias=None, gate=None, keep_first: int = 0, sigmoid: bool = False):
+    """``bias``, ``gate``, ``keep_first`` and ``sigmoid`` (see :func:`ops.paged_attention`) are served by the tcgen05 kernels and the
+    generic one.  ``stable_metadata``: the caller promises that ``block_tables`` / ``seq_lens`` / ``query_start_loc`` were
     filled by host copies before the step's first kernel (as the engine's runner does) and that the cache rows of
     the old context come from earlier steps; the decode kernel then starts fetching KV tiles while the kernel in
     front of it is still running."""
@@ -81,12 +81,14 @@ def paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_l
     g = Hq // Hkv
     B = seq_lens.shape[0]
     decode_layout = max_query_len * g <= 16
-    extras = bias is not None or gate is not None
+    extras = bias is not None or gate is not None or keep_first > 0 or sigmoid
+    if sigmoid and (bias is None or sinks is not None):
+        raise ValueError("sigmoid weights need a bias and take no sinks")
     if (q.dtype == torch.float32 or D not in (64, 128, 256) or (decode_layout and kv_cache.shape[3] % 16)
             or (extras and (D != 128 or kv_cache.shape[3] % 64))):
         # fp32 models, and head sizes (or cache blocks) that the tensor-core kernels do not take
         _ext.C().paged_attention_generic(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, 0,
-                                         window or 0, scale, bias, gate)
+                                         window or 0, scale, bias, gate, keep_first, sigmoid)
         return out
     if (decode_layout and (UMMA_DECODE[0] or extras) and D == 128 and kv_cache.shape[3] % 64 == 0
             and q.dtype in (torch.bfloat16, torch.float16)):
@@ -101,17 +103,18 @@ def paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_l
                 workspace = AttnWorkspace(T, Hq, D, num_splits, q.device)
             ws_o, ws_lse = workspace.o, workspace.lse
         _ext.C().decode_attention_umma(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, ws_o, ws_lse,
-                                       max_query_len, num_splits, window or 0, scale, bool(stable_metadata), bias, gate)
+                                       max_query_len, num_splits, window or 0, scale, bool(stable_metadata), bias, gate,
+                                       keep_first, sigmoid)
         return out
     if (not decode_layout and (UMMA_PREFILL[0] or extras) and D == 128 and kv_cache.shape[3] % 64 == 0 and kv_cache.dim() == 5
             and q.dtype in (torch.bfloat16, torch.float16) and q.is_contiguous() and out.is_contiguous()
             and kv_cache.is_contiguous()):
         # prefill / chunked prefill on tcgen05: 128 query rows of one head per CTA, S and O in TMEM
         _ext.C().prefill_attention_umma(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, None,
-                                        max_query_len, window or 0, scale, bias, gate)
+                                        max_query_len, window or 0, scale, bias, gate, keep_first, sigmoid)
         return out
     if extras:
-        raise ValueError("a score bias or an output gate needs contiguous q, out and cache")
+        raise ValueError("a score bias, an output gate, kept keys or sigmoid weights need contiguous q, out and cache")
     if num_splits is None:
         if decode_layout:
             num_splits = plan_splits(B, Hkv, 1, max_seq_len, q.device,

@@ -18,7 +18,8 @@ DECODE_GEMM = [os.environ.get("B200_DECODE_GEMM", "1") != "0"]
 PEER = None  # PeerBuffers of the tensor-parallel group once its sequence-parallel buffers exist
 
 
-ACT_CODES = {None: 0, "silu": 1, "gelu_tanh": 2, "swigluoai": 3}
+ACT_CODES = {None: 0, "silu": 1, "gelu_tanh": 2, "swigluoai": 3, "relu2": 4}
+UNGATED = (None, "relu2")
 
 
 def interleave_gate_up(w: torch.Tensor, inverse: bool = False) -> torch.Tensor:
@@ -37,13 +38,14 @@ def interleave_gate_up(w: torch.Tensor, inverse: bool = False) -> torch.Tensor:
 def gemm_bf16(x: torch.Tensor, weight: torch.Tensor, bias=None, out=None, splits: int = 0, bn: int = 0,
               stages: int = 0, ctas_per_sm: int = 0, act=None):
     """``act``: gated activation fused into the epilogue; ``weight`` (and ``bias``) rows are then interleaved per
-    tile (:func:`interleave_gate_up`) and the output has ``N / 2`` features."""
+    tile (:func:`interleave_gate_up`) and the output has ``N / 2`` features.  ``"relu2"`` is no gate: it applies to every output
+    of a plain projection."""
     global LAUNCHES
     lead = x.shape[:-1]
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(-1) != 1 or (x2.stride(0) % 8) or (x2.data_ptr() % 16):
         x2 = x2.contiguous()
-    N = weight.shape[0] // 2 if act else weight.shape[0]
+    N = weight.shape[0] if act in UNGATED else weight.shape[0] // 2
     if out is None:
         out = torch.empty(x2.shape[0], N, dtype=x.dtype, device=x.device)
     out2 = out.reshape(-1, N)

@@ -14,8 +14,8 @@ _MODES = {"softmax": 0, "sigmoid": 1, "softmax_after_topk": 2}
 _STATE: dict = {}
 
 
-def moe_route_cuda(logits, k, scoring, renormalize, bias, n_group, topk_group, scale):
-    w, ids = _ext.C().moe_route(logits, bias, k, _MODES[scoring], renormalize, n_group, topk_group, scale)
+def moe_route_cuda(logits, k, scoring, renormalize, bias, n_group, topk_group, scale, group_top):
+    w, ids = _ext.C().moe_route(logits, bias, k, _MODES[scoring], renormalize, n_group, topk_group, scale, group_top)
     return w, ids
 
 
@@ -74,24 +74,25 @@ def fused_moe_cuda(x, w13, w2, topk_weights, topk_ids, act="silu", b13=None, b2=
     return out
 
 
-def experts_on_weighted_input_cuda(x, w13, w2, topk_weights, topk_ids, act, limit):
-    """Rows of ``expert(weight * x)`` in expert order and the row of every (token, choice) pair."""
+def expert_rows_cuda(x, w_in, w_out, topk_ids, act, limit, factors, choices):
+    """Rows of ``expert(factor * x)`` in expert order and the row of every (token, choice) pair."""
     from . import act_and_mul
     C = _ext.C()
     T, k = topk_ids.shape
-    E = w13.shape[0]
-    ids, w = topk_ids.contiguous(), topk_weights.contiguous()
+    E = w_in.shape[0]
+    ids, f = topk_ids.contiguous(), None if factors is None else factors.contiguous()
     if 0 < T * k <= _small_pairs() and SMALL_BATCH_FUSION[0]:
-        xs, pos, lod, _ = C.moe_prepare_small(x, ids, None, E, E, False, w)
+        xs, pos, lod, _ = C.moe_prepare_small(x, ids, None, E, choices, False, f)
     else:
-        xs, pos, lod = C.moe_permute(x, ids, None, E, E, _state(x.device, E), 0, w)
+        xs, pos, lod = C.moe_permute(x, ids, None, E, choices, _state(x.device, E), 0, f)
 
-    def gemm(a, weight):
+    def gemm(a, weight, relu2=False):
         out = torch.empty(a.shape[0], weight.shape[1], dtype=a.dtype, device=a.device)
         if a.dtype == torch.float32:
-            C.gemm_f32_grouped(out, a, weight, lod)
+            C.gemm_f32_grouped(out, a, weight, lod, relu2)
         else:
-            C.grouped_gemm(out, a, weight, lod, None, None, None, 0)
+            C.grouped_gemm(out, a, weight, lod, None, None, None, 0, 4 if relu2 else 0)
         return out
 
-    return gemm(act_and_mul(gemm(xs, w13), act, limit), w2), pos
+    h = gemm(xs, w_in, True) if act == "relu2" else act_and_mul(gemm(xs, w_in), act, limit)
+    return gemm(h, w_out), pos

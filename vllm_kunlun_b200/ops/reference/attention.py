@@ -160,10 +160,11 @@ def copy_blocks(caches, mapping):
 # ----------------------------------------------------------------------------- GQA attention
 
 def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int], sinks, return_lse=False,
-            softcap: float = 0.0, bias=None):
+            softcap: float = 0.0, bias=None, keep_first: int = 0, sigmoid: bool = False):
     """q [Lq, Hq, D], k/v [Lk, Hkv, D(v)].  Query row i sits at absolute position
     ``causal_offset + i`` and sees keys ``<=`` that position (None = no mask).  ``bias [Hq, n]``: added to the scores by
-    distance, the last entry for every distance from ``n - 1`` on."""
+    distance, the last entry for every distance from ``n - 1`` on.  ``keep_first``: positions that a window never hides;
+    ``sigmoid``: weights are sigmoids of the scores, not normalised."""
     Lq, Hq, D = q.shape
     Lk, Hkv = k.shape[0], k.shape[1]
     g = Hq // Hkv
@@ -180,8 +181,10 @@ def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int],
         if bias is not None:
             s = s + bias.float()[:, (qpos - kpos).clamp(0, bias.shape[1] - 1)].reshape(Hkv, g, Lq, Lk)
         if window is not None:
-            mask &= kpos > qpos - window
+            mask &= (kpos > qpos - window) | (kpos < keep_first)
         s = s.masked_fill(~mask, float("-inf"))
+    if sigmoid:
+        return torch.matmul(torch.sigmoid(s), vf).permute(2, 0, 1, 3).reshape(Lq, Hq, -1)
     m = s.amax(-1, keepdim=True)
     if sinks is not None:
         sk = sinks.float().reshape(Hkv, g, 1, 1)
@@ -209,7 +212,8 @@ def gather_paged_kv(kv_cache, block_table_row, seq_len: int):
 
 
 def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
-                    window: Optional[int] = None, sinks=None, softcap: float = 0.0, bias=None, gate=None):
+                    window: Optional[int] = None, sinks=None, softcap: float = 0.0, bias=None, gate=None,
+                    keep_first: int = 0, sigmoid: bool = False):
     """Unified varlen paged attention: covers ``kunlun_ops.prefill_attention`` (with prefix cache,
     ``kunlun_attn.py:849-891``) and ``kunlun_ops.speculative_attention`` (decode with
     ``q_len >= 1``, ``kunlun_attn.py:926-947``).  K/V for all ``seq_lens[r]`` positions are read
@@ -221,7 +225,8 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
             continue
         L = int(seq_lens[r])
         k, v = gather_paged_kv(kv_cache, block_tables[r], L)
-        o = _attend(q[qs:qe], k, v, scale, L - (qe - qs), window, sinks, softcap=softcap, bias=bias)
+        o = _attend(q[qs:qe], k, v, scale, L - (qe - qs), window, sinks, softcap=softcap, bias=bias,
+                    keep_first=keep_first, sigmoid=sigmoid)
         if gate is not None:
             o = o * torch.sigmoid(gate[qs:qe].float()).unsqueeze(-1)
         out[qs:qe] = o.to(q.dtype)

@@ -351,6 +351,10 @@ def gptq_dequantize(qweight, scales, qzeros, g_idx, bits: int = 4):
     return ((w - z[g_idx.long()]).float() * scales.float()[g_idx.long()]).to(scales.dtype)
 
 
+def relu2(x):
+    return torch.relu(x.float()).square().to(x.dtype)
+
+
 def linear(x, weight, bias=None):
     out = x.float() @ weight.float().T
     if bias is not None:

@@ -31,14 +31,20 @@ def route_sigmoid_group_topk(logits, bias, k: int, n_group: int, topk_group: int
     Scores = sigmoid(logits); selection uses ``scores + bias``; each group is ranked by the sum of
     its top-2 biased scores, the best ``topk_group`` groups stay; final weights are the *unbiased*
     scores of the chosen experts, normalised and multiplied by ``scale``."""
-    T, E = logits.shape
-    s = torch.sigmoid(logits.float())
-    sel = s + bias.float() if bias is not None else s
-    g = sel.reshape(T, n_group, E // n_group)
-    gscore = g.topk(min(2, E // n_group), -1).values.sum(-1)
-    gidx = gscore.topk(topk_group, -1).indices
-    gmask = torch.zeros(T, n_group, dtype=torch.bool).scatter_(1, gidx, True)
-    masked = g.masked_fill(~gmask.unsqueeze(-1), float("-inf")).reshape(T, E)
+    return route_group_topk(torch.sigmoid(logits.float()), bias, k, n_group, topk_group, renormalize, scale, 2)
+
+
+def route_group_topk(s, bias, k: int, n_group: int, topk_group: int, renormalize: bool, scale: float, group_top: int):
+    """Choice by ``s + bias`` inside the ``topk_group`` groups whose ``group_top`` best members add up to most (0: no groups);
+    weights are the scores ``s [T, E]`` of the chosen ones."""
+    T, E = s.shape
+    masked = s + bias.float() if bias is not None else s
+    if group_top and n_group > 1:
+        g = masked.reshape(T, n_group, E // n_group)
+        gscore = g.topk(min(group_top, E // n_group), -1).values.sum(-1)
+        gidx = gscore.topk(topk_group, -1).indices
+        gmask = torch.zeros(T, n_group, dtype=torch.bool).scatter_(1, gidx, True)
+        masked = g.masked_fill(~gmask.unsqueeze(-1), float("-inf")).reshape(T, E)
     ids = masked.topk(k, -1).indices
     w = s.gather(1, ids)
     if renormalize:
