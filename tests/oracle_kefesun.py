@@ -148,3 +148,60 @@ def forward(tokens, w, cfg, layers_out=None):
         if layers_out is not None:
             layers_out.append(x)
     return layer_norm(x, w["final.norm"], eps) @ w["embed"].T
+
+
+def tensor_shapes(cfg):
+    W, V, n = cfg["width"], cfg["vocab"], cfg["canon"]["taps"]
+    out = {"embed": (V, W), "final.norm": (W,)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer.get("mlp")
+        out.update({p + "norm1": (W,), p + "canon1": (W, n)})
+        if layer["type"] == "attention":
+            H, G, D, Dv = (m[k] for k in ("heads", "kv_heads", "dim", "vdim"))
+            mix = {"q": (H * D, W), "q.b": (H * D,), "k": (G * D, W), "k.b": (G * D,), "v": (G * Dv, W), "v.b": (G * Dv,),
+                   "q.norm": (D,), "k.norm": (D,), "pb": (H,), "o": (W, H * Dv)}
+        else:
+            d = m["width"]
+            mix = {"z": (d, W), "z.b": (d,), "x": (d, W), "x.b": (d,), "g": (d, W), "o": (W, d)}
+        out.update({p + "mix." + k: s for k, s in mix.items()})
+        if f is None:
+            continue
+        rt, ff = f["router"], f["expert"]["ff"]
+        outputs = rt["experts"] + rt["identity"]
+        out.update({p + "norm2": (W,), p + "canon2": (W, n), p + "mlp.router": (outputs, W), p + "mlp.correction": (outputs,),
+                    p + "mlp.shared.up": (f["shared"]["ff"], W), p + "mlp.shared.down": (W, f["shared"]["ff"])})
+        for e in range(rt["experts"]):
+            out.update({f"{p}mlp.e{e}.up": (ff, W), f"{p}mlp.e{e}.down": (W, ff)})
+    return out
+
+
+def random_weights(cfg, seed=0, dtype=torch.float64):
+    """Seeded weights, already rounded to bfloat16 (what a checkpoint stores).  Scores spread widely around a low bias, so that few
+    keys count; half of the blend gates hardly move, so that early tokens still show late; corrections of both signs."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in sorted(tensor_shapes(cfg).items()):
+        z = torch.randn(shape, generator=g)
+        leaf = name.rsplit(".", 1)[-1]
+        if name.endswith((".q.norm", ".k.norm")):
+            t = 1.5 + 0.3 * z
+        elif leaf.startswith("norm"):
+            t = 1.0 + 0.15 * z
+        elif leaf.startswith("canon"):
+            t = 0.4 * z
+        elif leaf == "pb":
+            t = z - 2.5
+        elif name.endswith(".z.b"):
+            t = torch.where(torch.arange(shape[0]) % 2 == 0, z - 5.0, z)
+        elif leaf == "b":
+            t = 0.5 * z
+        elif leaf == "correction":
+            t = 0.3 * z - 0.2
+        elif leaf == "embed":
+            t = z / math.sqrt(shape[-1])
+        elif leaf == "router":
+            t = z * 2.0 / math.sqrt(shape[-1])
+        else:
+            t = z * 1.3 / math.sqrt(shape[-1])
+        out[name] = t.to(torch.bfloat16).to(dtype)
+    return out

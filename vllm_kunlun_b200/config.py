@@ -189,7 +189,7 @@ class ModelConfig:
         """Some layer keeps a per-request state besides (or instead of) the paged cache."""
         if self.linear_attn_pattern > 0:
             return True
-        if self.token_shift or self.bigram or self.input_conv_taps > 1:
+        if self.token_shift or self.bigram or self.input_conv_taps:
             return True
         if not self.layer_specs:
             return False
