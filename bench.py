@@ -78,11 +78,12 @@ def parse():
     ap.add_argument("--layers", type=int, default=0,
                     help="debugging only: run with this many layers (the JSON line then says so and is not a result)")
     ap.add_argument("--layer-bench", nargs="?", const="all", default=None, metavar="SIZE",
-                    help="instead of the headline run: prefill and decode throughput of Bolopel, Seturax and Petipel layers, "
-                         "each beside the closest other model (Qwen3-Next and DeepSeek with dense feed-forwards, Qwen3-Next "
-                         "with experts in every other layer) at equal sizes; one JSON line per size and model (SIZE: small | large | all)")
+                    help="instead of the headline run: prefill and decode throughput of Bolopel, Seturax, Petipel and "
+                         "Kefesun layers, each beside the closest other model (Qwen3-Next and DeepSeek with dense feed-forwards, "
+                         "Qwen3-Next with experts in every other layer, Petipel with experts in every layer) at equal sizes; one JSON line per size and model (SIZE: small | large | all)")
     ap.add_argument("--layer-bench-model", default="all",
-                    choices=["all", "bolopel", "qwen3-next", "seturax", "deepseek", "petipel", "qwen3-next-moe"])
+                    choices=["all", "bolopel", "qwen3-next", "seturax", "deepseek", "petipel", "qwen3-next-moe", "kefesun",
+                             "petipel-moe"])
     a = ap.parse_args()
     c = CONFIGS[a.config]
     a.model = a.model or c["model"]
@@ -166,8 +167,8 @@ def reference_arm(args):
 
 # Sizes of the layer benchmark: width, feed-forward, query / key-value heads of the softmax attention, heads of the
 # recurrent layers (head size 128 throughout), layers (every 4th one of the hybrids differs in kind), window, query latent
-# of the latent-attention models (their key / value latent is 512, their rotated part 64), experts of every other layer of
-# Petipel and its neighbour, experts per token and their width.
+# of the latent-attention models (their key / value latent is 512, their rotated part 64), experts of a routed layer, experts per
+# token and their width.
 LAYER_SIZES = {
     "small": dict(width=2048, ff=6144, heads=16, kv_heads=4, lin_heads=16, layers=8, window=1024, q_rank=768,
                   experts=32, top=4, expert_ff=768),
@@ -181,7 +182,8 @@ def layer_models(size):
     """The models of one size, all with dense feed-forwards of the same width: Bolopel (3 of 4 layers 'parallel', 1
     'channel_delta') and Qwen3-Next (3 of 4 layers gated delta net, 1 gated full attention); Seturax (windowed latent
     attention) and DeepSeek (latent attention over all positions).  Petipel (HGRN2 with experts and attention with a dense
-    feed-forward in turn) and Qwen3-Next with the same order of layers (gated delta net with experts, gated full attention)."""
+    feed-forward in turn) and Qwen3-Next with the same order of layers (gated delta net with experts, gated full attention).
+    Kefesun (minGRU and windowed sigmoid attention in turn, experts everywhere) and Petipel with experts everywhere."""
     import dataclasses
 
     from vllm_kunlun_b200.config import LayerSpec, ModelConfig
@@ -224,8 +226,20 @@ def layer_models(size):
                           LayerSpec("hgrn2", dict(heads=H, dim=128, vdim=128), dict(routed)) for i in range(z["layers"])))
     qwen_moe = dataclasses.replace(like, name=f"qwen3-next-moe-{size}", linear_attn_pattern=2, moe_layer_freq=2,
                                    num_experts=z["experts"], num_experts_per_tok=z["top"], moe_intermediate_size=z["expert_ff"])
+    sigmoid = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5,
+                   mask=dict(size=z["window"], keep_first=4), rot=dict(base=10000.0, dims=64))
+    corrected = dict(kind="moe", expert=dict(ff=z["expert_ff"]), shared=dict(ff=z["expert_ff"]),
+                     router=dict(experts=z["experts"] - 4, identity=4, top=z["top"], scale=2.5, groups=dict(count=4, keep=2)))
+    kefesun = dataclasses.replace(
+        own, architecture="Kefesun", name=f"kefesun-{size}", hidden_act="relu2", tie_word_embeddings=True, input_conv_taps=3,
+        embedding_scale=z["width"] ** 0.5,
+        layer_specs=tuple(LayerSpec("sigmoid_attention", dict(sigmoid), dict(corrected)) if i % 2 else
+                          LayerSpec("mingru", dict(width=128 * H), dict(corrected)) for i in range(z["layers"])))
+    petipel_moe = dataclasses.replace(
+        petipel, name=f"petipel-moe-{size}",
+        layer_specs=tuple(LayerSpec(s.type, dict(s.mixer), dict(routed)) for s in petipel.layer_specs))
     return {"bolopel": own, "qwen3-next": like, "seturax": seturax, "deepseek": deepseek, "petipel": petipel,
-            "qwen3-next-moe": qwen_moe}
+            "qwen3-next-moe": qwen_moe, "kefesun": kefesun, "petipel-moe": petipel_moe}
 
 
 def layer_bench(args):

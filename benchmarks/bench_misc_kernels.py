@@ -1,7 +1,7 @@
 """Device timings of the sampling, gated-delta-net, conv, LoRA and MTP-glue kernels (CUDA events, L2 flushed
 between iterations, 3 warm-ups), reported against the algorithmic bytes and the measured copy bandwidth.
 
-    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|sandwich|latent|conv|lora|all] [--small]
+    python benchmarks/bench_misc_kernels.py [--case sample|gdn|recurrence|stream|sandwich|postnorm|latent|conv|lora|all] [--small]
 
 ``--small`` shrinks every case to a few hundred MB so that a profiler capture of one launch ends quickly."""
 import argparse
@@ -196,6 +196,82 @@ def case_sandwich(small):
             report(f"experts ({name})", sec, touched + T * W * 4, f"{tag}; {T * k * 6 * ff * W / sec / 1e12:.0f} TFLOP/s")
 
 
+def case_postnorm(small):
+    """Norms on the sublayers' outputs with convolutions of their inputs, minGRU, sigmoid attention (32 / 8 heads of 128, window of
+    1024 and 4 kept keys, or all keys) beside softmax attention, corrected routing, ungated experts: 4 prompts of 2048 tokens, 16
+    tokens behind 2080."""
+    from vllm_kunlun_b200.attention.metadata import AttentionMetadata
+    W, H, G, D, E, I, k, ff, taps = 4096, 32, 8, 128, 28, 4, 4, 1536, 3
+    dev, bf = "cuda", torch.bfloat16
+
+    def rnd(*shape):
+        return torch.randn(*shape, device=dev).to(bf)
+
+    w, conv_w, corr = torch.rand(W, device=dev), torch.randn(taps, W, device=dev), torch.randn(E + I, device=dev) * 0.01
+    up, down, router = rnd(E, ff, W) * 0.02, rnd(E, W, ff) * 0.02, rnd(E + I, W) * 0.02
+    qn, pb = torch.rand(D, device=dev), torch.full((H, 1), -3.0, device=dev)
+    turns = ops.position_turns(64, 10000.0).to(dev)
+    for tag, B, n, ctx in (("prompts", 4, 2048 if not small else 512, 0), ("single tokens", 16, 1, 2080)):
+        T, blocks = B * n, -(-(ctx + n) // 64)
+        i32 = lambda t: t.to(torch.int32)  # noqa: E731
+        p = (torch.arange(T, device=dev) % n) + ctx
+        bt = i32(torch.arange(B * blocks, device=dev)).view(B, blocks)
+        lens, qsl = i32(torch.full((B,), ctx + n, device=dev)), i32(torch.arange(0, T + 1, n, device=dev))
+        idx, init = i32(torch.arange(B, device=dev)), i32(torch.ones(B, device=dev))
+        slots = torch.cat([bt[b].long()[p[b * n:(b + 1) * n] // 64] * 64 + p[b * n:(b + 1) * n] % 64 for b in range(B)])
+        md = AttentionMetadata(num_tokens=T, num_reqs=B, positions=p, slot_mapping=slots, block_tables=bt, seq_lens=lens,
+                               query_start_loc=qsl, max_query_len=n, max_seq_len=ctx + n, state_indices=idx,
+                               has_initial_state=init)
+        nd = B if n == 1 else 0
+        x, y, h = torch.randn(T, W, device=dev), rnd(T, W), rnd(T, W)
+        conv = (conv_w, torch.zeros(B, taps - 1, W, device=dev))
+        ids = torch.cat([torch.randperm(E + I, device=dev)[:k].view(1, k) for _ in range(T)]).int()
+        wt = torch.rand(T, k, device=dev)
+        rows, places = ops.expert_rows(h, up, down, ids, "relu2", choices=E + I)
+        parts = ops.ChoicesSum(y, rows, places, wt, h)
+        kept = 12 * (taps - 1) / n                        # state of a request, read and written
+        for name, part, nbytes in (("row", y, 10), ("experts", parts, 10 + 2 * k)):
+            if n == 1:
+                sec = timeit(lambda: ops.postnorm_input_conv(x, part, w, 1e-5, bf, conv, md))
+                report(f"postnorm_kernel with convolution ({name})", sec, T * W * (nbytes + 2 + kept), tag)
+            else:
+                sec = timeit(lambda: ops._c().postnorm(x, None, *(part if isinstance(part, ops.ChoicesSum) else (part,) + (None,) * 4),
+                                                       w, 1e-5, None, None, None, None, None, None))
+                report(f"postnorm_kernel ({name})", sec, T * W * nbytes, tag)
+        if n > 1:
+            report("input_conv_kernel", timeit(lambda: ops.input_conv(x, bf, conv, md)), T * W * 6, tag)
+        sec = timeit(lambda: ops.layernorm_residual(x, bf, [(y, 1.0)], w, 1e-5))
+        report("layernorm_residual_kernel", sec, T * W * 12, tag)
+        z = rnd(T, 3 * W)
+        zb, state, out = torch.full((W,), -2.0, device=dev), torch.zeros(B, W, device=dev), torch.empty(T, W, dtype=bf, device=dev)
+        sec = timeit(lambda: ops.gated_blend(z[:, :W], z[:, W:2 * W], z[:, 2 * W:], zb, zb, state, qsl, idx, init, out, n, nd))
+        report("gated_blend", sec, T * W * 8 + B * W * 8, tag)
+        proj, cache = rnd(T, (H + 2 * G) * D), rnd(B * blocks, 2, G, 64, D)
+        table = ops.rotary_table(p, turns)
+        split = (proj[:, :H * D], proj[:, H * D:(H + G) * D], proj[:, (H + G) * D:])
+        sec = timeit(lambda: ops.attn_prep_cache(*split, cache, slots, p, H, G, 1e-5, v_norm=False, qk_norm=(qn, qn), table=table))
+        report("attn_prep_cache_kernel (norms, rotation)", sec, 2 * T * (H + 2 * G) * D * 2, tag)
+        sec = timeit(lambda: ops.attn_prep_cache(*split, cache, slots, p, H, G, 1e-5))
+        report("attn_prep_cache_kernel (value norm)", sec, 2 * T * (H + 2 * G) * D * 2, tag)
+        q = rnd(T, H, D)
+        for window, keep in ((None, 0), (1024, 4)):
+            seen = lambda i: i + 1 if window is None else min(i + 1, window + keep)  # noqa: E731
+            flops = sum(seen(i) for i in range(ctx, ctx + n)) * B * H * D * 4
+            keys = ctx + n if window is None or n > 1 else window + keep
+            for name, kw in (("sigmoid", dict(bias=pb, sigmoid=True, keep_first=keep)), ("softmax", {})):
+                sec = timeit(lambda: ops.paged_attention(q, cache, bt, lens, qsl, 0.09, n, keys, window, num_decodes=nd,
+                                                         num_decode_tokens=nd, **kw))
+                report(f"attention ({name}, window {window})", sec, B * keys * G * D * 4 + T * H * D * 4,
+                       f"{tag}; {flops / sec / 1e12:.0f} TFLOP/s of visible scores")
+        for name, kw in (("groups, correction", dict(bias=corr, n_group=4, topk_group=2, group_top=1)), ("plain", {})):
+            sec = timeit(lambda: ops.router_and_route(h, router, None, k, "softmax", False, fp32=True, **kw))
+            report(f"router + route ({name})", sec, T * W * 2 + (E + I) * W * 2, tag)
+        touched = min(E, T * k) * 2 * ff * W * 2
+        sec = timeit(lambda: ops.expert_rows(h, up, down, ids, "relu2", choices=E + I))
+        report("experts (squared relu)", sec, touched + T * W * 2 + T * k * W * 2,
+               f"{tag}; {int((places >= 0).sum()) * 4 * ff * W / sec / 1e12:.0f} TFLOP/s")
+
+
 def case_latent(small):
     """Kernels around latent attention (32 heads, 128 + 64 / 128, latents of 1536 and 512) and the gated fp32 stream of
     width 4096: 4 prompts of 2048 tokens, and 16 single tokens behind a context of 2080."""
@@ -321,7 +397,8 @@ if __name__ == "__main__":
     ap.add_argument("--case", default="all")
     ap.add_argument("--small", action="store_true")
     a = ap.parse_args()
-    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "sandwich": case_sandwich, "latent": case_latent, "conv": case_conv, "lora": case_lora}
+    cases = {"sample": case_sample, "gdn": case_gdn, "recurrence": case_recurrence, "stream": case_stream, "sandwich": case_sandwich,
+             "postnorm": case_postnorm, "latent": case_latent, "conv": case_conv, "lora": case_lora}
     explicit = {"gemm_splits": case_gemm_splits}  # not part of "all"
     with torch.inference_mode():
         for n, fn in cases.items():

@@ -17,7 +17,7 @@
 //              shared-memory exchange between the four warps), exp2, P^T to one of two shared-memory buffers
 //              (16-bit, K-major, swizzled) for the second MMA; the same threads own output dim t in the epilogue
 // `kSigmoid` (with `kBias`): a visible key counts with sigmoid(score + bias), not normalised - no maxima, no row sums, splits add
-// up.  `keep_first`: with a window, the first keys stay visible; their tiles come first in the tile list.
+// up.  `kKeep` (with `kBias`): with a window, the first keys stay visible; their tiles come first in the tile list.
 // Split-KV partials go through the fp32 workspace and are merged by the last CTA of a (request, head) to arrive.
 // Every wait is bounded: on time-out the status word is set, the CTA drains its copies, frees TMEM and returns.
 #include <cuda.h>
@@ -96,7 +96,7 @@ template <> __device__ __forceinline__ uint16_t to_bits16<__half>(float v) { ret
 // maximum exceeds it by more than kMaxSlack (in log2 units), so p = exp2(s - m_used) stays below 2^kMaxSlack and the
 // result O / l is unchanged; in the common case O^T needs no rescale and the softmax warps never wait for the
 // previous P.V to finish - they run ahead into a second P buffer while the tensor core works.
-template <typename T, int D, int NR, bool kBias, bool kSigmoid>
+template <typename T, int D, int NR, bool kBias, bool kSigmoid, bool kKeep>
 __global__ void __launch_bounds__(kThreads)
 decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_constant__ Params p) {
   constexpr int KB = D / 64;                       // 64-dim blocks
@@ -175,8 +175,8 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   if (p.window > 0) kv_begin = max(0, ctx - p.window + 1) / kTileKeys * kTileKeys;
   const bool served = q_len > 0 && rows_total <= NR;
   // tiles of the kept first keys that lie in front of the window's first tile
-  const int kept = p.window > 0 ? p.keep_first : 0;
-  const int n_head = min((kept + kTileKeys - 1) / kTileKeys, kv_begin / kTileKeys);
+  const int kept = kKeep && p.window > 0 ? p.keep_first : 0;
+  const int n_head = kKeep ? min((kept + kTileKeys - 1) / kTileKeys, kv_begin / kTileKeys) : 0;
   const int n_tiles_all = served ? n_head + (kv_end - kv_begin + kTileKeys - 1) / kTileKeys : 0;
   const int per_split = (n_tiles_all + p.num_splits - 1) / p.num_splits;
   const int tile_lo = split * per_split;
@@ -184,7 +184,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   const int n_tiles = max(0, tile_hi - tile_lo);
   auto tile_key = [&](int i) {   // first key of this CTA's tile i
     i += tile_lo;
-    return i < n_head ? i * kTileKeys : kv_begin + (i - n_head) * kTileKeys;
+    return kKeep && i < n_head ? i * kTileKeys : kv_begin + (i - n_head) * kTileKeys;
   };
 
   if (warp == 0) {
@@ -373,7 +373,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
       const int key0 = tile_key(i);
       const int key = key0 + lane_id;
       const bool full = key0 + kTileKeys - 1 <= pos_min && key0 + kTileKeys <= kv_end &&
-                        (p.window <= 0 || key0 > pos_max - p.window || key0 + kTileKeys <= kept);
+                        (p.window <= 0 || key0 > pos_max - p.window || (kKeep && key0 + kTileKeys <= kept));
       // nearest distance of the tile: beyond the table's last entry the bias is one constant per row
       const bool near_tile = kBias && p.bias_len > 1 && pos_min - (key0 + kTileKeys - 1) < p.bias_len - 1;
       float sc[NR];
@@ -384,7 +384,7 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
         if constexpr (kBias)
           v += near_tile ? bias[r][min(max(pos[r] - key, 0), p.bias_len - 1)] * 1.4426950408889634f : far_bias[r];
         if (!full) {
-          const bool in = key < kv_end && key <= pos[r] && (p.window <= 0 || key > pos[r] - p.window || key < kept);
+          const bool in = key < kv_end && key <= pos[r] && (p.window <= 0 || key > pos[r] - p.window || (kKeep && key < kept));
           v = in ? v : -INFINITY;
         } else if (NR > 4 && pos[r] < 0) {
           v = -INFINITY;
@@ -594,10 +594,10 @@ decode_umma_kernel(const __grid_constant__ CUtensorMap tmKV, const __grid_consta
   }
 }
 
-template <typename T, int NR, bool kBias, bool kSigmoid>
+template <typename T, int NR, bool kBias, bool kSigmoid, bool kKeep>
 static int launch_nr(const Params& p0, const CUtensorMap& tm, int B, cudaStream_t st) {
   constexpr int D = 128;
-  auto kern = decode_umma_kernel<T, D, NR, kBias, kSigmoid>;
+  auto kern = decode_umma_kernel<T, D, NR, kBias, kSigmoid, kKeep>;
   Params p = p0;
   constexpr int kStageBytes = 2 * (D / 64) * kTileKeys * 128;
   p.num_stages = 3;
@@ -611,13 +611,14 @@ static int launch_nr(const Params& p0, const CUtensorMap& tm, int B, cudaStream_
 
 template <typename T>
 static int launch(const Params& p, const CUtensorMap& tm, int B, int max_rows, bool sigmoid, cudaStream_t st) {
-#define B200_DA_LAUNCH(BIAS, SIGMOID)                                              \
-  if (max_rows <= 4) return launch_nr<T, 4, BIAS, SIGMOID>(p, tm, B, st);           \
-  if (max_rows <= 8) return launch_nr<T, 8, BIAS, SIGMOID>(p, tm, B, st);           \
-  return launch_nr<T, 16, BIAS, SIGMOID>(p, tm, B, st);
-  if (sigmoid) { B200_DA_LAUNCH(true, true) }
-  if (p.bias != nullptr) { B200_DA_LAUNCH(true, false) }
-  B200_DA_LAUNCH(false, false)
+#define B200_DA_LAUNCH(BIAS, SIGMOID, KEEP)                                        \
+  if (max_rows <= 4) return launch_nr<T, 4, BIAS, SIGMOID, KEEP>(p, tm, B, st);     \
+  if (max_rows <= 8) return launch_nr<T, 8, BIAS, SIGMOID, KEEP>(p, tm, B, st);     \
+  return launch_nr<T, 16, BIAS, SIGMOID, KEEP>(p, tm, B, st);
+  if (sigmoid) { B200_DA_LAUNCH(true, true, true) }
+  if (p.keep_first > 0) { B200_DA_LAUNCH(true, false, true) }
+  if (p.bias != nullptr) { B200_DA_LAUNCH(true, false, false) }
+  B200_DA_LAUNCH(false, false, false)
 #undef B200_DA_LAUNCH
 }
 
@@ -648,7 +649,8 @@ extern "C" int b200_decode_attention_umma(void* out, const void* q, const void* 
   p.num_stages = 3;
   p.early_meta = early_meta;
   p.bias = bias; p.bias_len = bias_len; p.gate = gate; p.gate_stride = gate_stride;
-  if ((bias != nullptr && bias_len < 1) || keep_first < 0 || (sigmoid && (bias == nullptr || sinks != nullptr))) return 2;
+  if ((bias != nullptr && bias_len < 1) || keep_first < 0 || (keep_first > 0 && bias == nullptr) ||
+      (sigmoid && (bias == nullptr || sinks != nullptr))) return 2;
   p.keep_first = keep_first;
   const CUtensorMap& tm = *reinterpret_cast<const CUtensorMap*>(tmap);
   const int max_rows = max_query_len * (Hq / Hkv);

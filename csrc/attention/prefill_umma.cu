@@ -17,8 +17,9 @@
 // entry serves every farther distance.  A tile that lies farther away altogether adds that constant inside the exponent; for
 // a nearer one the softmax warps put the 255 entries the tile can meet into shared memory (two buffers, one per tile parity).
 // `kSigmoid` (with `kBias`): a visible key counts with sigmoid(score + bias), not normalised - no maximum, no row sum and no
-// rescale; P.V accumulates as it is.
-// `keep_first`: with a window, the first keys of a request stay visible.  Their tiles come first in the tile list, which then
+// rescale; P.V accumulates as it is.  Rows need no statistics, so eight warps share the tile, two per 32 rows with half of the
+// keys (and, at the end, of the output dims) each.
+// `kKeep` (with `kBias`): with a window, the first keys of a request stay visible.  Their tiles come first in the tile list, which then
 // jumps to the window's first tile.
 // The MLA instantiation (`kMla`) is the compute-friendly prefill form of multi-head latent attention
 // (v1/attention/backends/mla/common.py:1782-1843): 192-dim q / k (128 "nope" dims per head + 64 rotary dims shared
@@ -41,7 +42,8 @@
 namespace b200 {
 namespace pattn {
 
-constexpr int kThreads = 192;
+constexpr int soft_warps(bool sigmoid) { return sigmoid ? 8 : 4; }
+constexpr int threads(bool sigmoid) { return 64 + 32 * soft_warps(sigmoid); }
 constexpr int kQTile = 128, kKTile = 128, kPage = 64, kD = 128;
 constexpr int kHalfBytes = 128 * 128;          // one 64-dim block of a 128-row operand tile
 constexpr int kOpBytes = 2 * kHalfBytes;       // Q, K, V or P tile: 32 KB
@@ -139,11 +141,12 @@ template <> __device__ __forceinline__ uint32_t pack2<__half>(float a, float b) 
   return (uint32_t)__half_as_ushort(__float2half(a)) | ((uint32_t)__half_as_ushort(__float2half(b)) << 16);
 }
 
-template <typename T, bool kMla, bool kBias, bool kSigmoid>
-__global__ void __launch_bounds__(kThreads)
+template <typename T, bool kMla, bool kBias, bool kSigmoid, bool kKeep>
+__global__ void __launch_bounds__(threads(kSigmoid))
 prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                     const __grid_constant__ CUtensorMap tmKpe, const __grid_constant__ Params p) {
   static_assert(!kSigmoid || (kBias && !kMla));
+  constexpr int kSoftWarps = soft_warps(kSigmoid);
   constexpr int kQBlocks = Cfg<kMla>::kQBlocks, kKBytes = Cfg<kMla>::kKBytes, kVStages = Cfg<kMla>::kVStages;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -156,7 +159,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint64_t* k_empty = bars + 3;        // [2] S of the tile has been computed
   uint64_t* s_full = bars + 5;         // [2]
   uint64_t* s_empty = bars + 7;        // [2]
-  uint64_t* p_ready = bars + 9;        // [1] 4 arrivals (one per softmax warp)
+  uint64_t* p_ready = bars + 9;        // [1] one arrival per softmax warp
   uint64_t* p_free = bars + 10;        // [1]
   uint64_t* o_done = bars + 11;        // [1] one phase per P.V
   uint64_t* o_final = bars + 12;       // [1] once, after the last P.V
@@ -176,9 +179,9 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     for (int b = 0; b < 2; ++b) {
       mbar_init(&k_full[b], 1); mbar_init(&k_empty[b], 1);
       mbar_init(&v_full[b], 1); mbar_init(&v_empty[b], 1);
-      mbar_init(&s_full[b], 1); mbar_init(&s_empty[b], 4);
+      mbar_init(&s_full[b], 1); mbar_init(&s_empty[b], kSoftWarps);
     }
-    mbar_init(p_ready, 4); mbar_init(p_free, 1); mbar_init(o_done, 1); mbar_init(o_final, 1);
+    mbar_init(p_ready, kSoftWarps); mbar_init(p_free, 1); mbar_init(o_done, 1); mbar_init(o_final, 1);
     mbar_fence_init();
     prefetch_tmap(&tmQ);
     prefetch_tmap(&tmKV);
@@ -209,10 +212,10 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, pos_first - p.window + 1) / kKTile * kKTile;
   // tiles of the kept first keys that lie in front of the window's first tile
-  const int kept = p.window > 0 ? p.keep_first : 0;
-  const int n_head = min((kept + kKTile - 1) / kKTile, kv_begin / kKTile);
+  const int kept = kKeep && p.window > 0 ? p.keep_first : 0;
+  const int n_head = kKeep ? min((kept + kKTile - 1) / kKTile, kv_begin / kKTile) : 0;
   const int n_tiles = n_rows > 0 ? n_head + (kv_end - kv_begin + kKTile - 1) / kKTile : 0;
-  auto tile_key = [&](int i) { return i < n_head ? i * kKTile : kv_begin + (i - n_head) * kKTile; };
+  auto tile_key = [&](int i) { return kKeep && i < n_head ? i * kKTile : kv_begin + (i - n_head) * kKTile; };
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
@@ -356,7 +359,9 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
   } else {
     // ------------------------------------------------------------------ softmax + epilogue: thread = query row
+    constexpr int kCols = kSigmoid ? kKTile / 2 : kKTile, kDims = kSigmoid ? kD / 2 : kD;   // keys, output dims of a warp
     const int quarter = warp & 3;
+    const int part = kSigmoid ? (warp - 2) >> 2 : 0, col0 = part * kCols;
     const int r = quarter * 32 + lane;                 // row of the tile = TMEM lane
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     const uint32_t tS = tmem_base + lane_off, tO = tmem_base + 2 * kKTile + lane_off;
@@ -377,7 +382,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (threadIdx.x == 64 && i == 20) trace_mark(p.trace, cta_id, 8);
       const int key0 = tile_key(i);
       const bool full_tile = key0 + kKTile - 1 <= pos_first && key0 + kKTile <= kv_end &&
-                             (p.window <= 0 || key0 > pos_last - p.window || key0 + kKTile <= kept);
+                             (p.window <= 0 || key0 > pos_last - p.window || (kKeep && key0 + kKTile <= kept));
       // nearest distance of the tile: beyond the table's last entry its bias is one constant
       const bool near_tile = kBias && p.bias_len > 1 && pos_first - (key0 + kKTile - 1) < p.bias_len - 1;
       if constexpr (kBias) {
@@ -385,16 +390,17 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           float* dst = sBias + (i & 1) * 256;
           const int tid = threadIdx.x - 64, d0 = pos_first - key0 - (kKTile - 1);
 #pragma unroll
-          for (int d = 0; d < 256; d += 128) dst[tid + d] = bias[min(max(d0 + tid + d, 0), p.bias_len - 1)] * kLog2e;
-          asm volatile("bar.sync 3, 128;" ::: "memory");
+          for (int d = 0; d < 256; d += 32 * kSoftWarps)
+            dst[tid + d] = bias[min(max(d0 + tid + d, 0), p.bias_len - 1)] * kLog2e;
+          asm volatile("bar.sync 3, %0;" ::"n"(32 * kSoftWarps) : "memory");
         }
       }
       // ---- the whole row (128 scores) in one TMEM round trip: a tcgen05.ld + wait pair costs several hundred
       // nanoseconds whatever its width, so all four 32-column loads are issued before the single wait, and the
       // S buffer goes back to the tensor core at once
-      uint32_t v[kKTile];
+      uint32_t v[kCols];
 #pragma unroll
-      for (int c = 0; c < kKTile; c += 32) tmem_ld_x32_p(tS + buf * kKTile + c, v + c);
+      for (int c = 0; c < kCols; c += 32) tmem_ld_x32_p(tS + buf * kKTile + col0 + c, v + c);
       tmem_ld_wait();
       if (threadIdx.x == 64 && i == 4) trace_mark(p.trace, cta_id, 11);
       tc_fence_before_sync();
@@ -406,18 +412,18 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       float sc = p.scale_log2, off = far_bias;     // exponent = raw score * sc + off - maximum
       if constexpr (kBias) {
         if (near_tile) {
-          const float* src = sBias + (i & 1) * 256 + (kKTile - 1) + r;
+          const float* src = sBias + (i & 1) * 256 + (kKTile - 1) + r - col0;
 #pragma unroll
-          for (int e = 0; e < kKTile; ++e) v[e] = __float_as_uint(fmaf(__uint_as_float(v[e]), p.scale_log2, src[-e]));
+          for (int e = 0; e < kCols; ++e) v[e] = __float_as_uint(fmaf(__uint_as_float(v[e]), p.scale_log2, src[-e]));
           sc = 1.f;
           off = 0.f;
         }
       }
       if (!full_tile) {
 #pragma unroll
-        for (int e = 0; e < kKTile; ++e) {
-          const int key = key0 + e;
-          const bool in = key < kv_end && key <= pos && (p.window <= 0 || key > pos - p.window || key < kept);
+        for (int e = 0; e < kCols; ++e) {
+          const int key = key0 + col0 + e;
+          const bool in = key < kv_end && key <= pos && (p.window <= 0 || key > pos - p.window || (kKeep && key < kept));
           v[e] = in ? v[e] : 0xff800000u;   // -inf
         }
       }
@@ -425,7 +431,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         // P (one buffer): the previous P.V must have read it
         if (i >= 1 && !fail && !wait_or_abort(p_free, (i - 1) & 1, ab, 806)) fail = true;
 #pragma unroll
-        for (int c = 0; c < kKTile; c += 32) {
+        for (int c = 0; c < kCols; c += 32) {
           uint32_t pk[16];
 #pragma unroll
           for (int e = 0; e < 32; e += 2) {
@@ -440,7 +446,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           if (!fail) {
 #pragma unroll
             for (int q4 = 0; q4 < 4; ++q4) {
-              const int q = c / 8 + q4;
+              const int q = (col0 + c) / 8 + q4;
               *reinterpret_cast<uint4*>(sP + (q >> 3) * kHalfBytes + r * 128 + (((q & 7) ^ (r & 7)) << 4)) =
                   make_uint4(pk[q4 * 4], pk[q4 * 4 + 1], pk[q4 * 4 + 2], pk[q4 * 4 + 3]);
             }
@@ -452,7 +458,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         __syncwarp();
         if (lane == 0 && !warp_failed) mbar_arrive(p_ready);
         continue;
-      }
+      } else {
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
       for (int e = 0; e < kKTile; e += 4) {
@@ -520,6 +526,7 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       __syncwarp();
       if (lane == 0 && !warp_failed) mbar_arrive(p_ready);
       if (threadIdx.x == 64 && i == 4) trace_mark(p.trace, cta_id, 5);
+      }
     }
     if (threadIdx.x == 64) trace_mark(p.trace, cta_id, 6);
     // ---- epilogue
@@ -540,13 +547,14 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         inv = inv / (1.f + __expf(-g));
       }
       T* dst = reinterpret_cast<T*>(p.out) + orow * kD;
-      uint32_t o[kD];
+      dst += part * kDims;
+      uint32_t o[kDims];
 #pragma unroll
-      for (int c = 0; c < kD; c += 32) tmem_ld_x32_p(tO + c, o + c);   // warp-collective: every lane loads
+      for (int c = 0; c < kDims; c += 32) tmem_ld_x32_p(tO + part * kDims + c, o + c);   // warp-collective: every lane loads
       tmem_ld_wait();
       if (row_ok) {
 #pragma unroll
-        for (int q4 = 0; q4 < kD / 8; ++q4) {
+        for (int q4 = 0; q4 < kDims / 8; ++q4) {
           uint32_t w4[4];
 #pragma unroll
           for (int u = 0; u < 4; ++u)
@@ -567,15 +575,15 @@ prefill_umma_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
 }
 
-template <typename T, bool kMla, bool kBias, bool kSigmoid>
+template <typename T, bool kMla, bool kBias, bool kSigmoid, bool kKeep>
 static int launch(const Params& p, const CUtensorMap& tmQ, const CUtensorMap& tmKV, const CUtensorMap& tmKpe, int B,
                   int max_query_len, cudaStream_t st) {
-  auto kern = prefill_umma_kernel<T, kMla, kBias, kSigmoid>;
+  auto kern = prefill_umma_kernel<T, kMla, kBias, kSigmoid, kKeep>;
   const size_t smem = Cfg<kMla>::kSmem + (kBias ? Cfg<kMla>::kBiasSmem : 0);
   cudaError_t e = ensure_dynamic_smem((const void*)kern, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid((unsigned)((max_query_len + kQTile - 1) / kQTile), (unsigned)p.Hq, (unsigned)B);
-  return (int)launch_pdl(kern, grid, dim3(kThreads), smem, st, tmQ, tmKV, tmKpe, p);
+  return (int)launch_pdl(kern, grid, dim3(threads(kSigmoid)), smem, st, tmQ, tmKV, tmKpe, p);
 }
 
 }  // namespace pattn
@@ -585,7 +593,7 @@ static int launch(const Params& p, const CUtensorMap& tmQ, const CUtensorMap& tm
 // [T, Hq * 128] 16-bit tensor with 64-column x 128-row boxes; `tmKV`: the cache as [rows, 128] with 64 x 64 boxes;
 // both with 128-byte swizzle.  `bias` [Hq][bias_len] (or null): score bias by distance, the last entry for all farther ones;
 // `gate` [T][>= Hq] (or null): raw output gates; `sigmoid`: weights without a softmax (needs a bias; no sinks, no lse);
-// `keep_first`: keys that a window never hides.  Returns 3 for shapes it does not serve.
+// `keep_first`: keys that a window never hides (needs a bias).  Returns 3 for shapes it does not serve.
 extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tmQ, const void* tmKV,
                                            const int* block_tables, const int* seq_lens, const int* qsl,
                                            const float* sinks, int* status, int B, int Hq, int Hkv, int D, int block_size,
@@ -596,6 +604,7 @@ extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tm
   using namespace b200;
   if (B == 0 || max_query_len <= 0) return 0;
   if ((bias != nullptr && bias_len < 1) || keep_first < 0) return 2;
+  if (keep_first > 0 && bias == nullptr) return 2;
   if (sigmoid && (bias == nullptr || sinks != nullptr || lse != nullptr)) return 2;
   if (D != 128 || Hq % Hkv || block_size % pattn::kPage || B > 65535 || Hq > 65535) return 3;
   pattn::Params p;
@@ -606,9 +615,10 @@ extern "C" int b200_prefill_attention_umma(void* out, float* lse, const void* tm
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
 #define B200_PA_LAUNCH(T)                                                                            \
-  (sigmoid           ? pattn::launch<T, false, true, true>(p, q, kv, kv, B, max_query_len, st)        \
-   : bias != nullptr ? pattn::launch<T, false, true, false>(p, q, kv, kv, B, max_query_len, st)       \
-                     : pattn::launch<T, false, false, false>(p, q, kv, kv, B, max_query_len, st))
+  (sigmoid           ? pattn::launch<T, false, true, true, true>(p, q, kv, kv, B, max_query_len, st)  \
+   : keep_first > 0  ? pattn::launch<T, false, true, false, true>(p, q, kv, kv, B, max_query_len, st) \
+   : bias != nullptr ? pattn::launch<T, false, true, false, false>(p, q, kv, kv, B, max_query_len, st) \
+                     : pattn::launch<T, false, false, false, false>(p, q, kv, kv, B, max_query_len, st))
   if (dtype == 1) return B200_PA_LAUNCH(__nv_bfloat16);
   if (dtype == 2) return B200_PA_LAUNCH(__half);
 #undef B200_PA_LAUNCH
@@ -638,7 +648,7 @@ extern "C" int b200_mla_prefill_umma(void* out, float* lse, const void* tmQ, con
   const CUtensorMap& q = *reinterpret_cast<const CUtensorMap*>(tmQ);
   const CUtensorMap& kv = *reinterpret_cast<const CUtensorMap*>(tmKV);
   const CUtensorMap& kpe = *reinterpret_cast<const CUtensorMap*>(tmKpe);
-  if (dtype == 1) return pattn::launch<__nv_bfloat16, true, false, false>(p, q, kv, kpe, B, max_query_len, st);
-  if (dtype == 2) return pattn::launch<__half, true, false, false>(p, q, kv, kpe, B, max_query_len, st);
+  if (dtype == 1) return pattn::launch<__nv_bfloat16, true, false, false, false>(p, q, kv, kpe, B, max_query_len, st);
+  if (dtype == 2) return pattn::launch<__half, true, false, false, false>(p, q, kv, kpe, B, max_query_len, st);
   return 3;
 }

@@ -216,14 +216,22 @@ __global__ void __launch_bounds__(256) attn_prep_cache_kernel(AttnPrepArgs a, in
   } else {
     src = reinterpret_cast<const T*>(is_v ? a.v : a.k) + t * a.stride + (int64_t)kvh * n;
     const int64_t slot = a.slots[t];
-    if (slot >= 0 && slot < a.num_blocks * a.block_size)
+    if (slot >= 0 && slot < a.num_blocks * a.block_size) {      // fewer than 2^31 slots: 32-bit division
+      const uint32_t block = (uint32_t)slot / (uint32_t)a.block_size, cell = (uint32_t)slot % (uint32_t)a.block_size;
       dst = reinterpret_cast<T*>(a.cache) +
-            ((((slot / a.block_size) * 2 + (is_v ? 1 : 0)) * Hkv + kvh) * a.block_size + slot % a.block_size) * (int64_t)Dc;
+            (((int64_t)block * 2 + (is_v ? 1 : 0)) * Hkv + kvh) * ((int64_t)a.block_size * Dc) + (int64_t)cell * Dc;
+    }
   }
   const float* w = is_v ? nullptr : is_q ? a.q_norm : a.k_norm;
+  // heads that fit one quad per lane stay in registers; their rotation partners come from another lane
+  const bool held = vec && Dc <= 128;
+  float own[4] = {0.f, 0.f, 0.f, 0.f};
+  if (held && lane * 4 < n) load4(own, src + lane * 4);
   if (is_v ? a.v_norm != 0 : w != nullptr) {
     float ss = 0.f;
-    if (vec) {
+    if (held) {
+      ss = own[0] * own[0] + own[1] * own[1] + own[2] * own[2] + own[3] * own[3];
+    } else if (vec) {
       for (int i = lane * 4; i < n; i += 128) {
         float x[4];
         load4(x, src + i);
@@ -239,7 +247,39 @@ __global__ void __launch_bounds__(256) attn_prep_cache_kernel(AttnPrepArgs a, in
   const int64_t vo = (t * Hkv + kvh) * (int64_t)a.Dv;
   const T* mix = is_v && a.v_in != nullptr ? reinterpret_cast<const T*>(a.v_in) + vo : nullptr;
   T* keep = is_v && a.v_out != nullptr ? reinterpret_cast<T*>(a.v_out) + vo : nullptr;
-  if (vec) {
+  if (held) {
+    const int i = lane * 4, shift = pairs / 4;
+    const bool lower = i < pairs;
+    float x[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) x[j] = own[j] * (w == nullptr || i >= n ? f : f * w[i + j]);
+    if (pairs > 0) {        // the same for the whole warp
+#pragma unroll
+      for (int j = 0; j < 4; ++j) own[j] = __shfl_sync(0xffffffffu, x[j], (lower ? lane + shift : lane - shift) & 31);
+      if (i < 2 * pairs) {
+        const float* cs = turn + 2 * (lower ? i : i - pairs);
+        float c[4], s[4];
+        load4(c, cs);
+        load4(s, cs + 4);
+        const float sg = lower ? -1.f : 1.f;
+        x[0] = x[0] * c[0] + sg * own[0] * c[1];
+        x[1] = x[1] * c[2] + sg * own[1] * c[3];
+        x[2] = x[2] * s[0] + sg * own[2] * s[1];
+        x[3] = x[3] * s[2] + sg * own[3] * s[3];
+      }
+    }
+    if (i >= Dc) return;
+    if (i < n) {
+      if (keep != nullptr) store4(keep + i, x);
+      if (mix != nullptr) {
+        float b[4];
+        load4(b, mix + i);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] = (1.f - a.share) * x[j] + a.share * b[j];
+      }
+    }
+    if (dst != nullptr) store4(dst + i, x);
+  } else if (vec) {
     auto scaled = [&](float (&x)[4], int i) {
       load4(x, src + i);
 #pragma unroll
@@ -348,6 +388,7 @@ extern "C" int b200_attn_prep_cache(const AttnPrepArgs* args, int64_t T_, int dt
   const AttnPrepArgs& a = *args;
   if (T_ == 0) return 0;
   if (a.D > a.Dc || a.Dv > a.Dc || (a.table != nullptr && 2 * a.pairs > a.D)) return 3;
+  if (a.num_blocks * a.block_size >= ((int64_t)1 << 31)) return 3;
   const uintptr_t al = (uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.v_out | (uintptr_t)a.v_in;
   const int vec = a.D % 4 == 0 && a.Dv % 4 == 0 && a.Dc % 4 == 0 && a.stride % 4 == 0 && al % 16 == 0 &&
                   (a.table == nullptr || a.pairs % 4 == 0);

@@ -3,9 +3,9 @@
 //   out_t = S_t * silu(g)
 // over raw projections zr, ur, g; the state [slots][W] is fp32 and carried per request.
 // A token is the map S -> a S + b with a = 1 - z = sigmoid(-(zr + bz)), b = z c, and maps compose: a' a, a' b + b'.  One CTA takes
-// 32 columns (two channels each) of one request; its 16 warps take consecutive runs of tokens of a block, compose their run,
-// meet over shared memory and apply the map of everything in front.  Products only: no logarithms, no quotients, so gates near
-// zero and one are safe.  Single tokens: a thread per channel.
+// 32 channels of one request, a lane each; its 16 warps take consecutive runs of tokens of a block, compose their run, meet over
+// shared memory and apply the map of everything in front, while the next block's projections are on their way.  Products only: no
+// logarithms, no quotients of gates, so gates near zero and one are safe.  Single tokens: a thread per channel.
 // Launched with programmatic dependent launch: no __restrict__ on what a predecessor writes.  Compiled without fast-math.
 #include "../api.h"
 #include "../common/launch.cuh"
@@ -16,40 +16,29 @@ namespace {
 
 constexpr int kWarps = 16, kRun = 8, kBlock = kWarps * kRun;   // tokens per warp and per block of tokens
 
-template <typename T> struct alignas(2 * sizeof(T)) Pair { T v[2]; };
-template <typename T> __device__ __forceinline__ float2 load2(const T* p) {
-  const Pair<T> r = *reinterpret_cast<const Pair<T>*>(p);
-  return make_float2(to_f(r.v[0]), to_f(r.v[1]));
-}
-template <typename T> __device__ __forceinline__ void store2(T* p, float a, float b) {
-  Pair<T> r;
-  r.v[0] = from_f<T>(a);
-  r.v[1] = from_f<T>(b);
-  *reinterpret_cast<Pair<T>*>(p) = r;
-}
-// sigmoid(-x) and sigmoid(x), both without cancellation
-__device__ __forceinline__ void sigmoids(float x, float& neg, float& pos) {
-  const float e = expf(-fabsf(x)), r = 1.f / (1.f + e);
-  pos = x >= 0.f ? r : e * r;
-  neg = x >= 0.f ? e * r : r;
-}
-__device__ __forceinline__ void token_map(float zr, float ur, float bz, float bu, float& a, float& b) {
-  float z, n;
-  sigmoids(zr + bz, a, z);
-  const float u = ur + bu;
-  float c = u + 0.5f;
-  if (u < 0.f) sigmoids(u, n, c);
-  b = z * c;
-}
-__device__ __forceinline__ float silu(float g) {
-  float n, p;
-  sigmoids(g, n, p);
-  return g * p;
+// A token's map S -> a S + b and its output gate silu(g).  sigmoid(x) and sigmoid(-x) come from exp(-|x|) without cancellation.
+// 16-bit models use the hardware exponential and one hardware reciprocal for the three denominators, which lie between one and two
+// (a few units in the last place of fp32).
+template <typename T>
+__device__ __forceinline__ void token(float zr, float ur, float g, float bz, float bu, float& a, float& b, float& gate) {
+  const float z = zr + bz, u = ur + bu;
+  float ez, eu, eg, rz, ru, rg;
+  if constexpr (sizeof(T) == 4) {
+    ez = expf(-fabsf(z)); eu = expf(-fabsf(u)); eg = expf(-fabsf(g));
+    rz = 1.f / (1.f + ez); ru = 1.f / (1.f + eu); rg = 1.f / (1.f + eg);
+  } else {
+    ez = __expf(-fabsf(z)); eu = __expf(-fabsf(u)); eg = __expf(-fabsf(g));
+    const float dz = 1.f + ez, du = 1.f + eu, dg = 1.f + eg, zu = dz * du, r = __fdividef(1.f, zu * dg), t = r * dg;
+    rz = t * du; ru = t * dz; rg = r * zu;
+  }
+  a = z >= 0.f ? ez * rz : rz;
+  b = (z >= 0.f ? rz : ez * rz) * (u >= 0.f ? u + 0.5f : eu * ru);
+  gate = g * (g >= 0.f ? rg : eg * rg);
 }
 
 template <typename T>
-__global__ void __launch_bounds__(kWarps * 32) blend_scan_kernel(BlendArgs p) {
-  __shared__ float2 sa[kWarps][32], sb[kWarps][32];
+__global__ void __launch_bounds__(kWarps * 32, 2) blend_scan_kernel(BlendArgs p) {
+  __shared__ float sa[2][kWarps][32], sb[2][kWarps][32];
   griddep_launch();
   griddep_wait();
   const int req = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -57,64 +46,56 @@ __global__ void __launch_bounds__(kWarps * 32) blend_scan_kernel(BlendArgs p) {
   int64_t slot = p.slots[req];
   if (slot >= p.num_slots) slot = -1;
   if (q0 >= q1 || slot < 0) return;
-  const int c = (blockIdx.x * 32 + lane) * 2;
-  const bool on = c < p.width, both = c + 1 < p.width;    // the projections' columns are padded to an even number
-  float2 bz = make_float2(0.f, 0.f), bu = bz, S = bz;
-  if (on) {
-    bz.x = p.z_bias[c]; bu.x = p.x_bias[c];
-    if (both) { bz.y = p.z_bias[c + 1]; bu.y = p.x_bias[c + 1]; }
-    if (p.has_init[req]) {
-      S.x = p.state[slot * p.width + c];
-      if (both) S.y = p.state[slot * p.width + c + 1];
-    }
-  }
+  const int c = blockIdx.x * 32 + lane;
+  const bool on = c < p.width;
+  const float bz = on ? p.z_bias[c] : 0.f, bu = on ? p.x_bias[c] : 0.f;
+  float S = on && p.has_init[req] ? p.state[slot * p.width + c] : 0.f;
   const T* z = reinterpret_cast<const T*>(p.z) + c;
   const T* x = reinterpret_cast<const T*>(p.x) + c;
   const T* g = reinterpret_cast<const T*>(p.g) + c;
   T* out = reinterpret_cast<T*>(p.out) + c;
-  for (int64_t base = q0; base < q1; base += kBlock) {
-    const int64_t t0 = base + warp * kRun;
-    const int n = on ? (int)max((int64_t)0, min((int64_t)kRun, q1 - t0)) : 0;
-    float2 a[kRun], b[kRun];
-    float2 zr[kRun], ur[kRun];
+  T zr[kRun], ur[kRun], gr[kRun];
+  auto rows = [&](int64_t base) {      // tokens of this warp's run
+    return on ? (int)max((int64_t)0, min((int64_t)kRun, q1 - base - warp * kRun)) : 0;
+  };
+  auto fetch = [&](int64_t base) {
+    const int n = rows(base);
+    const int64_t o = (base + warp * kRun) * p.stride;
 #pragma unroll
     for (int i = 0; i < kRun; ++i)
-      if (i < n) { zr[i] = load2(z + (t0 + i) * p.stride); ur[i] = load2(x + (t0 + i) * p.stride); }
-    float2 A = make_float2(1.f, 1.f), B = make_float2(0.f, 0.f);
+      if (i < n) { zr[i] = z[o + i * p.stride]; ur[i] = x[o + i * p.stride]; gr[i] = g[o + i * p.stride]; }
+  };
+  fetch(q0);
+  int buf = 0;
+  for (int64_t base = q0; base < q1; base += kBlock, buf ^= 1) {
+    const int n = rows(base);
+    float a[kRun], b[kRun], gate[kRun], A = 1.f, B = 0.f;
 #pragma unroll
     for (int i = 0; i < kRun; ++i) {
       if (i >= n) break;
-      token_map(zr[i].x, ur[i].x, bz.x, bu.x, a[i].x, b[i].x);
-      token_map(zr[i].y, ur[i].y, bz.y, bu.y, a[i].y, b[i].y);
-      B.x = fmaf(a[i].x, B.x, b[i].x); B.y = fmaf(a[i].y, B.y, b[i].y);
-      A.x *= a[i].x; A.y *= a[i].y;
+      token<T>(to_f(zr[i]), to_f(ur[i]), to_f(gr[i]), bz, bu, a[i], b[i], gate[i]);
+      B = fmaf(a[i], B, b[i]);
+      A *= a[i];
     }
-    sa[warp][lane] = A;
-    sb[warp][lane] = B;
-    __syncthreads();
-    // state in front of this warp's run, and behind the block
-    float2 mine = S;
+    if (base + kBlock < q1) fetch(base + kBlock);
+    sa[buf][warp][lane] = A;
+    sb[buf][warp][lane] = B;
+    __syncthreads();      // buffers alternate: one barrier per block
+    float mine = S;       // state in front of this warp's run; S moves on to the end of the block
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) {
       if (w == warp) mine = S;
-      const float2 wa = sa[w][lane], wb = sb[w][lane];
-      S.x = fmaf(wa.x, S.x, wb.x); S.y = fmaf(wa.y, S.y, wb.y);
+      S = fmaf(sa[buf][w][lane], S, sb[buf][w][lane]);
     }
-    __syncthreads();      // the maps are overwritten by the next block
-#pragma unroll
-    for (int i = 0; i < kRun; ++i)
-      if (i < n) zr[i] = load2(g + (t0 + i) * p.stride);
+    T* o = out + (base + warp * kRun) * p.out_stride;
 #pragma unroll
     for (int i = 0; i < kRun; ++i) {
       if (i >= n) break;
-      mine.x = fmaf(a[i].x, mine.x, b[i].x); mine.y = fmaf(a[i].y, mine.y, b[i].y);
-      store2(out + (t0 + i) * p.out_stride, mine.x * silu(zr[i].x), both ? mine.y * silu(zr[i].y) : 0.f);
+      mine = fmaf(a[i], mine, b[i]);
+      o[i * p.out_stride] = from_f<T>(mine * gate[i]);
     }
   }
-  if (warp == 0 && on) {
-    p.state[slot * p.width + c] = S.x;
-    if (both) p.state[slot * p.width + c + 1] = S.y;
-  }
+  if (warp == 0 && on) p.state[slot * p.width + c] = S;
 }
 
 // A thread per channel walks the request's tokens: requests of one token (or a few).
@@ -130,12 +111,12 @@ __global__ void __launch_bounds__(128) blend_step_kernel(BlendArgs p) {
   float S = slot >= 0 && p.has_init[req] ? p.state[slot * p.width + c] : 0.f;
   const float bz = p.z_bias[c], bu = p.x_bias[c];
   for (int64_t t = q0; t < q1; ++t) {
-    float a, b;
-    token_map(to_f(reinterpret_cast<const T*>(p.z)[t * p.stride + c]), to_f(reinterpret_cast<const T*>(p.x)[t * p.stride + c]), bz,
-              bu, a, b);
+    float a, b, gate;
+    const int64_t o = t * p.stride + c;
+    token<T>(to_f(reinterpret_cast<const T*>(p.z)[o]), to_f(reinterpret_cast<const T*>(p.x)[o]),
+             to_f(reinterpret_cast<const T*>(p.g)[o]), bz, bu, a, b, gate);
     S = fmaf(a, S, b);
-    reinterpret_cast<T*>(p.out)[t * p.out_stride + c] =
-        from_f<T>(S * silu(to_f(reinterpret_cast<const T*>(p.g)[t * p.stride + c])));
+    reinterpret_cast<T*>(p.out)[t * p.out_stride + c] = from_f<T>(S * gate);
   }
   if (slot >= 0) p.state[slot * p.width + c] = S;
 }
@@ -148,13 +129,11 @@ extern "C" int b200_gated_blend(const BlendArgs* args, int dtype, cudaStream_t s
   const BlendArgs& a = *args;
   if (a.R == 0 || a.width == 0) return 0;
   if (a.R > 65535) return 3;
-  const uintptr_t al = (uintptr_t)a.z | (uintptr_t)a.x | (uintptr_t)a.g | (uintptr_t)a.out;
-  if (!a.steps && (al % 8 || a.stride % 2 || a.out_stride % 2 || a.out_stride < (a.width + 1) / 2 * 2)) return 3;
   B200_DISPATCH_DTYPE(dtype, {
     if (a.steps)
       launch_pdl(blend_step_kernel<T>, dim3((a.width + 127) / 128, a.R), dim3(128), 0, st, a);
     else
-      launch_pdl(blend_scan_kernel<T>, dim3((a.width + 63) / 64, a.R), dim3(kWarps * 32), 0, st, a);
+      launch_pdl(blend_scan_kernel<T>, dim3((a.width + 31) / 32, a.R), dim3(kWarps * 32), 0, st, a);
   });
   return (int)cudaGetLastError();
 }

@@ -20,20 +20,19 @@ constexpr int kMaxTopK = 16;
 
 // mode: 0 softmax->topk, 1 sigmoid->topk, 2 topk->softmax.  Modes 0 and 1 choose by score + bias.  group_top: how many of a
 // group's best selection scores add up to the group's score (1 or 2); 0 = choose without groups
-// One warp routes one token; `row` holds the token's E router logits (global or shared memory).
-template <typename T>
+// One warp routes one token; `row` holds the token's E <= 32 PER router logits (global or shared memory).
+template <typename T, int PER>
 __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __restrict__ out_ids, const T* row,
                                           const float* __restrict__ bias, int64_t t, int lane, int E, int k, int mode,
                                           int renorm, int n_group, int topk_group, int group_top, float scale) {
-  const int per = (E + 31) / 32;
-  float score[kMaxEPerLane];  // unbiased weight source
-  float sel[kMaxEPerLane];    // selection score
+  float score[PER];  // unbiased weight source
+  float sel[PER];    // selection score
   // expert e lives on lane e % 32, slot e / 32
   float mx = -INFINITY;
 #pragma unroll
-  for (int s = 0; s < kMaxEPerLane; ++s) {
+  for (int s = 0; s < PER; ++s) {
     int e = s * 32 + lane;
-    float v = (s < per && e < E) ? to_f(row[e]) : -INFINITY;
+    float v = (e < E) ? to_f(row[e]) : -INFINITY;
     score[s] = v;
     mx = fmaxf(mx, v);
   }
@@ -41,30 +40,30 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
     mx = warp_max(mx);
     float sum = 0.f;
 #pragma unroll
-    for (int s = 0; s < kMaxEPerLane; ++s) {
+    for (int s = 0; s < PER; ++s) {
       float p = (score[s] == -INFINITY) ? 0.f : __expf(score[s] - mx);
       sum += p;
       score[s] = p;
     }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int s = 0; s < kMaxEPerLane; ++s) {
+    for (int s = 0; s < PER; ++s) {
       int e = s * 32 + lane;
-      score[s] = (s < per && e < E) ? score[s] / sum : -INFINITY;
-      sel[s] = (bias && s < per && e < E) ? score[s] + bias[e] : score[s];
+      score[s] = (e < E) ? score[s] / sum : -INFINITY;
+      sel[s] = (bias && e < E) ? score[s] + bias[e] : score[s];
     }
   } else if (mode == 1) {
 #pragma unroll
-    for (int s = 0; s < kMaxEPerLane; ++s) {
+    for (int s = 0; s < PER; ++s) {
       int e = s * 32 + lane;
-      bool ok = s < per && e < E;
+      bool ok = e < E;
       float sg = ok ? 1.f / (1.f + __expf(-score[s])) : -INFINITY;
       score[s] = sg;
       sel[s] = ok ? sg + (bias ? bias[e] : 0.f) : -INFINITY;
     }
   } else {
 #pragma unroll
-    for (int s = 0; s < kMaxEPerLane; ++s) sel[s] = score[s];
+    for (int s = 0; s < PER; ++s) sel[s] = score[s];
   }
   if (mode != 2 && n_group > 1 && group_top > 0) {
     // group score = sum of the group_top best selection scores in the group; keep the best topk_group groups
@@ -73,9 +72,9 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
     for (int g = 0; g < n_group; ++g) {
       float b1 = -INFINITY, b2 = -INFINITY;
 #pragma unroll
-      for (int s = 0; s < kMaxEPerLane; ++s) {
+      for (int s = 0; s < PER; ++s) {
         int e = s * 32 + lane;
-        if (s < per && e < E && e / gsz == g) {
+        if (e < E && e / gsz == g) {
           float v = sel[s];
           if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
         }
@@ -105,9 +104,9 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
       if (lane == idx) gscore_mine = -INFINITY;
     }
 #pragma unroll
-    for (int s = 0; s < kMaxEPerLane; ++s) {
+    for (int s = 0; s < PER; ++s) {
       int e = s * 32 + lane;
-      if (s < per && e < E && !((keep >> (e / gsz)) & 1u)) sel[s] = -INFINITY;
+      if (e < E && !((keep >> (e / gsz)) & 1u)) sel[s] = -INFINITY;
     }
   }
   // k rounds of warp arg-max over sel
@@ -119,9 +118,9 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
     int idx = 0x7fffffff;
     float sc = 0.f;
 #pragma unroll
-    for (int s = 0; s < kMaxEPerLane; ++s) {
+    for (int s = 0; s < PER; ++s) {
       int e = s * 32 + lane;
-      if (s < per && e < E && (sel[s] > v || (sel[s] == v && e < idx))) { v = sel[s]; idx = e; sc = score[s]; }
+      if (e < E && (sel[s] > v || (sel[s] == v && e < idx))) { v = sel[s]; idx = e; sc = score[s]; }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -154,7 +153,7 @@ __device__ __forceinline__ void route_row(float* __restrict__ out_w, int* __rest
 }
 
 
-template <typename T>
+template <typename T, int PER>
 __global__ void moe_route_kernel(float* __restrict__ out_w, int* __restrict__ out_ids, const T* __restrict__ logits,
                                  const float* __restrict__ bias, int64_t T_, int E, int k, int mode, int renorm,
                                  int n_group, int topk_group, int group_top, float scale, int64_t stride) {
@@ -162,13 +161,13 @@ __global__ void moe_route_kernel(float* __restrict__ out_w, int* __restrict__ ou
   griddep_wait();
   const int64_t t = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T_) return;
-  route_row<T>(out_w, out_ids, logits + t * stride, bias, t, threadIdx.x & 31, E, k, mode, renorm, n_group, topk_group,
+  route_row<T, PER>(out_w, out_ids, logits + t * stride, bias, t, threadIdx.x & 31, E, k, mode, renorm, n_group, topk_group,
                group_top, scale);
 }
 
 // Router GEMM and routing in one launch for decode-sized batches: one CTA per token computes its E logits into
 // shared memory (each warp a slice of the experts, 16-byte loads of the router rows), then warp 0 routes the token.
-template <typename T>
+template <typename T, int PER>
 __global__ void __launch_bounds__(256) router_route_small_kernel(
     float* __restrict__ out_w, int* __restrict__ out_ids, const T* __restrict__ x, int64_t x_stride,
     const T* __restrict__ w, const T* __restrict__ wbias, const float* __restrict__ bias, int E, int K, int k, int mode,
@@ -195,7 +194,7 @@ __global__ void __launch_bounds__(256) router_route_small_kernel(
     if (lane == 0) slog[n] = acc + (wbias ? to_f(wbias[n]) : 0.f);
   }
   __syncthreads();
-  if (warp == 0) route_row<float>(out_w, out_ids, slog, bias, t, lane, E, k, mode, renorm, n_group, topk_group, group_top,
+  if (warp == 0) route_row<float, PER>(out_w, out_ids, slog, bias, t, lane, E, k, mode, renorm, n_group, topk_group, group_top,
                                   scale);
 }
 
@@ -504,16 +503,26 @@ __global__ void __launch_bounds__(256) router_gemm_small_kernel(float* __restric
 
 using namespace b200;
 
+// experts per lane, rounded up to what the routing kernels are built for
+#define B200_DISPATCH_PER(E, ...)                             \
+  do {                                                        \
+    if ((E) <= 32) { constexpr int PER = 1; __VA_ARGS__; }    \
+    else if ((E) <= 64) { constexpr int PER = 2; __VA_ARGS__; }   \
+    else if ((E) <= 128) { constexpr int PER = 4; __VA_ARGS__; }  \
+    else if ((E) <= 256) { constexpr int PER = 8; __VA_ARGS__; }  \
+    else { constexpr int PER = kMaxEPerLane; __VA_ARGS__; }       \
+  } while (0)
+
 extern "C" int b200_moe_route(float* out_w, int* out_ids, const void* logits, const float* bias, int64_t T_, int E,
                               int k, int mode, int renorm, int n_group, int topk_group, int group_top, float scale, int64_t stride,
                               int dtype, cudaStream_t st) {
   if (T_ == 0) return 0;
   if (E > 32 * kMaxEPerLane || k > kMaxTopK || n_group > 32 || (n_group > 1 && E % n_group)) return 2;
   const int wpb = 4;
-  B200_DISPATCH_DTYPE(dtype, {
-    launch_pdl(moe_route_kernel<T>, dim3((T_ + wpb - 1) / wpb), dim3(wpb * 32), 0, st, out_w, out_ids,
+  B200_DISPATCH_DTYPE(dtype, B200_DISPATCH_PER(E, {
+    launch_pdl(moe_route_kernel<T, PER>, dim3((T_ + wpb - 1) / wpb), dim3(wpb * 32), 0, st, out_w, out_ids,
                (const T*)logits, bias, T_, E, k, mode, renorm, n_group, topk_group, group_top, scale, stride);
-  });
+  }));
   return (int)cudaGetLastError();
 }
 
@@ -652,10 +661,11 @@ extern "C" int b200_router_route_small(float* out_w, int* out_ids, const void* x
   if (K % (16 / esz) || (x_stride * esz) % 16) return 2;
   const size_t smem = (((size_t)K * esz + 15) & ~(size_t)15) + (size_t)E * 4;
   if (smem > 96 * 1024) return 2;
-  B200_DISPATCH_DTYPE(dtype, {
-    if (smem > 48 * 1024) ensure_dynamic_smem((const void*)router_route_small_kernel<T>, 96 * 1024);
-    launch_pdl(router_route_small_kernel<T>, dim3((unsigned)T_), dim3(256), smem, st, out_w, out_ids, (const T*)x,
+  B200_DISPATCH_DTYPE(dtype, B200_DISPATCH_PER(E, {
+    const auto kern = router_route_small_kernel<T, PER>;
+    if (smem > 48 * 1024) ensure_dynamic_smem((const void*)kern, 96 * 1024);
+    launch_pdl(kern, dim3((unsigned)T_), dim3(256), smem, st, out_w, out_ids, (const T*)x,
                x_stride, (const T*)w, (const T*)wbias, bias, E, K, k, mode, renorm, n_group, topk_group, group_top, scale);
-  });
+  }));
   return (int)cudaGetLastError();
 }

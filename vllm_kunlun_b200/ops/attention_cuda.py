@@ -90,6 +90,8 @@ def paged_attention_cuda(out, q, kv_cache, block_tables, seq_lens, query_start_l
         _ext.C().paged_attention_generic(out, q, kv_cache, block_tables, seq_lens, query_start_loc, sinks, 0,
                                          window or 0, scale, bias, gate, keep_first, sigmoid)
         return out
+    if keep_first and bias is None:      # the instantiations that keep first keys read a bias
+        bias = torch.zeros(Hq, 1, dtype=torch.float32, device=q.device)
     if (decode_layout and (UMMA_DECODE[0] or extras) and D == 128 and kv_cache.shape[3] % 64 == 0
             and q.dtype in (torch.bfloat16, torch.float16)):
         if num_splits is None:
