@@ -3,8 +3,8 @@
 //   out_t = S_t * silu(g)
 // over raw projections zr, ur, g; the state [slots][W] is fp32 and carried per request.
 // A token is the map S -> a S + b with a = 1 - z = sigmoid(-(zr + bz)), b = z c, and maps compose: a' a, a' b + b'.  One CTA takes
-// 32 channels of one request, a lane each; its 16 warps take consecutive runs of tokens of a block, compose their run, meet over
-// shared memory and apply the map of everything in front, while the next block's projections are on their way.  Products only: no
+// 32 channels of one request, a lane each; its 16 warps take consecutive runs of tokens of a block and compose their run, one warp
+// applies the runs' maps to the state in turn, and every warp walks its run from the state in front of it, while the next block's projections are on their way.  Products only: no
 // logarithms, no quotients of gates, so gates near zero and one are safe.  Single tokens: a thread per channel.
 // Launched with programmatic dependent launch: no __restrict__ on what a predecessor writes.  Compiled without fast-math.
 #include "../api.h"
@@ -38,7 +38,7 @@ __device__ __forceinline__ void token(float zr, float ur, float g, float bz, flo
 
 template <typename T>
 __global__ void __launch_bounds__(kWarps * 32, 2) blend_scan_kernel(BlendArgs p) {
-  __shared__ float sa[2][kWarps][32], sb[2][kWarps][32];
+  __shared__ float sa[2][kWarps][32], sb[2][kWarps][32], ss[2][kWarps][32];
   griddep_launch();
   griddep_wait();
   const int req = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -46,54 +46,63 @@ __global__ void __launch_bounds__(kWarps * 32, 2) blend_scan_kernel(BlendArgs p)
   int64_t slot = p.slots[req];
   if (slot >= p.num_slots) slot = -1;
   if (q0 >= q1 || slot < 0) return;
-  const int c = blockIdx.x * 32 + lane;
-  const bool on = c < p.width;
-  const float bz = on ? p.z_bias[c] : 0.f, bu = on ? p.x_bias[c] : 0.f;
-  float S = on && p.has_init[req] ? p.state[slot * p.width + c] : 0.f;
-  const T* z = reinterpret_cast<const T*>(p.z) + c;
-  const T* x = reinterpret_cast<const T*>(p.x) + c;
-  const T* g = reinterpret_cast<const T*>(p.g) + c;
-  T* out = reinterpret_cast<T*>(p.out) + c;
+  // lanes behind the last channel compute the last one again and store nothing
+  const bool on = blockIdx.x * 32 + lane < p.width;
+  const int c = min(blockIdx.x * 32 + lane, p.width - 1);
+  const float bz = p.z_bias[c], bu = p.x_bias[c];
+  float S = p.has_init[req] ? p.state[slot * p.width + c] : 0.f;     // warp 0: state in front of the block
+  const int64_t first = q0 + warp * kRun;
+  const T* z = reinterpret_cast<const T*>(p.z) + first * p.stride + c;
+  const T* x = reinterpret_cast<const T*>(p.x) + first * p.stride + c;
+  const T* g = reinterpret_cast<const T*>(p.g) + first * p.stride + c;
+  T* out = reinterpret_cast<T*>(p.out) + first * p.out_stride + c;
+  const uint32_t row = (uint32_t)p.stride, out_row = (uint32_t)p.out_stride;
+  const int64_t block_step = (int64_t)kBlock * p.stride, out_step = (int64_t)kBlock * p.out_stride;
   T zr[kRun], ur[kRun], gr[kRun];
-  auto rows = [&](int64_t base) {      // tokens of this warp's run
-    return on ? (int)max((int64_t)0, min((int64_t)kRun, q1 - base - warp * kRun)) : 0;
-  };
-  auto fetch = [&](int64_t base) {
-    const int n = rows(base);
-    const int64_t o = (base + warp * kRun) * p.stride;
+  auto fetch = [&](int n) {             // n rows of this warp's run, then the pointers move on to the next block
+    if (n >= kRun) {
 #pragma unroll
-    for (int i = 0; i < kRun; ++i)
-      if (i < n) { zr[i] = z[o + i * p.stride]; ur[i] = x[o + i * p.stride]; gr[i] = g[o + i * p.stride]; }
+      for (int i = 0; i < kRun; ++i) { zr[i] = z[i * row]; ur[i] = x[i * row]; gr[i] = g[i * row]; }
+    } else {
+#pragma unroll
+      for (int i = 0; i < kRun; ++i)
+        if (i < n) { zr[i] = z[i * row]; ur[i] = x[i * row]; gr[i] = g[i * row]; }
+    }
+    z += block_step;
+    x += block_step;
+    g += block_step;
   };
-  fetch(q0);
+  int left = (int)(q1 - first);         // rows from this warp's run on
+  fetch(left);
   int buf = 0;
-  for (int64_t base = q0; base < q1; base += kBlock, buf ^= 1) {
-    const int n = rows(base);
+  for (int64_t base = q0; base < q1; base += kBlock, left -= kBlock, buf ^= 1) {
     float a[kRun], b[kRun], gate[kRun], A = 1.f, B = 0.f;
 #pragma unroll
     for (int i = 0; i < kRun; ++i) {
-      if (i >= n) break;
       token<T>(to_f(zr[i]), to_f(ur[i]), to_f(gr[i]), bz, bu, a[i], b[i], gate[i]);
+      if (i >= left) { a[i] = 1.f; b[i] = 0.f; }     // behind the request's end: nothing happens
       B = fmaf(a[i], B, b[i]);
       A *= a[i];
     }
-    if (base + kBlock < q1) fetch(base + kBlock);
+    if (base + kBlock < q1) fetch(left - kBlock);
     sa[buf][warp][lane] = A;
     sb[buf][warp][lane] = B;
-    __syncthreads();      // buffers alternate: one barrier per block
-    float mine = S;       // state in front of this warp's run; S moves on to the end of the block
+    __syncthreads();
+    if (warp == 0) {      // states in front of every warp's run; buffers alternate, so two barriers per block suffice
 #pragma unroll
-    for (int w = 0; w < kWarps; ++w) {
-      if (w == warp) mine = S;
-      S = fmaf(sa[buf][w][lane], S, sb[buf][w][lane]);
+      for (int w = 0; w < kWarps; ++w) {
+        ss[buf][w][lane] = S;
+        S = fmaf(sa[buf][w][lane], S, sb[buf][w][lane]);
+      }
     }
-    T* o = out + (base + warp * kRun) * p.out_stride;
+    __syncthreads();
+    float mine = ss[buf][warp][lane];
 #pragma unroll
     for (int i = 0; i < kRun; ++i) {
-      if (i >= n) break;
       mine = fmaf(a[i], mine, b[i]);
-      o[i * p.out_stride] = from_f<T>(mine * gate[i]);
+      if (on && i < left) out[i * out_row] = from_f<T>(mine * gate[i]);
     }
+    out += out_step;
   }
   if (warp == 0 && on) p.state[slot * p.width + c] = S;
 }
@@ -128,7 +137,7 @@ extern "C" int b200_gated_blend(const BlendArgs* args, int dtype, cudaStream_t s
   using namespace b200;
   const BlendArgs& a = *args;
   if (a.R == 0 || a.width == 0) return 0;
-  if (a.R > 65535) return 3;
+  if (a.R > 65535 || a.stride >= (1 << 28) || a.out_stride >= (1 << 28)) return 3;
   B200_DISPATCH_DTYPE(dtype, {
     if (a.steps)
       launch_pdl(blend_step_kernel<T>, dim3((a.width + 127) / 128, a.R), dim3(128), 0, st, a);
