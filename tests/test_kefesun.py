@@ -171,8 +171,8 @@ def plain_attention(q, k, v, lens, scale, pb, size, keep):
     out, off = [], 0
     for a, b in lens:
         s = slice(off, off + a + b)
-        out.append(oracle.sigmoid_attention(q[s], k[s][:, of], v[s][:, of], scale, pb,
-                                            oracle.visible(a + b, size if size else a + b, keep))[a:])
+        out.append(oracle.sigmoid_attention(q[s][a:], k[s][:, of], v[s][:, of], scale, pb,
+                                            oracle.visible(a + b, size if size else a + b, keep)[a:]))
         off += a + b
     return torch.cat(out)
 
@@ -182,7 +182,8 @@ def plain_attention(q, k, v, lens, scale, pb, size, keep):
 def test_sigmoid_attention(device, dtype, H, G, D, V):
     """Unequal requests, single tokens beside portions; windows and kept keys of every relation to pages and tiles."""
     g = torch.Generator().manual_seed(D)
-    for lens in ([(37, 1), (64, 1), (0, 1), (190, 1), (420, 1)], [(37, 1), (0, 130), (30, 41), (63, 2), (300, 3), (0, 1)]):
+    for lens in ([(37, 1), (64, 1), (0, 1), (190, 1), (420, 1)], [(37, 1), (0, 130), (30, 41), (63, 2), (300, 3), (0, 1)],
+                 [(2500, 1), (1700, 1)], [(1400, 140)]):
         T = sum(a + b for a, b in lens)
         q, k, v = rounded(dtype, torch.randn(T, H, D, generator=g) * 1.5, torch.randn(T, G, D, generator=g),
                           torch.randn(T, G, V, generator=g))

@@ -57,9 +57,13 @@ class KefesunDecoderLayer(ListedLayer):
         state = None if self.taps < 2 else get_forward_context().kv_caches[self.layer_idx][k - 1 - self.sublayers]
         return getattr(self, f"conv{k}"), state
 
+    def mix(self, h):
+        (y, _), = self.mixer(h)
+        return y
+
     def steps(self) -> list:
         """``(sublayer, its convolution, its norm weight)`` in order."""
-        out = [(lambda h: self.mixer(h)[0][0], self.conv(1), self.norm1.weight)]
+        out = [(self.mix, self.conv(1), self.norm1.weight)]
         return out if self.mlp is None else out + [(self.mlp, self.conv(2), self.norm2.weight)]
 
     def load_tensor(self, key: str, w: torch.Tensor):
